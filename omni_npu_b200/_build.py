@@ -1,9 +1,12 @@
 """In-tree build of the native libraries.
 
-Two shared objects are produced next to this file:
+Three shared objects are produced next to this file:
 
-* ``_C.so``       CUDA kernels for sm_100a (``csrc/**/*.cu``) + ``csrc/bindings.cpp``
-                  registering ``torch.ops.omni_b200.*``.
+* ``_C_core.so``  the kernels of ``CORE_SOURCES`` + ``csrc/bindings_core.cpp``: matrix products, MoE
+                  routing, sampling, gated / windowed attention, the 32-bit residual stream.  Some
+                  models run on this library alone (``ensure_core`` builds nothing else).
+* ``_C.so``       all other CUDA kernels for sm_100a (``csrc/**/*.cu``) + ``csrc/bindings.cpp``,
+                  linked against ``_C_core.so``.  Both register ``torch.ops.omni_b200.*``.
 * ``_runtime.so`` host-only C++ runtime pieces (``csrc/runtime``, ``csrc/alloc``):
                   KV block allocator, scheduler helpers, VMM sleep-mode allocator.
 
@@ -31,6 +34,14 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xptxas", "-v",
 ]
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function"]
+
+
+# sources of the core library, relative to csrc/
+CORE_SOURCES = [
+    "attn/gqa_gated.cu", "attn/gqa_gated_decode.cu", "attn/gqa_gated_prefill.cu", "attn/gqa_prefill_tcgen05.cu",
+    "gemm/gemm_simt.cu", "gemm/gemm_tcgen05.cu", "gemm/gemm_tcgen05_pair.cu", "moe/moe_ep.cu",
+    "norm_rope/residual_norm.cu", "sample/sampling.cu",
+]
 
 
 def _nvcc() -> str:
@@ -78,9 +89,35 @@ def runtime_sources() -> list[Path]:
     return out
 
 
-def build(force: bool = False, verbose: bool = False) -> dict:
-    """Compile everything that is out of date.  Returns the paths of the libraries."""
-    import torch  # noqa: F401  (import first: the headers' location comes from it)
+def core_is_current() -> bool:
+    """Whether ``_C_core.so`` exists and is newer than everything it is made of."""
+    lib = PKG / "_C_core.so"
+    if not lib.exists():
+        return False
+    t = lib.stat().st_mtime
+    srcs = [CSRC / x for x in CORE_SOURCES] + [CSRC / "bindings_core.cpp"]
+    return all(p.stat().st_mtime <= t for p in srcs) and _newest_header_mtime() <= t
+
+
+def ensure_core(verbose: bool = False) -> None:
+    """Build the core library alone when it is missing or older than its sources (one process at a
+    time; the others wait for it)."""
+    if core_is_current():
+        return
+    import fcntl
+    OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not core_is_current():
+            build(verbose=verbose, core_only=True)
+
+
+def build(force: bool = False, verbose: bool = False, core_only: bool = False) -> dict:
+    """Compile everything that is out of date (``core_only``: for the core library alone).  Returns
+    the paths of the libraries."""
+    import sysconfig
+
+    import torch  # (import first: the headers' location comes from it)
     from torch.utils import cpp_extension as ce
 
     OBJ.mkdir(parents=True, exist_ok=True)
@@ -88,35 +125,32 @@ def build(force: bool = False, verbose: bool = False) -> dict:
     nvcc = _nvcc()
     cuda_home = _cuda_home()
     jobs: list[tuple[list[str], Path | None]] = []
-    objs: list[Path] = []
+    objs: dict[str, list[Path]] = {"_C_core": [], "_C": [], "_runtime": []}
+    dirty: set[str] = set()
+
+    def compile_one(src: Path, lib: str, cmd: list[str], log: bool = False) -> None:
+        obj = OBJ / (src.relative_to(CSRC).as_posix().replace("/", "__") + ".o")
+        objs[lib].append(obj)
+        if force or _stale(src, obj, hdr_mtime):
+            dirty.add(lib)
+            jobs.append(([*cmd, "-c", str(src), "-o", str(obj)], obj.with_suffix(".log") if log else None))
 
     for src in cuda_sources():
-        obj = OBJ / (src.relative_to(CSRC).as_posix().replace("/", "__") + ".o")
-        objs.append(obj)
-        if force or _stale(src, obj, hdr_mtime):
-            jobs.append(([nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)],
-                         obj.with_suffix(".log")))
+        lib = "_C_core" if src.relative_to(CSRC).as_posix() in CORE_SOURCES else "_C"
+        if lib == "_C_core" or not core_only:
+            compile_one(src, lib, [nvcc, *NVCC_FLAGS, "-I", str(CSRC)], log=True)
 
     inc = []
     for p in ce.include_paths("cuda") if hasattr(ce, "include_paths") else []:
         inc += ["-I", p]
-    inc += ["-I", os.path.join(cuda_home, "include")]
-    import sysconfig
-    inc += ["-I", sysconfig.get_paths()["include"]]
+    inc += ["-I", os.path.join(cuda_home, "include"), "-I", sysconfig.get_paths()["include"]]
     abi = int(getattr(torch._C, "_GLIBCXX_USE_CXX11_ABI", 1))
-    bind_src = CSRC / "bindings.cpp"
-    bind_obj = OBJ / "bindings.cpp.o"
-    if force or _stale(bind_src, bind_obj, hdr_mtime):
-        jobs.append((["g++", *CXX_FLAGS, f"-D_GLIBCXX_USE_CXX11_ABI={abi}", *inc, "-c", str(bind_src),
-                      "-o", str(bind_obj)], None))
-
-    rt_objs: list[Path] = []
-    for src in runtime_sources():
-        obj = OBJ / (src.relative_to(CSRC).as_posix().replace("/", "__") + ".o")
-        rt_objs.append(obj)
-        if force or _stale(src, obj, hdr_mtime):
-            jobs.append((["g++", *CXX_FLAGS, "-I", os.path.join(cuda_home, "include"), "-I", str(CSRC),
-                          "-c", str(src), "-o", str(obj)], None))
+    cxx = ["g++", *CXX_FLAGS, f"-D_GLIBCXX_USE_CXX11_ABI={abi}", *inc]
+    compile_one(CSRC / "bindings_core.cpp", "_C_core", cxx)
+    if not core_only:
+        compile_one(CSRC / "bindings.cpp", "_C", cxx)
+        for src in runtime_sources():
+            compile_one(src, "_runtime", ["g++", *CXX_FLAGS, "-I", os.path.join(cuda_home, "include"), "-I", str(CSRC)])
 
     if jobs:
         if verbose:
@@ -124,17 +158,23 @@ def build(force: bool = False, verbose: bool = False) -> dict:
         with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 4)) as ex:
             list(ex.map(lambda j: _run(j[0], j[1]), jobs))
 
-    lib_c = PKG / "_C.so"
-    lib_rt = PKG / "_runtime.so"
     torch_lib = os.path.join(os.path.dirname(torch.__file__), "lib")
-    if jobs or not lib_c.exists():
-        _run(["g++", "-shared", "-o", str(lib_c), *map(str, objs), str(bind_obj),
-              f"-L{torch_lib}", "-lc10", "-ltorch_cpu", "-ltorch", "-lc10_cuda", "-ltorch_cuda",
-              f"-L{cuda_home}/lib64", "-lcudart", f"-Wl,-rpath,{torch_lib}",
-              f"-Wl,-rpath,{cuda_home}/lib64"])
-    if rt_objs and (jobs or not lib_rt.exists()):
-        _run(["g++", "-shared", "-o", str(lib_rt), *map(str, rt_objs), "-ldl", "-lpthread"])
-    return {"_C": lib_c, "_runtime": lib_rt if rt_objs else None}
+    libs = ["-lc10", "-ltorch_cpu", "-ltorch", "-lc10_cuda", "-ltorch_cuda", f"-L{cuda_home}/lib64", "-lcudart",
+            f"-Wl,-rpath,{torch_lib}", f"-Wl,-rpath,{cuda_home}/lib64"]
+
+    def link(name: str, extra: list[str]) -> Path:
+        out = PKG / f"{name}.so"
+        if name in dirty or not out.exists():
+            part = out.with_suffix(f".so.{os.getpid()}")      # in place in one step: others may be loading it
+            _run(["g++", "-shared", "-o", str(part), f"-Wl,-soname,{out.name}", *map(str, objs[name]), *extra])
+            os.replace(part, out)
+        return out
+
+    out = {"_C_core": link("_C_core", [f"-L{torch_lib}", *libs])}
+    if not core_only:
+        out["_C"] = link("_C", [f"-L{PKG}", "-l:_C_core.so", "-Wl,-rpath,$ORIGIN", f"-L{torch_lib}", *libs])
+        out["_runtime"] = link("_runtime", ["-ldl", "-lpthread"]) if objs["_runtime"] else None
+    return out
 
 
 if __name__ == "__main__":

@@ -113,3 +113,53 @@ class GQAAttention(torch.nn.Module):
         return ops.gqa_decode(q, k_cache, v_cache, md.block_tables, md.seq_lens, md.num_seqs,
                               self.num_heads, self.scale, md.q_len, self.window,
                               max_seq_len=md.max_seq_len)
+
+
+class GatedGQAAttention(torch.nn.Module):
+    """Attention with any head sizes (queries / keys ``head_dim``, values ``head_dim_v``), rotation of the
+    first ``rot_dim`` dimensions, an optional sliding window, an optional sink (a key of score ``sink``
+    without a value in every softmax) and an optional output gate.  The cache rows are padded to whole
+    tensor-core steps (``ops.gated_head_pad``)."""
+
+    def __init__(self, layer_idx: int, num_heads: int, num_kv_heads: int, head_dim: int, head_dim_v: int,
+                 scale: float, rot_dim: int, neox: bool = True, sliding_window: int = 0,
+                 sink: Optional[float] = None) -> None:
+        super().__init__()
+        self.layer_idx = layer_idx
+        self.num_heads, self.num_kv_heads = num_heads, num_kv_heads
+        self.head_dim, self.head_dim_v = head_dim, head_dim_v
+        self.scale, self.rot_dim, self.neox = scale, rot_dim, neox
+        self.window, self.sink = sliding_window, sink
+
+    def cache_widths(self, dtype: torch.dtype) -> Tuple[int, int]:
+        return ops.gated_head_pad(self.head_dim, dtype), ops.gated_head_pad(self.head_dim_v, dtype)
+
+    def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: Optional[torch.Tensor],
+                cos_sin: torch.Tensor, out_width: int = 0) -> torch.Tensor:
+        """q [T, Hq*D] (rotated in place), k [T, Hk*D], v [T, Hk*Dv], gate [T, Hq*Dv] or None: views into
+        the fused projection.  Returns [T, max(Hq*Dv, out_width)], zero beyond the heads."""
+        ctx = get_forward_context()
+        md: AttentionMetadata = ctx.attn_metadata
+        k_cache, v_cache = ctx.kv_caches[self.layer_idx]
+        ops.gated_rope_cache_(q, k, v, k_cache, v_cache, md.positions, md.slot_mapping, cos_sin, self.head_dim,
+                              self.head_dim_v, self.rot_dim, self.neox)
+        t, used = q.shape[0], self.num_heads * self.head_dim_v
+        out = q.new_zeros(t, out_width) if out_width > used else q.new_empty(t, used)
+
+        def run(rows: slice, seqs: slice, cu_q, n: int, max_q: int):
+            ops.gated_attention(q[rows], None if gate is None else gate[rows], k_cache, v_cache, out[rows],
+                                md.block_tables[seqs], cu_q, md.seq_lens[seqs], n, max_q, self.num_heads,
+                                self.head_dim, self.head_dim_v, self.scale, self.window, self.sink,
+                                max_seq_len=md.max_seq_len)
+
+        if not md.is_prefill:
+            run(slice(None), slice(None), None, md.num_seqs, md.q_len)
+            return out
+        nd = md.extra.get("num_decode_seqs", 0)
+        if nd:           # rows [0, nd): single new tokens of decoding sequences
+            run(slice(0, nd), slice(0, nd), None, nd, 1)
+            run(slice(nd, t), slice(nd, None), md.extra["cu_q_prefill"], md.num_seqs - nd,
+                md.extra["max_q_len_prefill"])
+        else:
+            run(slice(None), slice(None), md.cu_q, md.num_seqs, md.max_q_len)
+        return out

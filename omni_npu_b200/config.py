@@ -29,6 +29,49 @@ def to_dtype(x) -> torch.dtype:
     return _DTYPES[str(x).replace("torch.", "")]
 
 
+# ---- designs whose layers are listed one by one: what a layer is made of
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Grouped-query attention with its own sizes per layer."""
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    rotary_dim: int
+    rope_theta: float
+    scale: float
+    rope_neox: bool = False
+    sliding_window: int = 0               # 0 = every earlier key
+    sink: Optional[float] = None          # score of a key without a value in every softmax
+    output_gate: bool = False             # result times the sigmoid of its own projection
+
+
+@dataclass(frozen=True)
+class ExpertSpec:
+    """A gated feed-forward: width and activation ((0, 0) = silu, else slope and limit of the clamped form)."""
+    intermediate_size: int
+    act: Tuple[float, float] = (0.0, 0.0)
+
+
+@dataclass(frozen=True)
+class MoESpec:
+    num_experts: int
+    top_k: int
+    expert: ExpertSpec
+    shared: Optional[ExpertSpec] = None
+    scoring_func: str = "softmax"
+    renormalize: bool = True
+    scale: float = 1.0
+    n_group: int = 1
+    topk_group: int = 1
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    attention: AttentionSpec
+    mlp: Optional[MoESpec] = None
+
+
 @dataclass
 class ModelConfig:
     architecture: str = "LlamaForCausalLM"
@@ -80,6 +123,10 @@ class ModelConfig:
     # --- quantisation
     quant_method: Optional[str] = None    # None | "fp8" (128x128 block scales)
     weight_block_size: Tuple[int, int] = (128, 128)
+    # --- designs that list their layers
+    layer_specs: Tuple[LayerSpec, ...] = ()
+    embedding_scale: float = 1.0
+    norm_weight_offset: float = 0.0       # 1: norm weights are stored around zero
     # --- misc
     eos_token_id: Optional[int] = None
     hf_config: Dict[str, Any] = field(default_factory=dict)
@@ -105,6 +152,9 @@ class ModelConfig:
     def kv_bytes_per_token(self) -> int:
         """Bytes of KV cache one token occupies across all layers (per TP-1 rank)."""
         esz = self.dtype.itemsize
+        if self.layer_specs:
+            return esz * sum(s.attention.num_kv_heads * (s.attention.head_dim + s.attention.v_head_dim)
+                             for s in self.layer_specs)
         if self.use_mla:
             per = self.kv_lora_rank + self.qk_rope_head_dim + (self.index_head_dim if self.use_sparse else 0)
             return self.num_layers * per * esz
@@ -112,7 +162,11 @@ class ModelConfig:
 
     @classmethod
     def from_hf_dict(cls, d: Dict[str, Any], dtype=None) -> "ModelConfig":
-        """Build from the contents of an HF ``config.json``."""
+        """Build from the contents of a ``config.json``: HF keys, or the own keys of a design that names
+        itself under ``architecture`` and has a reader in the model registry."""
+        if "architectures" not in d and isinstance(d.get("architecture"), str):
+            from .models.registry import resolve_config_reader
+            return resolve_config_reader(d["architecture"])(d, dtype=dtype)
         if "text_config" in d and isinstance(d["text_config"], dict):
             merged = dict(d["text_config"])
             merged.setdefault("architectures", d.get("architectures"))

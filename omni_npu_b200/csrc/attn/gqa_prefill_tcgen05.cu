@@ -19,12 +19,14 @@
 // is in flight, frees its TMEM and returns (its output rows are then not valid).
 //
 // Same operation as gqa_prefill_kernel (which stays for other head sizes, sliding windows and
-// sinks); replaces npu_fused_infer_attention_score in its TND paged prefill form
+// sinks).  The EXT form adds what gqa_gated.cuh describes: a sliding window (tiles before it are
+// skipped), a softmax sink without a value, and the output gate; replaces npu_fused_infer_attention_score in its TND paged prefill form
 // (omni_npu/attention/backends/attention.py:216-281).
 
 #include <cstdlib>
 
 #include "attn_params.cuh"
+#include "gqa_gated.cuh"
 #include "../common/device_once.h"
 #include "../common/pdl.cuh"
 #include "../common/ptx.cuh"
@@ -98,11 +100,19 @@ __device__ __forceinline__ uint64_t desc_mnmajor(uint32_t smem_addr, uint32_t lb
 // Launch bounds name 256 threads although 192 are launched: the register file is split over the
 // four sub-partitions of an SM, and two CTAs of six warps put four warps on one of them, which only
 // fits with at most 128 registers per thread (the bound a 256-thread, two-per-SM kernel gets).
-template <int DQK>
+// What the EXT form takes beyond AttnParams.
+struct PrefillExt {
+  const __nv_bfloat16* gate;   // or null
+  long long g_stride;
+  int has_sink;
+  float sink_log2;
+};
+
+template <int DQK, bool EXT>
 __global__ void __launch_bounds__(256, tcp::Cfg<DQK>::CTAS_PER_SM)
 gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                       const __grid_constant__ CUtensorMap tm_v, const AttnParams p, const int box_rows,
-                      const int m_tiles) {
+                      const int m_tiles, const PrefillExt x) {
   using namespace tcp;
   using C = Cfg<DQK>;
   constexpr int OFF_Q = C::OFF_Q, OFF_K = C::OFF_K, OFF_V = C::OFF_V, OFF_P = C::OFF_P, OFF_BAR = C::OFF_BAR;
@@ -182,7 +192,9 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   const int kvh = h / (p.Hq / p.Hk);
   // keys this tile can see: causal rows reach position ctx + m0 + BM - 1 at most
   const int kv_hi = p.causal ? min(kv_len, ctx + m0 + BM) : kv_len;
-  const int n_tiles = active ? (kv_hi + BN - 1) / BN : 0;
+  // first tile: with a window, the one that holds the oldest key of the tile's first row
+  const int j0 = EXT && p.window > 0 ? max(0, ctx + m0 - p.window + 1) / BN : 0;
+  const int n_tiles = active ? (kv_hi + BN - 1) / BN - j0 : 0;
 
   int issued = 0;          // tiles whose copies were started (producer lane only)
   if (warp == 0) {
@@ -203,7 +215,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
             break;
           }
         }
-        const int n0 = j * BN;
+        const int n0 = (j0 + j) * BN;
         const int nvalid = min(BN, kv_len - n0);
         const int nboxes = (nvalid + box_rows - 1) / box_rows;
         const uint32_t box_bytes = static_cast<uint32_t>(nboxes * box_rows * 128);
@@ -285,7 +297,8 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const uint32_t lane_base = static_cast<uint32_t>(quarter * 32) << 16;
     const int q_pos = ctx + m0 + r;                       // position of this row's token
     const bool row_valid = m0 + r < q_len;
-    float row_max = -INFINITY, row_sum = 0.f;
+    // the sink is a key seen from the start
+    float row_max = EXT && x.has_sink ? x.sink_log2 : -INFINITY, row_sum = EXT && x.has_sink ? 1.f : 0.f;
     uint8_t* p_row = smem + OFF_P + r * 128;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
@@ -301,12 +314,13 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);
-      const int n0 = j * BN;
+      const int n0 = (j0 + j) * BN;
       float tile_max = -INFINITY;
       float s[64];
       // tiles that lie entirely below the diagonal and inside the sequence need no mask
       const int row_lo = ctx + m0 + quarter * 32;                      // smallest position in this warp
-      const bool interior = n0 + BN <= kv_len && (!p.causal || n0 + BN - 1 <= row_lo);
+      const bool interior = n0 + BN <= kv_len && (!p.causal || n0 + BN - 1 <= row_lo) &&
+                            (!EXT || p.window <= 0 || n0 > row_lo + 31 - p.window);
       if (interior) {
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
@@ -318,7 +332,8 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
           const int key = n0 + c;
-          const bool keep = key < kv_len && (!p.causal || key <= q_pos);
+          const bool keep = key < kv_len && (!p.causal || key <= q_pos) &&
+                            (!EXT || p.window <= 0 || key > q_pos - p.window);
           const float v = keep ? __uint_as_float(sv[c >> 5][c & 31]) * p.scale_log2 : -INFINITY;
           s[c] = v;
           tile_max = fmaxf(tile_max, v);
@@ -389,6 +404,24 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         tmem_ld_32x32b_x32(tmem_base + lane_base + COL_O + c * 32, ov);
         tmem_ld_wait();
         if (row_valid) {
+          if constexpr (EXT) {
+            if (x.gate) {
+              const uint4* g = reinterpret_cast<const uint4*>(x.gate + static_cast<long long>(q_begin + m0 + r) * x.g_stride +
+                                                              static_cast<long long>(h) * D + c * 32);
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const uint4 gv = g[i];
+                const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                  ov[i * 8 + 2 * k] = __float_as_uint(__uint_as_float(ov[i * 8 + 2 * k]) *
+                                                      gate_sigmoid(__uint_as_float(gw[k] << 16)));
+                  ov[i * 8 + 2 * k + 1] = __float_as_uint(__uint_as_float(ov[i * 8 + 2 * k + 1]) *
+                                                          gate_sigmoid(__uint_as_float(gw[k] & 0xffff0000u)));
+                }
+              }
+            }
+          }
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             uint4 v;
@@ -440,7 +473,7 @@ using namespace b200;
 // smem_bytes = 0: the kernel's own size; another value asks what a CTA of that size would get.
 extern "C" int b200_gqa_prefill_tc_ctas_per_sm(int smem_bytes) {
   int n = 0;
-  auto kern = gqa_prefill_tc_kernel<128>;
+  auto kern = gqa_prefill_tc_kernel<128, false>;
   if (smem_bytes <= 0) smem_bytes = tcp::Cfg<128>::SMEM;
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, tcp::Cfg<128>::SMEM);
   cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
@@ -453,7 +486,7 @@ extern "C" int b200_gqa_prefill_tc_ctas_per_sm(int smem_bytes) {
 // local (spill) bytes per thread.
 extern "C" int b200_gqa_prefill_tc_resources(int* out) {
   cudaFuncAttributes fa{};
-  if (cudaFuncGetAttributes(&fa, gqa_prefill_tc_kernel<128>) != cudaSuccess) return -1;
+  if (cudaFuncGetAttributes(&fa, gqa_prefill_tc_kernel<128, false>) != cudaSuccess) return -1;
   int dev = 0, v = 0;
   cudaGetDevice(&dev);
   out[0] = fa.numRegs;
@@ -471,10 +504,10 @@ extern "C" int b200_gqa_prefill_tc_resources(int* out) {
   return 0;
 }
 
-template <int DQK>
+template <int DQK, bool EXT = false>
 static int launch_prefill_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const AttnParams& p,
-                             int box_rows, dim3 grid, cudaStream_t stream) {
-  auto kern = gqa_prefill_tc_kernel<DQK>;
+                             int box_rows, dim3 grid, cudaStream_t stream, const PrefillExt& x = PrefillExt{}) {
+  auto kern = gqa_prefill_tc_kernel<DQK, EXT>;
   static DeviceOnce once;
   int dev = 0;
   if (once.needed(&dev)) {
@@ -484,7 +517,7 @@ static int launch_prefill_tc(const CUtensorMap& tq, const CUtensorMap& tk, const
     once.mark(dev);
   }
   return launch_pdl(kern, grid, dim3(tcp::THREADS), tcp::Cfg<DQK>::SMEM, stream, 1, tq, tk, tv, p, box_rows,
-                    static_cast<int>(grid.x)) == cudaSuccess
+                    static_cast<int>(grid.x), x) == cudaSuccess
              ? 0
              : -21;
 }
@@ -540,3 +573,54 @@ extern "C" int b200_gqa_prefill_tc(const void* q, const void* k_cache, const voi
   return Dqk == 128 ? launch_prefill_tc<128>(tq, tk, tv, p, box_rows, grid, stream)
                     : launch_prefill_tc<192>(tq, tk, tv, p, box_rows, grid, stream);
 }
+
+// The EXT form: gated, windowed attention with head sizes 128.  Returns 1 when the problem is not one it takes.
+namespace b200 {
+int gated_prefill_tc(const GatedAttnParams& g, int max_q_len, long long total_q_rows, int* status,
+                     cudaStream_t stream) {
+  const auto aligned = [](const void* ptr, long long stride) {
+    return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0 && ((stride * 2) & 15) == 0;
+  };
+  if (g.D != 128 || g.DV != 128 || g.DP != 128 || g.DVP != 128 || g.num_cache_blocks <= 0) return 1;
+  if (!((g.block_size % 8) == 0 &&
+        (g.block_size <= 64 ? (64 % g.block_size) == 0 : (g.block_size % 64) == 0)) ||
+      !aligned(g.k_cache, 0) || !aligned(g.v_cache, 0) || !aligned(g.q, g.q_stride) ||
+      !aligned(g.out, g.out_stride) || (g.gate && !aligned(g.gate, g.g_stride)))
+    return 1;
+  AttnParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(g.q);
+  p.k_cache = static_cast<const __nv_bfloat16*>(g.k_cache);
+  p.v_cache = static_cast<const __nv_bfloat16*>(g.v_cache);
+  p.out = static_cast<__nv_bfloat16*>(g.out);
+  p.block_tables = g.block_tables;
+  p.cu_q = g.cu_q;
+  p.seq_lens = g.seq_lens;
+  p.max_blocks = g.max_blocks;
+  p.block_size = g.block_size;
+  p.Hq = g.Hq;
+  p.Hk = g.Hk;
+  p.q_stride = g.q_stride;
+  p.out_stride = g.out_stride;
+  p.scale_log2 = g.scale_log2;
+  p.causal = 1;
+  p.window = g.window;
+  p.status = status;
+  p.num_cache_blocks = g.num_cache_blocks;
+  PrefillExt x{static_cast<const __nv_bfloat16*>(g.gate), g.g_stride, g.has_sink, g.sink_log2};
+  const int box_rows = g.block_size < 64 ? g.block_size : 64;
+  CUtensorMap tq, tk, tv;
+  int r = make_tensormap_2d(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, g.q, static_cast<uint64_t>(total_q_rows),
+                            static_cast<uint64_t>(g.Hq) * 128, static_cast<uint64_t>(g.q_stride), tcp::BM, 64,
+                            CU_TENSOR_MAP_SWIZZLE_128B);
+  if (r) return -1000;
+  const uint64_t rows = static_cast<uint64_t>(g.num_cache_blocks) * g.Hk * g.block_size;
+  r = make_tensormap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, g.k_cache, rows, 128, 128, box_rows, 64,
+                        CU_TENSOR_MAP_SWIZZLE_128B);
+  if (r) return -2000;
+  r = make_tensormap_2d(&tv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, g.v_cache, rows, 128, 128, box_rows, 64,
+                        CU_TENSOR_MAP_SWIZZLE_128B);
+  if (r) return -3000;
+  const dim3 grid((max_q_len + tcp::BM - 1) / tcp::BM, g.Hq, g.B);
+  return launch_prefill_tc<128, true>(tq, tk, tv, p, box_rows, grid, stream, x);
+}
+}  // namespace b200

@@ -9,21 +9,9 @@
 
 #include <tuple>
 
+#include "bindings_common.h"
+
 extern "C" {
-void b200_gemm_plan(int M, int N, int K, int elem_bytes, int swiglu, int force_bn, int force_splits,
-                    int* out_bn, int* out_splits, size_t* out_ws_bytes, int* out_counters,
-                    int* out_cluster);
-int b200_gemm(const void* A, const void* W, void* C, const void* bias, const void* residual, int M,
-              int N, int K, int lda, int ldw, int ldc, int dtype_fp8, int out_fp32, int swiglu,
-              int BN, int splits, int cluster_split, void* workspace, int* counters, int* status,
-              int max_ctas, cudaStream_t stream);
-int b200_gemm_pair(const void* A, const void* W, void* C, const void* bias, const void* residual,
-                   int M, int N, int K, int lda, int ldw, int ldc, int dtype_fp8, int out_fp32,
-                   int swiglu, int BN, int* status, int max_ctas, cudaStream_t stream);
-int b200_grouped_gemm(const void* A, const void* W, void* C, const int* expert_offsets,
-                      int num_experts, int total_rows, int N, int K, int lda, int ldc,
-                      int dtype_fp8, int swiglu, int BN, int* status, int max_ctas,
-                      cudaStream_t stream);
 int b200_lse_merge(void* out, float* lse_out, const void* outs, const float* lses, int N, long long T, int H, int D,
                    long long stride_n_out, long long stride_n_lse, cudaStream_t stream);
 int b200_gather_cache(void* dst, const void* cache, const int* block_tables, const int* cu_seq, int B,
@@ -108,30 +96,9 @@ int b200_mla_decode(const void* q, const void* cache, void* out, float* lse, con
                     int max_blocks, int block_size, int num_cache_blocks, long long q_stride,
                     long long out_stride, float scale, int splits, void* scratch, int* status,
                     cudaStream_t stream);
-int b200_moe_topk(const float* logits, const float* bias, int* topk_ids, float* topk_w, int T, int E,
-                  int k, int scoring, int n_group, int topk_group, int renorm, float scale,
-                  cudaStream_t stream);
-int b200_argmax(const void* logits, int* out, int B, int V, long long stride, int is_fp32,
-                cudaStream_t stream);
-int b200_sample(const void* logits, int* out, const float* temperature, const int* top_k,
-                const float* top_p, const long long* seeds, const long long* step_offset, int B,
-                int V, long long stride, int is_fp32, cudaStream_t stream);
 }
 
 namespace {
-
-using torch::Tensor;
-
-inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
-
-inline void check(int rc, const char* what) {
-  TORCH_CHECK(rc == 0, "omni_b200::", what, " failed with code ", rc);
-}
-
-#define CHECK_CUDA_BF16(t) \
-  TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kBFloat16, #t " must be a CUDA bf16 tensor")
-#define CHECK_I32(t) \
-  TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kInt && (t).is_contiguous(), #t " must be a contiguous CUDA int32 tensor")
 
 // Merge N partial attention results over disjoint key sets by their log-sum-exp.
 // outs [N, T, H, D] bf16, lses [N, T, H] fp32 -> (out [T, H, D], lse [T, H]).
@@ -187,117 +154,6 @@ std::tuple<Tensor, Tensor> spec_verify(const Tensor& draft, const Tensor& target
                          cur_stream()),
         "spec_verify");
   return {out, num};
-}
-
-// (BN, splits, workspace bytes, counters, cluster flag) for a problem.
-std::tuple<int64_t, int64_t, int64_t, int64_t, int64_t> gemm_plan(int64_t M, int64_t N, int64_t K,
-                                                                  int64_t elem_bytes, bool swiglu,
-                                                                  int64_t force_bn,
-                                                                  int64_t force_splits) {
-  int bn, sp, cnt, cl;
-  size_t ws;
-  b200_gemm_plan((int)M, (int)N, (int)K, (int)elem_bytes, swiglu ? 1 : 0, (int)force_bn,
-                 (int)force_splits, &bn, &sp, &ws, &cnt, &cl);
-  return {bn, sp, (int64_t)ws, cnt, cl};
-}
-
-// C = A @ W^T (+bias) (+residual).  A [M,K], W [N,K]; bf16 or float8_e4m3fn.
-Tensor gemm(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& bias,
-            const c10::optional<Tensor>& residual, bool out_fp32, bool swiglu, int64_t bn,
-            int64_t splits, bool cluster_split, const c10::optional<Tensor>& workspace,
-            const c10::optional<Tensor>& counters, const Tensor& status, int64_t max_ctas) {
-  TORCH_CHECK(a.is_cuda() && w.is_cuda() && a.dim() == 2 && w.dim() == 2, "gemm: 2-D CUDA tensors");
-  TORCH_CHECK(a.scalar_type() == w.scalar_type(), "gemm: dtype mismatch");
-  const bool fp8 = a.scalar_type() == at::kFloat8_e4m3fn;
-  TORCH_CHECK(fp8 || a.scalar_type() == at::kBFloat16, "gemm: bf16 or float8_e4m3fn inputs");
-  TORCH_CHECK(a.stride(1) == 1 && w.stride(1) == 1, "gemm: K must be contiguous");
-  const int M = a.size(0), K = a.size(1), N = w.size(0);
-  TORCH_CHECK(w.size(1) == K, "gemm: K mismatch");
-  c10::cuda::CUDAGuard guard(a.device());
-  const int n_out = swiglu ? N / 2 : N;
-  Tensor c = torch::empty({M, n_out}, a.options().dtype(out_fp32 ? at::kFloat : at::kBFloat16));
-  const void* bias_p = nullptr;
-  const void* res_p = nullptr;
-  if (bias.has_value()) {
-    CHECK_CUDA_BF16(*bias);
-    TORCH_CHECK(bias->numel() == N && bias->is_contiguous(), "gemm: bias [N]");
-    bias_p = bias->data_ptr();
-  }
-  if (residual.has_value()) {
-    CHECK_CUDA_BF16(*residual);
-    TORCH_CHECK(residual->is_contiguous() && residual->size(0) == M && residual->size(1) == n_out,
-                "gemm: residual [M,N] contiguous");
-    res_p = residual->data_ptr();
-  }
-  void* ws_p = nullptr;
-  int* cnt_p = nullptr;
-  if (splits > 1 && !cluster_split) {
-    TORCH_CHECK(workspace.has_value() && counters.has_value(), "gemm: split-K needs workspace");
-    ws_p = workspace->data_ptr();
-    cnt_p = counters->data_ptr<int>();
-  }
-  check(b200_gemm(a.data_ptr(), w.data_ptr(), c.data_ptr(), bias_p, res_p, M, N, K,
-                  (int)a.stride(0), (int)w.stride(0), n_out, fp8 ? 1 : 0, out_fp32 ? 1 : 0,
-                  swiglu ? 1 : 0, (int)bn, (int)splits, cluster_split ? 1 : 0, ws_p, cnt_p,
-                  status.data_ptr<int>(),
-                  (int)max_ctas, cur_stream()),
-        "gemm");
-  return c;
-}
-
-// Same contract as gemm() without split-K, run by CTA pairs: one 256 x BN tile per pair of SMs
-// (tcgen05 cta_group::2), each SM staging half of the weight tile.
-Tensor gemm_pair(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& bias,
-                 const c10::optional<Tensor>& residual, bool out_fp32, bool swiglu, int64_t bn,
-                 const Tensor& status, int64_t max_ctas) {
-  TORCH_CHECK(a.is_cuda() && w.is_cuda() && a.dim() == 2 && w.dim() == 2, "gemm_pair: 2-D CUDA tensors");
-  TORCH_CHECK(a.scalar_type() == w.scalar_type(), "gemm_pair: dtype mismatch");
-  const bool fp8 = a.scalar_type() == at::kFloat8_e4m3fn;
-  TORCH_CHECK(fp8 || a.scalar_type() == at::kBFloat16, "gemm_pair: bf16 or float8_e4m3fn inputs");
-  TORCH_CHECK(a.stride(1) == 1 && w.stride(1) == 1, "gemm_pair: K must be contiguous");
-  const int M = a.size(0), K = a.size(1), N = w.size(0);
-  TORCH_CHECK(w.size(1) == K, "gemm_pair: K mismatch");
-  c10::cuda::CUDAGuard guard(a.device());
-  const int n_out = swiglu ? N / 2 : N;
-  Tensor c = torch::empty({M, n_out}, a.options().dtype(out_fp32 ? at::kFloat : at::kBFloat16));
-  const void* bias_p = nullptr;
-  const void* res_p = nullptr;
-  if (bias.has_value()) {
-    CHECK_CUDA_BF16(*bias);
-    TORCH_CHECK(bias->numel() == N && bias->is_contiguous(), "gemm_pair: bias [N]");
-    bias_p = bias->data_ptr();
-  }
-  if (residual.has_value()) {
-    CHECK_CUDA_BF16(*residual);
-    TORCH_CHECK(residual->is_contiguous() && residual->size(0) == M && residual->size(1) == n_out,
-                "gemm_pair: residual [M,N] contiguous");
-    res_p = residual->data_ptr();
-  }
-  check(b200_gemm_pair(a.data_ptr(), w.data_ptr(), c.data_ptr(), bias_p, res_p, M, N, K,
-                       (int)a.stride(0), (int)w.stride(0), n_out, fp8 ? 1 : 0, out_fp32 ? 1 : 0,
-                       swiglu ? 1 : 0, (int)bn, status.data_ptr<int>(), (int)max_ctas, cur_stream()),
-        "gemm_pair");
-  return c;
-}
-
-Tensor grouped_gemm(const Tensor& a, const Tensor& w, const Tensor& expert_offsets, bool swiglu,
-                    int64_t bn, const Tensor& status, int64_t max_ctas) {
-  TORCH_CHECK(a.is_cuda() && w.is_cuda() && a.dim() == 2 && w.dim() == 3, "grouped_gemm: shapes");
-  TORCH_CHECK(a.scalar_type() == w.scalar_type(), "grouped_gemm: dtype mismatch");
-  const bool fp8 = a.scalar_type() == at::kFloat8_e4m3fn;
-  TORCH_CHECK(fp8 || a.scalar_type() == at::kBFloat16, "grouped_gemm: bf16 or fp8 inputs");
-  TORCH_CHECK(a.stride(1) == 1 && w.is_contiguous(), "grouped_gemm: contiguity");
-  CHECK_I32(expert_offsets);
-  const int E = w.size(0), N = w.size(1), K = w.size(2), rows = a.size(0);
-  TORCH_CHECK(a.size(1) == K && expert_offsets.numel() == E + 1, "grouped_gemm: size mismatch");
-  c10::cuda::CUDAGuard guard(a.device());
-  const int n_out = swiglu ? N / 2 : N;
-  Tensor c = torch::empty({rows, n_out}, a.options().dtype(at::kBFloat16));
-  check(b200_grouped_gemm(a.data_ptr(), w.data_ptr(), c.data_ptr(), expert_offsets.data_ptr<int>(),
-                          E, rows, N, K, (int)a.stride(0), n_out, fp8 ? 1 : 0, swiglu ? 1 : 0,
-                          (int)bn, status.data_ptr<int>(), (int)max_ctas, cur_stream()),
-        "grouped_gemm");
-  return c;
 }
 
 Tensor rms_norm(const Tensor& x, const Tensor& w, double eps) {
@@ -797,71 +653,13 @@ std::tuple<Tensor, Tensor> mla_decode(const Tensor& q, const Tensor& cache, cons
   return {out, lse};
 }
 
-// Router: gate logits [T,E] fp32 -> (top-k ids int32 [T,k], weights fp32 [T,k]).
-std::tuple<Tensor, Tensor> moe_topk(const Tensor& logits, const c10::optional<Tensor>& bias,
-                                    int64_t k, bool sigmoid, int64_t n_group, int64_t topk_group,
-                                    bool renorm, double scale) {
-  TORCH_CHECK(logits.is_cuda() && logits.scalar_type() == at::kFloat && logits.is_contiguous() &&
-                  logits.dim() == 2,
-              "moe_topk: logits [T,E] fp32 contiguous");
-  const int T = logits.size(0), E = logits.size(1);
-  c10::cuda::CUDAGuard guard(logits.device());
-  Tensor ids = torch::empty({T, k}, logits.options().dtype(at::kInt));
-  Tensor w = torch::empty({T, k}, logits.options());
-  const float* bp = nullptr;
-  if (bias.has_value()) {
-    TORCH_CHECK(bias->scalar_type() == at::kFloat && bias->numel() == E && bias->is_contiguous(),
-                "moe_topk: bias [E] fp32");
-    bp = bias->data_ptr<float>();
-  }
-  check(b200_moe_topk(logits.data_ptr<float>(), bp, ids.data_ptr<int>(), w.data_ptr<float>(), T, E,
-                      (int)k, sigmoid ? 1 : 0, (int)n_group, (int)topk_group, renorm ? 1 : 0,
-                      (float)scale, cur_stream()),
-        "moe_topk");
-  return {ids, w};
-}
-
-Tensor argmax(const Tensor& logits) {
-  TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1, "argmax: [B,V]");
-  const bool f32 = logits.scalar_type() == at::kFloat;
-  TORCH_CHECK(f32 || logits.scalar_type() == at::kBFloat16, "argmax: fp32 or bf16");
-  c10::cuda::CUDAGuard guard(logits.device());
-  Tensor out = torch::empty({logits.size(0)}, logits.options().dtype(at::kInt));
-  check(b200_argmax(logits.data_ptr(), out.data_ptr<int>(), (int)logits.size(0),
-                    (int)logits.size(1), logits.stride(0), f32 ? 1 : 0, cur_stream()),
-        "argmax");
-  return out;
-}
-
-Tensor sample(const Tensor& logits, const c10::optional<Tensor>& temperature,
-              const c10::optional<Tensor>& top_k, const c10::optional<Tensor>& top_p,
-              const c10::optional<Tensor>& seeds, const c10::optional<Tensor>& step_offset) {
-  TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1, "sample: [B,V]");
-  const bool f32 = logits.scalar_type() == at::kFloat;
-  TORCH_CHECK(f32 || logits.scalar_type() == at::kBFloat16, "sample: fp32 or bf16");
-  c10::cuda::CUDAGuard guard(logits.device());
-  Tensor out = torch::empty({logits.size(0)}, logits.options().dtype(at::kInt));
-  check(b200_sample(logits.data_ptr(), out.data_ptr<int>(),
-                    temperature.has_value() ? temperature->data_ptr<float>() : nullptr,
-                    top_k.has_value() ? top_k->data_ptr<int>() : nullptr,
-                    top_p.has_value() ? top_p->data_ptr<float>() : nullptr,
-                    seeds.has_value() ? (const long long*)seeds->data_ptr<int64_t>() : nullptr,
-                    step_offset.has_value() ? (const long long*)step_offset->data_ptr<int64_t>() : nullptr,
-                    (int)logits.size(0), (int)logits.size(1), logits.stride(0), f32 ? 1 : 0,
-                    cur_stream()),
-        "sample");
-  return out;
-}
-
 }  // namespace
 
-TORCH_LIBRARY(omni_b200, m) {
+// The namespace itself is defined by the core library (bindings_core.cpp), which this one links.
+TORCH_LIBRARY_FRAGMENT(omni_b200, m) {
   m.def("spec_verify", &spec_verify);
   m.def("lse_merge", &lse_merge);
   m.def("gather_cache", &gather_cache);
-  m.def("gemm_plan", &gemm_plan);
-  m.def("gemm", &gemm);
-  m.def("gemm_pair", &gemm_pair);
   m.def("gemm_scaled", &gemm_scaled);
   m.def("quant_int8_per_token", &quant_int8_per_token);
   m.def("rms_norm_quant", &rms_norm_quant);
@@ -869,7 +667,6 @@ TORCH_LIBRARY(omni_b200, m) {
   m.def("gemm_fp8_block", &gemm_fp8_block);
   m.def("grouped_gemm_fp8_block", &grouped_gemm_fp8_block);
   m.def("silu_and_mul_quant", &silu_and_mul_quant);
-  m.def("grouped_gemm", &grouped_gemm);
   m.def("rms_norm", &rms_norm);
   m.def("fused_add_rms_norm", &fused_add_rms_norm);
   m.def("silu_and_mul", &silu_and_mul);
@@ -888,7 +685,4 @@ TORCH_LIBRARY(omni_b200, m) {
   m.def("kv_p2p_copy", &kv_p2p_copy);
   m.def("mla_decode_scratch_bytes", &mla_decode_scratch_bytes);
   m.def("mla_decode", &mla_decode);
-  m.def("moe_topk", &moe_topk);
-  m.def("argmax", &argmax);
-  m.def("sample", &sample);
 }

@@ -32,6 +32,7 @@
 #include "../common/tensormap.h"
 #include "../common/device_once.h"
 #include "../comm/ll_protocol.cuh"
+#include "gated_act.cuh"
 
 namespace b200 {
 
@@ -75,7 +76,9 @@ struct GemmParams {
   int acc_stride;         // TMEM column distance between the two accumulators
   int ldc;                // row pitch of C in elements
   int out_fp32;           // 1: C is fp32, 0: bf16
-  int swiglu;             // 1: C[:, n/2] = silu(acc[gate]) * acc[up], gate/up interleaved per 16 cols
+  int swiglu;             // gated activation (gated_act.cuh): C[:, n/2] = act(acc[gate], acc[up]), gate/up interleaved per 16 cols
+  float act_alpha;        // constants of the clamped form
+  float act_limit;
   int num_experts;        // grouped: number of local experts (0 = dense)
   int cluster_split;      // 1: the `splits` CTAs of a cluster share one tile and reduce over DSMEM
   void* C;
@@ -912,8 +915,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            const float g = v[i];
-            o[i] = (g / (1.f + __expf(-g))) * v[8 + i];
+            o[i] = gated_act(p.swiglu, v[i], v[8 + i], p.act_alpha, p.act_limit);
           }
           __nv_bfloat16* dst =
               reinterpret_cast<__nv_bfloat16*>(p.C) + static_cast<size_t>(row) * p.ldc + ocol;
@@ -1387,7 +1389,7 @@ extern "C" void b200_gemm_plan(int M, int N, int K, int elem_bytes, int swiglu, 
 }
 
 // Dense GEMM.  A [M,K] (pitch lda), W [N,K] (pitch ldw), C [M,N or N/2 with
-// swiglu] (pitch ldc).  dtype_fp8 = 0: bf16 inputs; 1: e4m3 inputs (no scale
+// swiglu, the gated activation kind] (pitch ldc).  dtype_fp8 = 0: bf16 inputs; 1: e4m3 inputs (no scale
 // handling here; callers fold scales, see the block-scaled wrapper).
 // workspace / counters may be null when splits == 1 or cluster_split == 1.
 // Returns 0 on success.
@@ -1397,15 +1399,16 @@ static int gemm_impl(const void* A, const void* W, void* C, const void* bias, co
                      int splits, int cluster_split, void* workspace, int* counters, int* status,
                      int max_ctas, cudaStream_t stream, const float* a_scales, const float* w_scales,
                      const ArArgs* ar = nullptr, const struct AgArgs* ag = nullptr,
-                     const struct RsArgs* rs = nullptr);
+                     const struct RsArgs* rs = nullptr, float act_alpha = 0.f, float act_limit = 0.f);
 
 extern "C" int b200_gemm(const void* A, const void* W, void* C, const void* bias,
                          const void* residual, int M, int N, int K, int lda, int ldw, int ldc,
                          int dtype_fp8, int out_fp32, int swiglu, int BN, int splits,
                          int cluster_split, void* workspace, int* counters, int* status,
-                         int max_ctas, cudaStream_t stream) {
+                         int max_ctas, float act_alpha, float act_limit, cudaStream_t stream) {
   return gemm_impl(A, W, C, bias, residual, M, N, K, lda, ldw, ldc, dtype_fp8, out_fp32, swiglu, BN, splits,
-                   cluster_split, workspace, counters, status, max_ctas, stream, nullptr, nullptr);
+                   cluster_split, workspace, counters, status, max_ctas, stream, nullptr, nullptr, nullptr, nullptr,
+                   nullptr, act_alpha, act_limit);
 }
 
 // Quantised product with per-row (a_scales[M]) and per-column (w_scales[N]) scales applied to
@@ -1451,7 +1454,8 @@ static int gemm_impl(const void* A, const void* W, void* C, const void* bias, co
                      int N, int K, int lda, int ldw, int ldc, int dtype_fp8, int out_fp32, int swiglu, int BN,
                      int splits, int cluster_split, void* workspace, int* counters, int* status,
                      int max_ctas, cudaStream_t stream, const float* a_scales, const float* w_scales,
-                     const ArArgs* ar, const struct AgArgs* ag, const struct RsArgs* rs);
+                     const ArArgs* ar, const struct AgArgs* ag, const struct RsArgs* rs, float act_alpha,
+                     float act_limit);
 
 // Row-parallel projection of a tensor-parallel layer in ONE kernel: C = RMSNorm(residual +=
 // sum over ranks of (A @ W^T)) * norm_w  (norm_w null: C = sum (+ residual), residual untouched).
@@ -1544,7 +1548,7 @@ static int gemm_impl(const void* A, const void* W, void* C, const void* bias, co
                      int N, int K, int lda, int ldw, int ldc, int dtype_fp8, int out_fp32, int swiglu, int BN,
                      int splits, int cluster_split, void* workspace, int* counters, int* status,
                      int max_ctas, cudaStream_t stream, const float* a_scales, const float* w_scales,
-                     const ArArgs* ar, const AgArgs* ag, const RsArgs* rs) {
+                     const ArArgs* ar, const AgArgs* ag, const RsArgs* rs, float act_alpha, float act_limit) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const int eb = dtype_fp8 ? 1 : 2;
   if (BN < 16 || BN > 256 || (BN % 16) != 0) return -10;
@@ -1573,6 +1577,8 @@ static int gemm_impl(const void* A, const void* W, void* C, const void* bias, co
   p.ldc = ldc;
   p.out_fp32 = out_fp32;
   p.swiglu = swiglu;
+  p.act_alpha = act_alpha;
+  p.act_limit = act_limit;
   p.num_experts = 0;
   p.C = C;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
@@ -1653,7 +1659,7 @@ static int gemm_impl(const void* A, const void* W, void* C, const void* bias, co
 extern "C" int b200_grouped_gemm(const void* A, const void* W, void* C, const int* expert_offsets,
                                  int num_experts, int total_rows, int N, int K, int lda, int ldc,
                                  int dtype_fp8, int swiglu, int BN, int* status, int max_ctas,
-                                 cudaStream_t stream) {
+                                 float act_alpha, float act_limit, cudaStream_t stream) {
   if (total_rows <= 0 || num_experts <= 0) return 0;
   if (num_experts > kMaxExperts) return -13;
   const int eb = dtype_fp8 ? 1 : 2;
@@ -1678,6 +1684,8 @@ extern "C" int b200_grouped_gemm(const void* A, const void* W, void* C, const in
   p.ldc = ldc;
   p.out_fp32 = 0;
   p.swiglu = swiglu;
+  p.act_alpha = act_alpha;
+  p.act_limit = act_limit;
   p.num_experts = num_experts;
   p.C = C;
   p.expert_offsets = expert_offsets;

@@ -19,6 +19,7 @@
 #include <cstdlib>
 
 #include "../common/ptx.cuh"
+#include "gated_act.cuh"
 #include "../common/tensormap.h"
 #include "../common/device_once.h"
 
@@ -44,7 +45,8 @@ struct PairParams {
   int num_n_blocks;
   int elem_bytes;
   int tmem_cols, acc_stride;
-  int ldc, out_fp32, swiglu;
+  int ldc, out_fp32, swiglu;      // swiglu: gated activation kind (gated_act.cuh)
+  float act_alpha, act_limit;
   // timing diagnostics only (results are wrong), a bit mask: 1 stages are loaded once and then reused,
   // 2 no MMAs are issued, 4 the MMA thread does not wait for full barriers, 8 no empty-barrier
   // hand-back (the producer does not wait for it either), 16 one lane per epilogue warp polls,
@@ -322,8 +324,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            const float g = v[i];
-            o[i] = (g / (1.f + __expf(-g))) * v[8 + i];
+            o[i] = gated_act(p.swiglu, v[i], v[8 + i], p.act_alpha, p.act_limit);
           }
           __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + static_cast<size_t>(row) * p.ldc + ocol;
           uint4 pk;
@@ -465,7 +466,8 @@ extern "C" int b200_gemm_pair_prof(long long* out16) {
 // Same contract as b200_gemm (no split-K).  BN: multiple of 32 in [32, 256].
 extern "C" int b200_gemm_pair(const void* A, const void* W, void* C, const void* bias, const void* residual,
                               int M, int N, int K, int lda, int ldw, int ldc, int dtype_fp8, int out_fp32,
-                              int swiglu, int BN, int* status, int max_ctas, cudaStream_t stream) {
+                              int swiglu, int BN, int* status, int max_ctas, float act_alpha, float act_limit,
+                              cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const int eb = dtype_fp8 ? 1 : 2;
   if (BN < 32 || BN > 256 || (BN % 32) != 0) return -10;
@@ -492,6 +494,8 @@ extern "C" int b200_gemm_pair(const void* A, const void* W, void* C, const void*
   p.ldc = ldc;
   p.out_fp32 = out_fp32;
   p.swiglu = swiglu;
+  p.act_alpha = act_alpha;
+  p.act_limit = act_limit;
   p.C = C;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.residual = static_cast<const __nv_bfloat16*>(residual);

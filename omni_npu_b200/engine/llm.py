@@ -24,7 +24,8 @@ from .scheduler import Scheduler, SchedulerOutput
 
 class LLMEngine:
     def __init__(self, config: EngineConfig, local_rank: Optional[int] = None,
-                 rank: Optional[int] = None) -> None:
+                 rank: Optional[int] = None, before_capture=None) -> None:
+        """``before_capture``: called with the model runner before decode steps are captured."""
         import os
         self.config = config
         local_rank = int(os.environ.get("LOCAL_RANK", "0")) if local_rank is None else local_rank
@@ -35,6 +36,8 @@ class LLMEngine:
         self.worker.load_model()
         num_blocks = self.worker.determine_num_blocks()
         self.worker.initialize_from_config(num_blocks)
+        if before_capture is not None:
+            before_capture(self.worker.model_runner)
         self.worker.compile_or_warm_up_model()
         connector = None
         if config.kv_transfer is not None and config.kv_transfer.kv_connector:

@@ -233,6 +233,46 @@ class Scheduler:
         if req not in self.waiting:
             self.waiting.appendleft(req)
 
+    # ------------------------------------------------- steps put together by the caller
+    def schedule_portions(self, portions) -> SchedulerOutput:
+        """A step whose portions are given: ``portions`` = [(request, number of its next tokens)], the
+        tokens being known already (part of the request).  A request that is not running yet is
+        admitted, blocks are allocated as for any other step, decoding requests (one token, earlier
+        ones cached) come first in the batch.  Running out of sequence slots or blocks is an error:
+        nothing is evicted on the caller's behalf.  Returns the step; ``commit_portions`` books it."""
+        self._step += 1
+        out = SchedulerOutput(step_index=self._step)
+        decode: List[ScheduledSeq] = []
+        prompt: List[ScheduledSeq] = []
+        for req, n in portions:
+            if req not in self.running:
+                if len(self.running) >= self.cfg.max_num_seqs:
+                    raise RuntimeError(f"more than {self.cfg.max_num_seqs} live requests")
+                self.requests[req.request_id] = req
+                req.status = RequestStatus.RUNNING
+                self.running.append(req)
+            start = req.num_computed_tokens
+            if n < 1 or start + n > req.num_tokens:
+                raise ValueError(f"request {req.request_id}: {n} tokens from {start} of {req.num_tokens}")
+            if start + n > self.cfg.max_model_len:
+                raise ValueError(f"request {req.request_id} exceeds max_model_len {self.cfg.max_model_len}")
+            if not self._ensure_blocks(req, start + n):
+                raise RuntimeError("out of KV blocks")
+            seq = ScheduledSeq(req, start, n, start + n == req.num_tokens)
+            (decode if n == 1 and start > 0 else prompt).append(seq)
+        out.kind = "prefill" if prompt else "decode" if decode else "idle"
+        out.seqs = decode + prompt
+        out.num_decode_seqs = len(decode) if prompt else 0
+        out.num_tokens = sum(s.num_new_tokens for s in out.seqs)
+        if out.num_tokens > self.cfg.max_num_batched_tokens:
+            raise ValueError(f"{out.num_tokens} tokens in one step, at most {self.cfg.max_num_batched_tokens}")
+        out.finished_req_ids, self._finished_since_last = self._finished_since_last, []
+        return out
+
+    def commit_portions(self, out: SchedulerOutput) -> None:
+        for s in out.seqs:
+            s.request.num_computed_tokens = s.start + s.num_new_tokens
+
     # -------------------------------------------------------------- schedule
     def schedule(self) -> SchedulerOutput:
         self._step += 1

@@ -68,7 +68,8 @@ def gathered_gemm(layer: "LinearBase", x: torch.Tensor, swiglu: bool = False,
     projection of a sequence-sharded residual stream); None when the fused path does not apply."""
     symm = getattr(layer.group.comm, "symm", None)
     if (symm is None or not isinstance(layer.quant_method, UnquantizedLinearMethod) or x.dim() != 2
-            or out_dtype not in (None, torch.bfloat16) or not symm.can_all_gather_gemm(x, layer.weight)):
+            or out_dtype not in (None, torch.bfloat16) or getattr(layer, "gated_act", ops.SILU) != ops.SILU
+            or not symm.can_all_gather_gemm(x, layer.weight)):
         return None
     return symm.all_gather_gemm(x, layer.weight, layer.bias, swiglu)
 
@@ -86,7 +87,8 @@ class UnquantizedLinearMethod:
     def apply(self, layer: "LinearBase", x: torch.Tensor, bias: Optional[torch.Tensor],
               residual: Optional[torch.Tensor] = None, swiglu: bool = False,
               out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-        return ops.gemm(x, layer.weight, bias, residual, out_dtype, swiglu)
+        return ops.gemm(x, layer.weight, bias, residual, out_dtype, swiglu,
+                        act=getattr(layer, "gated_act", ops.SILU))
 
 
 class Fp8BlockLinearMethod:
@@ -198,7 +200,10 @@ class MergedColumnParallelLinear(LinearBase):
     """Several column-parallel projections sharing one input, stored as one
     weight so that one GEMM computes all of them (gate+up, q_a+kv_a, ...).
     With ``swiglu_interleave`` the two halves (gate, up) are stored interleaved
-    in groups of 8 rows so the GEMM epilogue can apply silu(gate)*up."""
+    in groups of 8 rows so the GEMM epilogue can apply silu(gate)*up (or the
+    gated activation set as ``gated_act``)."""
+
+    gated_act = ops.SILU
 
     def __init__(self, in_features, output_sizes: Sequence[int], bias=False, dtype=torch.bfloat16,
                  device=None, swiglu_interleave: bool = False, **kw):
@@ -312,6 +317,32 @@ class QKVParallelLinear(LinearBase):
         src = loaded.narrow(0, r * n, n)
         dst = param.data.narrow(0, off, n)
         dst.copy_(src if dst.dtype == torch.float8_e4m3fn else src.to(dst.dtype))
+
+
+class GatedQKVParallelLinear(QKVParallelLinear):
+    """q/k/v projection with an output gate of the value heads' width as a fourth part, all in one GEMM.
+    The gate is sharded like the query heads.  The output width is rounded up to whole 16-byte rows;
+    the extra rows of the weight are zero."""
+
+    def __init__(self, *args, output_gate: bool = True, **kw):
+        self.output_gate = output_gate
+        super().__init__(*args, **kw)
+
+    def _create(self, in_local: int, out_local: int, device) -> None:
+        self.gate_size = self.num_heads * self.head_dim_v if self.output_gate else 0
+        self.used_rows = out_local + self.gate_size
+        super()._create(in_local, (self.used_rows + 7) // 8 * 8, device)
+
+    def forward(self, x: torch.Tensor):
+        y = self.quant_method.apply(self, apply_transform(x, self.x_transform, self.group), self.bias)
+        q, k, v, g = y[:, : self.used_rows].split([self.q_size, self.k_size, self.v_size, self.gate_size], dim=1)
+        return q, k, v, (g if self.output_gate else None)
+
+    def weight_loader(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        if shard_id != "g":
+            return super().weight_loader(param, loaded, shard_id)
+        dst = param.data[self.used_rows - self.gate_size: self.used_rows]
+        dst.copy_(loaded.narrow(0, self.tp_rank * self.gate_size, self.gate_size).to(dst.dtype))
 
 
 class RowParallelLinear(LinearBase):

@@ -19,7 +19,7 @@ from .linear import MergedColumnParallelLinear, RowParallelLinear, row_parallel_
 class FusedMLP(nn.Module):
     def __init__(self, hidden_size: int, intermediate_size: int, dtype=torch.bfloat16, device=None,
                  quant_method_factory=None, prefix: str = "", group=None,
-                 reduce_results: bool = True, fuse_swiglu: bool = True) -> None:
+                 reduce_results: bool = True, fuse_swiglu: bool = True, act=None) -> None:
         super().__init__()
         qm = quant_method_factory or (lambda: None)
         self.fuse_swiglu = fuse_swiglu
@@ -27,6 +27,8 @@ class FusedMLP(nn.Module):
             hidden_size, [intermediate_size, intermediate_size], dtype=dtype, device=device,
             swiglu_interleave=fuse_swiglu, quant_method=qm(), prefix=f"{prefix}.gate_up_proj",
             group=group)
+        if act is not None:
+            self.gate_up_proj.gated_act = act        # applied in the GEMM epilogue (needs fuse_swiglu)
         self.down_proj = RowParallelLinear(intermediate_size, hidden_size, dtype=dtype, device=device,
                                            quant_method=qm(), prefix=f"{prefix}.down_proj",
                                            group=group, reduce_results=reduce_results)

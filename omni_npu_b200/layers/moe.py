@@ -45,6 +45,17 @@ def select_experts(router_logits: torch.Tensor, top_k: int, scoring_func: str = 
     return w, ids
 
 
+class RoutedRows:
+    """Expert outputs that still lie in expert order, for a consumer that brings them back to their
+    tokens itself: token t's share is sum_j weights[t, j] * y[slots[t * k + j]]."""
+
+    def __init__(self, y: torch.Tensor, slots: torch.Tensor, weights: torch.Tensor) -> None:
+        self.y, self.slots, self.weights = y, slots, weights
+
+    def __iter__(self):
+        return iter((self.y, self.slots, self.weights))
+
+
 class FusedMoE(nn.Module):
     def __init__(self, num_experts: int, top_k: int, hidden_size: int, intermediate_size: int,
                  dtype=torch.bfloat16, device=None, scoring_func: str = "softmax",
@@ -52,7 +63,8 @@ class FusedMoE(nn.Module):
                  topk_group: int = 1, router_bias: bool = False, num_shared_experts: int = 0,
                  shared_intermediate_size: Optional[int] = None, enable_expert_parallel: bool = True,
                  prefix: str = "", max_tokens: int = 8192, quant: Optional[str] = None,
-                 num_redundant_experts: int = 0, shared_quant_factory=None) -> None:
+                 num_redundant_experts: int = 0, shared_quant_factory=None,
+                 act: Tuple[float, float] = ops.SILU, shared_act: Optional[Tuple[float, float]] = None) -> None:
         super().__init__()
         self.num_experts, self.top_k = num_experts, top_k
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
@@ -61,6 +73,7 @@ class FusedMoE(nn.Module):
         self.n_group, self.topk_group = n_group, topk_group
         self.max_tokens = max_tokens
         self.dtype = dtype
+        self.act = act               # gated activation of the routed experts (ops.gemm); shared_act: of the shared one
         self.tp_group = pstate.get_tp_group()
         self.ep_group = pstate.get_ep_group() if enable_expert_parallel else None
         self.ep_size = self.ep_group.world_size if self.ep_group is not None else 1
@@ -102,7 +115,8 @@ class FusedMoE(nn.Module):
             self.shared_experts = FusedMLP(hidden_size, inter, dtype, device, prefix=f"{prefix}.shared_experts",
                                            quant_method_factory=shared_quant_factory,
                                            group=_solo_group() if self.ep_size > 1 else None,
-                                           reduce_results=False, fuse_swiglu=shared_quant_factory is None)
+                                           reduce_results=False, fuse_swiglu=shared_quant_factory is None,
+                                           act=shared_act)
         self.buffers: Optional[EpBuffers] = None
         self._side_stream: Optional[torch.cuda.Stream] = None
         self.expert_load: Optional[torch.Tensor] = None   # per-expert token counts (EPLB statistics)
@@ -114,12 +128,14 @@ class FusedMoE(nn.Module):
         if dev.type != "cuda" or self.buffers is not None:
             return
         fp8 = self.quant == "fp8" and self.hidden_size % 128 == 0
-        key = (id(self.ep_group), self.num_physical, self.hidden_size, self.top_k, fp8)
+        key = (id(self.ep_group), self.num_physical, self.hidden_size, self.top_k, fp8, self.max_tokens, self.dtype,
+               dev)
         shared = _SHARED_BUFFERS.get(key)
         if shared is None:
             group = self.ep_group if self.ep_group is not None else _solo_group()
             shared = EpBuffers(group, dev, self.num_physical if self.ep_size > 1 else self.local_experts,
-                               self.hidden_size, self.max_tokens, self.top_k, fp8_dispatch=fp8)
+                               self.hidden_size, self.max_tokens, self.top_k, fp8_dispatch=fp8,
+                               dtype=self.dtype)
             _SHARED_BUFFERS[key] = shared
         self.buffers = shared
         self._side_stream = torch.cuda.Stream(dev)
@@ -235,6 +251,29 @@ class FusedMoE(nn.Module):
             pass  # experts replicated: nothing to reduce
         return out
 
+    def forward_deferred(self, hidden: torch.Tensor):
+        """The layer with its last step left to the caller: (routed, dense) with ``routed`` the experts'
+        rows (:class:`RoutedRows`) or None, ``dense`` [T,H] the rest (shared expert) or None; the layer's
+        result is their sum.  With expert parallelism (and on the CPU) everything is in ``dense``."""
+        if not hidden.is_cuda or self.ep_size > 1 or self.quant == "fp8" or self.eplb is not None:
+            return None, self.forward(hidden)
+        w, ids = select_experts(self.gate(hidden, out_dtype=torch.float32), self.top_k, self.scoring_func,
+                                self.e_score_correction_bias, self.n_group, self.topk_group, self.renormalize,
+                                self.routed_scaling_factor)
+        if self.buffers is None:
+            self.init_ep_buffers()
+        cur = torch.cuda.current_stream(hidden.device)
+        shared_out = None
+        if self.shared_experts is not None:
+            self._side_stream.wait_stream(cur)
+            with torch.cuda.stream(self._side_stream):
+                shared_out = self.shared_experts(hidden)
+        rows, offsets, handle = ep_dispatch(None, hidden, ids, w, self.num_physical, self.buffers)
+        y = ops.grouped_gemm(ops.grouped_gemm(rows, self.w13, offsets, swiglu=True, act=self.act), self.w2, offsets)
+        if shared_out is not None:
+            cur.wait_stream(self._side_stream)
+        return RoutedRows(y, handle.slots, w), shared_out
+
     def _routed(self, x: torch.Tensor, w: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
         comm = self.ep_group.comm if self.ep_size > 1 else _Solo.comm
         shared_out = None
@@ -261,7 +300,7 @@ class FusedMoE(nn.Module):
                 hq, hs = ops.quant_fp8_1x128(h1)
                 y = ops.grouped_gemm_fp8_block(hq, hs, self.w2, self.w2_scale, offsets)
             else:
-                h1 = ops.grouped_gemm(rows, self.w13, offsets, swiglu=True)
+                h1 = ops.grouped_gemm(rows, self.w13, offsets, swiglu=True, act=self.act)
                 y = ops.grouped_gemm(h1, self.w2, offsets)
             self.buffers.expert_y[: y.shape[0]].copy_(y)
             if shared_out is not None:
@@ -271,7 +310,7 @@ class FusedMoE(nn.Module):
         if self.shared_experts is not None:
             shared_out = self.shared_experts(x)
         rows, offsets, handle = ep_dispatch(comm, x, ids, w, self.num_physical)
-        h1 = ops.grouped_gemm(rows, self.w13, offsets, swiglu=True)
+        h1 = ops.grouped_gemm(rows, self.w13, offsets, swiglu=True, act=self.act)
         y = ops.grouped_gemm(h1, self.w2, offsets)
         return ep_combine(comm, y, handle, shared_out)
 

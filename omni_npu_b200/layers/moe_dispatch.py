@@ -16,7 +16,6 @@ from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from pathlib import Path
 from typing import Optional
 
 import torch
@@ -34,8 +33,8 @@ class _EpHostArgs(ctypes.Structure):
 def _lib():
     global _LIB
     if _LIB is None:
-        ops.load_extension(required=True)
-        lib = ctypes.CDLL(str(Path(__file__).resolve().parent.parent / "_C.so"))
+        ops.load_extension(required=True, core_only=True)
+        lib = ctypes.CDLL(str(ops.CORE_LIB))
         vp, ci, ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
         lib.b200_ep_flag_words.restype = ci
         lib.b200_ep_dispatch.argtypes = [ctypes.POINTER(_EpHostArgs), ci, ci, ci, ci, vp, vp, ci, ci, ci, ll,
@@ -65,8 +64,8 @@ class DispatchHandle:
 
 class EpBuffers:
     def __init__(self, group, device: torch.device, num_experts: int, hidden: int, max_tokens: int,
-                 top_k: int, capacity_factor: float = 2.0, fp8_dispatch: bool = False) -> None:
-        from ..parallel.symm_mem import _lib as symm_lib
+                 top_k: int, capacity_factor: float = 2.0, fp8_dispatch: bool = False,
+                 dtype: torch.dtype = torch.bfloat16) -> None:
         self.group, self.device = group, device
         self.world, self.rank = group.world_size, group.rank_in_group
         self.num_experts, self.hidden, self.top_k = num_experts, hidden, top_k
@@ -75,11 +74,18 @@ class EpBuffers:
         factor = 1.0 if self.world == 1 else capacity_factor
         self.cap_rows = int(max(256, factor * max_tokens * top_k))
         self.max_tokens = max_tokens
-        lib = symm_lib()
         self._own, self._opened = [], []
-        self._symm_lib = lib
+        self.dtype = dtype
+        lib = self._symm_lib = None
+        if self.world > 1:                   # alone, nobody maps these buffers: ordinary tensors do
+            from ..parallel.symm_mem import _lib as symm_lib
+            lib = self._symm_lib = symm_lib()
 
         def alloc(nbytes):
+            if lib is None:
+                buf = torch.zeros(max(nbytes, 256), dtype=torch.uint8, device=device)
+                self._own.append(buf)
+                return ctypes.c_void_p(buf.data_ptr()), b""
             ptr = ctypes.c_void_p()
             handle = ctypes.create_string_buffer(64)
             rc = lib.b200_symm_alloc(max(nbytes, 2 << 20), ctypes.byref(ptr), handle)
@@ -88,7 +94,8 @@ class EpBuffers:
             self._own.append(ptr)
             return ptr, handle.raw
 
-        row_bytes = hidden * 2
+        row_bytes = hidden * dtype.itemsize
+        self.row_halves = row_bytes // 2     # what the row-moving kernels count in
         mine = [alloc(self.cap_rows * row_bytes), alloc(self.cap_rows * row_bytes),
                 alloc(self.world * num_experts * 4), alloc(_lib().b200_ep_flag_words() * 4)]
         # fp8 dispatch: rows arrive quantised (e4m3 + one fp32 scale per 128 columns) in two more
@@ -113,8 +120,8 @@ class EpBuffers:
                     table[r] = p.value
                     self._opened.append(p)
         # torch views of my own buffers (the grouped GEMMs read / write them in place)
-        self.recv_x = _as_tensor(mine[0][0].value, (self.cap_rows, hidden), torch.bfloat16, device)
-        self.expert_y = _as_tensor(mine[1][0].value, (self.cap_rows, hidden), torch.bfloat16, device)
+        self.recv_x = _as_tensor(mine[0][0].value, (self.cap_rows, hidden), dtype, device)
+        self.expert_y = _as_tensor(mine[1][0].value, (self.cap_rows, hidden), dtype, device)
         if self.fp8_dispatch:
             self.recv_q = _as_tensor(mine[4][0].value, (self.cap_rows, hidden), torch.uint8, device).view(torch.float8_e4m3fn)
             self.recv_s = _as_tensor(mine[5][0].value, (self.cap_rows, hidden // 128), torch.float32, device)
@@ -136,7 +143,8 @@ class EpBuffers:
         for p in self._opened:
             self._symm_lib.b200_symm_close(p)
         for p in self._own:
-            self._symm_lib.b200_symm_free(p)
+            if self._symm_lib is not None:
+                self._symm_lib.b200_symm_free(p)
         self._opened, self._own = [], []
 
 
@@ -178,10 +186,13 @@ def ep_dispatch(comm, hidden: torch.Tensor, topk_ids: torch.Tensor, topk_weights
         raise RuntimeError("expert-parallel buffers not initialised for this communicator")
     if t > buf.max_tokens:
         raise RuntimeError(f"{t} tokens exceed the dispatch capacity of {buf.max_tokens}")
+    if hidden.dtype != buf.dtype or hidden.shape[1] != buf.hidden:
+        raise RuntimeError(f"dispatch buffers hold {buf.hidden} x {buf.dtype} rows, got {tuple(hidden.shape)} {hidden.dtype}")
     stream = torch.cuda.current_stream(hidden.device).cuda_stream
+    halves = hidden.dtype.itemsize // 2
     common = (ctypes.byref(buf.args), buf.world, buf.rank, buf.num_experts,
               buf.cap_rows, hidden.data_ptr(), topk_ids.data_ptr(), t, k,
-              hidden.shape[1], hidden.stride(0), buf.expert_offsets.data_ptr(),
+              buf.row_halves, hidden.stride(0) * halves, buf.expert_offsets.data_ptr(),
               buf.send_base.data_ptr(), buf.cursors.data_ptr(), buf.slots.data_ptr(),
               buf.total_recv.data_ptr(), buf.status.data_ptr())
     if fp8:
@@ -210,6 +221,8 @@ def ep_combine(comm, expert_out: torch.Tensor, handle: DispatchHandle,
     buf = buffers or comm.ep_buffers
     t, k = handle.topk_ids.shape
     h = buf.hidden
+    if buf.dtype != torch.bfloat16:
+        raise RuntimeError("the combine kernel reduces bf16 rows (32-bit models combine in the residual kernel)")
     if expert_out.data_ptr() != buf.expert_y.data_ptr():
         buf.expert_y[: expert_out.shape[0]].copy_(expert_out)
     out = torch.empty((t, h), dtype=torch.bfloat16, device=buf.device) if out is None else out

@@ -54,7 +54,7 @@ class RotaryEmbedding(nn.Module):
     def __init__(self, head_dim: int, rot_dim: int, max_position: int, base: float,
                  is_neox: bool = True, inv_freq: Optional[torch.Tensor] = None, mscale: float = 1.0,
                  mrope_section: Optional[Tuple[int, int, int]] = None,
-                 mrope_interleaved: bool = False, device=None) -> None:
+                 mrope_interleaved: bool = False, device=None, exact_angles: bool = False) -> None:
         super().__init__()
         self.head_dim, self.rot_dim = head_dim, rot_dim
         self.max_position, self.base = max_position, base
@@ -63,7 +63,13 @@ class RotaryEmbedding(nn.Module):
         self.mrope_section = mrope_section
         self.mrope_interleaved = mrope_interleaved
         inv = inv_freq if inv_freq is not None else _base_inv_freq(rot_dim, base)
-        cache = ref.build_cos_sin_cache(rot_dim, max_position, base, inv, mscale)
+        if exact_angles:
+            # products p * f in double precision, so that the rounding of an angle does not grow with p
+            inv64 = float(base) ** (-torch.arange(0, rot_dim, 2, dtype=torch.float64) / max(rot_dim, 1))
+            a = torch.outer(torch.arange(max_position, dtype=torch.float64), inv64)
+            cache = torch.cat([a.cos() * mscale, a.sin() * mscale], dim=-1).float()
+        else:
+            cache = ref.build_cos_sin_cache(rot_dim, max_position, base, inv, mscale)
         self.register_buffer("cos_sin_cache", cache.to(device) if device is not None else cache,
                              persistent=False)
 
@@ -200,11 +206,11 @@ _ROPE_CACHE: Dict[Any, RotaryEmbedding] = {}
 
 def get_rope(head_dim: int, rot_dim: int, max_position: int, base: float, is_neox: bool = True,
              rope_scaling: Optional[Dict[str, Any]] = None, device=None,
-             dual_chunk_attention_config: Optional[Dict[str, Any]] = None) -> nn.Module:
+             dual_chunk_attention_config: Optional[Dict[str, Any]] = None, exact_angles: bool = False) -> nn.Module:
     dca = {k: v for k, v in (dual_chunk_attention_config or {}).items() if k in ("chunk_size", "local_size")}
     key = (head_dim, rot_dim, max_position, base, is_neox,
            tuple(sorted((k, str(v)) for k, v in (rope_scaling or {}).items())), str(device),
-           tuple(sorted(dca.items())))
+           tuple(sorted(dca.items())), exact_angles)
     hit = _ROPE_CACHE.get(key)
     if hit is not None:
         return hit
@@ -268,6 +274,6 @@ def get_rope(head_dim: int, rot_dim: int, max_position: int, base: float, is_neo
     else:
         rope = RotaryEmbedding(head_dim, rot_dim, max_pos, base, is_neox, inv, mscale,
                                tuple(mrope) if mrope else None,
-                               bool(rs.get("mrope_interleaved", False)), device)
+                               bool(rs.get("mrope_interleaved", False)), device, exact_angles)
     _ROPE_CACHE[key] = rope
     return rope

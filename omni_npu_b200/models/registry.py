@@ -24,8 +24,34 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "PanguProMoEV2ForCausalLM": ("omni_npu_b200.models.pangu", "PanguProMoEV2ForCausalLM"),
     "Qwen3VLForConditionalGeneration": ("omni_npu_b200.models.qwen3_vl", "Qwen3VLForConditionalGeneration"),
     "OpenPanguVLForConditionalGeneration": ("omni_npu_b200.models.openpangu_vl", "OpenPanguVLForConditionalGeneration"),
+    "Rivudra": ("omni_npu_b200.models.rivudra", "RivudraForCausalLM"),
     "MockModel": ("omni_npu_b200.models.mock", "MockModelForCausalLM"),
 }
+
+
+# designs whose config.json has keys of its own: name under "architecture" -> reader returning a ModelConfig
+_CONFIG_READERS: Dict[str, Tuple[str, str]] = {
+    "Rivudra": ("omni_npu_b200.models.rivudra", "read_config"),
+}
+
+
+# architectures whose kernels are all in the core library (_build.CORE_SOURCES)
+_CORE_LIBRARY_ONLY = {"Rivudra"}
+
+
+def runs_on_core_library(arch: str) -> bool:
+    return arch in _CORE_LIBRARY_ONLY
+
+
+def register_config_reader(arch: str, module: str, function: str) -> None:
+    _CONFIG_READERS[arch] = (module, function)
+
+
+def resolve_config_reader(arch: str):
+    if arch not in _CONFIG_READERS:
+        raise ValueError(f"no config reader for architecture {arch!r}; known: {sorted(_CONFIG_READERS)}")
+    module, name = _CONFIG_READERS[arch]
+    return getattr(importlib.import_module(module), name)
 
 
 def register_model(arch: str, module: str, cls_name: str) -> None:

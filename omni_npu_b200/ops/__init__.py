@@ -1,7 +1,7 @@
 """Device ops of the framework.
 
 Every function takes torch tensors.  CUDA tensors run the hand-written sm_100a
-kernels from ``_C.so`` (``torch.ops.omni_b200.*``); a missing extension on a
+kernels from ``_C_core.so`` / ``_C.so`` (``torch.ops.omni_b200.*``); a missing extension on a
 CUDA tensor is an error, never a silent fallback.  CPU tensors run the fp32
 PyTorch references in :mod:`omni_npu_b200.ops.ref`, which is what the gloo /
 no-GPU plumbing tests exercise.
@@ -22,34 +22,49 @@ from . import ref
 
 _PKG = Path(__file__).resolve().parent.parent
 _LIB = _PKG / "_C.so"
+CORE_LIB = _PKG / "_C_core.so"
 _loaded = False
+_core_loaded = False
 _load_error: Optional[str] = None
 _lock = threading.Lock()
 
 
-def load_extension(required: bool = False) -> bool:
-    """Load ``_C.so`` (idempotent).  Returns whether the ops are available."""
-    global _loaded, _load_error
-    if _loaded:
+def load_extension(required: bool = False, core_only: bool = False) -> bool:
+    """Load the kernel libraries (idempotent): ``_C.so``, which brings ``_C_core.so`` with it, or the
+    core library alone.  Returns whether the ops are available."""
+    global _loaded, _core_loaded, _load_error
+    if _loaded or (core_only and _core_loaded):
         return True
     with _lock:
-        if _loaded:
-            return True
-        if not _LIB.exists():
-            _load_error = f"{_LIB} not built (run `python -m omni_npu_b200._build`)"
+        lib = CORE_LIB if core_only else _LIB
+        if not lib.exists():
+            _load_error = f"{lib} not built (run `python -m omni_npu_b200._build`)"
         else:
             try:
-                torch.ops.load_library(str(_LIB))
-                _loaded = True
+                torch.ops.load_library(str(lib))
+                _core_loaded = True
+                _loaded = _loaded or not core_only
             except Exception as e:  # pragma: no cover - depends on the box
-                _load_error = f"loading {_LIB} failed: {e}"
-    if required and not _loaded:
+                _load_error = f"loading {lib} failed: {e}"
+    ok = _loaded or (core_only and _core_loaded)
+    if required and not ok:
         raise RuntimeError("omni_npu_b200 CUDA extension unavailable: " + str(_load_error))
-    return _loaded
+    return ok
+
+
+def full_library_built() -> bool:
+    return _LIB.exists()
 
 
 def _C():
     load_extension(required=True)
+    return torch.ops.omni_b200
+
+
+def _core():
+    """The ops of the core library (present too when the full one is loaded)."""
+    if not _core_loaded:
+        load_extension(required=True, core_only=True)
     return torch.ops.omni_b200
 
 
@@ -168,6 +183,7 @@ def check_status(device: Optional[torch.device] = None) -> None:
 
 
 # ------------------------------------------------------------------------ GEMM
+SILU = (0.0, 0.0)          # gated activation silu(gate) * up: no slope, no limit
 # smallest M routed to the CTA-pair GEMM (0 = never); prefill-sized problems only
 PAIR_MIN_M = int(os.environ.get("OMNI_B200_GEMM_PAIR_MIN_M", "1024"))
 # Plain bf16 products (no bias, residual, SwiGLU, scales or fused collective) of a decode-sized batch
@@ -192,17 +208,25 @@ def library_small_m(m: int, cluster_split_plan: bool, plain_bf16: bool) -> bool:
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
          swiglu: bool = False, bn: int = 0, splits: int = 0, max_ctas: int = 0,
-         pair: Optional[bool] = None) -> torch.Tensor:
+         pair: Optional[bool] = None, act: Tuple[float, float] = SILU) -> torch.Tensor:
     """``a[M,K] @ w[N,K].T`` (+bias, +residual).  bf16 or float8_e4m3fn inputs,
     fp32 accumulation, bf16 (default) or fp32 output.  ``swiglu`` fuses
-    silu(gate)*up for weights laid out by :func:`ref.interleave_gate_up`.
+    silu(gate)*up for weights laid out by :func:`ref.interleave_gate_up`; ``act`` = (slope, limit)
+    with a non-zero slope selects the clamped form of it (:func:`ref.gated_act`).  fp32 inputs run on
+    the CUDA cores, with no reduced-precision mode.
     ``splits`` > 1 forces split-K (as a thread-block cluster when it fits), a
     negative value forces the workspace variant with |splits| slices.
     ``pair`` selects the CTA-pair kernel (256-row tiles over two SMs); by default
     it runs for M >= PAIR_MIN_M when no split-K was asked for."""
     if not a.is_cuda:
-        return ref.gemm(a, w, bias, residual, out_dtype, swiglu)
-    C = _C()
+        return ref.gemm(a, w, bias, residual, out_dtype, swiglu, act)
+    C = _core()
+    if a.dtype == torch.float32:
+        _count(1)
+        y = C.gemm_simt(a, w, None, swiglu, act[0], act[1])
+        if bias is not None:
+            y = y + bias
+        return y if residual is None else y + residual
     st = device_state(a.device)
     m, k = a.shape
     n = w.shape[0]
@@ -212,7 +236,8 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         n_eff = n
         pbn = bn if bn > 0 else (256 if n_eff >= 256 else max(32, ((n_eff + 31) // 32) * 32))
         _count(1)
-        return C.gemm_pair(a, w, bias, residual, out_dtype == torch.float32, swiglu, pbn, st.status, max_ctas)
+        return C.gemm_pair(a, w, bias, residual, out_dtype == torch.float32, swiglu, pbn, st.status, max_ctas,
+                           act[0], act[1])
     key = (m, n, k, a.dtype.itemsize, swiglu, bn, splits)
     plan = st.plans.get(key)
     if plan is None:
@@ -227,7 +252,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         ws, cnt = st.gemm_workspace(torch.cuda.current_stream(a.device).cuda_stream, ws_bytes, ncnt)
     _count(1)
     return C.gemm(a, w, bias, residual, out_dtype == torch.float32, swiglu, pbn, psplits,
-                  bool(cluster), ws, cnt, st.status, max_ctas)
+                  bool(cluster), ws, cnt, st.status, max_ctas, act[0], act[1])
 
 
 def quant_int8_per_token(x: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -331,16 +356,21 @@ def gemm_scaled(a_q: torch.Tensor, w_q: torch.Tensor, a_scale: torch.Tensor, w_s
 
 
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
-                 swiglu: bool = False, bn: int = 0, max_ctas: int = 0) -> torch.Tensor:
-    """Per-expert GEMM: rows expert_offsets[e]:expert_offsets[e+1] of ``a`` times ``w[e].T``."""
+                 swiglu: bool = False, bn: int = 0, max_ctas: int = 0,
+                 act: Tuple[float, float] = SILU) -> torch.Tensor:
+    """Per-expert GEMM: rows expert_offsets[e]:expert_offsets[e+1] of ``a`` times ``w[e].T``
+    (``swiglu`` / ``act`` as in :func:`gemm`)."""
     if not a.is_cuda:
-        return ref.grouped_gemm(a, w, expert_offsets, swiglu)
+        return ref.grouped_gemm(a, w, expert_offsets, swiglu, act)
+    if a.dtype == torch.float32:
+        _count(1)
+        return _core().gemm_simt(a, w, expert_offsets, swiglu, act[0], act[1])
     if bn <= 0:
         n = w.shape[1]
         bn = 256 if n % 256 == 0 else (128 if n % 128 == 0 else (64 if n % 64 == 0 else 32))
     st = device_state(a.device)
     _count(1)
-    return _C().grouped_gemm(a, w, expert_offsets, swiglu, bn, st.status, max_ctas)
+    return _core().grouped_gemm(a, w, expert_offsets, swiglu, bn, st.status, max_ctas, act[0], act[1])
 
 
 # ------------------------------------------------------------- norm/activation
@@ -613,12 +643,91 @@ def gqa_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                         st.work_counter(stream_id) if persistent else None)
 
 
+# ------------------------------- attention with a window, a sink without a value and an output gate
+def gated_head_pad(dim: int, dtype: torch.dtype) -> int:
+    """Width of a cache row for a head size: whole 16-element steps of the bf16 products (the rest of
+    the row holds zeros)."""
+    return dim if dtype == torch.float32 else (dim + 15) // 16 * 16
+
+
+def gated_rope_cache_(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor,
+                      v_cache: torch.Tensor, positions: torch.Tensor, slot_mapping: torch.Tensor,
+                      cos_sin: torch.Tensor, head_dim: int, head_dim_v: int, rot_dim: int, neox: bool) -> None:
+    """RoPE on the first ``rot_dim`` dimensions of q (in place) and k; k / v stored into the paged cache,
+    whose rows may be wider than the heads."""
+    if not q.is_cuda:
+        return ref.gated_rope_cache_(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim,
+                                     head_dim_v, rot_dim, neox)
+    _count(1)
+    _core().gated_rope_cache(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim, head_dim_v,
+                             rot_dim, neox)
+
+
+def gated_decode_splits(num_seqs: int, num_kv_heads: int, keys: int, sms: int = 148) -> int:
+    """CTAs (of one cluster) that share the visible keys of a (sequence, key/value head): enough to
+    give every SM two, at least 128 keys each."""
+    base = max(1, num_seqs * num_kv_heads)
+    splits = 1
+    while splits < 8 and base * splits < 2 * sms and keys >= 256 * splits:
+        splits *= 2
+    return splits
+
+
+def gated_attention(q: torch.Tensor, gate: Optional[torch.Tensor], k_cache: torch.Tensor, v_cache: torch.Tensor,
+                    out: torch.Tensor, block_tables: torch.Tensor, cu_q: Optional[torch.Tensor],
+                    seq_lens: torch.Tensor, num_seqs: int, max_q_len: int, num_q_heads: int, head_dim: int,
+                    head_dim_v: int, scale: float, window: int = 0, sink: Optional[float] = None,
+                    max_seq_len: int = 0, splits: int = 0, variant: int = 0) -> None:
+    """Attention of rotated queries over the paged cache (see csrc/attn/gqa_gated.cuh), written into
+    ``out`` [T, >= Hq * Dv].  ``cu_q``: query offsets of prompt portions; None = decode step with
+    ``max_q_len`` rows per sequence.  ``sink``: score of a key without a value that joins every softmax
+    (None: none).  ``gate`` [T, Hq * Dv]: the result is multiplied by its sigmoid."""
+    if not q.is_cuda:
+        return ref.gated_attention(q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len,
+                                   num_q_heads, head_dim, head_dim_v, scale, window, sink)
+    if cu_q is None and splits <= 0:
+        keys = max_seq_len or block_tables.shape[1] * k_cache.shape[2]
+        splits = gated_decode_splits(num_seqs, k_cache.shape[1], min(keys, window) if window else keys)
+    _count(1)
+    _core().gated_attention(q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len,
+                            max_q_len, num_q_heads, head_dim, head_dim_v, scale, window, sink is not None,
+                            0.0 if sink is None else float(sink), max(1, splits), variant,
+                            device_state(q.device).status)
+
+
+# ----------------------------------------------------------- 32-bit residual stream
+def embed_residual_norm(residual: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, scale: float,
+                        weight: torch.Tensor, eps: float, weight_offset: float, true_width: int) -> torch.Tensor:
+    """residual [T,H] fp32 <- scale * table[ids]; returns its RMS norm times (weight_offset + weight).
+    ``true_width``: columns that count in the mean (the rest are zero padding)."""
+    if not residual.is_cuda:
+        return ref.embed_residual_norm(residual, ids, table, scale, weight, eps, weight_offset, true_width)
+    _count(1)
+    return _core().residual_norm(residual, ids, table, scale, None, None, None, None, None, weight, eps,
+                                 weight_offset, true_width, weight.dtype == torch.float32)
+
+
+def residual_add_norm(residual: torch.Tensor, a: Optional[torch.Tensor], b: Optional[torch.Tensor], routed,
+                      weight: Optional[torch.Tensor], eps: float, weight_offset: float, true_width: int):
+    """residual += a + b + routed (in place, fp32); returns its RMS norm times (weight_offset + weight),
+    or None without a weight.  ``routed`` = (y, slots, weights): expert outputs in expert order that are
+    brought back to their tokens here (layers/moe.py:RoutedRows), or None."""
+    if not residual.is_cuda:
+        return ref.residual_add_norm(residual, a, b, routed, weight, eps, weight_offset, true_width)
+    y, slots, w = routed if routed is not None else (None, None, None)
+    like = next(x for x in (weight, a, b, y) if x is not None)
+    _count(1)
+    out = _core().residual_norm(residual, None, None, 1.0, a, b, y, slots, w, weight, eps, weight_offset, true_width,
+                                like.dtype == torch.float32)
+    return out if weight is not None else None
+
+
 # -------------------------------------------------------------------- sampling
 def argmax(logits: torch.Tensor) -> torch.Tensor:
     if not logits.is_cuda:
         return ref.argmax(logits)
     _count(1)
-    return _C().argmax(logits)
+    return _core().argmax(logits)
 
 
 def sample(logits: torch.Tensor, temperature: Optional[torch.Tensor] = None,
@@ -629,7 +738,7 @@ def sample(logits: torch.Tensor, temperature: Optional[torch.Tensor] = None,
     if not logits.is_cuda:
         return ref.sample(logits, temperature, top_k, top_p, generator, seeds, step_offset)
     _count(1)
-    return _C().sample(logits, temperature, top_k, top_p, seeds, step_offset)
+    return _core().sample(logits, temperature, top_k, top_p, seeds, step_offset)
 
 
 def spec_verify(draft: torch.Tensor, target: torch.Tensor, bonus: torch.Tensor, cu: torch.Tensor,
@@ -651,7 +760,7 @@ def moe_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], k: int, sigmoid
     if not logits.is_cuda:
         return ref.moe_topk(logits, bias, k, sigmoid, n_group, topk_group, renorm, scale)
     _count(1)
-    return _C().moe_topk(logits.contiguous(), bias, k, sigmoid, n_group, topk_group, renorm, scale)
+    return _core().moe_topk(logits.contiguous(), bias, k, sigmoid, n_group, topk_group, renorm, scale)
 
 
 def mla_decode(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, seq_lens: torch.Tensor,

@@ -15,14 +15,14 @@ import torch.nn.functional as F
 
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-         swiglu: bool = False) -> torch.Tensor:
+         swiglu: bool = False, act: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
     """``a @ w.T`` with fp32 accumulation.  With ``swiglu`` the N columns are
-    interpreted as interleaved groups of 8 gate / 8 up columns."""
+    interpreted as interleaved groups of 8 gate / 8 up columns, joined by :func:`gated_act`."""
     out = a.float() @ w.float().t()
     if swiglu:
         n = out.shape[-1]
         g = out.view(*out.shape[:-1], n // 16, 2, 8)
-        out = (F.silu(g[..., 0, :]) * g[..., 1, :]).reshape(*out.shape[:-1], n // 2)
+        out = gated_act(g[..., 0, :], g[..., 1, :], act).reshape(*out.shape[:-1], n // 2)
     if bias is not None:
         out = out + bias.float()
     if residual is not None:
@@ -30,6 +30,16 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
     if out_dtype is None:
         out_dtype = torch.bfloat16 if a.dtype.itemsize == 1 else a.dtype
     return out.to(out_dtype)
+
+
+def gated_act(gate: torch.Tensor, up: torch.Tensor, act: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
+    """silu(gate) * up; with ``act`` = (slope, limit), slope non-zero:
+    g * sigmoid(slope * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    slope, limit = act
+    if slope == 0.0:
+        return F.silu(gate) * up
+    g = gate.clamp(max=limit)
+    return g * torch.sigmoid(slope * g) * (up.clamp(-limit, limit) + 1)
 
 
 def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor:
@@ -43,7 +53,7 @@ def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor
 
 
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
-                 swiglu: bool = False) -> torch.Tensor:
+                 swiglu: bool = False, act: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
     e = w.shape[0]
     offs = expert_offsets.tolist()
     n_out = w.shape[1] // 2 if swiglu else w.shape[1]
@@ -52,7 +62,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
     for i in range(e):
         lo, hi = offs[i], offs[i + 1]
         if hi > lo:
-            out[lo:hi] = gemm(a[lo:hi], w[i], swiglu=swiglu, out_dtype=out.dtype)
+            out[lo:hi] = gemm(a[lo:hi], w[i], swiglu=swiglu, out_dtype=out.dtype, act=act)
     return out
 
 
@@ -219,6 +229,56 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         out[qs:qe] = o.reshape(ql, hq * dv).to(q.dtype)
         lse[qs:qe] = l.t()
     return (out, lse) if return_lse else out
+
+
+def gated_rope_cache_(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim, head_dim_v, rot_dim,
+                      neox) -> None:
+    """RoPE on q (in place) and k, then k / v into cache rows that may be wider than the heads."""
+    qo, ko = rope_qk(q, k, positions, cos_sin, head_dim, rot_dim, neox)
+    q.copy_(qo)
+    gqa_cache_write(ko, v, k_cache[..., :head_dim], v_cache[..., :head_dim_v], slot_mapping)
+
+
+def gated_attention(q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len, num_q_heads,
+                    head_dim, head_dim_v, scale, window=0, sink=None) -> None:
+    """Windowed paged attention; a sink of score ``sink`` scales a row's plain result by
+    L / (L + exp(sink)) with L its sum of exponentials; then the sigmoid gate."""
+    if cu_q is None:
+        cu_q = torch.arange(0, (num_seqs + 1) * max_q_len, max_q_len, dtype=torch.int32)
+    o, lse = paged_attention(q, k_cache[..., :head_dim], v_cache[..., :head_dim_v], block_tables[:num_seqs],
+                             cu_q[: num_seqs + 1], seq_lens[:num_seqs], num_q_heads, scale, True, window, True)
+    y = o.float().view(q.shape[0], num_q_heads, head_dim_v)
+    if sink is not None:
+        y = y * torch.sigmoid(lse - sink).unsqueeze(-1)
+    y = y.reshape(q.shape[0], -1)
+    if gate is not None:
+        y = y * torch.sigmoid(gate.float())
+    out[:, : y.shape[1]].copy_(y)
+
+
+def embed_residual_norm(residual, ids, table, scale, weight, eps, weight_offset, true_width):
+    residual.copy_(table[ids.long()].float() * scale)
+    return _unit_norm(residual, weight, eps, weight_offset, true_width)
+
+
+def residual_add_norm(residual, a, b, routed, weight, eps, weight_offset, true_width):
+    add = torch.zeros_like(residual)
+    if routed is not None:
+        y, slots, w = routed
+        t, k = w.shape
+        rows = y[slots[: t * k].long().clamp_min(0)].float().view(t, k, -1)
+        live = (slots[: t * k] >= 0).view(t, k, 1)
+        add += (rows * w.unsqueeze(-1) * live).sum(1)
+    for x in (b, a):
+        if x is not None:
+            add += x.float()
+    residual += add
+    return _unit_norm(residual, weight, eps, weight_offset, true_width) if weight is not None else None
+
+
+def _unit_norm(x, weight, eps, weight_offset, true_width):
+    inv = torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / true_width + eps)
+    return (x * inv * (weight_offset + weight.float())).to(weight.dtype)
 
 
 def argmax(logits: torch.Tensor) -> torch.Tensor:

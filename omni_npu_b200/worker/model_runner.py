@@ -87,6 +87,11 @@ class ModelRunner:
         # device, and the result by index in the step's seqs: (position of the first entry, entries)
         self._plp_plan = None
         self._plp_capture = None
+        # logits at chosen rows of a step (trace replay): the rows asked for, and what was computed there
+        self.keep_logits = False              # captured decode graphs also keep their logits
+        self._graph_logits: Dict[int, torch.Tensor] = {}
+        self._want_rows: Optional[List[int]] = None
+        self.last_logits: Optional[torch.Tensor] = None
         self.last_prompt_logprobs: Dict[int, Tuple[int, list]] = {}
         self.step_counter = torch.zeros(1, dtype=torch.int64, device=device)
         self.d2h_bytes_last = 0
@@ -243,6 +248,14 @@ class ModelRunner:
             logits = self.model.compute_logits(hidden)
             if self._plp_plan:
                 self._capture_prompt_logprobs(hidden_all)
+            if self._want_rows:
+                if idx is None:
+                    self.last_logits = logits
+                else:
+                    rows = torch.tensor(self._want_rows, dtype=torch.long, device=hidden_all.device)
+                    self.last_logits = self.model.compute_logits(hidden_all.index_select(0, rows))
+            elif self.keep_logits and not md.is_prefill:
+                self._graph_logits[num_samples] = logits
             if self._logits_fn is not None:
                 logits = self._logits_fn(logits)
             # (no step offset: the staged seed of a row already carries the index of the token it samples)
@@ -722,6 +735,26 @@ class ModelRunner:
         finally:
             self._logits_fn = None
             self._plp_plan = self._plp_capture = None
+
+    def execute_with_logits(self, out: SchedulerOutput, rows: Sequence[int]) -> Optional[torch.Tensor]:
+        """Run one scheduled step (prefill or decode, through ``execute_model``: same batch, graphs and
+        kernels) and return the logits at the given rows of its flat batch, fp32 [len(rows), vocab] on
+        the host; None when no row is asked for.  Decode graphs must have been captured with
+        ``keep_logits`` set."""
+        self.last_logits = None
+        self._want_rows = list(rows)
+        try:
+            self.execute_model(out)
+            if not rows:
+                return None
+            got = self.last_logits
+            if out.kind == "decode":
+                if got is None:                     # the step ran as a graph
+                    got = self._graph_logits[self._pad_decode_size(len(out.seqs))]
+                got = got.index_select(0, torch.tensor(self._want_rows, dtype=torch.long, device=got.device))
+            return got.float().cpu()
+        finally:
+            self._want_rows = self.last_logits = None
 
     def _execute_scheduled(self, out: SchedulerOutput, ib, n: int, ev) -> List[int]:
         if out.kind == "spec_decode":

@@ -50,7 +50,10 @@ class Worker:
         if want_cuda:
             torch.cuda.set_device(self.local_rank)
             self.device = torch.device("cuda", self.local_rank)
-            ops.load_extension(required=True)
+            # models that run on the core library alone need nothing else loaded (or built)
+            from ..models.registry import runs_on_core_library
+            ops.load_extension(required=True, core_only=not ops.full_library_built()
+                               and runs_on_core_library(self.config.model.architecture))
             self._init_free, self._init_total = torch.cuda.mem_get_info(self.device)
         else:
             self.device = torch.device("cpu")

@@ -53,6 +53,10 @@ def parse_args():
                     help="decoding requests ride along in prefill steps (default: prompts first)")
     ap.add_argument("--profile", default=None,
                     help="write a per-kernel time table (torch profiler, one extra untimed pass) to this file")
+    ap.add_argument("--design", default=None, choices=["rivudra"],
+                    help="instead of the workload: steps and kernels of this design beside the closest existing "
+                         "model at equal size, one JSON line per size (one GPU)")
+    ap.add_argument("--design-size", default=None, help="with --design: only the sizes whose name contains this")
     args = ap.parse_args()
     n, i, o = WORKLOADS.get(args.model, WORKLOADS["llama-3-8b"])
     args.num_requests = args.num_requests or n
@@ -374,7 +378,10 @@ def _shutdown(llm, world: int) -> None:
 
 def main() -> None:
     args = parse_args()
-    if args.impl == "reference":
+    if args.design:
+        from omni_npu_b200.ops import bench_design
+        bench_design.run(args.design, args.design_size)
+    elif args.impl == "reference":
         run_reference(args)
     else:
         run_ours(args)

@@ -25,8 +25,9 @@ template <>
 __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float x) { return __float2bfloat16(x); }
 
 // ------------------------------------------------------------- rotation + cache write
-// q is rotated in place, k is rotated into the cache, v is copied into the cache.  One CTA per token;
-// a work item is two neighbouring elements (interleaved pairs, or no rotation) or one pair (i, i + rot/2).
+// q is rotated in place, k is rotated into the cache, v is copied into the cache.  One warp per
+// (token, head): query heads first, then key heads, then value heads.  With interleaved pairs and
+// aligned rows a lane takes four elements at a time.
 struct RopeCacheParams {
   void* q;
   const void* k;
@@ -41,46 +42,82 @@ struct RopeCacheParams {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(256) gated_rope_cache_kernel(const RopeCacheParams p) {
+struct Quad;
+template <>
+struct Quad<float> {
+  static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
+  static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+};
+template <>
+struct Quad<__nv_bfloat16> {
+  static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xffff0000u));
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  }
+};
+
+static constexpr int kRopeWarps = 4;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kRopeWarps * 32) gated_rope_cache_kernel(const RopeCacheParams p) {
   pdl_trigger();
   pdl_wait();
   const long long t = blockIdx.x;
+  const int lane = threadIdx.x & 31;
+  int h = blockIdx.y * kRopeWarps + (threadIdx.x >> 5);
+  if (h >= p.Hq + 2 * p.Hk) return;
+  const bool is_q = h < p.Hq;
+  const bool is_v = h >= p.Hq + p.Hk;
+  const int slot = is_q ? 0 : p.slots[t];
+  if (slot < 0) return;
+  const T* src;
+  T* dst;
+  int dim = p.D;
+  if (is_q) {
+    dst = static_cast<T*>(p.q) + t * p.q_stride + static_cast<long long>(h) * p.D;
+    src = dst;
+  } else {
+    const long long blk = slot / p.block_size, off = slot % p.block_size;
+    h -= is_v ? p.Hq + p.Hk : p.Hq;
+    const long long row = (blk * p.Hk + h) * p.block_size + off;
+    if (is_v) {
+      dim = p.DV;
+      src = static_cast<const T*>(p.v) + t * p.v_stride + static_cast<long long>(h) * p.DV;
+      dst = static_cast<T*>(p.v_cache) + row * p.DVP;
+    } else {
+      src = static_cast<const T*>(p.k) + t * p.k_stride + static_cast<long long>(h) * p.D;
+      dst = static_cast<T*>(p.k_cache) + row * p.DP;
+    }
+  }
+  const int rot = is_v ? 0 : p.rot, half = p.rot >> 1;
   int pos = p.positions[t];
   pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
-  const int slot = p.slots[t];
   const float* cs = p.cos_sin + static_cast<long long>(pos) * p.rot;
-  const int half = p.rot >> 1;
-  T* q = static_cast<T*>(p.q) + t * p.q_stride;
-  for (int i = threadIdx.x; i < p.Hq * half; i += blockDim.x) {
-    const int h = i / half, j = i % half;
-    T* x = q + static_cast<long long>(h) * p.D + (p.neox ? j : 2 * j);
-    const int o = p.neox ? half : 1;
-    const float c = cs[j], s = cs[half + j], u = to_f(x[0]), w = to_f(x[o]);
-    x[0] = from_f<T>(u * c - w * s);
-    x[o] = from_f<T>(w * c + u * s);
-  }
-  if (slot < 0) return;
-  const long long blk = slot / p.block_size, off = slot % p.block_size;
-  const T* k = static_cast<const T*>(p.k) + t * p.k_stride;
-  T* kc = static_cast<T*>(p.k_cache);
-  for (int i = threadIdx.x; i < p.Hk * p.D; i += blockDim.x) {
-    const int h = i / p.D, d = i % p.D;
-    const T* x = k + static_cast<long long>(h) * p.D;
-    T y = x[d];
-    if (d < p.rot) {
-      const bool second = p.neox ? d >= half : (d & 1) != 0;
-      const int j = p.neox ? (second ? d - half : d) : d >> 1;
-      const float c = cs[j], s = cs[half + j];
-      const float a = to_f(x[d]), o = to_f(x[p.neox ? (second ? d - half : d + half) : d ^ 1]);
-      y = from_f<T>(second ? a * c + o * s : a * c - o * s);
+  if constexpr (VEC) {                       // interleaved pairs; D, DV and rot are multiples of four
+    for (int d = lane * 4; d < dim; d += 128) {
+      if (is_q && d >= rot) break;           // nothing to do for the rest of a query head
+      float4 x = Quad<T>::load(src + d);
+      if (d < rot) {
+        const int j = d >> 1;
+        const float c0 = cs[j], c1 = cs[j + 1], s0 = cs[half + j], s1 = cs[half + j + 1];
+        x = make_float4(x.x * c0 - x.y * s0, x.y * c0 + x.x * s0, x.z * c1 - x.w * s1, x.w * c1 + x.z * s1);
+      }
+      Quad<T>::store(dst + d, x);
     }
-    kc[((blk * p.Hk + h) * p.block_size + off) * p.DP + d] = y;
-  }
-  const T* v = static_cast<const T*>(p.v) + t * p.v_stride;
-  T* vc = static_cast<T*>(p.v_cache);
-  for (int i = threadIdx.x; i < p.Hk * p.DV; i += blockDim.x) {
-    const int h = i / p.DV, d = i % p.DV;
-    vc[((blk * p.Hk + h) * p.block_size + off) * p.DVP + d] = v[static_cast<long long>(h) * p.DV + d];
+  } else {
+    for (int j = lane; j < (rot >> 1); j += 32) {
+      const int a = p.neox ? j : 2 * j, b = a + (p.neox ? half : 1);
+      const float c = cs[j], s = cs[half + j], u = to_f(src[a]), w = to_f(src[b]);
+      dst[a] = from_f<T>(u * c - w * s);
+      dst[b] = from_f<T>(w * c + u * s);
+    }
+    if (!is_q)
+      for (int d = rot + lane; d < dim; d += 32) dst[d] = src[d];
   }
 }
 
@@ -200,9 +237,20 @@ extern "C" int b200_gated_rope_cache(void* q, const void* k, const void* v, void
   if (rot < 0 || rot > D || (rot & 1) || DP < D || DVP < DV) return -1;
   RopeCacheParams p{q, k, v, k_cache, v_cache, positions, slots, cos_sin, Hq, Hk, D, DV, DP, DVP, rot, neox,
                     block_size, max_pos, q_stride, k_stride, v_stride};
-  const cudaError_t e = is_fp32
-      ? launch_pdl(gated_rope_cache_kernel<float>, dim3(T), dim3(256), 0, stream, 1, p)
-      : launch_pdl(gated_rope_cache_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, 1, p);
+  const dim3 grid(T, (Hq + 2 * Hk + kRopeWarps - 1) / kRopeWarps), block(kRopeWarps * 32);
+  const uintptr_t need = is_fp32 ? 15 : 7;           // four elements of a row in one access
+  const auto ok = [&](const void* ptr, long long stride) {
+    return (reinterpret_cast<uintptr_t>(ptr) & need) == 0 && (stride & 3) == 0;
+  };
+  const bool vec = !neox && (D & 3) == 0 && (DV & 3) == 0 && (rot & 3) == 0 && ok(q, q_stride) && ok(k, k_stride) &&
+                   ok(v, v_stride) && ok(k_cache, DP) && ok(v_cache, DVP);
+  cudaError_t e;
+  if (is_fp32)
+    e = vec ? launch_pdl(gated_rope_cache_kernel<float, true>, grid, block, 0, stream, 1, p)
+            : launch_pdl(gated_rope_cache_kernel<float, false>, grid, block, 0, stream, 1, p);
+  else
+    e = vec ? launch_pdl(gated_rope_cache_kernel<__nv_bfloat16, true>, grid, block, 0, stream, 1, p)
+            : launch_pdl(gated_rope_cache_kernel<__nv_bfloat16, false>, grid, block, 0, stream, 1, p);
   return e == cudaSuccess ? 0 : -3;
 }
 
@@ -230,6 +278,9 @@ extern "C" int b200_gated_attention(const void* q, const void* gate, const void*
   p.max_blocks = max_blocks;
   p.block_size = block_size;
   p.num_cache_blocks = num_cache_blocks;
+  p.bs_shift = -1;
+  for (int i = 0; i < 30; ++i)
+    if ((1 << i) == block_size) p.bs_shift = i;
   p.Hq = Hq;
   p.Hk = Hk;
   p.D = D;

@@ -24,6 +24,7 @@ struct GatedAttnParams {
   const int* cu_q;             // [B + 1]; null: every sequence has q_len rows
   const int* seq_lens;         // [B] keys including this step's
   int B, max_blocks, block_size, num_cache_blocks;
+  int bs_shift;                // log2(block_size), -1 when it is not a power of two
   int Hq, Hk, D, DV, DP, DVP;
   long long q_stride, g_stride, out_stride;
   float scale_log2;            // scale * log2(e)

@@ -25,7 +25,7 @@ constexpr int WARPS = 4, THREADS = WARPS * 32, KEYS = 16, ROWS = 16;
 // DM: upper bound of the padded head sizes (64, 128 or 256)
 template <int DM>
 struct Cfg {
-  static constexpr int STAGES = DM > 128 ? 3 : 4;
+  static constexpr int STAGES = 3;                              // (DM 128: two CTAs per SM)
   static constexpr int TILE = KEYS * DM * 2;                    // one K or V tile of a warp
   static constexpr int RING = WARPS * STAGES * 2 * TILE;
   static constexpr int Q_BYTES = ROWS * DM * 2;
@@ -78,6 +78,12 @@ __global__ void __launch_bounds__(gdec::THREADS) gqa_gated_decode_kernel(const G
 
   const int kchunks = p.DP >> 3, vchunks = p.DVP >> 3;
   const int key_row = lane >> 1;
+  // the cache block of this lane's key is looked up one tile ahead of its copies
+  auto block_of = [&](int i) {
+    const int key = (t_begin + warp + i * WARPS) * KEYS + key_row;
+    return i < mine && key < hi ? bt[p.bs_shift >= 0 ? key >> p.bs_shift : key / p.block_size] : 0;
+  };
+  int blk = block_of(0);
   auto issue = [&](int i) {
     if (i < mine) {
       const int key = (t_begin + warp + i * WARPS) * KEYS + key_row;
@@ -85,20 +91,25 @@ __global__ void __launch_bounds__(gdec::THREADS) gqa_gated_decode_kernel(const G
       const __nv_bfloat16* ks = kc;
       const __nv_bfloat16* vs = vc;
       if (ok) {
-        const long long row = (static_cast<long long>(bt[key / p.block_size]) * p.Hk + kvh) * p.block_size +
-                              key % p.block_size;
+        const int off = p.bs_shift >= 0 ? key & (p.block_size - 1) : key % p.block_size;
+        const long long row = (static_cast<long long>(blk) * p.Hk + kvh) * p.block_size + off;
         ks = kc + row * p.DP;
         vs = vc + row * p.DVP;
       }
+      blk = block_of(i + 1);
       const int sz = ok ? 16 : 0;
       const uint32_t kt = smem_u32(ring + (warp * C::STAGES + i % C::STAGES) * 2 * C::TILE);
       const uint32_t vt = kt + C::TILE;
-      for (int c = lane & 1; c < kchunks; c += 2)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(kt + tile_offset<DM>(key_row, c)),
-                     "l"(ks + c * 8), "r"(sz) : "memory");
-      for (int c = lane & 1; c < vchunks; c += 2)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vt + tile_offset<DM>(key_row, c)),
-                     "l"(vs + c * 8), "r"(sz) : "memory");
+#pragma unroll
+      for (int c = lane & 1, u = 0; u < DM / 16; ++u, c += 2)
+        if (c < kchunks)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(kt + tile_offset<DM>(key_row, c)),
+                       "l"(ks + c * 8), "r"(sz) : "memory");
+#pragma unroll
+      for (int c = lane & 1, u = 0; u < DM / 16; ++u, c += 2)
+        if (c < vchunks)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vt + tile_offset<DM>(key_row, c)),
+                       "l"(vs + c * 8), "r"(sz) : "memory");
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -106,7 +117,17 @@ __global__ void __launch_bounds__(gdec::THREADS) gqa_gated_decode_kernel(const G
   for (int i = 0; i < C::STAGES - 1; ++i) issue(i);
 
   // query rows -> shared (zero beyond the head size and the last row)
-  for (int idx = tid; idx < ROWS * p.DP; idx += THREADS) {
+  const bool vec_q = (p.D & 7) == 0 && (p.q_stride & 7) == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0;
+  if (vec_q) {
+    // eight threads per row
+    const int r = tid >> 3, R = r0 + r;
+    const __nv_bfloat16* src =
+        q + (R < rows_all ? (q_begin + R / per) * p.q_stride + static_cast<long long>(kvh * per + R % per) * p.D : 0);
+    for (int c = tid & 7; c < kchunks; c += 8)
+      *reinterpret_cast<uint4*>(sQ + tile_offset<DM>(r, c)) =
+          R < rows_all && c * 8 < p.D ? *reinterpret_cast<const uint4*>(src + c * 8) : make_uint4(0u, 0u, 0u, 0u);
+  }
+  for (int idx = tid; !vec_q && idx < ROWS * p.DP; idx += THREADS) {
     const int r = idx / p.DP, d = idx % p.DP;
     const int R = r0 + r;
     __nv_bfloat16 v = __float2bfloat16(0.f);
@@ -216,22 +237,31 @@ __global__ void __launch_bounds__(gdec::THREADS) gqa_gated_decode_kernel(const G
             make_float2(o_acc[i][2 * r], o_acc[i][2 * r + 1]);
   }
   __syncthreads();
-  // ---- joined in the first warp's area, scaled to the CTA's maximum
-  for (int idx = tid; idx < ROWS * p.DVP; idx += THREADS) {
-    const int row = idx / p.DVP, d = idx % p.DVP;
-    float m = -INFINITY;
+  // ---- joined in the first warp's area, scaled to the CTA's maximum: eight threads per row
+  {
+    const int row = tid >> 3;
+    float m = -INFINITY, f[WARPS], l = 0.f;
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) m = fmaxf(m, stat[(w * ROWS + row) * 2]);
-    float o = 0.f, l = 0.f;
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) {
       const float mw = stat[(w * ROWS + row) * 2];
-      const float f = mw == -INFINITY ? 0.f : exp2f(mw - m);
-      o += f * part[(w * ROWS + row) * DM + d];
-      l += f * stat[(w * ROWS + row) * 2 + 1];
+      f[w] = mw == -INFINITY ? 0.f : exp2f(mw - m);
+      l += f[w] * stat[(w * ROWS + row) * 2 + 1];
     }
-    part[row * DM + d] = o;
-    if (d == 0) {
+    if (r0 + row < rows_all) {
+      for (int d = (tid & 7) * 2; d < p.DVP; d += 16) {
+        float2 o = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int w = 0; w < WARPS; ++w) {
+          const float2 x = *reinterpret_cast<const float2*>(part + (w * ROWS + row) * DM + d);
+          o.x += f[w] * x.x;
+          o.y += f[w] * x.y;
+        }
+        *reinterpret_cast<float2*>(part + row * DM + d) = o;
+      }
+    }
+    if ((tid & 7) == 0) {
       cta_stat[row * 2] = m;
       cta_stat[row * 2 + 1] = l;
     }
@@ -240,31 +270,44 @@ __global__ void __launch_bounds__(gdec::THREADS) gqa_gated_decode_kernel(const G
   if (p.splits > 1) cluster.sync();
   else __syncthreads();
 
-  // ---- rows are dealt out over the CTAs of the cluster
-  for (int idx = tid; idx < ROWS * p.DV; idx += THREADS) {
-    const int row = idx / p.DV, d = idx % p.DV;
-    const int R = r0 + row;
-    if (R >= rows_all || row % p.splits != split) continue;
-    float m = p.has_sink ? p.sink_log2 : -INFINITY;
-    for (int c = 0; c < p.splits; ++c) {
-      const float* st = p.splits > 1 ? cluster.map_shared_rank(cta_stat, c) : cta_stat;
-      m = fmaxf(m, st[row * 2]);
+  // ---- rows are dealt out over the CTAs of the cluster, eight threads per row and `splits` rows apart
+  {
+    const int row = tid >> 3, R = r0 + row;
+    if (R < rows_all && row % p.splits == split) {
+      float m = p.has_sink ? p.sink_log2 : -INFINITY;
+      float mc[8];
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {
+        mc[c] = -INFINITY;
+        if (c < p.splits) mc[c] = (p.splits > 1 ? cluster.map_shared_rank(cta_stat, c) : cta_stat)[row * 2];
+        m = fmaxf(m, mc[c]);
+      }
+      float l = p.has_sink ? exp2f(p.sink_log2 - m) : 0.f;
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {
+        if (mc[c] == -INFINITY) {
+          mc[c] = 0.f;
+          continue;
+        }
+        mc[c] = exp2f(mc[c] - m);
+        l += mc[c] * (p.splits > 1 ? cluster.map_shared_rank(cta_stat, c) : cta_stat)[row * 2 + 1];
+      }
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const long long tok = q_begin + R / per;
+      const long long col = static_cast<long long>(kvh * per + R % per) * p.DV;
+      const __nv_bfloat16* gate = p.gate ? static_cast<const __nv_bfloat16*>(p.gate) + tok * p.g_stride + col : nullptr;
+      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + tok * p.out_stride + col;
+      for (int d = tid & 7; d < p.DV; d += 8) {
+        float o = 0.f;
+#pragma unroll
+        for (int c = 0; c < 8; ++c)
+          if (c < p.splits && mc[c] != 0.f)
+            o += mc[c] * (p.splits > 1 ? cluster.map_shared_rank(part, c) : part)[row * DM + d];
+        o *= inv;
+        if (gate) o *= gate_sigmoid(__bfloat162float(gate[d]));
+        dst[d] = __float2bfloat16(o);
+      }
     }
-    float o = 0.f, l = p.has_sink ? exp2f(p.sink_log2 - m) : 0.f;
-    for (int c = 0; c < p.splits; ++c) {
-      const float* st = p.splits > 1 ? cluster.map_shared_rank(cta_stat, c) : cta_stat;
-      const float* po = p.splits > 1 ? cluster.map_shared_rank(part, c) : part;
-      const float mc = st[row * 2];
-      if (mc == -INFINITY) continue;
-      const float f = exp2f(mc - m);
-      o += f * po[row * DM + d];
-      l += f * st[row * 2 + 1];
-    }
-    o = l > 0.f ? o / l : 0.f;
-    const long long tok = q_begin + R / per;
-    const long long col = static_cast<long long>(kvh * per + R % per) * p.DV + d;
-    if (p.gate) o *= gate_sigmoid(__bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[tok * p.g_stride + col]));
-    static_cast<__nv_bfloat16*>(p.out)[tok * p.out_stride + col] = __float2bfloat16(o);
   }
   if (p.splits > 1) cluster.sync();                        // no CTA leaves while its memory is being read
 }

@@ -17,6 +17,7 @@ divide by the true width.
 """
 from __future__ import annotations
 
+import os
 import re
 from typing import Any, Dict, Iterable, List, Optional, Tuple
 
@@ -33,6 +34,9 @@ from ..layers.rope import get_rope
 from ..parallel import state as pstate
 from .utils import IntermediateTensors, PPMissingLayer, build_pipeline_layers
 
+# Steps of at most this many rows run the two sublayers on two streams: each leaves most of the GPU idle
+# there, and neither needs the other's result.
+OVERLAP_ROWS = int(os.environ.get("OMNI_B200_PARALLEL_SUBLAYER_ROWS", "256"))
 SIGMOID_SLOPE = 1.702          # of the experts' gate
 SINK_SCORE = 0.0
 NORM_WEIGHT_OFFSET = 1.0
@@ -126,6 +130,15 @@ class RivudraMixer(nn.Module):
         return self.o_proj(self.attn(q, k, v, g, self.rotary.cos_sin_cache, self.o_proj.in_local))
 
 
+_SIDE_STREAMS: Dict[torch.device, torch.cuda.Stream] = {}
+
+
+def _side_stream(device: torch.device) -> torch.cuda.Stream:
+    if device not in _SIDE_STREAMS:
+        _SIDE_STREAMS[device] = torch.cuda.Stream(device)
+    return _SIDE_STREAMS[device]
+
+
 class RivudraLayer(nn.Module):
     def __init__(self, engine: EngineConfig, spec: LayerSpec, layer_idx: int, device) -> None:
         super().__init__()
@@ -153,8 +166,16 @@ class RivudraLayer(nn.Module):
         """The layer's share of the residual from its normed input: (dense, dense or None, routed or None)."""
         if self.mlp is None:
             return self.mix(hidden), None, None
+        if not hidden.is_cuda or hidden.shape[0] > OVERLAP_ROWS or self.mix.qkvg_proj.tp_size > 1:
+            routed, dense = self.mlp.forward_deferred(hidden)
+            return self.mix(hidden), dense, routed
+        cur, side = torch.cuda.current_stream(hidden.device), _side_stream(hidden.device)
+        side.wait_stream(cur)
+        with torch.cuda.stream(side):
+            mixed = self.mix(hidden)
         routed, dense = self.mlp.forward_deferred(hidden)
-        return self.mix(hidden), dense, routed
+        cur.wait_stream(side)
+        return mixed, dense, routed
 
 
 class RivudraForCausalLM(nn.Module):

@@ -664,11 +664,11 @@ def gated_rope_cache_(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache
 
 
 def gated_decode_splits(num_seqs: int, num_kv_heads: int, keys: int, sms: int = 148) -> int:
-    """CTAs (of one cluster) that share the visible keys of a (sequence, key/value head): enough to
-    give every SM two, at least 128 keys each."""
+    """CTAs (of one cluster) that share the visible keys of a (sequence, key/value head): as many as
+    are resident at once (two per SM), at least 128 keys each."""
     base = max(1, num_seqs * num_kv_heads)
     splits = 1
-    while splits < 8 and base * splits < 2 * sms and keys >= 256 * splits:
+    while splits < 8 and base * splits <= sms and keys >= 256 * splits:
         splits *= 2
     return splits
 

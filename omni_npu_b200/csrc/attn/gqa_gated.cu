@@ -25,9 +25,9 @@ template <>
 __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float x) { return __float2bfloat16(x); }
 
 // ------------------------------------------------------------- rotation + cache write
-// q is rotated in place, k is rotated into the cache, v is copied into the cache.  One warp per
-// (token, head): query heads first, then key heads, then value heads.  With interleaved pairs and
-// aligned rows a lane takes four elements at a time.
+// q is rotated in place, k is rotated into the cache, v is copied into the cache.  Aligned rows with
+// interleaved pairs go 16 bytes at a time, a token per CTA row (split over gridDim.y CTAs when there are
+// few tokens); anything else takes one warp per (token, head).
 struct RopeCacheParams {
   void* q;
   const void* k;
@@ -41,29 +41,107 @@ struct RopeCacheParams {
   long long q_stride, k_stride, v_stride;
 };
 
+// 16 bytes of a row as floats
 template <typename T>
-struct Quad;
+struct Chunk;
 template <>
-struct Quad<float> {
-  static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
-  static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-};
-template <>
-struct Quad<__nv_bfloat16> {
-  static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
-                       __uint_as_float(u.y & 0xffff0000u));
+struct Chunk<float> {
+  static constexpr int W = 4;
+  static __device__ __forceinline__ void load(const float* p, float (&x)[4]) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
   }
-  static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  static __device__ __forceinline__ void store(float* p, const float (&x)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
   }
 };
+template <>
+struct Chunk<__nv_bfloat16> {
+  static constexpr int W = 8;
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&x)[8]) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t r[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      x[2 * i] = __uint_as_float(r[i] << 16);
+      x[2 * i + 1] = __uint_as_float(r[i] & 0xffff0000u);
+    }
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&x)[8]) {
+    uint4 u;
+    uint32_t* r = reinterpret_cast<uint32_t*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const __nv_bfloat162 v = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+      r[i] = *reinterpret_cast<const uint32_t*>(&v);
+    }
+    *reinterpret_cast<uint4*>(p) = u;
+  }
+};
+
+static constexpr int kRopeThreads = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kRopeThreads) gated_rope_cache_vec_kernel(const RopeCacheParams p) {
+  constexpr int W = Chunk<T>::W;
+  pdl_trigger();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const int slot = p.slots[t];
+  int pos = p.positions[t];
+  pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
+  const float* cs = p.cos_sin + static_cast<long long>(pos) * p.rot;
+  const int half = p.rot >> 1;
+  const int qc = p.rot / W, kc = p.D / W, vc = p.DV / W;         // chunks per head (q: rotated part only)
+  const int nq = p.Hq * qc, nk = p.Hk * kc, nv = p.Hk * vc;
+  const int total = slot < 0 ? nq : nq + nk + nv;
+  const long long blk = slot < 0 ? 0 : slot / p.block_size;
+  const int off = slot < 0 ? 0 : slot % p.block_size;
+  for (int i = blockIdx.y * kRopeThreads + threadIdx.x; i < total; i += gridDim.y * kRopeThreads) {
+    const T* src;
+    T* dst;
+    int d;
+    bool turn = true;
+    if (i < nq) {
+      const int h = i / qc;
+      d = (i - h * qc) * W;
+      dst = static_cast<T*>(p.q) + t * p.q_stride + static_cast<long long>(h) * p.D + d;
+      src = dst;
+    } else if (i < nq + nk) {
+      const int h = (i - nq) / kc;
+      d = (i - nq - h * kc) * W;
+      src = static_cast<const T*>(p.k) + t * p.k_stride + static_cast<long long>(h) * p.D + d;
+      dst = static_cast<T*>(p.k_cache) + ((blk * p.Hk + h) * p.block_size + off) * p.DP + d;
+      turn = d < p.rot;
+    } else {
+      const int h = (i - nq - nk) / vc;
+      d = (i - nq - nk - h * vc) * W;
+      src = static_cast<const T*>(p.v) + t * p.v_stride + static_cast<long long>(h) * p.DV + d;
+      dst = static_cast<T*>(p.v_cache) + ((blk * p.Hk + h) * p.block_size + off) * p.DVP + d;
+      turn = false;
+    }
+    float x[W];
+    Chunk<T>::load(src, x);
+    if (turn) {
+      const float2* c2 = reinterpret_cast<const float2*>(cs + (d >> 1));
+      const float2* s2 = reinterpret_cast<const float2*>(cs + half + (d >> 1));
+#pragma unroll
+      for (int j = 0; j < W / 4; ++j) {
+        const float2 c = c2[j], s = s2[j];
+        const float u0 = x[4 * j], w0 = x[4 * j + 1], u1 = x[4 * j + 2], w1 = x[4 * j + 3];
+        x[4 * j] = u0 * c.x - w0 * s.x;
+        x[4 * j + 1] = w0 * c.x + u0 * s.x;
+        x[4 * j + 2] = u1 * c.y - w1 * s.y;
+        x[4 * j + 3] = w1 * c.y + u1 * s.y;
+      }
+    }
+    Chunk<T>::store(dst, x);
+  }
+}
 
 static constexpr int kRopeWarps = 4;
 
-template <typename T, bool VEC>
+template <typename T>
 __global__ void __launch_bounds__(kRopeWarps * 32) gated_rope_cache_kernel(const RopeCacheParams p) {
   pdl_trigger();
   pdl_wait();
@@ -98,27 +176,14 @@ __global__ void __launch_bounds__(kRopeWarps * 32) gated_rope_cache_kernel(const
   int pos = p.positions[t];
   pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
   const float* cs = p.cos_sin + static_cast<long long>(pos) * p.rot;
-  if constexpr (VEC) {                       // interleaved pairs; D, DV and rot are multiples of four
-    for (int d = lane * 4; d < dim; d += 128) {
-      if (is_q && d >= rot) break;           // nothing to do for the rest of a query head
-      float4 x = Quad<T>::load(src + d);
-      if (d < rot) {
-        const int j = d >> 1;
-        const float c0 = cs[j], c1 = cs[j + 1], s0 = cs[half + j], s1 = cs[half + j + 1];
-        x = make_float4(x.x * c0 - x.y * s0, x.y * c0 + x.x * s0, x.z * c1 - x.w * s1, x.w * c1 + x.z * s1);
-      }
-      Quad<T>::store(dst + d, x);
-    }
-  } else {
-    for (int j = lane; j < (rot >> 1); j += 32) {
-      const int a = p.neox ? j : 2 * j, b = a + (p.neox ? half : 1);
-      const float c = cs[j], s = cs[half + j], u = to_f(src[a]), w = to_f(src[b]);
-      dst[a] = from_f<T>(u * c - w * s);
-      dst[b] = from_f<T>(w * c + u * s);
-    }
-    if (!is_q)
-      for (int d = rot + lane; d < dim; d += 32) dst[d] = src[d];
+  for (int j = lane; j < (rot >> 1); j += 32) {
+    const int a = p.neox ? j : 2 * j, b = a + (p.neox ? half : 1);
+    const float c = cs[j], s = cs[half + j], u = to_f(src[a]), w = to_f(src[b]);
+    dst[a] = from_f<T>(u * c - w * s);
+    dst[b] = from_f<T>(w * c + u * s);
   }
+  if (!is_q)
+    for (int d = rot + lane; d < dim; d += 32) dst[d] = src[d];
 }
 
 // ------------------------------------------------------------- one CTA per (token, head), fp32 math
@@ -237,20 +302,24 @@ extern "C" int b200_gated_rope_cache(void* q, const void* k, const void* v, void
   if (rot < 0 || rot > D || (rot & 1) || DP < D || DVP < DV) return -1;
   RopeCacheParams p{q, k, v, k_cache, v_cache, positions, slots, cos_sin, Hq, Hk, D, DV, DP, DVP, rot, neox,
                     block_size, max_pos, q_stride, k_stride, v_stride};
-  const dim3 grid(T, (Hq + 2 * Hk + kRopeWarps - 1) / kRopeWarps), block(kRopeWarps * 32);
-  const uintptr_t need = is_fp32 ? 15 : 7;           // four elements of a row in one access
+  const int W = is_fp32 ? 4 : 8;
   const auto ok = [&](const void* ptr, long long stride) {
-    return (reinterpret_cast<uintptr_t>(ptr) & need) == 0 && (stride & 3) == 0;
+    return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0 && stride % W == 0;
   };
-  const bool vec = !neox && (D & 3) == 0 && (DV & 3) == 0 && (rot & 3) == 0 && ok(q, q_stride) && ok(k, k_stride) &&
-                   ok(v, v_stride) && ok(k_cache, DP) && ok(v_cache, DVP);
   cudaError_t e;
-  if (is_fp32)
-    e = vec ? launch_pdl(gated_rope_cache_kernel<float, true>, grid, block, 0, stream, 1, p)
-            : launch_pdl(gated_rope_cache_kernel<float, false>, grid, block, 0, stream, 1, p);
-  else
-    e = vec ? launch_pdl(gated_rope_cache_kernel<__nv_bfloat16, true>, grid, block, 0, stream, 1, p)
-            : launch_pdl(gated_rope_cache_kernel<__nv_bfloat16, false>, grid, block, 0, stream, 1, p);
+  if (!neox && D % W == 0 && DV % W == 0 && rot % W == 0 && ok(q, q_stride) && ok(k, k_stride) && ok(v, v_stride) &&
+      ok(k_cache, DP) && ok(v_cache, DVP)) {
+    const int chunks = (Hq * rot + Hk * (D + DV)) / W;
+    int ny = (chunks + kRopeThreads - 1) / kRopeThreads;
+    if (T >= 512) ny = 1;                              // enough tokens: fewer, longer CTAs
+    const dim3 grid(T, ny), block(kRopeThreads);
+    e = is_fp32 ? launch_pdl(gated_rope_cache_vec_kernel<float>, grid, block, 0, stream, 1, p)
+                : launch_pdl(gated_rope_cache_vec_kernel<__nv_bfloat16>, grid, block, 0, stream, 1, p);
+  } else {
+    const dim3 grid(T, (Hq + 2 * Hk + kRopeWarps - 1) / kRopeWarps), block(kRopeWarps * 32);
+    e = is_fp32 ? launch_pdl(gated_rope_cache_kernel<float>, grid, block, 0, stream, 1, p)
+                : launch_pdl(gated_rope_cache_kernel<__nv_bfloat16>, grid, block, 0, stream, 1, p);
+  }
   return e == cudaSuccess ? 0 : -3;
 }
 

@@ -164,3 +164,28 @@ def test_server_command_line_takes_the_model(setup):
 def test_config_file_is_plain_json(setup):
     with open(setup[0] / "config.json") as f:
         assert json.load(f)["architecture"] == "Rivudra"
+
+
+@pytest.mark.parametrize("pp", [1, 2])
+def test_two_ranks(tmp_path, pp, monkeypatch):
+    """Tensor parallel (heads and experts sharded, one key/value head replicated) and two pipeline stages
+    (the fp32 residual crosses the boundary)."""
+    from dist_utils import run_ranks
+    monkeypatch.delenv("OMNI_B200_PP_LAYER_PARTITION", raising=False)
+    cfg = cases.model(96, 203, [
+        cases.attn_layer(4, 2, 24, 40, 16, 10, mlp=cases.moe(8, 3, 40, 0.8, 4, 2, 1.7, shared=(24, 1.1))),
+        cases.attn_layer(6, 1, 16, 16, 8, 33),
+        cases.attn_layer(2, 2, 48, 24, 48, 17, mlp=cases.moe(6, 1, 16, 2.5))])
+    (tmp_path / "model").mkdir()
+    w = cases.write_model(tmp_path / "model", cfg, seed=9)
+    prompts = [cases.tokens(n, cfg["vocab"], n) for n in (20, 33, 70)]
+    (tmp_path / "prompts.json").write_text(json.dumps(prompts))
+    (tmp_path / "pipeline_parallel").write_text(str(pp))
+    res = run_ranks("tp_engine", 2, str(tmp_path))
+    assert res[0]["tokens"] == res[1]["tokens"]
+    for p, out in zip(prompts, res[0]["tokens"]):
+        seq = list(p)
+        for t in out:
+            logits = oracle.forward(seq, w, cfg)[-1]
+            assert float(logits.max() - logits[t]) < 1e-3
+            seq.append(t)

@@ -39,9 +39,13 @@ CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function"]
 # sources of the core library, relative to csrc/
 CORE_SOURCES = [
     "attn/gqa_gated.cu", "attn/gqa_gated_decode.cu", "attn/gqa_gated_prefill.cu", "attn/gqa_prefill_tcgen05.cu",
+    "attn/latent_attn.cu", "attn/mla_decode.cu",
     "gemm/gemm_simt.cu", "gemm/gemm_tcgen05.cu", "gemm/gemm_tcgen05_pair.cu", "moe/moe_ep.cu",
-    "norm_rope/residual_norm.cu", "sample/sampling.cu",
+    "norm_rope/hyper_norm.cu", "norm_rope/residual_norm.cu", "recurrent/recurrent.cu", "sample/sampling.cu",
 ]
+
+# sources whose fp32 functions and divisions keep their full accuracy
+PRECISE_SOURCES = ["attn/latent_attn.cu", "norm_rope/hyper_norm.cu", "recurrent/recurrent.cu"]
 
 
 def _nvcc() -> str:
@@ -137,8 +141,11 @@ def build(force: bool = False, verbose: bool = False, core_only: bool = False) -
 
     for src in cuda_sources():
         lib = "_C_core" if src.relative_to(CSRC).as_posix() in CORE_SOURCES else "_C"
+        flags = NVCC_FLAGS
+        if src.relative_to(CSRC).as_posix() in PRECISE_SOURCES:
+            flags = [f for f in flags if f != "--use_fast_math"]
         if lib == "_C_core" or not core_only:
-            compile_one(src, lib, [nvcc, *NVCC_FLAGS, "-I", str(CSRC)], log=True)
+            compile_one(src, lib, [nvcc, *flags, "-I", str(CSRC)], log=True)
 
     inc = []
     for p in ce.include_paths("cuda") if hasattr(ce, "include_paths") else []:

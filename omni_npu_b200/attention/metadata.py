@@ -31,16 +31,20 @@ class AttentionMetadata:
     cu_q: torch.Tensor            # [num_seqs + 1] int32 query offsets
     num_actual_tokens: int = 0    # tokens that are not padding
     num_actual_seqs: int = 0
+    # models with recurrent state
+    seq_idx: Optional[torch.Tensor] = None        # [num_tokens] int32, sequence of each row
+    state_slots: Optional[torch.Tensor] = None    # [num_seqs] int32, -1 for padded sequences
     extra: Dict[str, Any] = field(default_factory=dict)
 
 
 class ForwardContext:
     def __init__(self, attn_metadata: Optional[AttentionMetadata], kv_caches, config=None,
-                 in_graph_capture: bool = False) -> None:
+                 in_graph_capture: bool = False, states=None) -> None:
         self.attn_metadata = attn_metadata
         self.kv_caches = kv_caches
         self.config = config
         self.in_graph_capture = in_graph_capture
+        self.states = states              # recurrent state per layer run (models that have one)
 
 
 _ctx: Optional[ForwardContext] = None
@@ -54,10 +58,10 @@ def get_forward_context() -> ForwardContext:
 
 @contextlib.contextmanager
 def set_forward_context(attn_metadata: Optional[AttentionMetadata], kv_caches, config=None,
-                        in_graph_capture: bool = False):
+                        in_graph_capture: bool = False, states=None):
     global _ctx
     prev = _ctx
-    _ctx = ForwardContext(attn_metadata, kv_caches, config, in_graph_capture)
+    _ctx = ForwardContext(attn_metadata, kv_caches, config, in_graph_capture, states)
     try:
         yield _ctx
     finally:

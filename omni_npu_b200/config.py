@@ -14,7 +14,7 @@ import dataclasses
 import json
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Sequence, Tuple
+from typing import Any, Dict, List, Optional, Sequence, Tuple, Union
 
 import torch
 
@@ -67,9 +67,67 @@ class MoESpec:
 
 
 @dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Attention over a cached latent (``kv_rank``, normed) and one rotated key part that all heads share."""
+    num_heads: int
+    nope_dim: int
+    rope_dim: int
+    v_head_dim: int
+    kv_rank: int
+    rope_theta: float
+    scale: float
+    rope_neox: bool = True
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    """Linear attention whose forget gate f (per channel) also decides what is written: keys are 1 - f."""
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+
+
+@dataclass(frozen=True)
+class DeltaRuleSpec:
+    """Gated delta rule with a decay per head and key channel, short convolutions before q / k / v and
+    low-rank projections for decay and output gate."""
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    conv_taps: int
+    decay_rank: int
+    gate_rank: int
+    unit_eps: float = 1e-6                # of the unit norm of q and k
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    """A feed-forward without experts: down(act(up(h)))."""
+    intermediate_size: int
+    act: str = "xielu"
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    attention: AttentionSpec
-    mlp: Optional[MoESpec] = None
+    attention: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, DeltaRuleSpec]
+    mlp: Union[MoESpec, DenseSpec, None] = None
+
+    @property
+    def kv_elems(self) -> int:
+        """Cached elements per token (recurrent layers keep a state per sequence instead)."""
+        a = self.attention
+        if isinstance(a, AttentionSpec):
+            return a.num_kv_heads * (a.head_dim + a.v_head_dim)
+        return a.kv_rank + a.rope_dim if isinstance(a, LatentAttentionSpec) else 0
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start`` .. ``stop`` - 1 run ``times`` times in a row with the same weights."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass
@@ -127,6 +185,9 @@ class ModelConfig:
     layer_specs: Tuple[LayerSpec, ...] = ()
     embedding_scale: float = 1.0
     norm_weight_offset: float = 0.0       # 1: norm weights are stored around zero
+    layer_loop: Optional[LoopSpec] = None
+    residual_streams: int = 1             # parallel residual streams joined by hyper-connections
+    logit_scale: float = 1.0
     # --- misc
     eos_token_id: Optional[int] = None
     hf_config: Dict[str, Any] = field(default_factory=dict)
@@ -149,24 +210,31 @@ class ModelConfig:
         return (self.is_moe and idx >= self.first_k_dense
                 and (idx - self.first_k_dense) % max(1, self.moe_layer_freq) == 0)
 
+    def layer_order(self) -> List[int]:
+        """The layer of every run through the model; each run has a cache or state of its own."""
+        n, loop = self.num_layers, self.layer_loop
+        if loop is None:
+            return list(range(n))
+        return [*range(loop.start), *list(range(loop.start, loop.stop)) * loop.times, *range(loop.stop, n)]
+
     def kv_bytes_per_token(self) -> int:
         """Bytes of KV cache one token occupies across all layers (per TP-1 rank)."""
         esz = self.dtype.itemsize
         if self.layer_specs:
-            return esz * sum(s.attention.num_kv_heads * (s.attention.head_dim + s.attention.v_head_dim)
-                             for s in self.layer_specs)
+            return esz * sum(self.layer_specs[i].kv_elems for i in self.layer_order())
         if self.use_mla:
             per = self.kv_lora_rank + self.qk_rope_head_dim + (self.index_head_dim if self.use_sparse else 0)
             return self.num_layers * per * esz
         return self.num_layers * 2 * self.num_kv_heads * self.head_dim * esz
 
     @classmethod
-    def from_hf_dict(cls, d: Dict[str, Any], dtype=None) -> "ModelConfig":
+    def from_hf_dict(cls, d: Dict[str, Any], dtype=None, path: Optional[str] = None) -> "ModelConfig":
         """Build from the contents of a ``config.json``: HF keys, or the own keys of a design that names
-        itself under ``architecture`` and has a reader in the model registry."""
+        itself under ``architecture`` and has a reader in the model registry.  ``path``: the directory the
+        weights lie in, for readers that take sizes from the shapes of tensors."""
         if "architectures" not in d and isinstance(d.get("architecture"), str):
             from .models.registry import resolve_config_reader
-            return resolve_config_reader(d["architecture"])(d, dtype=dtype)
+            return resolve_config_reader(d["architecture"])(d, dtype=dtype, path=path)
         if "text_config" in d and isinstance(d["text_config"], dict):
             merged = dict(d["text_config"])
             merged.setdefault("architectures", d.get("architectures"))
@@ -233,7 +301,7 @@ class ModelConfig:
     @classmethod
     def from_pretrained(cls, path: str, dtype=None) -> "ModelConfig":
         with open(os.path.join(path, "config.json")) as f:
-            return cls.from_hf_dict(json.load(f), dtype=dtype)
+            return cls.from_hf_dict(json.load(f), dtype=dtype, path=path)
 
 
 # ----------------------------------------------------------------- presets

@@ -236,7 +236,8 @@ __global__ void __launch_bounds__(kPlainThreads) gated_plain_kernel(const GatedA
     float s = -INFINITY;
     long long row = 0;
     if (key < hi) {
-      row = (static_cast<long long>(bt[key / p.block_size]) * p.Hk + kvh) * p.block_size + key % p.block_size;
+      row = p.contiguous ? static_cast<long long>(bt[0] + key) * p.Hk + kvh
+                         : (static_cast<long long>(bt[key / p.block_size]) * p.Hk + kvh) * p.block_size + key % p.block_size;
       const T* k = kc + row * p.DP;
       float acc = 0.f;
       for (int d = 0; d < p.D; ++d) acc = fmaf(sq[d], to_f(k[d]), acc);
@@ -331,7 +332,7 @@ extern "C" int b200_gated_attention(const void* q, const void* gate, const void*
                                     int num_cache_blocks, int Hq, int Hk, int D, int DV, int DP, int DVP,
                                     long long q_stride, long long g_stride, long long out_stride, float scale,
                                     int window, int has_sink, float sink, int splits, int is_fp32, int variant,
-                                    int* status, cudaStream_t stream) {
+                                    int* status, int contiguous, cudaStream_t stream) {
   if (B <= 0 || total_rows <= 0) return 0;
   if (Hk <= 0 || Hq % Hk != 0) return -1;
   GatedAttnParams p{};
@@ -341,6 +342,7 @@ extern "C" int b200_gated_attention(const void* q, const void* gate, const void*
   p.v_cache = v_cache;
   p.out = out;
   p.block_tables = block_tables;
+  p.contiguous = contiguous;
   p.cu_q = cu_q;
   p.seq_lens = seq_lens;
   p.B = B;
@@ -368,8 +370,8 @@ extern "C" int b200_gated_attention(const void* q, const void* gate, const void*
   const bool tensor = !is_fp32 && variant != 2 && (DP & 15) == 0 && (DVP & 15) == 0 && DP <= 256 && DVP <= 256;
   if (!tensor) return is_fp32 ? launch_plain<float>(p, total_rows, stream)
                               : launch_plain<__nv_bfloat16>(p, total_rows, stream);
-  if (cu_q == nullptr) return gated_decode(p, stream);
-  if (variant == 0) {
+  if (cu_q == nullptr) return contiguous ? -3 : gated_decode(p, stream);
+  if (variant == 0 && !contiguous) {
     const int rc = gated_prefill_tc(p, max_q_len, total_rows, status, stream);
     if (rc <= 0) return rc;
   }

@@ -20,7 +20,8 @@ struct GatedAttnParams {
   const void* k_cache;         // [blocks, Hk, block_size, DP]
   const void* v_cache;         // [blocks, Hk, block_size, DVP]
   void* out;                   // [T, Hq * DV], row pitch out_stride
-  const int* block_tables;     // [B, max_blocks]
+  const int* block_tables;     // [B, max_blocks]; with contiguous set: [B], the first row of a sequence
+  int contiguous;              // keys lie in rows one after another, [keys, Hk, DP]: no blocks
   const int* cu_q;             // [B + 1]; null: every sequence has q_len rows
   const int* seq_lens;         // [B] keys including this step's
   int B, max_blocks, block_size, num_cache_blocks;

@@ -1,4 +1,5 @@
-// Prompt portions of the gated, windowed attention (gqa_gated.cuh), bf16, any head sizes up to 256.
+// Prompt portions of the gated, windowed attention (gqa_gated.cuh), bf16, any head sizes up to 256, keys in
+// cache blocks or contiguous.
 //
 // One CTA = 128 rows of one (sequence, key/value head): a row is one (token, head of the group), so a
 // tile covers 128 / group tokens and its keys serve all heads of the group; with a window that is short
@@ -26,13 +27,16 @@ struct Cfg {
 
 template <int DM>
 __device__ __forceinline__ void load_gated_tile(uint32_t dst, const __nv_bfloat16* cache, const int* bt, int n0,
-                                                int hi, int kvh, int Hk, int block_size, int width, int tid) {
+                                                int hi, int kvh, int Hk, int block_size, int width, int contiguous,
+                                                int tid) {
   // four threads per key row, 16-byte chunks dealt out in turn
   const int row = tid >> 2;
   const int key = n0 + row;
   const bool ok = key < hi;
   const __nv_bfloat16* src = cache;
-  if (ok)
+  if (ok && contiguous)
+    src = cache + (static_cast<long long>(bt[0] + key) * Hk + kvh) * width;
+  else if (ok)
     src = cache + ((static_cast<long long>(bt[key / block_size]) * Hk + kvh) * block_size + key % block_size) * width;
   const int sz = ok ? 16 : 0;
   for (int c = tid & 3; c < (width >> 3); c += 4)
@@ -76,8 +80,8 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
   const int lo = p.window > 0 ? max(0, ctx + m0 - p.window + 1) / BN * BN : 0;
   const int tiles = (hi - lo + BN - 1) / BN;
 
-  load_gated_tile<DM>(kv0, kc, bt, lo, hi, kvh, p.Hk, p.block_size, p.DP, tid);
-  load_gated_tile<DM>(kv0 + 2 * C::T_BYTES, vc, bt, lo, hi, kvh, p.Hk, p.block_size, p.DVP, tid);
+  load_gated_tile<DM>(kv0, kc, bt, lo, hi, kvh, p.Hk, p.block_size, p.DP, p.contiguous, tid);
+  load_gated_tile<DM>(kv0 + 2 * C::T_BYTES, vc, bt, lo, hi, kvh, p.Hk, p.block_size, p.DVP, p.contiguous, tid);
   asm volatile("cp.async.commit_group;" ::: "memory");
 
   // ---- query rows -> shared: two threads per row
@@ -128,8 +132,8 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
     const int st = it & 1;
     if (it + 1 < tiles) {
       const int nn = lo + (it + 1) * BN;
-      load_gated_tile<DM>(kv0 + (st ^ 1) * C::T_BYTES, kc, bt, nn, hi, kvh, p.Hk, p.block_size, p.DP, tid);
-      load_gated_tile<DM>(kv0 + (2 + (st ^ 1)) * C::T_BYTES, vc, bt, nn, hi, kvh, p.Hk, p.block_size, p.DVP, tid);
+      load_gated_tile<DM>(kv0 + (st ^ 1) * C::T_BYTES, kc, bt, nn, hi, kvh, p.Hk, p.block_size, p.DP, p.contiguous, tid);
+      load_gated_tile<DM>(kv0 + (2 + (st ^ 1)) * C::T_BYTES, vc, bt, nn, hi, kvh, p.Hk, p.block_size, p.DVP, p.contiguous, tid);
       asm volatile("cp.async.commit_group;" ::: "memory");
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {

@@ -1,16 +1,19 @@
 // Multi-head latent attention, absorbed (MQA) form, over the paged latent cache.
 //
-//   cache row  = [ c_kv (512) | k_pe (64) ]                 one row per token, shared by all heads
-//   query row  = [ q_nope . W_UK (512) | q_pe (64) ]       per head
-//   out[h]     = softmax(q[h] . cache^T * scale) . c_kv     (512 wide; W_UV is applied by the caller)
+//   cache row  = [ c_kv (rank) | k_pe ]                     one row per token, shared by all heads
+//   query row  = [ q_nope . W_UK (rank) | q_pe ]           per head
+//   out[h]     = softmax(q[h] . cache^T * scale) . c_kv     (rank wide; W_UV is applied by the caller)
+//
+// The row is 512 + 64 elements for the DeepSeek family (sizes known to the compiler) or any size up to
+// 640 with a rank up to 512 (b200_latent_decode; the row holds zeros behind its last element).
 //
 // One CTA handles 16 query rows (heads) of one sequence (and one query token for
-// multi-token decode) over one split of the keys.  K tiles of 64 tokens x 576
-// dims come in through TMA (nine 64-column slabs, 128B swizzle) into a two-stage
+// multi-token decode) over one split of the keys.  K tiles of 64 tokens x one row
+// come in through TMA (64-column slabs, 128B swizzle) into a two-stage
 // ring, issued by a producer warp.  Four compute warps:
-//   QK^T : warp w scores keys 16w..16w+15 of the tile (K = 576),
+//   QK^T : warp w scores keys 16w..16w+15 of the tile,
 //   softmax: tile-wide row max / sum through shared memory, P stored as bf16,
-//   P.V  : warp w accumulates output columns 128w..128w+127 over all 64 keys.
+//   P.V  : warp w accumulates a quarter of the output columns over all 64 keys.
 // Split-KV partials are merged by a second kernel.  All waits are bounded.
 //
 // Replaces the decode call of npu_fused_infer_attention_score over the latent
@@ -28,18 +31,17 @@ static constexpr float kMlaLog2e = 1.4426950408889634f;
 static constexpr int kLat = 512;
 static constexpr int kRope = 64;
 static constexpr int kRow = kLat + kRope;     // 576
-static constexpr int kSlabs = kRow / 64;      // 9
 static constexpr int kMlaBN = 64;
 static constexpr int kMlaStages = 2;
 static constexpr int kSlabBytes = kMlaBN * 128;           // 8 KB
-static constexpr int kTileBytes = kSlabs * kSlabBytes;    // 72 KB
-static constexpr int kQBytes = kSlabs * 16 * 128;         // 18 KB
 static constexpr int kPBytes = 16 * kMlaBN * 2;           // 2 KB
-static constexpr int kMlaSmem = 1024 + kMlaStages * kTileBytes + kQBytes + kPBytes + 4096;
+
+// shared memory for rows of `slabs` 64-column slabs: two key tiles, the queries, P, scratch
+static constexpr int mla_smem(int slabs) { return 1024 + slabs * (kMlaStages * kSlabBytes + 16 * 128) + kPBytes + 4096; }
 
 struct MlaParams {
-  const __nv_bfloat16* q;        // [T, N, 576]
-  __nv_bfloat16* out;            // [T, N, 512]
+  const __nv_bfloat16* q;        // [T, N, row]
+  __nv_bfloat16* out;            // [T, N, rank]
   float* lse;                    // [T, N] or null
   const int* block_tables;       // [B, max_blocks]
   const int* seq_lens;           // [B]
@@ -51,7 +53,8 @@ struct MlaParams {
   long long q_stride, out_stride;  // elements between tokens
   float scale_log2;
   int splits;
-  float* o_part;                 // [B*q_len, head_tiles, splits, 16, 512]
+  int row, rank;                 // used by the instantiations whose sizes are not built in
+  float* o_part;                 // [B*q_len, head_tiles, splits, 16, 64 * CT]
   float* ml_part;                // [.., 16, 2]
   int* status;
 };
@@ -62,14 +65,20 @@ __device__ __forceinline__ uint32_t mla_off(int row, int chunk, int rows_per_sla
                                (((chunk & 7) ^ (row & 7)) << 4));
 }
 
+// ROW: elements of a cache row, 0 = p.row.  CT: 16-column output tiles of a warp (4 * 16 * CT >= rank).
+template <int ROW, int CT>
 __global__ void __launch_bounds__(160)
 mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, const int box_rows) {
+  const int row_elems = ROW ? ROW : p.row;
+  const int rank = ROW ? kLat : p.rank;
+  const int slabs = ROW ? ROW / 64 : (p.row + 63) >> 6;
+  const int tile_bytes = slabs * kSlabBytes, q_bytes = slabs * 16 * 128;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
   uint8_t* sKV = smem;
-  uint8_t* sQ = sKV + kMlaStages * kTileBytes;
-  uint8_t* sP = sQ + kQBytes;                                  // [16][64] bf16, swizzled rows of 128 B
+  uint8_t* sQ = sKV + kMlaStages * tile_bytes;
+  uint8_t* sP = sQ + q_bytes;                                  // [16][64] bf16, swizzled rows of 128 B
   float* s_red = reinterpret_cast<float*>(sP + kPBytes);       // [2][4][16] max / sum exchange
   uint64_t* full_bar = reinterpret_cast<uint64_t*>(s_red + 128);
   uint64_t* empty_bar = full_bar + kMlaStages;
@@ -104,7 +113,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
   }
   {
     uint4* z = reinterpret_cast<uint4*>(sKV);
-    for (int i = tid; i < kMlaStages * kTileBytes / 16; i += 160) z[i] = make_uint4(0u, 0u, 0u, 0u);
+    for (int i = tid; i < kMlaStages * tile_bytes / 16; i += 160) z[i] = make_uint4(0u, 0u, 0u, 0u);
   }
   const int bt_first = sel ? 0 : (t_begin * kMlaBN) / p.block_size;
   const int bt_last = sel ? 0 : min(p.max_blocks, (min(kv_len, t_end * kMlaBN) + p.block_size - 1) / p.block_size);
@@ -131,30 +140,30 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
         }
         const int n0 = (t_begin + it) * kMlaBN;
         const int nvalid = min(kMlaBN, kv_len - n0);
-        uint8_t* dst_tile = sKV + stage * kTileBytes;
+        uint8_t* dst_tile = sKV + stage * tile_bytes;
         if (!sel) {
           const int nboxes = (nvalid + box_rows - 1) / box_rows;
-          mbar_arrive_expect_tx(&full_bar[stage], static_cast<uint32_t>(nboxes * box_rows * 128 * kSlabs));
+          mbar_arrive_expect_tx(&full_bar[stage], static_cast<uint32_t>(nboxes * box_rows * 128 * slabs));
           for (int j = 0; j < nboxes; ++j) {
             const int key = n0 + j * box_rows;
             const int bi = key / p.block_size;
             const int blk = bt_cached ? s_bt[bi - bt_first] : bt[bi];
             const int row = blk * p.block_size + key % p.block_size;
 #pragma unroll
-            for (int s = 0; s < kSlabs; ++s)
+            for (int s = 0; s < slabs; ++s)
               tma_load_2d(dst_tile + s * kSlabBytes + j * box_rows * 128, &tm_c, &full_bar[stage], s * 64, row);
           }
         } else {
           // sparse: one row per selected token (negative index = hole, left zero-scored)
           int nrows = 0;
           for (int j = 0; j < nvalid; ++j) nrows += sel[n0 + j] >= 0 ? 1 : 0;
-          mbar_arrive_expect_tx(&full_bar[stage], static_cast<uint32_t>(nrows * 128 * kSlabs));
+          mbar_arrive_expect_tx(&full_bar[stage], static_cast<uint32_t>(nrows * 128 * slabs));
           for (int j = 0; j < nvalid; ++j) {
             const int pos = sel[n0 + j];
             if (pos < 0) continue;
             const int row = bt[pos / p.block_size] * p.block_size + pos % p.block_size;
 #pragma unroll
-            for (int s = 0; s < kSlabs; ++s)
+            for (int s = 0; s < slabs; ++s)
               tma_load_2d(dst_tile + s * kSlabBytes + j * 128, &tm_c, &full_bar[stage], s * 64, row);
           }
         }
@@ -171,19 +180,20 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
   }
 
   // -------------------------------------------------------------- consumers
-  for (int idx = tid; idx < 16 * 72; idx += 128) {
-    const int row = idx / 72, c = idx % 72;
+  const int chunks = slabs * 8;
+  for (int idx = tid; idx < 16 * chunks; idx += 128) {
+    const int row = idx / chunks, c = idx % chunks;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (head0 + row < p.N)
+    if (head0 + row < p.N && c * 8 < row_elems)
       v = *reinterpret_cast<const uint4*>(p.q + static_cast<long long>(tok) * p.q_stride +
-                                          static_cast<long long>(head0 + row) * kRow + c * 8);
+                                          static_cast<long long>(head0 + row) * row_elems + c * 8);
     *reinterpret_cast<uint4*>(sQ + mla_off(row, c, 16)) = v;
   }
   asm volatile("bar.sync 1, 128;" ::: "memory");
 
-  float o_acc[16][4];
+  float o_acc[2 * CT][4];
 #pragma unroll
-  for (int i = 0; i < 16; ++i)
+  for (int i = 0; i < 2 * CT; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) o_acc[i][j] = 0.f;
   float row_max[2] = {-INFINITY, -INFINITY};
@@ -215,13 +225,13 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
           : "memory");
       if (!all_ok) break;
     }
-    const uint32_t kt = smem_u32(sKV + stage * kTileBytes);
+    const uint32_t kt = smem_u32(sKV + stage * tile_bytes);
     const int n0 = (t_begin + it) * kMlaBN;
 
     // ---- S = Q K^T for this warp's 16 keys
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll 4
-    for (int ks = 0; ks < kRow / 16; ++ks) {
+    for (int ks = 0; ks < (row_elems + 15) / 16; ++ks) {
       uint32_t qf[4], kf[4];
       ldmatrix_x4(qf, smem_u32(sQ) + mla_off(lane & 15, ks * 2 + (lane >> 4), 16));
       const int krow = warp * 16 + (lane & 7) + ((lane >> 4) << 3);
@@ -288,13 +298,13 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
       row_sum[r] = row_sum[r] * corr[r] + s_red[64 + row] + s_red[80 + row] + s_red[96 + row] + s_red[112 + row];
     }
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < 2 * CT; ++i) {
       o_acc[i][0] *= corr[0];
       o_acc[i][1] *= corr[0];
       o_acc[i][2] *= corr[1];
       o_acc[i][3] *= corr[1];
     }
-    // ---- O[:, 128w : 128w+128] += P V
+    // ---- O (this warp's columns) += P V
 #pragma unroll
     for (int ks = 0; ks < kMlaBN / 16; ++ks) {
       uint32_t pf[4];
@@ -304,10 +314,11 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
         ldmatrix_x4(pf, smem_u32(sP) + prow * 128 + ((pchunk ^ (prow & 7)) << 4));
       }
 #pragma unroll
-      for (int dt = 0; dt < 8; ++dt) {
+      for (int dt = 0; dt < CT; ++dt) {
+        if (!ROW && (warp * CT + dt) * 16 >= rank) continue;
         uint32_t vf[4];
         const int vrow = ks * 16 + (lane & 15);
-        const int vchunk = warp * 16 + dt * 2 + (lane >> 4);
+        const int vchunk = warp * 2 * CT + dt * 2 + (lane >> 4);
         ldmatrix_x4_trans(vf, kt + mla_off(vrow, vchunk, kMlaBN));
         mma_bf16_16816(o_acc[2 * dt], pf, vf[0], vf[1]);
         mma_bf16_16816(o_acc[2 * dt + 1], pf, vf[2], vf[3]);
@@ -321,7 +332,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
   __syncthreads();
   if (*abort_flag) return;
 
-  // ---- write: every thread owns rows r_a, r_a+8 and 32 columns of its warp's slice
+  // ---- write: every thread owns rows r_a, r_a+8 and two columns in eight of its warp's slice
   const size_t part_row = ((static_cast<size_t>(tok) * gridDim.y + blockIdx.y) * p.splits + split) * 16;
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
@@ -331,19 +342,25 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
     if (p.splits == 1) {
       const float inv = l > 0.f ? 1.f / l : 0.f;
       __nv_bfloat16* dst = p.out + static_cast<long long>(tok) * p.out_stride +
-                           static_cast<long long>(head0 + row) * kLat + warp * 128;
+                           static_cast<long long>(head0 + row) * rank;
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const int col = i * 8 + (lane & 3) * 2;
-        *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(o_acc[i][2 * r] * inv, o_acc[i][2 * r + 1] * inv);
+      for (int i = 0; i < 2 * CT; ++i) {
+        const int col = warp * 16 * CT + i * 8 + (lane & 3) * 2;
+        const float o0 = o_acc[i][2 * r] * inv, o1 = o_acc[i][2 * r + 1] * inv;
+        if (ROW || (col + 1 < rank && (rank & 1) == 0)) {
+          *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(o0, o1);
+        } else {
+          if (col < rank) dst[col] = __float2bfloat16(o0);
+          if (col + 1 < rank) dst[col + 1] = __float2bfloat16(o1);
+        }
       }
       if (p.lse && warp == 0 && (lane & 3) == 0)
         p.lse[static_cast<long long>(tok) * p.N + head0 + row] =
             l > 0.f ? (row_max[r] + log2f(l)) / kMlaLog2e : -INFINITY;
     } else {
-      float* dst = p.o_part + (part_row + row) * kLat + warp * 128;
+      float* dst = p.o_part + (part_row + row) * (64 * CT) + warp * 16 * CT;
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
+      for (int i = 0; i < 2 * CT; ++i) {
         const int col = i * 8 + (lane & 3) * 2;
         *reinterpret_cast<float2*>(dst + col) = make_float2(o_acc[i][2 * r], o_acc[i][2 * r + 1]);
       }
@@ -356,6 +373,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const MlaParams p, c
 }
 
 // one warp per (token, head): merge split partials
+template <int CT>
 __global__ void __launch_bounds__(128)
 mla_merge_kernel(const MlaParams p, int total_tokens, int head_tiles) {
   const long long gw = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
@@ -367,54 +385,82 @@ mla_merge_kernel(const MlaParams p, int total_tokens, int head_tiles) {
   float m = -INFINITY;
   for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.ml_part[(base + static_cast<size_t>(s) * 16) * 2]);
   float l = 0.f;
-  float acc[16];
+  float acc[2 * CT];
 #pragma unroll
-  for (int i = 0; i < 16; ++i) acc[i] = 0.f;
+  for (int i = 0; i < 2 * CT; ++i) acc[i] = 0.f;
   for (int s = 0; s < p.splits; ++s) {
     const size_t pr = base + static_cast<size_t>(s) * 16;
     const float ms = p.ml_part[pr * 2];
     const float f = ms == -INFINITY ? 0.f : exp2f(ms - m);
     l += p.ml_part[pr * 2 + 1] * f;
+    if (f == 0.f) continue;                  // (a split without keys has left its columns unwritten or zero)
 #pragma unroll
-    for (int i = 0; i < 16; ++i) acc[i] += p.o_part[pr * kLat + i * 32 + lane] * f;
+    for (int i = 0; i < 2 * CT; ++i) acc[i] += p.o_part[pr * (64 * CT) + i * 32 + lane] * f;
   }
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  __nv_bfloat16* dst = p.out + static_cast<long long>(tok) * p.out_stride + static_cast<long long>(head) * kLat;
+  __nv_bfloat16* dst = p.out + static_cast<long long>(tok) * p.out_stride + static_cast<long long>(head) * p.rank;
 #pragma unroll
-  for (int i = 0; i < 16; ++i) dst[i * 32 + lane] = __float2bfloat16(acc[i] * inv);
+  for (int i = 0; i < 2 * CT; ++i)
+    if (i * 32 + lane < p.rank) dst[i * 32 + lane] = __float2bfloat16(acc[i] * inv);
   if (p.lse && lane == 0)
     p.lse[static_cast<long long>(tok) * p.N + head] = l > 0.f ? (m + log2f(l)) / kMlaLog2e : -INFINITY;
+}
+
+
+static int mla_tiles_per_warp(int rank) { return rank <= 128 ? 2 : rank <= 256 ? 4 : 8; }
+
+template <int ROW, int CT>
+static int launch_mla(const MlaParams& p, const void* cache, int num_cache_blocks, int T, cudaStream_t stream) {
+  auto kern = mla_decode_kernel<ROW, CT>;
+  const int slabs = (p.row + 63) / 64, smem = mla_smem(slabs);
+  static DeviceOnce once;
+  int cur_dev = 0;
+  if (once.needed(&cur_dev)) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, mla_smem(ROW ? ROW / 64 : 10)) !=
+        cudaSuccess)
+      return -20;
+    once.mark(cur_dev);
+  }
+  const int tiles = (p.N + 15) / 16;
+  const int box_rows = p.topk_indices ? 1 : (p.block_size < 64 ? p.block_size : 64);
+  CUtensorMap tm;
+  const uint64_t rows = num_cache_blocks > 0 ? static_cast<uint64_t>(num_cache_blocks) * p.block_size : (1ull << 31);
+  int r = make_tensormap_2d(&tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cache, rows, p.row, p.row, box_rows, 64,
+                            CU_TENSOR_MAP_SWIZZLE_128B);
+  if (r) return r - 2000;
+  kern<<<dim3(T, tiles, p.splits), 160, smem, stream>>>(tm, p, box_rows);
+  if (cudaGetLastError() != cudaSuccess) return -21;
+  if (p.splits > 1) {
+    const long long warps = static_cast<long long>(T) * p.N;
+    mla_merge_kernel<CT><<<static_cast<unsigned>((warps + 3) / 4), 128, 0, stream>>>(p, T, tiles);
+    if (cudaGetLastError() != cudaSuccess) return -22;
+  }
+  return 0;
 }
 
 }  // namespace b200
 
 using namespace b200;
 
-extern "C" size_t b200_mla_decode_scratch_bytes(int total_tokens, int N, int splits) {
+extern "C" size_t b200_latent_decode_scratch_bytes(int total_tokens, int N, int rank, int splits) {
   if (splits <= 1) return 0;
   const size_t tiles = (N + 15) / 16;
-  return static_cast<size_t>(total_tokens) * tiles * splits * 16 * (kLat + 2) * sizeof(float);
+  return static_cast<size_t>(total_tokens) * tiles * splits * 16 * (64 * mla_tiles_per_warp(rank) + 2) * sizeof(float);
 }
 
-// q [T, N*576]; cache [num_blocks, block_size, 576]; out [T, N*512].  T = B * q_len.
-// topk_indices (optional) [T, topk]: attend only to these token positions.
-extern "C" int b200_mla_decode(const void* q, const void* cache, void* out, float* lse,
-                               const int* block_tables, const int* seq_lens, const int* topk_indices,
-                               int topk, int B, int q_len, int N, int max_blocks, int block_size,
-                               int num_cache_blocks, long long q_stride, long long out_stride,
-                               float scale, int splits, void* scratch, int* status,
-                               cudaStream_t stream) {
+extern "C" size_t b200_mla_decode_scratch_bytes(int total_tokens, int N, int splits) {
+  return b200_latent_decode_scratch_bytes(total_tokens, N, kLat, splits);
+}
+
+static int mla_decode_any(const void* q, const void* cache, void* out, float* lse, const int* block_tables,
+                          const int* seq_lens, const int* topk_indices, int topk, int B, int q_len, int N, int row,
+                          int rank, int max_blocks, int block_size, int num_cache_blocks, long long q_stride,
+                          long long out_stride, float scale, int splits, void* scratch, int* status,
+                          cudaStream_t stream) {
   if (B <= 0) return 0;
   if (splits < 1) splits = 1;
   if (splits > 1 && scratch == nullptr) return -3;
   if ((block_size % 8) != 0 || !(block_size <= 64 ? (64 % block_size) == 0 : (block_size % 64) == 0)) return -4;
-  static DeviceOnce once;
-  int cur_dev = 0;
-  if (once.needed(&cur_dev)) {
-    if (cudaFuncSetAttribute(mla_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMlaSmem) != cudaSuccess)
-      return -20;
-    once.mark(cur_dev);
-  }
   MlaParams p{};
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.out = static_cast<__nv_bfloat16*>(out);
@@ -431,26 +477,43 @@ extern "C" int b200_mla_decode(const void* q, const void* cache, void* out, floa
   p.out_stride = out_stride;
   p.scale_log2 = scale * kMlaLog2e;
   p.splits = splits;
+  p.row = row;
+  p.rank = rank;
   p.status = status;
   const int T = B * q_len;
-  const int tiles = (N + 15) / 16;
   if (splits > 1) {
     p.o_part = static_cast<float*>(scratch);
-    p.ml_part = p.o_part + static_cast<size_t>(T) * tiles * splits * 16 * kLat;
+    p.ml_part = p.o_part + static_cast<size_t>(T) * ((N + 15) / 16) * splits * 16 * 64 * mla_tiles_per_warp(rank);
   }
-  const int box_rows = topk_indices ? 1 : (block_size < 64 ? block_size : 64);
-  CUtensorMap tm;
-  const uint64_t rows = num_cache_blocks > 0 ? static_cast<uint64_t>(num_cache_blocks) * block_size : (1ull << 31);
-  int r = make_tensormap_2d(&tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cache, rows, kRow, kRow, box_rows, 64,
-                            CU_TENSOR_MAP_SWIZZLE_128B);
-  if (r) return r - 2000;
-  dim3 grid(T, tiles, splits);
-  mla_decode_kernel<<<grid, 160, kMlaSmem, stream>>>(tm, p, box_rows);
-  if (cudaGetLastError() != cudaSuccess) return -21;
-  if (splits > 1) {
-    const long long warps = static_cast<long long>(T) * N;
-    mla_merge_kernel<<<static_cast<unsigned>((warps + 3) / 4), 128, 0, stream>>>(p, T, tiles);
-    if (cudaGetLastError() != cudaSuccess) return -22;
+  if (row == kRow && rank == kLat) return launch_mla<kRow, 8>(p, cache, num_cache_blocks, T, stream);
+  switch (mla_tiles_per_warp(rank)) {
+    case 2: return launch_mla<0, 2>(p, cache, num_cache_blocks, T, stream);
+    case 4: return launch_mla<0, 4>(p, cache, num_cache_blocks, T, stream);
+    default: return launch_mla<0, 8>(p, cache, num_cache_blocks, T, stream);
   }
-  return 0;
+}
+
+// q [T, N*576]; cache [num_blocks, block_size, 576]; out [T, N*512].  T = B * q_len.
+// topk_indices (optional) [T, topk]: attend only to these token positions.
+extern "C" int b200_mla_decode(const void* q, const void* cache, void* out, float* lse,
+                               const int* block_tables, const int* seq_lens, const int* topk_indices,
+                               int topk, int B, int q_len, int N, int max_blocks, int block_size,
+                               int num_cache_blocks, long long q_stride, long long out_stride,
+                               float scale, int splits, void* scratch, int* status,
+                               cudaStream_t stream) {
+  return mla_decode_any(q, cache, out, lse, block_tables, seq_lens, topk_indices, topk, B, q_len, N, kRow, kLat,
+                        max_blocks, block_size, num_cache_blocks, q_stride, out_stride, scale, splits, scratch, status,
+                        stream);
+}
+
+// Single new tokens, rows of any size: q [B, N*row]; cache [num_blocks, block_size, row], row a multiple of
+// 8 and at most 640, rank at most 512; out [B, N*rank].
+extern "C" int b200_latent_decode(const void* q, const void* cache, void* out, const int* block_tables,
+                                  const int* seq_lens, int B, int N, int row, int rank, int max_blocks, int block_size,
+                                  int num_cache_blocks, float scale, int splits, void* scratch, int* status,
+                                  cudaStream_t stream) {
+  if ((row & 7) || row > 640 || rank > 512 || rank > row) return -5;
+  return mla_decode_any(q, cache, out, nullptr, block_tables, seq_lens, nullptr, 0, B, 1, N, row, rank, max_blocks,
+                        block_size, num_cache_blocks, static_cast<long long>(N) * row, static_cast<long long>(N) * rank,
+                        scale, splits, scratch, status, stream);
 }

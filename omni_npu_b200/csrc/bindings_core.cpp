@@ -48,14 +48,47 @@ int b200_gated_attention(const void* q, const void* gate, const void* k_cache, c
                          int q_len, int max_q_len, int max_blocks, int block_size, int num_cache_blocks, int Hq,
                          int Hk, int D, int DV, int DP, int DVP, long long q_stride, long long g_stride,
                          long long out_stride, float scale, int window, int has_sink, float sink, int splits,
-                         int is_fp32, int variant, int* status, cudaStream_t stream);
+                         int is_fp32, int variant, int* status, int contiguous, cudaStream_t stream);
+int b200_hyper_norm(const float* streams, float* streams_out, const int* ids, const void* table, int table_rows,
+                    const void* y, long long y_stride, const void* ls, const float* mix, const float* w_out,
+                    const float* w_in, const void* norm_w, const void* norm_b, float eps, float out_scale,
+                    const void* mu, float* state, const int* seq_idx, const int* state_slots, const int* cu_q,
+                    const int* seq_lens, void* out, int T, int N, int W, int n_true, int is_fp32, cudaStream_t stream);
+int b200_gated_linear_prep(const void* proj, long long stride, int q_off, int f_off, int heads, int dim,
+                           const float* f_bias, const float* lower, float* q, float* k, int T, int is_fp32,
+                           cudaStream_t stream);
+int b200_delta_prep(const void* proj, long long stride, const void* low, long long low_stride, int q_off, int k_off,
+                    int v_off, int b_off, int heads, int groups, int dim, int vdim, int taps, int channels,
+                    const void* conv_w, const void* conv_state, const float* dt_bias, const float* a_log,
+                    float unit_eps, float q_scale, const int* seq_idx, const int* state_slots, const int* cu_q,
+                    const int* seq_lens, float* q, float* k, float* g, void* v, float* beta, int T, int is_fp32,
+                    cudaStream_t stream);
+int b200_recurrent_scan(const float* q, const float* k, const float* g, const void* v, long long v_stride,
+                        const float* beta, float* state, float* o, const int* state_slots, const int* cu_q,
+                        const int* seq_lens, int B, int H, int G, int E, int DP, const void* proj,
+                        long long proj_stride, void* conv_state, int keep, int channels, int is_fp32,
+                        cudaStream_t stream);
+int b200_head_norm_gate(const float* o, const void* w, const void* gate, long long gate_stride, void* out,
+                        int out_width, int T, int H, int E, float eps, int is_fp32, cudaStream_t stream);
+int b200_latent_prep(void* q, long long q_stride, const void* kv, long long kv_stride, const void* norm_w, float eps,
+                     void* cache, const int* positions, const int* slots, const float* cos_sin, int max_pos, int T,
+                     int H, int dim, int rot, int rank, int row, int neox, void* q_latent, int num_latent, int is_fp32,
+                     cudaStream_t stream);
+int b200_head_gemm(const void* a, long long a_t, long long a_h, const void* w, void* out, long long o_t, long long o_h,
+                   int T, int H, int N, int K, int is_fp32, cudaStream_t stream);
+int b200_latent_gather(const void* cache, void* out, const int* block_tables, const int* seq_lens, const int* start,
+                       int B, int max_len, int max_blocks, int block_size, int row_bytes, int total,
+                       cudaStream_t stream);
+size_t b200_latent_decode_scratch_bytes(int total_tokens, int N, int rank, int splits);
+int b200_latent_decode(const void* q, const void* cache, void* out, const int* block_tables, const int* seq_lens, int B,
+                       int N, int row, int rank, int max_blocks, int block_size, int num_cache_blocks, float scale,
+                       int splits, void* scratch, int* status, cudaStream_t stream);
 }
 
 namespace {
 
-// Gated activation of the GEMM epilogues (gemm/gated_act.cuh): none, silu(gate) * up, or the clamped
-// form when a slope is given.
-inline int act_kind(bool gated, double act_alpha) { return gated ? (act_alpha != 0.0 ? 2 : 1) : 0; }
+// Activation kinds of the GEMM epilogues are those of gemm/gated_act.cuh; 1 and 2 join pairs of columns.
+inline bool gated(int64_t act) { return act == 1 || act == 2; }
 
 // (BN, splits, workspace bytes, counters, cluster flag) for a problem.
 std::tuple<int64_t, int64_t, int64_t, int64_t, int64_t> gemm_plan(int64_t M, int64_t N, int64_t K,
@@ -71,7 +104,7 @@ std::tuple<int64_t, int64_t, int64_t, int64_t, int64_t> gemm_plan(int64_t M, int
 
 // C = A @ W^T (+bias) (+residual).  A [M,K], W [N,K]; bf16 or float8_e4m3fn.
 Tensor gemm(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& bias,
-            const c10::optional<Tensor>& residual, bool out_fp32, bool swiglu, int64_t bn,
+            const c10::optional<Tensor>& residual, bool out_fp32, int64_t act, int64_t bn,
             int64_t splits, bool cluster_split, const c10::optional<Tensor>& workspace,
             const c10::optional<Tensor>& counters, const Tensor& status, int64_t max_ctas, double act_alpha,
             double act_limit) {
@@ -83,7 +116,7 @@ Tensor gemm(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& bias,
   const int M = a.size(0), K = a.size(1), N = w.size(0);
   TORCH_CHECK(w.size(1) == K, "gemm: K mismatch");
   c10::cuda::CUDAGuard guard(a.device());
-  const int n_out = swiglu ? N / 2 : N;
+  const int n_out = gated(act) ? N / 2 : N;
   Tensor c = torch::empty({M, n_out}, a.options().dtype(out_fp32 ? at::kFloat : at::kBFloat16));
   const void* bias_p = nullptr;
   const void* res_p = nullptr;
@@ -107,7 +140,7 @@ Tensor gemm(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& bias,
   }
   check(b200_gemm(a.data_ptr(), w.data_ptr(), c.data_ptr(), bias_p, res_p, M, N, K,
                   (int)a.stride(0), (int)w.stride(0), n_out, fp8 ? 1 : 0, out_fp32 ? 1 : 0,
-                  act_kind(swiglu, act_alpha), (int)bn, (int)splits, cluster_split ? 1 : 0, ws_p, cnt_p,
+                  (int)act, (int)bn, (int)splits, cluster_split ? 1 : 0, ws_p, cnt_p,
                   status.data_ptr<int>(), (int)max_ctas, (float)act_alpha, (float)act_limit, cur_stream()),
         "gemm");
   return c;
@@ -116,7 +149,7 @@ Tensor gemm(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& bias,
 // Same contract as gemm() without split-K, run by CTA pairs: one 256 x BN tile per pair of SMs
 // (tcgen05 cta_group::2), each SM staging half of the weight tile.
 Tensor gemm_pair(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& bias,
-                 const c10::optional<Tensor>& residual, bool out_fp32, bool swiglu, int64_t bn,
+                 const c10::optional<Tensor>& residual, bool out_fp32, int64_t act, int64_t bn,
                  const Tensor& status, int64_t max_ctas, double act_alpha, double act_limit) {
   TORCH_CHECK(a.is_cuda() && w.is_cuda() && a.dim() == 2 && w.dim() == 2, "gemm_pair: 2-D CUDA tensors");
   TORCH_CHECK(a.scalar_type() == w.scalar_type(), "gemm_pair: dtype mismatch");
@@ -126,7 +159,7 @@ Tensor gemm_pair(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& 
   const int M = a.size(0), K = a.size(1), N = w.size(0);
   TORCH_CHECK(w.size(1) == K, "gemm_pair: K mismatch");
   c10::cuda::CUDAGuard guard(a.device());
-  const int n_out = swiglu ? N / 2 : N;
+  const int n_out = gated(act) ? N / 2 : N;
   Tensor c = torch::empty({M, n_out}, a.options().dtype(out_fp32 ? at::kFloat : at::kBFloat16));
   const void* bias_p = nullptr;
   const void* res_p = nullptr;
@@ -143,13 +176,13 @@ Tensor gemm_pair(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& 
   }
   check(b200_gemm_pair(a.data_ptr(), w.data_ptr(), c.data_ptr(), bias_p, res_p, M, N, K,
                        (int)a.stride(0), (int)w.stride(0), n_out, fp8 ? 1 : 0, out_fp32 ? 1 : 0,
-                       act_kind(swiglu, act_alpha), (int)bn, status.data_ptr<int>(), (int)max_ctas,
+                       (int)act, (int)bn, status.data_ptr<int>(), (int)max_ctas,
                        (float)act_alpha, (float)act_limit, cur_stream()),
         "gemm_pair");
   return c;
 }
 
-Tensor grouped_gemm(const Tensor& a, const Tensor& w, const Tensor& expert_offsets, bool swiglu,
+Tensor grouped_gemm(const Tensor& a, const Tensor& w, const Tensor& expert_offsets, int64_t act,
                     int64_t bn, const Tensor& status, int64_t max_ctas, double act_alpha, double act_limit) {
   TORCH_CHECK(a.is_cuda() && w.is_cuda() && a.dim() == 2 && w.dim() == 3, "grouped_gemm: shapes");
   TORCH_CHECK(a.scalar_type() == w.scalar_type(), "grouped_gemm: dtype mismatch");
@@ -160,10 +193,10 @@ Tensor grouped_gemm(const Tensor& a, const Tensor& w, const Tensor& expert_offse
   const int E = w.size(0), N = w.size(1), K = w.size(2), rows = a.size(0);
   TORCH_CHECK(a.size(1) == K && expert_offsets.numel() == E + 1, "grouped_gemm: size mismatch");
   c10::cuda::CUDAGuard guard(a.device());
-  const int n_out = swiglu ? N / 2 : N;
+  const int n_out = gated(act) ? N / 2 : N;
   Tensor c = torch::empty({rows, n_out}, a.options().dtype(at::kBFloat16));
   check(b200_grouped_gemm(a.data_ptr(), w.data_ptr(), c.data_ptr(), expert_offsets.data_ptr<int>(),
-                          E, rows, N, K, (int)a.stride(0), n_out, fp8 ? 1 : 0, act_kind(swiglu, act_alpha), (int)bn,
+                          E, rows, N, K, (int)a.stride(0), n_out, fp8 ? 1 : 0, (int)act, (int)bn,
                           status.data_ptr<int>(), (int)max_ctas, (float)act_alpha, (float)act_limit, cur_stream()),
         "grouped_gemm");
   return c;
@@ -234,7 +267,7 @@ inline bool is_f32(const Tensor& t) {
   TORCH_CHECK((t).is_cuda() && (t).scalar_type() == (dt) && (t).dim() == 2 && (t).stride(1) == 1, #t ": 2-D rows of the call's type")
 
 // fp32 A [M,K] @ W [N,K]^T; with expert_offsets W is [E,N,K] and rows belong to experts in order.
-Tensor gemm_simt(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& expert_offsets, bool swiglu,
+Tensor gemm_simt(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& expert_offsets, int64_t act,
                  double act_alpha, double act_limit) {
   CHECK_ROWS(a, at::kFloat);
   TORCH_CHECK(w.is_cuda() && w.scalar_type() == at::kFloat && w.is_contiguous(), "gemm_simt: fp32 weights");
@@ -247,10 +280,10 @@ Tensor gemm_simt(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& 
   }
   const int M = a.size(0), N = w.size(-2), K = a.size(1);
   c10::cuda::CUDAGuard guard(a.device());
-  const int n_out = swiglu ? N / 2 : N;
+  const int n_out = gated(act) ? N / 2 : N;
   Tensor c = torch::empty({M, n_out}, a.options());
   check(b200_gemm_simt(a.data_ptr<float>(), w.data_ptr<float>(), c.data_ptr<float>(), M, N, K, a.stride(0), K, n_out,
-                       grouped ? expert_offsets->data_ptr<int>() : nullptr, E, act_kind(swiglu, act_alpha),
+                       grouped ? expert_offsets->data_ptr<int>() : nullptr, E, (int)act,
                        (float)act_alpha, (float)act_limit, cur_stream()),
         "gemm_simt");
   return c;
@@ -366,7 +399,7 @@ void gated_attention(const Tensor& q, const c10::optional<Tensor>& gate, const T
                      Tensor out, const Tensor& block_tables, const c10::optional<Tensor>& cu_q,
                      const Tensor& seq_lens, int64_t num_seqs, int64_t q_len, int64_t max_q_len, int64_t num_q_heads,
                      int64_t head_dim, int64_t head_dim_v, double scale, int64_t window, bool has_sink, double sink,
-                     int64_t splits, int64_t variant, const Tensor& status) {
+                     int64_t splits, int64_t variant, const Tensor& status, bool contiguous) {
   const auto dt = q.scalar_type();
   const bool f32 = is_f32(q);
   CHECK_ROWS(q, dt);
@@ -402,8 +435,313 @@ void gated_attention(const Tensor& q, const c10::optional<Tensor>& gate, const T
                              (int)k_cache.size(0), (int)num_q_heads, (int)k_cache.size(1), (int)head_dim,
                              (int)head_dim_v, (int)k_cache.size(3), (int)v_cache.size(3), q.stride(0), gs,
                              out.stride(0), (float)scale, (int)window, has_sink ? 1 : 0, (float)sink, (int)splits,
-                             f32 ? 1 : 0, (int)variant, status.data_ptr<int>(), cur_stream()),
+                             f32 ? 1 : 0, (int)variant, status.data_ptr<int>(), contiguous ? 1 : 0, cur_stream()),
         "gated_attention");
+}
+
+#define CHECK_F32(t) TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kFloat && (t).is_contiguous(), #t ": contiguous fp32")
+#define CHECK_VEC(t, dt, n) \
+  TORCH_CHECK((t).is_cuda() && (t).scalar_type() == (dt) && (t).is_contiguous() && (t).numel() == (n), #t ": vector of the call's type and width")
+
+// Joins y to the streams (or starts them from the table), reads and normalises: (streams, rows).
+std::tuple<Tensor, Tensor> hyper_norm(const c10::optional<Tensor>& streams, const c10::optional<Tensor>& ids,
+                                      const c10::optional<Tensor>& table, int64_t N, const c10::optional<Tensor>& y,
+                                      const c10::optional<Tensor>& ls, const c10::optional<Tensor>& mix,
+                                      const c10::optional<Tensor>& w_out, const Tensor& w_in, const Tensor& norm_w,
+                                      const Tensor& norm_b, double eps, int64_t n_true, double out_scale,
+                                      const c10::optional<Tensor>& mu, const c10::optional<Tensor>& state,
+                                      const c10::optional<Tensor>& seq_idx, const c10::optional<Tensor>& state_slots,
+                                      const c10::optional<Tensor>& cu_q, const c10::optional<Tensor>& seq_lens,
+                                      bool keep) {
+  const auto dt = norm_w.scalar_type();
+  const bool f32 = is_f32(norm_w);
+  const int64_t W = norm_w.numel();
+  CHECK_VEC(norm_w, dt, W);
+  CHECK_VEC(norm_b, dt, W);
+  CHECK_F32(w_in);
+  TORCH_CHECK(w_in.numel() == N && N >= 1 && N <= 8, "hyper_norm: 1 to 8 streams");
+  c10::cuda::CUDAGuard guard(norm_w.device());
+  int64_t T;
+  const float *x = nullptr, *mix_p = nullptr, *out_p = nullptr;
+  const int* ids_p = nullptr;
+  const void *table_p = nullptr, *y_p = nullptr, *ls_p = nullptr;
+  int table_rows = 0;
+  long long ys = 0;
+  if (ids.has_value()) {
+    CHECK_I32(*ids);
+    TORCH_CHECK(table.has_value() && table->is_cuda() && table->scalar_type() == dt && table->is_contiguous() &&
+                    table->dim() == 2 && table->size(1) == W && table->size(0) > 0, "hyper_norm: table [rows, W]");
+    T = ids->numel();
+    ids_p = ids->data_ptr<int>();
+    table_p = table->data_ptr();
+    table_rows = (int)table->size(0);
+  } else {
+    TORCH_CHECK(streams.has_value() && y.has_value() && ls.has_value() && mix.has_value() && w_out.has_value(),
+                "hyper_norm: streams with a sublayer's result");
+    CHECK_F32(*streams);
+    CHECK_F32(*mix);
+    CHECK_F32(*w_out);
+    CHECK_ROWS(*y, dt);
+    CHECK_VEC(*ls, dt, W);
+    T = streams->size(0);
+    TORCH_CHECK(streams->dim() == 3 && streams->size(1) == N && streams->size(2) == W && y->size(0) == T &&
+                    y->size(1) == W && mix->numel() == N * N && w_out->numel() == N, "hyper_norm: shapes");
+    x = streams->data_ptr<float>();
+    y_p = y->data_ptr();
+    ys = y->stride(0);
+    ls_p = ls->data_ptr();
+    mix_p = mix->data_ptr<float>();
+    out_p = w_out->data_ptr<float>();
+  }
+  const void* mu_p = nullptr;
+  float* st = nullptr;
+  const int *si = nullptr, *ss = nullptr, *cu = nullptr, *sl = nullptr;
+  if (mu.has_value()) {
+    TORCH_CHECK(state.has_value() && seq_idx.has_value() && state_slots.has_value() && cu_q.has_value() &&
+                    seq_lens.has_value(), "hyper_norm: token shift arguments");
+    CHECK_VEC(*mu, dt, W);
+    CHECK_F32(*state);
+    CHECK_I32(*seq_idx);
+    CHECK_I32(*state_slots);
+    CHECK_I32(*cu_q);
+    CHECK_I32(*seq_lens);
+    TORCH_CHECK(state->dim() == 2 && state->size(1) == W && seq_idx->numel() >= T, "hyper_norm: state [slots, W]");
+    mu_p = mu->data_ptr();
+    st = state->data_ptr<float>();
+    si = seq_idx->data_ptr<int>();
+    ss = state_slots->data_ptr<int>();
+    cu = cu_q->data_ptr<int>();
+    sl = seq_lens->data_ptr<int>();
+  }
+  Tensor out = torch::empty({T, W}, norm_w.options());
+  Tensor next = torch::empty(keep ? std::vector<int64_t>{T, N, W} : std::vector<int64_t>{0}, w_in.options());
+  check(b200_hyper_norm(x, keep ? next.data_ptr<float>() : nullptr, ids_p, table_p, table_rows, y_p, ys, ls_p, mix_p,
+                        out_p, w_in.data_ptr<float>(), norm_w.data_ptr(), norm_b.data_ptr(), (float)eps,
+                        (float)out_scale, mu_p, st, si, ss, cu, sl, out.data_ptr(), (int)T, (int)N, (int)W, (int)n_true,
+                        f32 ? 1 : 0, cur_stream()),
+        "hyper_norm");
+  return {next, out};
+}
+
+std::tuple<Tensor, Tensor> gated_linear_prep(const Tensor& proj, int64_t q_off, int64_t f_off, int64_t heads,
+                                             int64_t dim, const Tensor& f_bias, const Tensor& lower) {
+  const bool f32 = is_f32(proj);
+  CHECK_ROWS(proj, proj.scalar_type());
+  CHECK_F32(f_bias);
+  CHECK_F32(lower);
+  const int64_t T = proj.size(0), n = heads * dim;
+  TORCH_CHECK(f_bias.numel() == n && lower.numel() == n && q_off >= 0 && f_off >= 0 && q_off + n <= proj.size(1) &&
+                  f_off + n <= proj.size(1), "gated_linear_prep: shapes");
+  c10::cuda::CUDAGuard guard(proj.device());
+  Tensor q = torch::empty({T, heads, (dim + 3) / 4 * 4}, f_bias.options()), k = torch::empty_like(q);
+  check(b200_gated_linear_prep(proj.data_ptr(), proj.stride(0), (int)q_off, (int)f_off, (int)heads, (int)dim,
+                               f_bias.data_ptr<float>(), lower.data_ptr<float>(), q.data_ptr<float>(),
+                               k.data_ptr<float>(), (int)T, f32 ? 1 : 0, cur_stream()),
+        "gated_linear_prep");
+  return {q, k};
+}
+
+std::tuple<Tensor, Tensor, Tensor, Tensor, Tensor> delta_prep(
+    const Tensor& proj, const Tensor& low, int64_t q_off, int64_t k_off, int64_t v_off, int64_t b_off, int64_t heads,
+    int64_t groups, int64_t dim, int64_t vdim, const Tensor& conv_w, const Tensor& conv_state, const Tensor& dt_bias,
+    const Tensor& a_log, double unit_eps, const Tensor& seq_idx, const Tensor& state_slots, const Tensor& cu_q,
+    const Tensor& seq_lens) {
+  const auto dt = proj.scalar_type();
+  const bool f32 = is_f32(proj);
+  CHECK_ROWS(proj, dt);
+  CHECK_ROWS(low, dt);
+  CHECK_F32(dt_bias);
+  CHECK_F32(a_log);
+  CHECK_I32(seq_idx);
+  CHECK_I32(state_slots);
+  CHECK_I32(cu_q);
+  CHECK_I32(seq_lens);
+  const int64_t T = proj.size(0), channels = conv_w.size(0), taps = conv_w.size(1);
+  TORCH_CHECK(conv_w.is_cuda() && conv_w.scalar_type() == dt && conv_w.is_contiguous() && conv_state.is_cuda() &&
+                  conv_state.scalar_type() == dt && conv_state.is_contiguous() && conv_state.dim() == 3 &&
+                  conv_state.size(1) == taps - 1 && conv_state.size(2) == channels, "delta_prep: convolution");
+  TORCH_CHECK(low.size(0) == T && low.size(1) == heads * dim && dt_bias.numel() == heads * dim &&
+                  a_log.numel() == heads && seq_idx.numel() >= T && b_off + heads <= proj.size(1) &&
+                  channels <= proj.size(1) && q_off + groups * dim <= channels && k_off + groups * dim <= channels &&
+                  v_off + heads * vdim <= channels && heads % groups == 0, "delta_prep: shapes");
+  c10::cuda::CUDAGuard guard(proj.device());
+  const int64_t DP = (dim + 3) / 4 * 4;
+  Tensor q = torch::empty({T, groups, DP}, dt_bias.options()), k = torch::empty_like(q);
+  Tensor g = torch::empty({T, heads, DP}, dt_bias.options()), beta = torch::empty({T, heads}, dt_bias.options());
+  Tensor v = torch::empty({T, heads * vdim}, proj.options());
+  check(b200_delta_prep(proj.data_ptr(), proj.stride(0), low.data_ptr(), low.stride(0), (int)q_off, (int)k_off,
+                        (int)v_off, (int)b_off, (int)heads, (int)groups, (int)dim, (int)vdim, (int)taps, (int)channels,
+                        conv_w.data_ptr(), conv_state.data_ptr(), dt_bias.data_ptr<float>(), a_log.data_ptr<float>(),
+                        (float)unit_eps, 1.f / sqrtf((float)dim), seq_idx.data_ptr<int>(), state_slots.data_ptr<int>(),
+                        cu_q.data_ptr<int>(), seq_lens.data_ptr<int>(), q.data_ptr<float>(), k.data_ptr<float>(),
+                        g.data_ptr<float>(), v.data_ptr(), beta.data_ptr<float>(), (int)T, f32 ? 1 : 0, cur_stream()),
+        "delta_prep");
+  return {q, k, g, v, beta};
+}
+
+Tensor recurrent_scan(const Tensor& q, const Tensor& k, const c10::optional<Tensor>& g, const Tensor& v,
+                      const c10::optional<Tensor>& beta, Tensor state, int64_t heads, int64_t vdim,
+                      const Tensor& state_slots, const Tensor& cu_q, const Tensor& seq_lens, int64_t num_seqs,
+                      const c10::optional<Tensor>& proj, const c10::optional<Tensor>& conv_state) {
+  CHECK_F32(q);
+  CHECK_F32(k);
+  CHECK_F32(state);
+  CHECK_ROWS(v, v.scalar_type());
+  CHECK_I32(state_slots);
+  CHECK_I32(cu_q);
+  CHECK_I32(seq_lens);
+  const bool f32 = is_f32(v);
+  TORCH_CHECK(q.dim() == 3 && q.sizes() == k.sizes(), "recurrent_scan: q, k [T, G, d]");
+  const int64_t T = q.size(0), G = q.size(1), DP = q.size(2);
+  TORCH_CHECK(v.size(0) == T && v.size(1) == heads * vdim && state.dim() == 4 && state.size(1) == heads &&
+                  state.size(2) == vdim && state.size(3) == DP && heads % G == 0 && state_slots.numel() >= num_seqs &&
+                  cu_q.numel() >= num_seqs + 1 && seq_lens.numel() >= num_seqs, "recurrent_scan: shapes");
+  TORCH_CHECK(g.has_value() == beta.has_value(), "recurrent_scan: decays and step sizes come together");
+  if (g.has_value()) {
+    CHECK_F32(*g);
+    CHECK_F32(*beta);
+    TORCH_CHECK(g->numel() == T * heads * DP && beta->numel() == T * heads, "recurrent_scan: g [T, H, d], beta [T, H]");
+  }
+  const void* proj_p = nullptr;
+  void* cs = nullptr;
+  long long ps = 0;
+  int keep = 0, channels = 0;
+  if (proj.has_value() && conv_state.has_value()) {
+    CHECK_ROWS(*proj, v.scalar_type());
+    TORCH_CHECK(conv_state->is_cuda() && conv_state->scalar_type() == v.scalar_type() && conv_state->is_contiguous() &&
+                    conv_state->dim() == 3 && conv_state->size(0) == state.size(0) &&
+                    conv_state->size(2) <= proj->size(1) && proj->size(0) == T, "recurrent_scan: convolution inputs");
+    proj_p = proj->data_ptr();
+    ps = proj->stride(0);
+    cs = conv_state->data_ptr();
+    keep = (int)conv_state->size(1);
+    channels = (int)conv_state->size(2);
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor o = torch::empty({T, heads, vdim}, q.options());
+  check(b200_recurrent_scan(q.data_ptr<float>(), k.data_ptr<float>(), g.has_value() ? g->data_ptr<float>() : nullptr,
+                            v.data_ptr(), v.stride(0), beta.has_value() ? beta->data_ptr<float>() : nullptr,
+                            state.data_ptr<float>(), o.data_ptr<float>(), state_slots.data_ptr<int>(),
+                            cu_q.data_ptr<int>(), seq_lens.data_ptr<int>(), (int)num_seqs, (int)heads, (int)G,
+                            (int)vdim, (int)DP, proj_p, ps, cs, keep, channels, f32 ? 1 : 0, cur_stream()),
+        "recurrent_scan");
+  return o;
+}
+
+Tensor head_norm_gate(const Tensor& o, const Tensor& weight, double eps, const c10::optional<Tensor>& gate,
+                      int64_t out_width) {
+  CHECK_F32(o);
+  const auto dt = weight.scalar_type();
+  const bool f32 = is_f32(weight);
+  TORCH_CHECK(o.dim() == 3 && out_width >= o.size(1) * o.size(2), "head_norm_gate: o [T, H, E]");
+  CHECK_VEC(weight, dt, o.size(2));
+  const void* gp = nullptr;
+  long long gs = 0;
+  if (gate.has_value()) {
+    CHECK_ROWS(*gate, dt);
+    TORCH_CHECK(gate->size(0) == o.size(0) && gate->size(1) == o.size(1) * o.size(2), "head_norm_gate: gate");
+    gp = gate->data_ptr();
+    gs = gate->stride(0);
+  }
+  c10::cuda::CUDAGuard guard(o.device());
+  Tensor out = torch::empty({o.size(0), out_width}, weight.options());
+  check(b200_head_norm_gate(o.data_ptr<float>(), weight.data_ptr(), gp, gs, out.data_ptr(), (int)out_width,
+                            (int)o.size(0), (int)o.size(1), (int)o.size(2), (float)eps, f32 ? 1 : 0, cur_stream()),
+        "head_norm_gate");
+  return out;
+}
+
+void latent_prep(Tensor q, const Tensor& kv, const Tensor& norm_w, double eps, Tensor cache, const Tensor& positions,
+                 const Tensor& slots, const Tensor& cos_sin, int64_t heads, int64_t dim, int64_t rot, int64_t rank,
+                 bool neox, const c10::optional<Tensor>& q_latent, int64_t num_latent) {
+  const auto dt = q.scalar_type();
+  const bool f32 = is_f32(q);
+  CHECK_ROWS(q, dt);
+  CHECK_ROWS(kv, dt);
+  CHECK_VEC(norm_w, dt, rank);
+  CHECK_I32(positions);
+  CHECK_I32(slots);
+  const int64_t T = q.size(0);
+  TORCH_CHECK(cache.is_cuda() && cache.scalar_type() == dt && cache.is_contiguous() && cache.dim() == 3,
+              "latent_prep: cache [blocks, block_size, row]");
+  TORCH_CHECK(q.size(1) >= heads * (dim + rot) && kv.size(0) == T && kv.size(1) >= rank + rot &&
+                  cache.size(2) >= rank + rot && positions.numel() >= T && slots.numel() >= T, "latent_prep: shapes");
+  TORCH_CHECK(cos_sin.is_cuda() && cos_sin.scalar_type() == at::kFloat && cos_sin.is_contiguous() &&
+                  cos_sin.dim() == 2 && cos_sin.size(1) == rot, "latent_prep: cos_sin [max_pos, rot] fp32");
+  void* ql = nullptr;
+  if (num_latent > 0) {
+    TORCH_CHECK(q_latent.has_value() && q_latent->is_cuda() && q_latent->scalar_type() == dt &&
+                    q_latent->is_contiguous() && q_latent->dim() == 3 && q_latent->size(0) >= num_latent &&
+                    q_latent->size(1) == heads && q_latent->size(2) == cache.size(2), "latent_prep: q_latent");
+    ql = q_latent->data_ptr();
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  check(b200_latent_prep(q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), norm_w.data_ptr(), (float)eps,
+                         cache.data_ptr(), positions.data_ptr<int>(), slots.data_ptr<int>(), cos_sin.data_ptr<float>(),
+                         (int)cos_sin.size(0), (int)T, (int)heads, (int)dim, (int)rot, (int)rank, (int)cache.size(2),
+                         neox ? 1 : 0, ql, (int)num_latent, f32 ? 1 : 0, cur_stream()),
+        "latent_prep");
+}
+
+void head_gemm(const Tensor& a, const Tensor& w, Tensor out) {
+  const auto dt = a.scalar_type();
+  const bool f32 = is_f32(a);
+  TORCH_CHECK(a.is_cuda() && w.is_cuda() && out.is_cuda() && w.scalar_type() == dt && out.scalar_type() == dt &&
+                  a.dim() == 3 && w.dim() == 3 && out.dim() == 3 && a.stride(2) == 1 && out.stride(2) == 1 &&
+                  w.is_contiguous(), "head_gemm: a [T, H, K], w [H, N, K], out [T, H, N]");
+  TORCH_CHECK(a.size(1) == w.size(0) && a.size(2) == w.size(2) && out.size(0) == a.size(0) &&
+                  out.size(1) == a.size(1) && out.size(2) == w.size(1), "head_gemm: shapes");
+  c10::cuda::CUDAGuard guard(a.device());
+  check(b200_head_gemm(a.data_ptr(), a.stride(0), a.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0),
+                       out.stride(1), (int)a.size(0), (int)a.size(1), (int)w.size(1), (int)w.size(2), f32 ? 1 : 0,
+                       cur_stream()),
+        "head_gemm");
+}
+
+Tensor latent_gather(const Tensor& cache, const Tensor& block_tables, const Tensor& seq_lens, const Tensor& start,
+                     int64_t num_seqs, int64_t total, int64_t max_len) {
+  TORCH_CHECK(cache.is_cuda() && cache.is_contiguous() && cache.dim() == 3, "latent_gather: cache [blocks, size, row]");
+  TORCH_CHECK(block_tables.is_cuda() && block_tables.scalar_type() == at::kInt && block_tables.dim() == 2 &&
+                  block_tables.stride(1) == 1 && block_tables.size(0) >= num_seqs, "latent_gather: block tables");
+  CHECK_I32(seq_lens);
+  CHECK_I32(start);
+  TORCH_CHECK(seq_lens.numel() >= num_seqs && start.numel() >= num_seqs, "latent_gather: sequences");
+  c10::cuda::CUDAGuard guard(cache.device());
+  Tensor out = torch::empty({total, cache.size(2)}, cache.options());
+  check(b200_latent_gather(cache.data_ptr(), out.data_ptr(), block_tables.data_ptr<int>(), seq_lens.data_ptr<int>(),
+                           start.data_ptr<int>(), (int)num_seqs, (int)max_len, (int)block_tables.stride(0),
+                           (int)cache.size(1), (int)(cache.size(2) * cache.element_size()), (int)total, cur_stream()),
+        "latent_gather");
+  return out;
+}
+
+int64_t latent_decode_scratch_bytes(int64_t T, int64_t N, int64_t rank, int64_t splits) {
+  return (int64_t)b200_latent_decode_scratch_bytes((int)T, (int)N, (int)rank, (int)splits);
+}
+
+void latent_decode(const Tensor& q, const Tensor& cache, const Tensor& block_tables, const Tensor& seq_lens,
+                   int64_t num_seqs, int64_t heads, int64_t rank, double scale, int64_t splits,
+                   const c10::optional<Tensor>& scratch, const Tensor& status, Tensor out) {
+  TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && q.is_contiguous() && q.dim() == 3 &&
+                  cache.is_cuda() && cache.scalar_type() == at::kBFloat16 && cache.is_contiguous() && cache.dim() == 3 &&
+                  out.is_cuda() && out.scalar_type() == at::kBFloat16 && out.is_contiguous(), "latent_decode: bf16");
+  TORCH_CHECK(q.size(0) >= num_seqs && q.size(1) == heads && q.size(2) == cache.size(2) &&
+                  out.numel() >= num_seqs * heads * rank, "latent_decode: shapes");
+  TORCH_CHECK(block_tables.is_cuda() && block_tables.scalar_type() == at::kInt && block_tables.dim() == 2 &&
+                  block_tables.stride(1) == 1 && block_tables.size(0) >= num_seqs, "latent_decode: block tables");
+  CHECK_I32(seq_lens);
+  void* sc = nullptr;
+  if (splits > 1) {
+    TORCH_CHECK(scratch.has_value() && (int64_t)scratch->nbytes() >=
+                    latent_decode_scratch_bytes(num_seqs, heads, rank, splits), "latent_decode: scratch too small");
+    sc = scratch->data_ptr();
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  check(b200_latent_decode(q.data_ptr(), cache.data_ptr(), out.data_ptr(), block_tables.data_ptr<int>(),
+                           seq_lens.data_ptr<int>(), (int)num_seqs, (int)heads, (int)cache.size(2), (int)rank,
+                           (int)block_tables.stride(0), (int)cache.size(1), (int)cache.size(0), (float)scale,
+                           (int)splits, sc, status.data_ptr<int>(), cur_stream()),
+        "latent_decode");
 }
 
 }  // namespace
@@ -420,4 +758,14 @@ TORCH_LIBRARY(omni_b200, m) {
   m.def("residual_norm", &residual_norm);
   m.def("gated_rope_cache", &gated_rope_cache);
   m.def("gated_attention", &gated_attention);
+  m.def("hyper_norm", &hyper_norm);
+  m.def("gated_linear_prep", &gated_linear_prep);
+  m.def("delta_prep", &delta_prep);
+  m.def("recurrent_scan", &recurrent_scan);
+  m.def("head_norm_gate", &head_norm_gate);
+  m.def("latent_prep", &latent_prep);
+  m.def("head_gemm", &head_gemm);
+  m.def("latent_gather", &latent_gather);
+  m.def("latent_decode_scratch_bytes", &latent_decode_scratch_bytes);
+  m.def("latent_decode", &latent_decode);
 }

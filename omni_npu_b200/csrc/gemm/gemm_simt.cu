@@ -1,5 +1,5 @@
 // fp32 products on the CUDA cores: C[M,N] = A[M,K] * W[N,K]^T, dense or grouped by expert, with the
-// gated activations of the tensor-core kernels.  It serves models that are run entirely in 32-bit
+// activations of the tensor-core kernels.  It serves models that are run entirely in 32-bit
 // (no reduced-precision tensor-core mode); any M, N, K.
 //
 // One CTA = a 64 x 64 tile, 256 threads x (4 x 4) outputs, K in steps of 16 through shared memory.
@@ -89,7 +89,7 @@ __global__ void __launch_bounds__(simt::THREADS) gemm_simt_kernel(const SimtGemm
     }
     __syncthreads();
   }
-  if (p.act == kActNone) {
+  if (!act_is_gated(p.act)) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int row = m0 + ty * 4 + i;
@@ -97,7 +97,7 @@ __global__ void __launch_bounds__(simt::THREADS) gemm_simt_kernel(const SimtGemm
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int col = n0 + tx * 4 + j;
-        if (col < p.N) p.C[row * p.ldc + col] = acc[i][j];
+        if (col < p.N) p.C[row * p.ldc + col] = p.act == kActXielu ? xielu(acc[i][j], p.act_alpha, p.act_limit) : acc[i][j];
       }
     }
     return;
@@ -123,7 +123,7 @@ extern "C" int b200_gemm_simt(const float* A, const float* W, float* C, int M, i
                               long long ldw, long long ldc, const int* expert_offsets, int num_experts, int act,
                               float act_alpha, float act_limit, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (act != kActNone && (N % 16) != 0) return -11;
+  if (act_is_gated(act) && (N % 16) != 0) return -11;
   SimtGemmParams p{A, W, C, M, N, K, lda, ldw, ldc, expert_offsets, num_experts, act, act_alpha, act_limit};
   // grouped: every expert may end in a partly filled tile
   const long long tiles = (M + simt::BM - 1) / simt::BM + (expert_offsets ? num_experts : 0);

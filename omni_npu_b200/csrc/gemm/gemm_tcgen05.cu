@@ -909,7 +909,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
           }
           continue;
         }
-        if (p.swiglu) {
+        if (p.swiglu == kActXielu) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) v[i] = xielu(v[i], p.act_alpha, p.act_limit);
+        } else if (p.swiglu) {
           // Columns [c, c+8) hold gate values, [c+8, c+16) the matching up values.
           const int ocol = col >> 1;
           float o[8];
@@ -1552,7 +1555,7 @@ static int gemm_impl(const void* A, const void* W, void* C, const void* bias, co
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const int eb = dtype_fp8 ? 1 : 2;
   if (BN < 16 || BN > 256 || (BN % 16) != 0) return -10;
-  if (swiglu && ((N % 16) != 0 || splits != 1)) return -11;
+  if (swiglu && ((act_is_gated(swiglu) && (N % 16) != 0) || splits != 1)) return -11;
   if (splits <= 1) cluster_split = 0;
   if (cluster_split && (splits > 8 || BN > 128 || (kBM % splits) != 0)) return -14;
   if (splits > 1 && !cluster_split && (workspace == nullptr || counters == nullptr)) return -12;
@@ -1664,7 +1667,7 @@ extern "C" int b200_grouped_gemm(const void* A, const void* W, void* C, const in
   if (num_experts > kMaxExperts) return -13;
   const int eb = dtype_fp8 ? 1 : 2;
   if (BN < 16 || BN > 256 || (BN % 16) != 0) return -10;
-  if (swiglu && (N % 16) != 0) return -11;
+  if (act_is_gated(swiglu) && (N % 16) != 0) return -11;
   GemmParams p{};
   p.M = total_rows;
   p.N = N;

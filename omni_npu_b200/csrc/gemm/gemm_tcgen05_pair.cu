@@ -319,7 +319,10 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
         for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
         const int col = n0 + c;
         if (!row_ok || col >= p.N) continue;
-        if (p.swiglu) {
+        if (p.swiglu == kActXielu) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) v[i] = xielu(v[i], p.act_alpha, p.act_limit);
+        } else if (p.swiglu) {
           const int ocol = col >> 1;
           float o[8];
 #pragma unroll
@@ -471,7 +474,7 @@ extern "C" int b200_gemm_pair(const void* A, const void* W, void* C, const void*
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const int eb = dtype_fp8 ? 1 : 2;
   if (BN < 32 || BN > 256 || (BN % 32) != 0) return -10;
-  if (swiglu && (N % 16) != 0) return -11;
+  if (act_is_gated(swiglu) && (N % 16) != 0) return -11;
   PairParams p{};
   p.M = M;
   p.N = N;

@@ -16,48 +16,11 @@
 #include <stdint.h>
 
 #include "../common/pdl.cuh"
+#include "../common/rows.cuh"
 
 namespace b200 {
 
 static constexpr int kResThreads = 256;
-
-template <typename T>
-struct Row8;
-template <>
-struct Row8<__nv_bfloat16> {
-  static __device__ __forceinline__ void load(const void* base, long long vec, float (&v)[8]) {
-    const uint4 u = reinterpret_cast<const uint4*>(base)[vec];
-    const uint32_t r[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      v[2 * i] = __uint_as_float(r[i] << 16);
-      v[2 * i + 1] = __uint_as_float(r[i] & 0xffff0000u);
-    }
-  }
-  static __device__ __forceinline__ void store(void* base, long long vec, const float (&v)[8]) {
-    uint4 u;
-    uint32_t* r = reinterpret_cast<uint32_t*>(&u);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const __nv_bfloat162 p = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-      r[i] = *reinterpret_cast<const uint32_t*>(&p);
-    }
-    reinterpret_cast<uint4*>(base)[vec] = u;
-  }
-};
-template <>
-struct Row8<float> {
-  static __device__ __forceinline__ void load(const void* base, long long vec, float (&v)[8]) {
-    const float4 a = reinterpret_cast<const float4*>(base)[2 * vec];
-    const float4 b = reinterpret_cast<const float4*>(base)[2 * vec + 1];
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-  }
-  static __device__ __forceinline__ void store(void* base, long long vec, const float (&v)[8]) {
-    reinterpret_cast<float4*>(base)[2 * vec] = make_float4(v[0], v[1], v[2], v[3]);
-    reinterpret_cast<float4*>(base)[2 * vec + 1] = make_float4(v[4], v[5], v[6], v[7]);
-  }
-};
 
 struct ResidualNormParams {
   float* residual;

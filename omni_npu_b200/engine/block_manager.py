@@ -152,3 +152,27 @@ class BlockPool:
     @property
     def num_parked(self) -> int:
         return len(self._delayed)
+
+
+class StateSlotPool:
+    """Slots of per-sequence recurrent state (one fixed-size record per running request, beside the
+    paged blocks).  A slot is handed out as it is: a sequence that starts at position 0 takes its state
+    as zero, whatever the slot held before."""
+
+    def __init__(self, num_slots: int) -> None:
+        self.num_slots = num_slots
+        self._free: List[int] = list(range(num_slots - 1, -1, -1))
+
+    @property
+    def num_free(self) -> int:
+        return len(self._free)
+
+    def allocate(self) -> int:
+        if not self._free:
+            raise RuntimeError("out of state slots")
+        return self._free.pop()
+
+    def free(self, slot: int) -> None:
+        if slot in self._free:
+            raise RuntimeError(f"state slot {slot} freed twice")
+        self._free.append(slot)

@@ -58,8 +58,15 @@ class LLMEngine:
                                  "speculative decoding")
         if config.speculative.method in ("mtp", "deepseek_mtp") and config.speculative.num_speculative_tokens > 1:
             config.scheduler.num_lookahead_tokens = config.speculative.num_speculative_tokens - 1
+        state_slots = self.worker.model_runner.num_state_slots
+        if state_slots and (connector is not None or config.cache.enable_prefix_caching
+                            or config.parallel.prefill_context_parallel_size > 1
+                            or (config.speculative.method and config.speculative.num_speculative_tokens)):
+            raise ValueError("a model with recurrent state is not combined with prefix caching, KV connectors, "
+                             "speculative decoding or prefill context parallelism: its state is kept for the "
+                             "newest token of a sequence only")
         self.scheduler = Scheduler(config.scheduler, config.cache, num_blocks, reserved, connector,
-                                   context_parallel_size=dcp)
+                                   context_parallel_size=dcp, num_state_slots=state_slots)
         self._ids = itertools.count()
         self.stats = {"steps": 0, "prefill_steps": 0, "decode_steps": 0, "spec_decode_steps": 0,
                       "h2d_bytes": 0, "d2h_bytes": 0, "output_tokens": 0}

@@ -72,7 +72,7 @@ class Request:
                  "block_ids", "num_computed_tokens", "arrival_time", "first_token_time",
                  "finish_time", "kv_transfer_params", "eos_token_id", "num_preemptions",
                  "spec_token_ids", "client_index", "num_external_tokens", "_block_hashes",
-                 "_registered_blocks", "logprobs", "prompt_logprobs")
+                 "_registered_blocks", "logprobs", "prompt_logprobs", "state_slot")
 
     def __init__(self, request_id: str, prompt_token_ids: Sequence[int],
                  sampling_params: Optional[SamplingParams] = None,
@@ -84,6 +84,7 @@ class Request:
         self.output_token_ids: List[int] = []
         self.status = RequestStatus.WAITING
         self.block_ids: List[int] = []
+        self.state_slot = -1                  # slot of the recurrent state while running (models that have one)
         self.num_computed_tokens = 0
         self.arrival_time = time.monotonic() if arrival_time is None else arrival_time
         self.first_token_time: Optional[float] = None

@@ -16,7 +16,7 @@ from dataclasses import dataclass, field
 from typing import Any, Deque, Dict, List, Optional, Tuple
 
 from ..config import CacheConfig, SchedulerConfig
-from .block_manager import BlockPool
+from .block_manager import BlockPool, StateSlotPool
 from .request import Request, RequestStatus
 
 
@@ -50,7 +50,8 @@ class SchedulerOutput:
 
 class Scheduler:
     def __init__(self, sched_cfg: SchedulerConfig, cache_cfg: CacheConfig, num_blocks: int,
-                 num_reserved_blocks: int = 0, kv_connector=None, context_parallel_size: int = 1) -> None:
+                 num_reserved_blocks: int = 0, kv_connector=None, context_parallel_size: int = 1,
+                 num_state_slots: int = 0) -> None:
         self.cfg = sched_cfg
         # With decode context parallelism every rank stores 1 / world of a sequence's tokens
         # (token p on rank p % world), so one block id covers block_size * world tokens.
@@ -60,6 +61,8 @@ class Scheduler:
         self.pool = BlockPool(num_blocks, self.block_size, num_reserved_blocks,
                               prefix_caching=bool(getattr(cache_cfg, "enable_prefix_caching", False))
                               and kv_connector is None)
+        # models with recurrent state: every running request owns a slot (as many as it can run at once)
+        self.state_pool = StateSlotPool(num_state_slots) if num_state_slots else None
         self.prefix_stats = {"requests": 0, "hit_tokens": 0}
         self.waiting: Deque[Request] = deque()
         self.running: List[Request] = []
@@ -125,6 +128,18 @@ class Scheduler:
             return False
         req.block_ids.extend(self.pool.allocate(need))
         return True
+
+    def _admit(self, req: Request) -> None:
+        req.status = RequestStatus.RUNNING
+        self.running.append(req)
+        if self.state_pool is not None:
+            req.state_slot = self.state_pool.allocate()
+
+    def _release_state(self, req: Request) -> None:
+        """Give the state slot back (the request ended, or will be recomputed from its first token)."""
+        if req.state_slot >= 0:
+            self.state_pool.free(req.state_slot)
+            req.state_slot = -1
 
     # ------------------------------------------------------------ prefix caching
     def _attach_cached_prefix(self, req: Request) -> bool:
@@ -193,6 +208,7 @@ class Scheduler:
         else:
             self.pool.free(req.block_ids)
         req.block_ids = []
+        self._release_state(req)
         self._finished_since_last.append(req.request_id)
         self.requests.pop(req.request_id, None)      # a long-running server must not keep every request it ever saw
 
@@ -208,6 +224,7 @@ class Scheduler:
             self.running.remove(victim)
             self.pool.free(victim.block_ids)
             victim.block_ids = []
+            self._release_state(victim)
             victim.num_computed_tokens = 0
             victim._registered_blocks = 0
             victim.status = RequestStatus.PREEMPTED
@@ -224,6 +241,7 @@ class Scheduler:
             self.running.remove(req)
         self.pool.free(req.block_ids)
         req.block_ids = []
+        self._release_state(req)
         req.num_computed_tokens = 0
         req._registered_blocks = 0
         req.spec_token_ids = []
@@ -249,8 +267,7 @@ class Scheduler:
                 if len(self.running) >= self.cfg.max_num_seqs:
                     raise RuntimeError(f"more than {self.cfg.max_num_seqs} live requests")
                 self.requests[req.request_id] = req
-                req.status = RequestStatus.RUNNING
-                self.running.append(req)
+                self._admit(req)
             start = req.num_computed_tokens
             if n < 1 or start + n > req.num_tokens:
                 raise ValueError(f"request {req.request_id}: {n} tokens from {start} of {req.num_tokens}")
@@ -392,8 +409,7 @@ class Scheduler:
                     self._detach_cached_prefix(req)
                 break
             self.waiting.popleft()
-            req.status = RequestStatus.RUNNING
-            self.running.append(req)
+            self._admit(req)
             prefill.append(ScheduledSeq(req, req.num_computed_tokens, n, n == remaining))
             budget -= n
         if prefill:

@@ -345,6 +345,45 @@ class GatedQKVParallelLinear(QKVParallelLinear):
         dst.copy_(loaded.narrow(0, self.tp_rank * self.gate_size, self.gate_size).to(dst.dtype))
 
 
+class SegmentedLinear(LinearBase):
+    """Several projections of one input as one product, each with its own rows: ``segments`` = name ->
+    (rows, sharded).  Sharded segments are split over the group, the others are whole on every rank.  A
+    segment starts at a whole 16-byte column of the result (``offsets``); the rows between are zero."""
+
+    def __init__(self, in_features: int, segments, dtype=torch.bfloat16, device=None, **kw) -> None:
+        super().__init__(in_features, sum(n for n, _ in segments.values()), False, dtype, device, **kw)
+        self.sharded = {k: sh for k, (_, sh) in segments.items()}
+        self.rows = {}
+        self.offsets = {}
+        off = 0
+        for name, (n, sh) in segments.items():
+            if sh and n % self.tp_size:
+                raise ValueError(f"{self.prefix}: {n} rows of {name!r} do not split over {self.tp_size} ranks")
+            self.rows[name] = n // self.tp_size if sh else n
+            self.offsets[name] = off
+            off += (self.rows[name] + 7) // 8 * 8
+        self._create(in_features, off, device)
+        self.weight.data.zero_()
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return self.quant_method.apply(self, x, None)
+
+    def segment(self, y: torch.Tensor, name: str) -> torch.Tensor:
+        return y[:, self.offsets[name]: self.offsets[name] + self.rows[name]]
+
+    def padding_rows(self) -> torch.Tensor:
+        """Indices of the rows that belong to no segment."""
+        used = torch.zeros(self.weight.shape[0], dtype=torch.bool)
+        for name, n in self.rows.items():
+            used[self.offsets[name]: self.offsets[name] + n] = True
+        return (~used).nonzero().view(-1)
+
+    def weight_loader(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
+        n, off = self.rows[shard_id], self.offsets[shard_id]
+        src = loaded.narrow(0, self.tp_rank * n, n) if self.sharded[shard_id] else loaded
+        param.data[off: off + n, : src.shape[1]] = src.to(param.dtype).to(param.device)
+
+
 class RowParallelLinear(LinearBase):
     """Input features sharded across the group; partial sums are reduced
     (all-reduce, or reduce-scatter when the residual stream is token-sharded)."""

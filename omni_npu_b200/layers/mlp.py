@@ -13,7 +13,8 @@ import torch
 from torch import nn
 
 from .activation import SiluAndMul
-from .linear import MergedColumnParallelLinear, RowParallelLinear, row_parallel_add_rms_norm
+from .. import ops
+from .linear import ColumnParallelLinear, MergedColumnParallelLinear, RowParallelLinear, row_parallel_add_rms_norm
 
 
 class FusedMLP(nn.Module):
@@ -51,3 +52,27 @@ class FusedMLP(nn.Module):
         else:
             h = self.act(self.gate_up_proj(x))
         return row_parallel_add_rms_norm(self.down_proj, h, norm, residual)
+
+
+class XieluMLP(nn.Module):
+    """down(xielu(up(x))): one up projection, the activation in its epilogue.  ``act_params`` (p, q) gives
+    xielu(z) = softplus(p) z^2 + z / 2 above zero and (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 below."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int, dtype=torch.bfloat16, device=None,
+                 prefix: str = "") -> None:
+        super().__init__()
+        self.up_proj = ColumnParallelLinear(hidden_size, intermediate_size, dtype=dtype, device=device,
+                                            prefix=f"{prefix}.up_proj")
+        self.down_proj = RowParallelLinear(intermediate_size, hidden_size, dtype=dtype, device=device,
+                                           prefix=f"{prefix}.down_proj")
+        self.act_params = nn.Parameter(torch.zeros(2, dtype=torch.float32, device=device), requires_grad=False)
+        self.constants = (0.0, 0.0)
+
+    @torch.no_grad()
+    def fix_constants(self) -> None:
+        """The activation's two factors as host numbers (after loading)."""
+        p, q = torch.nn.functional.softplus(self.act_params.double().cpu()).tolist()
+        self.constants = (p, 0.5 + q)
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return self.down_proj(ops.gemm(x, self.up_proj.weight, xielu=self.constants))

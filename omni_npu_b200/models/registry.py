@@ -25,6 +25,7 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "Qwen3VLForConditionalGeneration": ("omni_npu_b200.models.qwen3_vl", "Qwen3VLForConditionalGeneration"),
     "OpenPanguVLForConditionalGeneration": ("omni_npu_b200.models.openpangu_vl", "OpenPanguVLForConditionalGeneration"),
     "Rivudra": ("omni_npu_b200.models.rivudra", "RivudraForCausalLM"),
+    "Fuvirax": ("omni_npu_b200.models.fuvirax", "FuviraxForCausalLM"),
     "MockModel": ("omni_npu_b200.models.mock", "MockModelForCausalLM"),
 }
 
@@ -32,11 +33,12 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
 # designs whose config.json has keys of its own: name under "architecture" -> reader returning a ModelConfig
 _CONFIG_READERS: Dict[str, Tuple[str, str]] = {
     "Rivudra": ("omni_npu_b200.models.rivudra", "read_config"),
+    "Fuvirax": ("omni_npu_b200.models.fuvirax", "read_config"),
 }
 
 
 # architectures whose kernels are all in the core library (_build.CORE_SOURCES)
-_CORE_LIBRARY_ONLY = {"Rivudra"}
+_CORE_LIBRARY_ONLY = {"Rivudra", "Fuvirax"}
 
 
 def runs_on_core_library(arch: str) -> bool:

@@ -74,7 +74,7 @@ def _layer_spec(d: Dict[str, Any]) -> LayerSpec:
     return LayerSpec(attn, moe)
 
 
-def read_config(d: Dict[str, Any], dtype=None) -> ModelConfig:
+def read_config(d: Dict[str, Any], dtype=None, path: Optional[str] = None) -> ModelConfig:
     """``ModelConfig`` from the design's own config.json keys."""
     specs = tuple(_layer_spec(x) for x in d["layers"])
     first = specs[0].attention

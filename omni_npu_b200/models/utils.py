@@ -86,6 +86,17 @@ def iter_safetensors(path: str) -> Iterator[Tuple[str, torch.Tensor]]:
                 yield k, f.get_tensor(k)
 
 
+def safetensors_shapes(path: str) -> Dict[str, Tuple[int, ...]]:
+    """Name -> shape of every tensor under a directory, read from the files' headers alone."""
+    from safetensors import safe_open
+    out: Dict[str, Tuple[int, ...]] = {}
+    for fn in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(fn, framework="pt", device="cpu") as f:
+            for k in f.keys():
+                out[k] = tuple(f.get_slice(k).get_shape())
+    return out
+
+
 @torch.no_grad()
 def random_init_(model: nn.Module, seed: int = 0, std: float = 0.02, by_name: Optional[bool] = None) -> None:
     """Deterministic random initialisation (normal, std 0.02; norm weights 1).

@@ -197,6 +197,13 @@ PAIR_MIN_M = int(os.environ.get("OMNI_B200_GEMM_PAIR_MIN_M", "1024"))
 SMALL_M_GEMM = os.environ.get("OMNI_B200_SMALL_M_GEMM", "library")
 SMALL_M_LIBRARY_ROWS = (64, 256)
 
+def _act_kind(swiglu: bool, act: Tuple[float, float], xielu: Optional[Tuple[float, float]]) -> Tuple[int, float, float]:
+    """(kind, constants) of a GEMM epilogue's activation as csrc/gemm/gated_act.cuh numbers them."""
+    if xielu is not None:
+        return (3, *xielu)
+    return (0, *act) if not swiglu else (2 if act[0] != 0.0 else 1, *act)
+
+
 def library_small_m(m: int, cluster_split_plan: bool, plain_bf16: bool) -> bool:
     """Whether ``gemm`` hands a product to cuBLAS: only a plain bf16 product (nothing fused, no forced
     tile or split), only when this package's plan for it is a cluster split-K, only for the row
@@ -208,22 +215,25 @@ def library_small_m(m: int, cluster_split_plan: bool, plain_bf16: bool) -> bool:
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
          swiglu: bool = False, bn: int = 0, splits: int = 0, max_ctas: int = 0,
-         pair: Optional[bool] = None, act: Tuple[float, float] = SILU) -> torch.Tensor:
+         pair: Optional[bool] = None, act: Tuple[float, float] = SILU,
+         xielu: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """``a[M,K] @ w[N,K].T`` (+bias, +residual).  bf16 or float8_e4m3fn inputs,
     fp32 accumulation, bf16 (default) or fp32 output.  ``swiglu`` fuses
     silu(gate)*up for weights laid out by :func:`ref.interleave_gate_up`; ``act`` = (slope, limit)
-    with a non-zero slope selects the clamped form of it (:func:`ref.gated_act`).  fp32 inputs run on
-    the CUDA cores, with no reduced-precision mode.
+    with a non-zero slope selects the clamped form of it (:func:`ref.gated_act`).  ``xielu`` = (a, b)
+    applies :func:`ref.xielu` to every output.  fp32 inputs run on the CUDA cores, with no
+    reduced-precision mode.
     ``splits`` > 1 forces split-K (as a thread-block cluster when it fits), a
     negative value forces the workspace variant with |splits| slices.
     ``pair`` selects the CTA-pair kernel (256-row tiles over two SMs); by default
     it runs for M >= PAIR_MIN_M when no split-K was asked for."""
     if not a.is_cuda:
-        return ref.gemm(a, w, bias, residual, out_dtype, swiglu, act)
+        return ref.gemm(a, w, bias, residual, out_dtype, swiglu, act, xielu)
     C = _core()
+    kind = _act_kind(swiglu, act, xielu)
     if a.dtype == torch.float32:
         _count(1)
-        y = C.gemm_simt(a, w, None, swiglu, act[0], act[1])
+        y = C.gemm_simt(a, w, None, *kind)
         if bias is not None:
             y = y + bias
         return y if residual is None else y + residual
@@ -236,23 +246,24 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         n_eff = n
         pbn = bn if bn > 0 else (256 if n_eff >= 256 else max(32, ((n_eff + 31) // 32) * 32))
         _count(1)
-        return C.gemm_pair(a, w, bias, residual, out_dtype == torch.float32, swiglu, pbn, st.status, max_ctas,
-                           act[0], act[1])
-    key = (m, n, k, a.dtype.itemsize, swiglu, bn, splits)
+        return C.gemm_pair(a, w, bias, residual, out_dtype == torch.float32, kind[0], pbn, st.status, max_ctas,
+                           kind[1], kind[2])
+    fused = kind[0] != 0
+    key = (m, n, k, a.dtype.itemsize, fused, bn, splits)
     plan = st.plans.get(key)
     if plan is None:
-        plan = C.gemm_plan(m, n, k, a.dtype.itemsize, swiglu, bn, 1 if swiglu else splits)
+        plan = C.gemm_plan(m, n, k, a.dtype.itemsize, fused, bn, 1 if fused else splits)
         st.plans[key] = plan
     pbn, psplits, ws_bytes, ncnt, cluster = plan
-    if library_small_m(m, bool(cluster), bias is None and residual is None and not swiglu and bn == 0
+    if library_small_m(m, bool(cluster), bias is None and residual is None and not fused and bn == 0
                        and splits == 0 and a.dtype == torch.bfloat16 and out_dtype in (None, torch.bfloat16)):
         return torch.nn.functional.linear(a, w)          # a library kernel: not counted as a launch of ours
     ws = cnt = None
     if psplits > 1 and not cluster:
         ws, cnt = st.gemm_workspace(torch.cuda.current_stream(a.device).cuda_stream, ws_bytes, ncnt)
     _count(1)
-    return C.gemm(a, w, bias, residual, out_dtype == torch.float32, swiglu, pbn, psplits,
-                  bool(cluster), ws, cnt, st.status, max_ctas, act[0], act[1])
+    return C.gemm(a, w, bias, residual, out_dtype == torch.float32, kind[0], pbn, psplits,
+                  bool(cluster), ws, cnt, st.status, max_ctas, kind[1], kind[2])
 
 
 def quant_int8_per_token(x: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -364,13 +375,14 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
         return ref.grouped_gemm(a, w, expert_offsets, swiglu, act)
     if a.dtype == torch.float32:
         _count(1)
-        return _core().gemm_simt(a, w, expert_offsets, swiglu, act[0], act[1])
+        return _core().gemm_simt(a, w, expert_offsets, *_act_kind(swiglu, act, None))
     if bn <= 0:
         n = w.shape[1]
         bn = 256 if n % 256 == 0 else (128 if n % 128 == 0 else (64 if n % 64 == 0 else 32))
     st = device_state(a.device)
     _count(1)
-    return _core().grouped_gemm(a, w, expert_offsets, swiglu, bn, st.status, max_ctas, act[0], act[1])
+    kind, c0, c1 = _act_kind(swiglu, act, None)
+    return _core().grouped_gemm(a, w, expert_offsets, kind, bn, st.status, max_ctas, c0, c1)
 
 
 # ------------------------------------------------------------- norm/activation
@@ -692,7 +704,7 @@ def gated_attention(q: torch.Tensor, gate: Optional[torch.Tensor], k_cache: torc
     _core().gated_attention(q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len,
                             max_q_len, num_q_heads, head_dim, head_dim_v, scale, window, sink is not None,
                             0.0 if sink is None else float(sink), max(1, splits), variant,
-                            device_state(q.device).status)
+                            device_state(q.device).status, False)
 
 
 # ----------------------------------------------------------- 32-bit residual stream
@@ -720,6 +732,148 @@ def residual_add_norm(residual: torch.Tensor, a: Optional[torch.Tensor], b: Opti
     out = _core().residual_norm(residual, None, None, 1.0, a, b, y, slots, w, weight, eps, weight_offset, true_width,
                                 like.dtype == torch.float32)
     return out if weight is not None else None
+
+
+# ------------------------------------ several residual streams, layer norm and token shift in one pass
+def hyper_norm(streams: Optional[torch.Tensor], ids: Optional[torch.Tensor], table: Optional[torch.Tensor],
+               num_streams: int, y: Optional[torch.Tensor], conn, w_in: torch.Tensor, norm_w: torch.Tensor,
+               norm_b: torch.Tensor, eps: float, true_width: int, out_scale: float = 1.0, shift=None, keep: bool = True):
+    """Join a sublayer's result to the residual streams and read them for the next one
+    (csrc/norm_rope/hyper_norm.cu).  ``streams`` [T, N, W] fp32; ``conn`` = (layer scale [W], mix [N, N] indexed
+    [from, to], out [N]) of the sublayer that gave ``y`` [T, W]; or ``ids`` / ``table``: every stream starts as
+    an embedding row.  Then u = sum_s w_in[s] x_s, layer norm, times ``out_scale``, and with ``shift`` = (mu,
+    state [slots, W] fp32, seq_idx, state_slots, cu_q, seq_lens, num_seqs) the blend with the previous token's
+    row.  Returns (new streams, or None unless ``keep``; rows [T, W])."""
+    if not norm_w.is_cuda:
+        return ref.hyper_norm(streams, ids, table, num_streams, y, conn, w_in, norm_w, norm_b, eps, true_width, out_scale,
+                              shift, keep)
+    ls, mix, w_out = conn if conn is not None else (None, None, None)
+    mu, state, seq_idx, slots, cu_q, seq_lens, _ = shift if shift is not None else (None,) * 7
+    _count(1)
+    new, h = _core().hyper_norm(streams, ids, table, num_streams, y, ls, mix, w_out, w_in, norm_w, norm_b, eps,
+                                true_width, out_scale, mu, state, seq_idx, slots, cu_q, seq_lens, keep)
+    return (new if keep else None), h
+
+
+# ------------------------------------------------------------------ recurrent layers
+def gated_linear_prep(proj: torch.Tensor, q_off: int, f_off: int, heads: int, dim: int, f_bias: torch.Tensor,
+                      lower: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+    """(silu(q), keys 1 - forget gate), fp32 [T, heads, dim rounded up to 4] (:func:`ref.gated_linear_prep`)."""
+    if not proj.is_cuda:
+        return ref.gated_linear_prep(proj, q_off, f_off, heads, dim, f_bias, lower)
+    _count(1)
+    return _core().gated_linear_prep(proj, q_off, f_off, heads, dim, f_bias, lower)
+
+
+def delta_prep(proj: torch.Tensor, low: torch.Tensor, offs, heads: int, kv_heads: int, dim: int, vdim: int,
+               conv_w: torch.Tensor, conv_state: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+               unit_eps: float, seq_idx: torch.Tensor, state_slots: torch.Tensor, cu_q: torch.Tensor,
+               seq_lens: torch.Tensor, num_seqs: int):
+    """Short convolutions with silu, unit norms, decays and step sizes of the delta rule
+    (:func:`ref.delta_prep`): q, k, g fp32, v in the projection's type, beta fp32."""
+    if not proj.is_cuda:
+        return ref.delta_prep(proj, low, offs, heads, kv_heads, dim, vdim, conv_w, conv_state, dt_bias, a_log, unit_eps,
+                              seq_idx, state_slots, cu_q, seq_lens, num_seqs)
+    _count(1)
+    return _core().delta_prep(proj, low, offs["q"], offs["k"], offs["v"], offs["b"], heads, kv_heads, dim, vdim, conv_w,
+                              conv_state, dt_bias, a_log, unit_eps, seq_idx, state_slots, cu_q, seq_lens)
+
+
+def recurrent_scan(q: torch.Tensor, k: torch.Tensor, g: Optional[torch.Tensor], v: torch.Tensor,
+                   beta: Optional[torch.Tensor], state: torch.Tensor, heads: int, vdim: int, state_slots: torch.Tensor,
+                   cu_q: torch.Tensor, seq_lens: torch.Tensor, num_seqs: int, conv=None) -> torch.Tensor:
+    """Carry the state of every sequence over its tokens of this step (:func:`ref.recurrent_scan`);
+    o [T, heads, vdim] fp32."""
+    if not q.is_cuda:
+        return ref.recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, conv)
+    proj, cs = conv if conv is not None else (None, None)
+    _count(1)
+    return _core().recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, proj, cs)
+
+
+def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor],
+                   out_width: int) -> torch.Tensor:
+    """RMS norm per head, times the sigmoid of ``gate``: [T, out_width], zero beyond the heads."""
+    if not o.is_cuda:
+        return ref.head_norm_gate(o, weight, eps, gate, out_width)
+    _count(1)
+    return _core().head_norm_gate(o, weight, eps, gate, out_width)
+
+
+# ------------------------------------------------------- latent attention with run-time sizes
+def latent_prep_(q: torch.Tensor, kv_a: torch.Tensor, norm_w: torch.Tensor, eps: float, cache: torch.Tensor,
+                 positions: torch.Tensor, slot_mapping: torch.Tensor, cos_sin: torch.Tensor, heads: int, dim: int,
+                 rot: int, rank: int, neox: bool, q_latent: Optional[torch.Tensor] = None, num_latent: int = 0) -> None:
+    """RMS norm of the latent and rotation of the shared key part into the cache row
+    [latent | rotated | zeros]; rotation of the queries: in place, but for the first ``num_latent`` rows into
+    columns ``rank`` .. of ``q_latent`` [num_latent.., heads, row]."""
+    if not q.is_cuda:
+        for rows, lat in ((slice(0, num_latent), q_latent), (slice(num_latent, q.shape[0]), None)):
+            ref.latent_prep_(q[rows], kv_a[rows], norm_w, eps, cache, positions[: q.shape[0]][rows],
+                             slot_mapping[: q.shape[0]][rows], cos_sin, heads, dim, rot, rank, neox, lat)
+        return
+    _count(1)
+    _core().latent_prep(q, kv_a, norm_w, eps, cache, positions, slot_mapping, cos_sin, heads, dim, rot, rank, neox,
+                        q_latent, num_latent)
+
+
+def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t, h] = w[h] @ a[t, h] for every head: a [T, H, K], w [H, N, K], out [T, H, N] (views with any
+    token and head pitch)."""
+    if not a.is_cuda:
+        return ref.head_gemm(a, w, out)
+    _count(1)
+    _core().head_gemm(a, w, out)
+
+
+def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, seq_lens: torch.Tensor, start: torch.Tensor,
+                  num_seqs: int, total: int, max_len: int) -> torch.Tensor:
+    """Cached rows of all sequences, one after another: [total, row]; sequence b begins at ``start[b]``."""
+    if not cache.is_cuda:
+        return ref.latent_gather(cache, block_tables, seq_lens, num_seqs)
+    _count(1)
+    return _core().latent_gather(cache, block_tables, seq_lens, start, num_seqs, total, max_len)
+
+
+def contiguous_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor,
+                         start: torch.Tensor, seq_lens: torch.Tensor, num_seqs: int, max_q_len: int, heads: int,
+                         head_dim: int, head_dim_v: int, scale: float) -> None:
+    """Causal attention of prompt portions over keys that lie contiguously: k [keys, heads, 1, >= head_dim],
+    sequence b's from row ``start[b]``."""
+    if not q.is_cuda:
+        bt = start[:num_seqs, None].long() + torch.arange(int(seq_lens[:num_seqs].max()))[None, :]
+        return ref.gated_attention(q, None, k, v, out, bt.clamp(max=k.shape[0] - 1), cu_q, seq_lens, num_seqs, max_q_len,
+                                   heads, head_dim, head_dim_v, scale)
+    _count(1)
+    _core().gated_attention(q, None, k, v, out, start.view(-1, 1), cu_q, seq_lens, num_seqs, max_q_len, max_q_len, heads,
+                            head_dim, head_dim_v, scale, 0, False, 0.0, 1, 0, device_state(q.device).status, True)
+
+
+def latent_decode(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, seq_lens: torch.Tensor,
+                  num_seqs: int, heads: int, rank: int, scale: float, out: torch.Tensor, max_seq_len: int = 0,
+                  splits: int = 0) -> None:
+    """Single new tokens over the latent cache: q [B, heads, row], cache [blocks, block_size, row]; the values
+    are a row's first ``rank`` columns.  out [B, heads, rank]."""
+    if not q.is_cuda:
+        return ref.latent_decode(q, cache, block_tables, seq_lens, num_seqs, heads, rank, scale, out)
+    st = device_state(q.device)
+    row = cache.shape[2]
+    if q.dtype == torch.float32 or rank > 512 or row > 640 or cache.shape[1] % 8:
+        c = cache.unsqueeze(1)                  # the plain kernel: one key/value head, values inside the key rows
+        _count(1)
+        _core().gated_attention(q.view(num_seqs, -1), None, c, c, out.view(num_seqs, -1), block_tables, None, seq_lens,
+                                num_seqs, 1, 1, heads, row, rank, scale, 0, False, 0.0, 1, 2, st.status, False)
+        return
+    tiles = (heads + 15) // 16
+    if splits <= 0:
+        bound = max_seq_len if max_seq_len > 0 else block_tables.shape[1] * cache.shape[1]
+        splits = max(1, min((2 * 148 + num_seqs * tiles - 1) // max(1, num_seqs * tiles), max(1, bound // 256), 16))
+    scratch = None
+    if splits > 1:
+        nbytes = _core().latent_decode_scratch_bytes(num_seqs, heads, rank, splits)
+        scratch = st.decode_scratch(torch.cuda.current_stream(q.device).cuda_stream, nbytes)
+    _count(2 if splits > 1 else 1)
+    _core().latent_decode(q, cache, block_tables, seq_lens, num_seqs, heads, rank, scale, splits, scratch, st.status, out)
 
 
 # -------------------------------------------------------------------- sampling

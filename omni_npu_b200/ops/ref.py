@@ -15,14 +15,18 @@ import torch.nn.functional as F
 
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-         swiglu: bool = False, act: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
+         swiglu: bool = False, act: Tuple[float, float] = (0.0, 0.0),
+         xielu_ab: Optional[Tuple[float, float]] = None) -> torch.Tensor:
     """``a @ w.T`` with fp32 accumulation.  With ``swiglu`` the N columns are
-    interpreted as interleaved groups of 8 gate / 8 up columns, joined by :func:`gated_act`."""
+    interpreted as interleaved groups of 8 gate / 8 up columns, joined by :func:`gated_act`;
+    ``xielu_ab`` applies :func:`xielu`."""
     out = a.float() @ w.float().t()
     if swiglu:
         n = out.shape[-1]
         g = out.view(*out.shape[:-1], n // 16, 2, 8)
         out = gated_act(g[..., 0, :], g[..., 1, :], act).reshape(*out.shape[:-1], n // 2)
+    if xielu_ab is not None:
+        out = xielu(out, xielu_ab)
     if bias is not None:
         out = out + bias.float()
     if residual is not None:
@@ -30,6 +34,12 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
     if out_dtype is None:
         out_dtype = torch.bfloat16 if a.dtype.itemsize == 1 else a.dtype
     return out.to(out_dtype)
+
+
+def xielu(z: torch.Tensor, ab: Tuple[float, float]) -> torch.Tensor:
+    """a z^2 + z / 2 above zero, b (exp(z) - 1 - z) + z / 2 below."""
+    neg = z.clamp(max=0)
+    return torch.where(z > 0, ab[0] * z * z, ab[1] * (torch.expm1(neg) - neg)) + z / 2
 
 
 def gated_act(gate: torch.Tensor, up: torch.Tensor, act: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
@@ -576,3 +586,157 @@ def grouped_gemm_fp8_block(a_q, a_scale, w_q, w_scale, expert_offsets, swiglu=Fa
             y = (torch.nn.functional.silu(y[:, :, 0]) * y[:, :, 1]).reshape(-1, half)
         out[offs[i]: offs[i + 1]] = y
     return out.to(torch.bfloat16)
+
+
+# ------------------------------------------- residual streams, token shift, recurrent layers
+def _portions(cu_q, seq_lens, state_slots, num_seqs):
+    """(first row, one past the last row, first position, state slot) of every sequence of a step."""
+    cu, lens, slots = cu_q.tolist(), seq_lens.tolist(), state_slots.tolist()
+    for b in range(num_seqs):
+        yield cu[b], cu[b + 1], lens[b] - (cu[b + 1] - cu[b]), slots[b]
+
+
+def hyper_norm(streams, ids, table, num_streams, y, conn, w_in, norm_w, norm_b, eps, true_width, out_scale, shift,
+               keep):
+    if ids is not None:
+        x = table[ids.long()].float()
+        new = x.unsqueeze(1).expand(-1, num_streams, -1).contiguous()
+    else:
+        ls, mix, w_out = conn
+        new = torch.einsum("tsw,sr->trw", streams, mix) + w_out[None, :, None] * (y.float() * ls.float())[:, None, :]
+    u = torch.einsum("tsw,s->tw", new, w_in)[:, :true_width]
+    c = u - u.mean(-1, keepdim=True)
+    n = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps)
+    h = torch.zeros_like(new[:, 0])
+    h[:, :true_width] = (n * norm_w[:true_width].float() + norm_b[:true_width].float()) * out_scale
+    if shift is not None:
+        mu, state, _, state_slots, cu_q, seq_lens, num_seqs = shift
+        before = torch.zeros_like(h)
+        before[1:] = h[:-1]
+        for lo, hi, start, slot in _portions(cu_q, seq_lens, state_slots, num_seqs):
+            before[lo] = state[slot] if start > 0 and slot >= 0 else 0
+            if slot >= 0:
+                state[slot] = h[hi - 1]
+        h = h + (before - h) * mu.float()
+    return (new if keep else None), h.to(norm_w.dtype)
+
+
+def gated_linear_prep(proj, q_off, f_off, heads, dim, f_bias, lower):
+    """q = silu(projection) and the keys 1 - f = (1 - lower) * sigmoid(-(projection + bias)), fp32
+    [T, heads, dim rounded up to 4]."""
+    t, n = proj.shape[0], heads * dim
+    q = F.silu(proj[:, q_off: q_off + n].float())
+    k = (1 - lower) * torch.sigmoid(-(proj[:, f_off: f_off + n].float() + f_bias))
+    return tuple(F.pad(x.view(t, heads, dim), (0, -dim % 4)) for x in (q, k))
+
+
+def delta_prep(proj, low, offs, heads, kv_heads, dim, vdim, conv_w, conv_state, dt_bias, a_log, unit_eps, seq_idx,
+               state_slots, cu_q, seq_lens, num_seqs):
+    """Short convolutions + silu of q / k / v, unit norms, decays and step sizes: q, k [T, G, dim],
+    g [T, H, dim] (dim rounded up to 4) and beta [T, H] in fp32, v [T, H * vdim] in the projection's type."""
+    t, taps, c = proj.shape[0], conv_w.shape[1], conv_w.shape[0]
+    x = proj[:, :c].float()
+    y = torch.zeros_like(x)
+    for lo, hi, start, slot in _portions(cu_q, seq_lens, state_slots, num_seqs):
+        before = conv_state[slot].float() if start > 0 and slot >= 0 else x.new_zeros(taps - 1, c)
+        ext = torch.cat([before, x[lo:hi]])
+        for j in range(taps):
+            y[lo:hi] += conv_w[:, j].float() * ext[j: j + hi - lo]
+    y = F.silu(y)
+
+    def heads_of(name, n, d):
+        return y[:, offs[name]: offs[name] + n * d].reshape(t, n, d)
+
+    def unit(z):
+        return z * torch.rsqrt(z.pow(2).sum(-1, keepdim=True) + unit_eps)
+
+    q = unit(heads_of("q", kv_heads, dim)) * dim ** -0.5
+    k = unit(heads_of("k", kv_heads, dim))
+    v = heads_of("v", heads, vdim).reshape(t, heads * vdim).to(proj.dtype)
+    rate = F.softplus(low[:, : heads * dim].float() + dt_bias).view(t, heads, dim)
+    g = torch.exp(-torch.exp(a_log)[None, :, None] * rate)
+    beta = torch.sigmoid(proj[:, offs["b"]: offs["b"] + heads].float())
+    pad = (0, -dim % 4)
+    return F.pad(q, pad), F.pad(k, pad), F.pad(g, pad), v, beta
+
+
+def recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, conv=None):
+    """Token by token, per head: S <- g S (g None: 1 - k), then S <- S + k u^T with u = v, or with ``beta``
+    u = beta (v - S^T k); o = S^T q.  q, k [T, G, d], v [T, heads * vdim] -> o [T, heads, vdim] fp32.
+    ``state`` [slots, heads, vdim, d] holds S^T; ``conv`` = (proj, conv_state): the newest convolution
+    inputs are stored too."""
+    per = heads // q.shape[1]
+    o = torch.zeros(q.shape[0], heads, vdim)
+    vv = v.float().view(-1, heads, vdim)
+    qq, kk = (x.repeat_interleave(per, dim=1) for x in (q, k))
+    for lo, hi, start, slot in _portions(cu_q, seq_lens, state_slots, num_seqs):
+        s = state[slot].clone() if start > 0 and slot >= 0 else torch.zeros(heads, vdim, q.shape[-1])
+        for t in range(lo, hi):
+            s = s * (g[t] if g is not None else 1 - kk[t])[:, None, :]
+            u = vv[t]
+            if beta is not None:
+                u = beta[t][:, None] * (u - torch.einsum("hed,hd->he", s, kk[t]))
+            s = s + u[:, :, None] * kk[t][:, None, :]
+            o[t] = torch.einsum("hed,hd->he", s, qq[t])
+        if slot < 0:
+            continue
+        state[slot] = s
+        if conv is not None:
+            proj, cs = conv
+            keep = cs.shape[1]
+            before = cs[slot] if start > 0 else torch.zeros_like(cs[slot])
+            ext = torch.cat([before, proj[lo:hi, : cs.shape[2]]])
+            cs[slot] = ext[ext.shape[0] - keep:]
+    return o
+
+
+def head_norm_gate(o, weight, eps, gate, out_width):
+    """Per-head RMS norm (plain weight), times the sigmoid of ``gate``; [T, out_width] in the weight's type."""
+    t, heads, d = o.shape
+    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+    y = y.reshape(t, heads * d)
+    if gate is not None:
+        y = y * torch.sigmoid(gate.float())
+    return F.pad(y, (0, out_width - heads * d)).to(weight.dtype)
+
+
+# ------------------------------------------------------------- latent attention of any size
+def latent_prep_(q, kv_a, norm_w, eps, cache, positions, slot_mapping, cos_sin, heads, dim, rot, rank, neox, q_latent):
+    t = q.shape[0]
+    half = rot // 2
+    cs = cos_sin[positions.long()]
+    cos, sin = cs[:, :half], cs[:, half:]
+    qv = q[:, : heads * (dim + rot)].unflatten(1, (heads, dim + rot))
+    q_rot = _rope_one(qv[..., dim:].contiguous(), cos, sin, rot, neox)
+    if q_latent is None:
+        qv[..., dim:] = q_rot
+    else:
+        q_latent[:t, :, rank: rank + rot] = q_rot
+        q_latent[:t, :, rank + rot:] = 0
+    c = kv_a[:, :rank].float()
+    c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
+    pe = _rope_one(kv_a[:, rank: rank + rot].reshape(t, 1, rot), cos, sin, rot, neox).view(t, rot)
+    row = F.pad(torch.cat([c.to(cache.dtype), pe.to(cache.dtype)], -1), (0, cache.shape[-1] - rank - rot))
+    paged_scatter_rows(cache, row, slot_mapping)
+
+
+def head_gemm(a, w, out):
+    out.copy_(torch.einsum("thk,hnk->thn", a.float(), w.float()))
+
+
+def latent_gather(cache, block_tables, seq_lens, num_seqs):
+    bs = cache.shape[1]
+    rows = []
+    for b in range(num_seqs):
+        pos = torch.arange(int(seq_lens[b]))
+        rows.append(cache.view(-1, cache.shape[-1])[block_tables[b][pos // bs].long() * bs + pos % bs])
+    return torch.cat(rows)
+
+
+def latent_decode(q, cache, block_tables, seq_lens, num_seqs, heads, rank, scale, out):
+    """Absorbed decode attention: q [B, heads, row], cache [blocks, bs, row]; the values are the first
+    ``rank`` columns of a row.  out [B, heads, rank]."""
+    for b in range(num_seqs):
+        kv = latent_gather(cache, block_tables[b:b + 1], seq_lens[b:b + 1], 1).float()
+        p = torch.softmax(q[b].float() @ kv.t() * scale, dim=-1)
+        out[b] = (p @ kv[:, :rank]).to(out.dtype)

@@ -5,7 +5,7 @@ of computed tokens, sampling parameters).  A step's device inputs are built with
 vectorised numpy operations into ONE pinned int32 staging buffer laid out as
 
     [ input_ids | positions | slot_mapping | seq_lens | cu_q | temperature(f32 bits)
-      | top_k | top_p(f32 bits) | block_table rows ]
+      | top_k | top_p(f32 bits) | sequence of each token | state slots | block_table rows ]
 
 and shipped with a single host-to-device copy.  For every CUDA-graph batch size
 the section offsets are fixed, so the captured graph reads the same device
@@ -39,6 +39,8 @@ class StepLayout:
     seeds: int = 0
     logits_idx: int = 0
     next_ids: int = 0
+    seq: int = 0
+    state: int = 0
     bt: int = 0
     total: int = 0
 
@@ -48,7 +50,7 @@ class StepLayout:
         off = 0
         for name, n in (("ids", T), ("pos", T), ("slot", T), ("seq_lens", S), ("cu_q", S + 1),
                         ("temp", S), ("top_k", S), ("top_p", S), ("seeds", 2 * S),
-                        ("logits_idx", S), ("next_ids", T), ("bt", S * max_blocks)):
+                        ("logits_idx", S), ("next_ids", T), ("seq", T), ("state", S), ("bt", S * max_blocks)):
             off = (off + 3) // 4 * 4           # 16-byte aligned sections
             setattr(lay, name, off)
             off += n
@@ -160,6 +162,8 @@ class InputBatch:
             "seeds": buf[lay.seeds: lay.seeds + 2 * S].view(torch.int64),
             "logits_idx": buf[lay.logits_idx: lay.logits_idx + S],
             "next_ids": buf[lay.next_ids: lay.next_ids + T],
+            "seq": buf[lay.seq: lay.seq + T],
+            "state": buf[lay.state: lay.state + S],
             "bt": buf[lay.bt: lay.bt + S * mb].view(S, mb),
         }
 
@@ -242,6 +246,9 @@ class InputBatch:
         h[lay.cu_q: lay.cu_q + lay.S + 1] = np.arange(lay.S + 1, dtype=np.int32) * q_len
         h[lay.logits_idx: lay.logits_idx + lay.S] = np.arange(lay.S, dtype=np.int32)
         h[lay.next_ids: lay.next_ids + lay.T] = -1
+        h[lay.seq: lay.seq + lay.T] = np.arange(lay.T, dtype=np.int32) // q_len
+        h[lay.state: lay.state + lay.S] = -1
+        h[lay.state: lay.state + n] = np.fromiter((r.state_slot for r in reqs), dtype=np.int32, count=n)
         self._fill_sampling(lay, rows, n, [len(r.output_token_ids) for r in reqs])
         bt = h[lay.bt: lay.bt + lay.S * lay.max_blocks].reshape(lay.S, lay.max_blocks)
         bt[:n] = self.block_table[rows]
@@ -276,6 +283,8 @@ class InputBatch:
             h[lay.pos + off: lay.pos + off + q] = p
             h[lay.slot + off: lay.slot + off + q] = self._slots(row, p)
             h[lay.seq_lens + i] = s.start + q
+            h[lay.seq + off: lay.seq + off + q] = i
+            h[lay.state + i] = req.state_slot
             off += q
             cu[i + 1] = off
             h[lay.logits_idx + i] = off - 1
@@ -321,6 +330,8 @@ class InputBatch:
             h[lay.next_ids + off: lay.next_ids + off + q - 1] = toks[1:]
             nxt = s.start + q
             h[lay.next_ids + off + q - 1] = req.token_at(nxt) if nxt < req.num_tokens else -1
+            h[lay.seq + off: lay.seq + off + q] = i
+            h[lay.state + i] = req.state_slot
             off += q
             cu[i + 1] = off
             h[lay.logits_idx + i] = off - 1

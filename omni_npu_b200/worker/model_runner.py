@@ -53,6 +53,7 @@ class ModelRunner:
         self.model_config = config.model
         self.model: Optional[torch.nn.Module] = None
         self.kv_caches: List = []
+        self.states: Optional[List] = None        # recurrent state per layer run (models that have one)
         self.num_blocks = 0
         sc = config.scheduler
         dcp = config.parallel.decode_context_parallel_size
@@ -207,7 +208,14 @@ class ModelRunner:
                     cc.block_size, n * spec.bytes_per_block / 2**30, peak / 2**30)
         return n
 
+    @property
+    def num_state_slots(self) -> int:
+        """Slots of recurrent state: one per sequence that can run at once, 0 without such a state."""
+        return self.config.scheduler.max_num_seqs if getattr(self.model, "has_recurrent_state", False) else 0
+
     def _init_kv_cache_tensors(self, num_blocks: int) -> None:
+        if self.states is None and self.num_state_slots:
+            self.states = self.model.allocate_states(self.num_state_slots, self.device)
         alloc = getattr(self.model, "allocate_kv_cache", None)
         if callable(alloc):
             self.kv_caches = alloc(num_blocks, self.config.cache.block_size, self.device)
@@ -233,7 +241,7 @@ class ModelRunner:
                                  positions=views["pos"], slot_mapping=views["slot"],
                                  block_tables=views["bt"], seq_lens=views["seq_lens"],
                                  cu_q=views["cu_q"], num_actual_tokens=actual_tokens,
-                                 num_actual_seqs=actual_seqs)
+                                 num_actual_seqs=actual_seqs, seq_idx=views["seq"], state_slots=views["state"])
 
     def _forward_and_sample(self, views, md: AttentionMetadata, num_samples: int) -> torch.Tensor:
         """Model forward + LM head + sampling for the staged step (device side only).
@@ -241,7 +249,7 @@ class ModelRunner:
         the sampled token and the k drafts for the tokens after it."""
         if self.pp_group is not None:
             return self._forward_and_sample_pipeline(views, md, num_samples)
-        with set_forward_context(md, self.kv_caches, self.config):
+        with set_forward_context(md, self.kv_caches, self.config, states=self.states):
             hidden_all = self.model(views["ids"], views["pos"])
             idx = views["logits_idx"][:num_samples].long() if md.is_prefill else None
             hidden = hidden_all.index_select(0, idx) if idx is not None else hidden_all[:num_samples]
@@ -830,12 +838,12 @@ class ModelRunner:
                     md, is_prefill=False, num_seqs=nd, num_tokens=nd, max_q_len=1, q_len=1,
                     positions=views["pos"][:nd], slot_mapping=views["slot"][:nd], block_tables=views["bt"][:nd],
                     seq_lens=views["seq_lens"][:nd], cu_q=views["cu_q"][: nd + 1], num_actual_tokens=nd,
-                    num_actual_seqs=nd, extra={"seq_lens_host": lens[:nd]})
+                    num_actual_seqs=nd, seq_idx=None, state_slots=None, extra={"seq_lens_host": lens[:nd]})
                 md.extra["md_prefill"] = dataclasses.replace(
                     md, num_seqs=n - nd, num_tokens=T - nd, max_q_len=md.extra["max_q_len_prefill"],
                     positions=views["pos"][nd:T], slot_mapping=views["slot"][nd:T], block_tables=views["bt"][nd:n],
                     seq_lens=views["seq_lens"][nd:n], cu_q=md.extra["cu_q_prefill"], num_actual_tokens=T - nd,
-                    num_actual_seqs=n - nd, extra={"seq_lens_host": lens[nd:]})
+                    num_actual_seqs=n - nd, seq_idx=None, state_slots=None, extra={"seq_lens_host": lens[nd:]})
             sampled = self._forward_and_sample(views, md, n)
         self.step_counter += 1
         self._event_stop(ev, out.kind)
@@ -974,6 +982,8 @@ class ModelRunner:
             h[lay.pos: lay.pos + T] = pos
             h[lay.slot: lay.slot + T] = -1
             h[lay.next_ids: lay.next_ids + T] = 0
+            h[lay.seq: lay.seq + T] = np.repeat(np.arange(n_seq, dtype=np.int32), per)
+            h[lay.state: lay.state + n_seq] = -1
             h[lay.seq_lens: lay.seq_lens + n_seq] = per
             h[lay.cu_q: lay.cu_q + n_seq + 1] = np.arange(n_seq + 1, dtype=np.int32) * per
             h[lay.logits_idx: lay.logits_idx + n_seq] = np.arange(1, n_seq + 1, dtype=np.int32) * per - 1

@@ -13,6 +13,7 @@ of host-side arguments: lengths live in device memory here.
 from __future__ import annotations
 
 import dataclasses
+import gc
 import os
 import weakref
 from typing import Any, Callable, Dict, Hashable, Optional
@@ -40,9 +41,17 @@ class CUDAGraphRunner:
         torch.cuda.current_stream(self.device).wait_stream(stream)
         torch.cuda.synchronize(self.device)
         self.graph = torch.cuda.CUDAGraph()
-        with ops.count_capture() as cc:
-            with torch.cuda.graph(self.graph, pool=self.pool):
-                self.output = self.fn()
+        # a graph of an earlier engine that the collector frees meanwhile would invalidate the capture
+        gc.collect()
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with ops.count_capture() as cc:
+                with torch.cuda.graph(self.graph, pool=self.pool):
+                    self.output = self.fn()
+        finally:
+            if collecting:
+                gc.enable()
         self.num_kernels = cc.kernels
         if self.pool is None:
             self.pool = self.graph.pool()

@@ -1,9 +1,11 @@
 """Throughput of a design beside the framework's closest existing model at equal size (random weights).
 
-``bench.py --design rivudra`` runs this on one GPU.  Per size it prints one JSON line with
+``bench.py --design rivudra`` or ``--design fuvirax`` runs this on one GPU.  Per size it prints one JSON line
+with
 
 * whole steps through the engine (device time of prompt and decode steps, CUDA events): Rivudra and a
-  Qwen3-MoE of the same width, heads, experts and window;
+  Qwen3-MoE of the same width, heads, experts and window, or Fuvirax and a dense DeepSeek-V2 of the same
+  width, heads, latent sizes and feed-forward;
 * single kernels: time, the fraction of the measured roofline (the slower of bytes / copy bandwidth and
   FLOPs / library bf16 GEMM throughput) and the same for the like kernel of the other model.  Between
   iterations a 256 MB buffer is written, so inputs come from HBM.
@@ -18,7 +20,8 @@ from typing import Callable, Dict, List, Optional, Tuple
 import torch
 
 from .. import ops
-from ..config import AttentionSpec, ExpertSpec, LayerSpec, ModelConfig, MoESpec
+from ..config import (AttentionSpec, DeltaRuleSpec, DenseSpec, ExpertSpec, GatedLinearSpec, LatentAttentionSpec, LayerSpec,
+                      ModelConfig, MoESpec)
 
 LAYERS = 4
 CLAMPED = (1.702, 7.0)
@@ -230,15 +233,217 @@ def kernels(size) -> List[dict]:
     return out
 
 
+# ----------------------------------------------------------------------------- Fuvirax
+# width, heads, head size (states and unrotated keys), value size, rotated keys, latent, feed-forward, streams
+FUVIRAX_SIZES: Dict[str, Tuple[int, ...]] = {
+    "2048x16h/128 ff8192 s2": (2048, 16, 128, 128, 64, 512, 8192, 2),
+    "4096x32h/128 ff12288 s4": (4096, 32, 128, 128, 64, 512, 12288, 4),
+    "3072x24h/128 ff8192 s3": (3072, 24, 128, 128, 64, 512, 8192, 3),
+}
+FUVIRAX_LAYERS = 6           # two of each mixer
+LOW_RANK = 128
+TAPS = 4
+# fp32 multiply-adds per second of the CUDA cores at the maximum clock: what bounds the recurrences
+FP32_FLOPS = 148 * 128 * 2 * 1.965e9
+
+
+def fuvirax(size) -> ModelConfig:
+    w, h, d, e, rot, rank, ff, streams = size
+    mlp = DenseSpec(ff)
+    specs = (LayerSpec(GatedLinearSpec(h, d, e), mlp), LayerSpec(DeltaRuleSpec(h, h, d, e, TAPS, LOW_RANK, LOW_RANK), mlp),
+             LayerSpec(LatentAttentionSpec(h, d, rot, e, rank, 1e4, (d + rot) ** -0.5), mlp))
+    return ModelConfig(architecture="Fuvirax", model_type="fuvirax", hidden_size=w, num_layers=FUVIRAX_LAYERS, num_heads=h,
+                       num_kv_heads=1, head_dim=e, vocab_size=VOCAB, max_position_embeddings=1 << 16,
+                       layer_specs=specs * (FUVIRAX_LAYERS // 3), residual_streams=streams, tie_word_embeddings=True)
+
+
+def deepseek_dense(size) -> ModelConfig:
+    w, h, d, e, rot, rank, ff, _ = size
+    return ModelConfig(architecture="DeepseekV2ForCausalLM", model_type="deepseek_v2", hidden_size=w,
+                       num_layers=FUVIRAX_LAYERS, num_heads=h, num_kv_heads=h, head_dim=d + rot, intermediate_size=ff,
+                       vocab_size=VOCAB, max_position_embeddings=1 << 16, rope_neox=False, use_mla=True,
+                       kv_lora_rank=rank, qk_nope_head_dim=d, qk_rope_head_dim=rot, v_head_dim=e)
+
+
+def fuvirax_kernels(size) -> List[dict]:
+    from ..attention.latent import LatentAttention
+    w, h, d, e, rot, rank, ff, ns = size
+    bw, fl = _peaks()
+    out: List[dict] = []
+    bf = dict(dtype=torch.bfloat16, device="cuda")
+    f32 = dict(dtype=torch.float32, device="cuda")
+    i32 = dict(dtype=torch.int32, device="cuda")
+
+    def entry(name: str, fn, nbytes: float, flops: float = 0.0, like: Optional[Tuple] = None, peak: float = fl):
+        ms = _time(fn)
+        bound = max(nbytes / bw, flops / peak) * 1e3
+        r = {"kernel": name, "ms": round(ms, 4), "roofline": round(bound / ms, 3)}
+        if like is not None:
+            lms = _time(like[0])
+            lb = max(like[1] / bw, like[2] / fl) * 1e3
+            r.update(like_ms=round(lms, 4), like_roofline=round(lb / lms, 3),
+                     distance=round((lb / lms) / (bound / ms), 2))
+        out.append(r)
+
+    bs, qk, row = 64, d + rot, rank + rot
+    for kind, n, rows in (("prefill", 8, 1024), ("decode b1", 1, 1), ("decode b16", 16, 1), ("decode b128", 128, 1)):
+        t, pre = n * rows, kind == "prefill"
+        ctx = rows if pre else CONTEXT
+        x = torch.randn(t, w, **bf)
+        gain, bias = torch.randn(w, **bf), torch.randn(w, **bf)
+        cu = torch.arange(0, (n + 1) * rows, rows, **i32)
+        lens = torch.full((n,), ctx, **i32)
+        slots, idx = torch.arange(n, **i32), torch.arange(n, **i32).repeat_interleave(rows)
+        states = (slots, cu, lens, n)
+        # ---- join + norm (+ token shift) against add + norm
+        st = torch.randn(t, ns, w, **f32)
+        conn = (gain, torch.eye(ns, **f32), torch.ones(ns, **f32))
+        w_in, shift_state = torch.ones(ns, **f32), torch.zeros(n, w, **f32)
+        shift = (gain, shift_state, idx, *states)
+        res16 = torch.randn(t, w, **bf)
+        like_norm = (lambda: ops.fused_add_rms_norm(x, res16, gain, 1e-6), t * w * 2 * 4, 0)
+        for label, sh in (("with token shift", shift), ("no shift", None)):
+            entry(f"join + norm {label}, {kind}",
+                  lambda sh=sh: ops.hyper_norm(st, None, None, ns, x, conn, w_in, gain, bias, 1e-5, w, 1.0, sh),
+                  t * w * (8 * ns + 4) + (n * w * 8 if sh else 0), 0, like_norm)
+        del st
+        # ---- products
+        def product(name, cols, like_cols=h * qk):
+            a, b = torch.randn(cols, w, **bf), torch.randn(like_cols, w, **bf)
+            entry(f"{name}, {kind}", lambda: ops.gemm(x, a), (a.numel() + x.numel() + t * cols) * 2, 2.0 * t * a.numel(),
+                  (lambda: ops.gemm(x, b), (b.numel() + x.numel() + t * like_cols) * 2, 2.0 * t * b.numel()))
+        delta_cols = h * (2 * d + e) + (h + 7) // 8 * 8 + 2 * LOW_RANK
+        product("projection, gated linear (like: q of MLA)", h * (2 * d + e))
+        product("projection, delta rule (like: q of MLA)", delta_cols)
+        product("projection, latent (like: q of MLA)", h * qk + row)
+        up, gu = torch.randn(ff, w, **bf), torch.randn(2 * ff, w, **bf)
+        entry(f"up + xielu (like: gate/up + silu), {kind}", lambda: ops.gemm(x, up, xielu=(0.7, 0.9)),
+              (up.numel() + x.numel() + t * ff) * 2, 2.0 * t * up.numel(),
+              (lambda: ops.gemm(x, gu, swiglu=True), (gu.numel() + x.numel() + t * ff) * 2, 2.0 * t * gu.numel()))
+        del up, gu
+        # ---- attention inputs: paged latent rows, queries
+        per = (ctx + bs - 1) // bs
+        cache = torch.randn(n * per, bs, row, **bf)
+        bt = torch.randperm(n * per, device="cuda").int().view(n, per)
+        pos = torch.arange(ctx - rows, ctx, **i32).repeat(n)
+        slot = (bt.long().gather(1, (pos.view(n, rows) // bs).long()) * bs + pos.view(n, rows) % bs).int().view(-1)
+        cs = torch.randn(CONTEXT + 128, rot, device="cuda")
+        q, kv_a = torch.randn(t, h * qk, **bf), torch.randn(t, row, **bf)
+        attn = LatentAttention(h, d, rot, e, rank, qk ** -0.5, True, 1e-5, torch.bfloat16, torch.device("cuda"))
+        attn.w_uk.data.normal_(std=0.02)
+        attn.w_uv.data.normal_(std=0.02)
+        attn.build_absorbed()
+        q_lat = torch.empty(t, h, row, **bf)
+        def like_prep():
+            ops.mla_kv_rmsnorm_rope_cache(kv_a[:, :rank], kv_a[:, rank:], attn.latent_norm, cache, pos, slot, cs, 1e-5, False)
+            pe = q.view(t, h, qk)[:, :, d:].reshape(t, h * rot).contiguous()
+            ops.rope_qk_(pe, pe.new_empty(t, 0), pos, cs, rot, rot, False)
+        moved = t * (2 * row + 2 * h * rot) * 2
+        entry(f"latent norm + rotation + cache, {kind}",
+              lambda: ops.latent_prep_(q, kv_a, attn.latent_norm, 1e-5, cache, pos, slot, cs, h, d, rot, rank, True,
+                                       None if pre else q_lat, 0 if pre else t), moved, 0, (like_prep, moved, 0))
+        pairs = n * h * sum(p + 1 for p in range(ctx - rows, ctx))
+        if pre:
+            start = (torch.cumsum(lens, 0) - lens).int()
+            def own_keys():
+                r = ops.latent_gather(cache, bt, lens, start, n, t, ctx)
+                return ops.gemm(r, attn.w_key), ops.gemm(r, attn.w_value)
+            kvb = torch.randn(h * (d + e), rank, **bf)
+            def like_keys():
+                lat = cache.index_select(0, bt.view(-1).long())
+                kv = ops.gemm(lat[..., :rank].reshape(-1, rank).contiguous(), kvb).view(-1, bs, h, d + e)
+                pe = lat[..., rank:].unsqueeze(2).expand(-1, bs, h, rot)
+                k = torch.cat([kv[..., :d], pe], -1).permute(0, 2, 1, 3).contiguous()
+                return k, kv[..., d:].permute(0, 2, 1, 3).contiguous()
+            kbytes, kflops = t * (row + h * (qk + e)) * 2 + kvb.numel() * 2, 2.0 * t * kvb.numel()
+            entry(f"keys and values from the latents, {kind}", own_keys, kbytes, kflops, (like_keys, kbytes, kflops))
+            k, v = own_keys()
+            o = torch.empty(t, h * e, **bf)
+            lk, lv = like_keys()
+            lbt = torch.arange(n * per, **i32).view(n, per)
+            abytes, aflops = t * h * (2 * qk + 2 * e) * 2, 2.0 * pairs * (qk + e)
+            like_attn = (lambda: ops.gqa_prefill(q, lk, lv, lbt, cu, lens, n, rows, h, 0.07, True, 0), abytes, aflops)
+            entry(f"attention, {kind}",
+                  lambda: ops.contiguous_attention(q, k.view(-1, h, 1, qk), v.view(-1, h, 1, e), o, cu, start, lens, n, rows,
+                                                   h, qk, e, 0.07), abytes, aflops, like_attn)
+        else:
+            lat_o, o = torch.empty(t, h, rank, **bf), torch.empty(t, h * e, **bf)
+            heads = q.view(t, h, qk)
+            uv = attn.w_uv.view(h, e, rank)
+            offs = torch.arange(0, (h + 1) * t, t, **i32)
+            def like_fold():
+                qn = heads[..., :d].transpose(0, 1).reshape(h * t, d).contiguous()
+                ql = ops.grouped_gemm(qn, attn.w_fold, offs).view(h, t, rank).transpose(0, 1)
+                return torch.cat([ql, q_lat[..., rank:]], -1).reshape(t, h * row).contiguous()
+            def like_unfold():
+                a = lat_o.transpose(0, 1).reshape(h * t, rank).contiguous()
+                return ops.grouped_gemm(a, uv, offs).view(h, t, e).transpose(0, 1).reshape(t, h * e).contiguous()
+            fb, ff_ = (h * d * rank + t * h * (d + rank)) * 2, 2.0 * t * h * d * rank
+            entry(f"queries into the latent space, {kind}",
+                  lambda: ops.head_gemm(heads[..., :d], attn.w_fold, q_lat[..., :rank]), fb, ff_, (like_fold, fb, ff_))
+            ub, uf = (h * e * rank + t * h * (e + rank)) * 2, 2.0 * t * h * e * rank
+            entry(f"results out of the latent space, {kind}", lambda: ops.head_gemm(lat_o, uv, o.view(t, h, e)), ub, uf,
+                  (like_unfold, ub, uf))
+            abytes, aflops = (n * ctx * row + t * h * (row + rank)) * 2, 2.0 * pairs * (row + rank)
+            q_flat = torch.randn(t, h * row, **bf)
+            like_attn = (lambda: ops.mla_decode(q_flat, cache, bt, lens, n, h, 0.07, 1, max_seq_len=CONTEXT), abytes, aflops)
+            entry(f"attention, {kind}",
+                  lambda: ops.latent_decode(q_flat.view(t, h, row), cache, bt, lens, n, h, rank, 0.07, lat_o,
+                                            max_seq_len=CONTEXT), abytes, aflops, like_attn)
+        # ---- recurrent layers; the like kernel of the scans is attention
+        proj = torch.randn(t, delta_cols, **bf)
+        fb_, low_ = torch.randn(h * d, **f32), torch.rand(h * d, **f32)
+        state = torch.zeros(n, h, e, d, **f32)
+        rw = n * h * e * d * 8                                  # the state is read and written once per step
+        entry(f"gated linear: q and keys (like: norm + rotation + cache of MLA), {kind}",
+              lambda: ops.gated_linear_prep(proj, 0, h * d, h, d, fb_, low_), t * h * d * (4 + 8), 0, (like_prep, moved, 0))
+        qf, kf = ops.gated_linear_prep(proj, 0, h * d, h, d, fb_, low_)
+        v = proj[:, 2 * h * d: 2 * h * d + h * e]
+        entry(f"gated linear: scan (like: attention), {kind}",
+              lambda: ops.recurrent_scan(qf, kf, None, v, None, state, h, e, *states),
+              t * h * (8 * d + 6 * e) + rw, 5.0 * t * h * d * e, like_attn, FP32_FLOPS)
+        offs_ = {"q": 0, "k": h * d, "v": 2 * h * d, "b": h * (2 * d + e)}
+        ch = offs_["b"]
+        conv_w, conv_state = torch.randn(ch, TAPS, **bf), torch.zeros(n, TAPS - 1, ch, **bf)
+        lowp = torch.randn(t, h * (d + e), **bf)
+        dt, a_log = torch.randn(h * d, **f32), torch.randn(h, **f32)
+        prep = lambda: ops.delta_prep(proj, lowp[:, : h * d], offs_, h, h, d, e, conv_w, conv_state, dt, a_log, 1e-6,  # noqa: E731
+                                      idx, *states)
+        entry(f"delta rule: convolutions, norms, decays (like: norm + rotation + cache of MLA), {kind}", prep,
+              t * h * ((2 * d + e) * 2 + 2 * d + 12 * d + 2 * e), 0, (like_prep, moved, 0))
+        qf, kf, gf, vf, beta = prep()
+        entry(f"delta rule: scan (like: attention), {kind}",
+              lambda: ops.recurrent_scan(qf, kf, gf, vf, beta, state, h, e, *states, conv=(proj, conv_state)),
+              t * h * (12 * d + 6 * e) + rw, 7.0 * t * h * d * e, like_attn, FP32_FLOPS)
+        low_w = torch.randn(h * (d + e), 2 * LOW_RANK, **bf)
+        lp = torch.randn(t, 2 * LOW_RANK, **bf)
+        entry(f"delta rule: low-rank product, {kind}", lambda: ops.gemm(lp, low_w),
+              (lp.numel() + low_w.numel() + t * h * (d + e)) * 2, 2.0 * t * low_w.numel())
+        of, gate, ow = torch.randn(t, h, e, **f32), lowp[:, h * d:], torch.randn(e, **bf)
+        flat = torch.randn(t, h * e, **bf)
+        fw = torch.randn(h * e, **bf)
+        entry(f"head norm + gate (like: norm), {kind}", lambda: ops.head_norm_gate(of, ow, 1e-5, gate, h * e), t * h * e * 8,
+              0, (lambda: ops.rms_norm(flat, fw, 1e-6), t * h * e * 4, 0))
+        del proj, lowp, cache, q, qf, kf, gf, vf, of
+        gc.collect()
+        torch.cuda.empty_cache()
+    ops.check_status()
+    return out
+
+
+DESIGNS = {
+    "rivudra": (SIZES, LAYERS, kernels, {"rivudra": rivudra, "qwen3-moe": qwen3_moe}),
+    "fuvirax": (FUVIRAX_SIZES, FUVIRAX_LAYERS, fuvirax_kernels, {"fuvirax": fuvirax, "deepseek-v2 dense": deepseek_dense}),
+}
+
+
 def run(design: str, only: Optional[str] = None) -> None:
-    if design != "rivudra":
-        raise SystemExit(f"no comparison for design {design!r}")
+    sizes, layers, kernel_table, models = DESIGNS[design]
     ops.load_extension(required=True)
-    for name, size in SIZES.items():
+    for name, size in sizes.items():
         if only and only not in name:
             continue
-        line = {"design": design, "size": name, "layers": LAYERS, "dtype": "bf16", "data": "random",
+        line = {"design": design, "size": name, "layers": layers, "dtype": "bf16", "data": "random",
                 "l2_policy": "kernels: 256 MB written before each; steps: weights and cache above L2",
-                "kernels": kernels(size), "steps": {"rivudra": model_steps(rivudra(size)),
-                                                    "qwen3-moe": model_steps(qwen3_moe(size))}}
+                "kernels": kernel_table(size), "steps": {k: model_steps(make(size)) for k, make in models.items()}}
         print(json.dumps(line), flush=True)

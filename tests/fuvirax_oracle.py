@@ -70,12 +70,12 @@ def rotate_halves(x: torch.Tensor, positions: torch.Tensor, base: float) -> torc
 
 
 # ------------------------------------------------------------------ mixers
-def latent_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> torch.Tensor:
-    t, heads, d, r, e, rank = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+def latent_core(q: torch.Tensor, down: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> torch.Tensor:
+    """Queries q [T, H * (dim + rot)] over latents down [T, rank + rot] -> heads [T, H * vdim]."""
+    t, heads, d, r, e, rank = q.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
     pos = torch.arange(t)
-    q = (h @ w["q"].T).view(t, heads, d + r)
+    q = q.view(t, heads, d + r)
     q_rot = rotate_halves(q[..., d:], pos, m["rot"]["base"])
-    down = h @ w["dkv"].T
     c = rms(down[:, :rank], eps) * w["dkv.norm"]
     k_rot = rotate_halves(down[:, None, rank:], pos, m["rot"]["base"])[:, 0]
     k = (c @ w["uk"].T).view(t, heads, d)
@@ -85,7 +85,11 @@ def latent_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: 
     for n in range(heads):
         s = (q[:, n, :d] @ k[:, n].T + q_rot[:, n] @ k_rot.T) * m["scale"]
         out.append(torch.softmax(s.masked_fill(hidden, -math.inf), -1) @ v[:, n])
-    return torch.cat(out, -1) @ w["o"].T
+    return torch.cat(out, -1)
+
+
+def latent_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> torch.Tensor:
+    return latent_core(h @ w["q"].T, h @ w["dkv"].T, w, m, eps) @ w["o"].T
 
 
 def gated_linear_scan(q: torch.Tensor, f: torch.Tensor, v: torch.Tensor) -> torch.Tensor:

@@ -116,6 +116,8 @@ def close(got: torch.Tensor, want: torch.Tensor, dtype: str) -> None:
 
 class Driver:
     """Requests with their oracle logits, fed in portions through a replay of the engine."""
+    oracle = oracle
+    close = staticmethod(close)
 
     def __init__(self, path, cfg, w, device, dtype, max_tokens=512, **kw) -> None:
         from omni_npu_b200.engine.trace_replay import TraceReplay
@@ -127,7 +129,7 @@ class Driver:
 
     def add(self, rid: str, n: int, seed: int) -> None:
         toks = tokens(n, self.cfg["vocab"], seed)
-        self.req[rid], self.at[rid] = (toks, oracle.forward(toks, self.w, self.cfg)), 0
+        self.req[rid], self.at[rid] = (toks, self.oracle.forward(toks, self.w, self.cfg)), 0
 
     def step(self, portions: Dict[str, int]) -> None:
         entries, end, rows = [], [], []
@@ -150,7 +152,7 @@ class Driver:
         self.replay.check()
         pool = self.replay.engine.scheduler.pool
         assert pool.num_free == pool.num_blocks - pool.num_reserved, "cache blocks were not given back"
-        close(torch.cat(self.got), torch.cat(self.want), self.dtype)
+        self.close(torch.cat(self.got), torch.cat(self.want), self.dtype)
 
 
 # ---------------------------------------------------------------------------- whole-model checks
@@ -198,7 +200,7 @@ def check_mixed(d: Driver, rounds: int = 3) -> None:
     d.finish()
 
 
-def check_generate(path, cfg, w, device, **kw) -> None:
+def check_generate(path, cfg, w, device, oracle=oracle, **kw) -> None:
     """Greedy generation through ``LLM.generate``: continuous batching over a small cache."""
     from omni_npu_b200 import LLM, SamplingParams
     prompts = [tokens(n, cfg["vocab"], 50 + n) for n in (1, 19, 40, 7, 28, 2)]
@@ -209,7 +211,7 @@ def check_generate(path, cfg, w, device, **kw) -> None:
         seq = list(p)
         for got in o.output_token_ids:
             logits = oracle.forward(seq, w, cfg)[-1]
-            assert float(logits.max() - logits[got]) < 1e-3          # the greedy token, or its equal
+            assert float(logits.max() - logits[got]) < 1e-3 * max(1.0, float(logits.std()))   # the greedy token, or its equal
             seq.append(got)
         assert len(o.output_token_ids) == 14
 

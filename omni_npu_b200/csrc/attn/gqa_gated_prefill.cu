@@ -17,11 +17,13 @@ namespace b200 {
 
 namespace gpre {
 constexpr int BM = 128, BN = 64, THREADS = 256;
-template <int DM>
+// DK, DV: upper bounds of the padded head sizes
+template <int DK, int DV>
 struct Cfg {
-  static constexpr int Q_BYTES = BM * DM * 2;
-  static constexpr int T_BYTES = BN * DM * 2;
-  static constexpr int SMEM = Q_BYTES + 4 * T_BYTES;
+  static constexpr int Q_BYTES = BM * DK * 2;
+  static constexpr int K_BYTES = BN * DK * 2;
+  static constexpr int V_BYTES = BN * DV * 2;
+  static constexpr int SMEM = Q_BYTES + 2 * K_BYTES + 2 * V_BYTES;
 };
 }  // namespace gpre
 
@@ -44,14 +46,16 @@ __device__ __forceinline__ void load_gated_tile(uint32_t dst, const __nv_bfloat1
                  "l"(src + c * 8), "r"(sz) : "memory");
 }
 
-template <int DM>
-__global__ void __launch_bounds__(gpre::THREADS, DM > 128 ? 1 : 2)
+// EXACT: the padded head sizes are DK and DV, and the query fragments stay in registers
+template <int DK, int DV, bool EXACT>
+__global__ void __launch_bounds__(gpre::THREADS, DK > 128 ? 1 : 2)
 gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
   using namespace gpre;
-  using C = Cfg<DM>;
+  using C = Cfg<DK, DV>;
+  const int DP = EXACT ? DK : p.DP, DVP = EXACT ? DV : p.DVP;
   extern __shared__ __align__(128) uint8_t smem[];
   uint8_t* sQ = smem;
-  const uint32_t kv0 = smem_u32(smem + C::Q_BYTES);
+  const uint32_t kv0 = smem_u32(smem + C::Q_BYTES), v0 = kv0 + 2 * C::K_BYTES;
 
   pdl_trigger();
   pdl_wait();
@@ -65,7 +69,7 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
   const long long q_begin = p.cu_q[b];
   const int q_len = static_cast<int>(p.cu_q[b + 1] - q_begin);
   // (the grid is laid out for heads_per_tile heads; a last, smaller chunk packs more tokens per tile)
-  const int m0 = blockIdx.x * tt;
+  const int m0 = (gridDim.x - 1 - blockIdx.x) * tt;                // (the tiles with most keys first)
   if (m0 >= q_len) return;
   const int kv_len = p.seq_lens[b];
   const int ctx = kv_len - q_len;
@@ -80,8 +84,8 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
   const int lo = p.window > 0 ? max(0, ctx + m0 - p.window + 1) / BN * BN : 0;
   const int tiles = (hi - lo + BN - 1) / BN;
 
-  load_gated_tile<DM>(kv0, kc, bt, lo, hi, kvh, p.Hk, p.block_size, p.DP, p.contiguous, tid);
-  load_gated_tile<DM>(kv0 + 2 * C::T_BYTES, vc, bt, lo, hi, kvh, p.Hk, p.block_size, p.DVP, p.contiguous, tid);
+  load_gated_tile<DK>(kv0, kc, bt, lo, hi, kvh, p.Hk, p.block_size, DP, p.contiguous, tid);
+  load_gated_tile<DV>(v0, vc, bt, lo, hi, kvh, p.Hk, p.block_size, DVP, p.contiguous, tid);
   asm volatile("cp.async.commit_group;" ::: "memory");
 
   // ---- query rows -> shared: two threads per row
@@ -92,7 +96,7 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
     const __nv_bfloat16* src = q + (ok ? (q_begin + tok) * p.q_stride +
                                              static_cast<long long>(kvh * per + head0 + r % hc) * p.D : 0);
     const bool vec = (p.D & 7) == 0 && ((p.q_stride & 7) == 0) && ((reinterpret_cast<uintptr_t>(q) & 15) == 0);
-    for (int c = tid & 1; c < (p.DP >> 3); c += 2) {
+    for (int c = tid & 1; c < (DP >> 3); c += 2) {
       uint4 u = make_uint4(0u, 0u, 0u, 0u);
       if (ok && vec) {
         if (c * 8 < p.D) u = *reinterpret_cast<const uint4*>(src + c * 8);
@@ -106,15 +110,16 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
           w[j] = static_cast<uint32_t>(__bfloat16_as_ushort(h[2 * j])) |
                  (static_cast<uint32_t>(__bfloat16_as_ushort(h[2 * j + 1])) << 16);
       }
-      *reinterpret_cast<uint4*>(sQ + tile_offset<DM>(r, c)) = u;
+      *reinterpret_cast<uint4*>(sQ + tile_offset<DK>(r, c)) = u;
     }
   }
 
-  float o_acc[DM / 8][4];
+  float o_acc[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < DM / 8; ++i)
+  for (int i = 0; i < DV / 8; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) o_acc[i][j] = 0.f;
+  uint32_t q_frag[EXACT ? DK / 16 : 1][4];
   // the sink is a key seen from the start: maximum = its score, sum = 1
   float row_max[2], row_sum[2];
   int pos[2];
@@ -132,33 +137,45 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
     const int st = it & 1;
     if (it + 1 < tiles) {
       const int nn = lo + (it + 1) * BN;
-      load_gated_tile<DM>(kv0 + (st ^ 1) * C::T_BYTES, kc, bt, nn, hi, kvh, p.Hk, p.block_size, p.DP, p.contiguous, tid);
-      load_gated_tile<DM>(kv0 + (2 + (st ^ 1)) * C::T_BYTES, vc, bt, nn, hi, kvh, p.Hk, p.block_size, p.DVP, p.contiguous, tid);
+      load_gated_tile<DK>(kv0 + (st ^ 1) * C::K_BYTES, kc, bt, nn, hi, kvh, p.Hk, p.block_size, DP, p.contiguous, tid);
+      load_gated_tile<DV>(v0 + (st ^ 1) * C::V_BYTES, vc, bt, nn, hi, kvh, p.Hk, p.block_size, DVP, p.contiguous, tid);
       asm volatile("cp.async.commit_group;" ::: "memory");
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
+    if constexpr (EXACT) {
+      if (it == 0) {
+#pragma unroll
+        for (int ks = 0; ks < DK / 16; ++ks)
+          ldmatrix_x4(q_frag[ks], smem_u32(sQ) + tile_offset<DK>(warp * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+      }
+    }
     const int n0 = lo + it * BN;
     // a warp none of whose rows sees a key of this tile has nothing to add
     const bool seen = n0 <= w_hi && (p.window <= 0 || n0 + BN - 1 > w_lo - p.window);
     if (seen) {
-      const uint32_t kt = kv0 + st * C::T_BYTES, vt = kv0 + (2 + st) * C::T_BYTES;
+      const uint32_t kt = kv0 + st * C::K_BYTES, vt = v0 + st * C::V_BYTES;
       float s[BN / 8][4];
 #pragma unroll
       for (int i = 0; i < BN / 8; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
 #pragma unroll
-      for (int ks = 0; ks < DM / 16; ++ks) {
-        if (ks * 16 < p.DP) {
+      for (int ks = 0; ks < DK / 16; ++ks) {
+        if (EXACT || ks * 16 < DP) {
           uint32_t qf[4];
-          ldmatrix_x4(qf, smem_u32(sQ) + tile_offset<DM>(warp * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+          if constexpr (EXACT) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) qf[j] = q_frag[ks][j];
+          } else {
+            ldmatrix_x4(qf, smem_u32(sQ) + tile_offset<DK>(warp * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+          }
 #pragma unroll
           for (int nt = 0; nt < BN / 16; ++nt) {
             uint32_t kf[4];
-            ldmatrix_x4(kf, kt + tile_offset<DM>(nt * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
+            ldmatrix_x4(kf, kt + tile_offset<DK>(nt * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
             mma_bf16_16816(s[2 * nt], qf, kf[0], kf[1]);
             mma_bf16_16816(s[2 * nt + 1], qf, kf[2], kf[3]);
           }
@@ -197,7 +214,7 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
         }
       if (corr[0] != 1.f || corr[1] != 1.f) {
 #pragma unroll
-        for (int i = 0; i < DM / 8; ++i)
+        for (int i = 0; i < DV / 8; ++i)
 #pragma unroll
           for (int j = 0; j < 4; ++j) o_acc[i][j] *= corr[j >> 1];
       }
@@ -209,10 +226,10 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
         pa[2] = pack_bf16x2(s[2 * ks + 1][0], s[2 * ks + 1][1]);
         pa[3] = pack_bf16x2(s[2 * ks + 1][2], s[2 * ks + 1][3]);
 #pragma unroll
-        for (int dt = 0; dt < DM / 16; ++dt) {
-          if (dt * 16 < p.DVP) {
+        for (int dt = 0; dt < DV / 16; ++dt) {
+          if (EXACT || dt * 16 < DVP) {
             uint32_t vf[4];
-            ldmatrix_x4_trans(vf, vt + tile_offset<DM>(ks * 16 + (lane & 15), dt * 2 + (lane >> 4)));
+            ldmatrix_x4_trans(vf, vt + tile_offset<DV>(ks * 16 + (lane & 15), dt * 2 + (lane >> 4)));
             mma_bf16_16816(o_acc[2 * dt], pa, vf[0], vf[1]);
             mma_bf16_16816(o_acc[2 * dt + 1], pa, vf[2], vf[3]);
           }
@@ -235,7 +252,7 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
     __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + tok * p.out_stride + col0;
     const bool pairs = (reinterpret_cast<uintptr_t>(dst) & 3) == 0 && (reinterpret_cast<uintptr_t>(g) & 3) == 0;
 #pragma unroll
-    for (int i = 0; i < DM / 8; ++i) {
+    for (int i = 0; i < DV / 8; ++i) {
       const int d = i * 8 + (lane & 3) * 2;
       if (d >= p.DV) continue;
       float o0 = o_acc[i][2 * r] * inv, o1 = o_acc[i][2 * r + 1] * inv;
@@ -254,13 +271,13 @@ gqa_gated_prefill_kernel(const GatedAttnParams p, const int heads_per_tile) {
   }
 }
 
-template <int DM>
+template <int DK, int DV, bool EXACT = false>
 static int launch_gated_prefill(const GatedAttnParams& p, int max_q_len, cudaStream_t stream) {
-  auto kern = gqa_gated_prefill_kernel<DM>;
+  auto kern = gqa_gated_prefill_kernel<DK, DV, EXACT>;
   static DeviceOnce once;
   int dev = 0;
   if (once.needed(&dev)) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, gpre::Cfg<DM>::SMEM) != cudaSuccess)
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, gpre::Cfg<DK, DV>::SMEM) != cudaSuccess)
       return -20;
     once.mark(dev);
   }
@@ -269,15 +286,17 @@ static int launch_gated_prefill(const GatedAttnParams& p, int max_q_len, cudaStr
   const int hchunks = (per + heads - 1) / heads;
   const int tt = gpre::BM / heads;
   const dim3 grid((max_q_len + tt - 1) / tt, p.Hk * hchunks, p.B);
-  return launch_pdl(kern, grid, dim3(gpre::THREADS), gpre::Cfg<DM>::SMEM, stream, 1, p, heads) == cudaSuccess ? 0
+  return launch_pdl(kern, grid, dim3(gpre::THREADS), gpre::Cfg<DK, DV>::SMEM, stream, 1, p, heads) == cudaSuccess ? 0
                                                                                                                : -21;
 }
 
 int gated_prefill(const GatedAttnParams& p, int max_q_len, cudaStream_t stream) {
   const int m = p.DP > p.DVP ? p.DP : p.DVP;
-  if (m <= 64) return launch_gated_prefill<64>(p, max_q_len, stream);
-  if (m <= 128) return launch_gated_prefill<128>(p, max_q_len, stream);
-  if (m <= 256) return launch_gated_prefill<256>(p, max_q_len, stream);
+  if (m <= 64) return launch_gated_prefill<64, 64>(p, max_q_len, stream);
+  if (m <= 128) return launch_gated_prefill<128, 128>(p, max_q_len, stream);
+  if (p.DP == 192 && p.DVP == 128) return launch_gated_prefill<192, 128, true>(p, max_q_len, stream);
+  if (p.DP <= 192 && p.DVP <= 128) return launch_gated_prefill<192, 128>(p, max_q_len, stream);
+  if (m <= 256) return launch_gated_prefill<256, 256>(p, max_q_len, stream);
   return -2;
 }
 

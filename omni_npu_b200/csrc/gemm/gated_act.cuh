@@ -18,7 +18,13 @@ __device__ __forceinline__ float gated_act(int kind, float g, float u, float alp
 }
 
 //   kActXielu       z > 0: alpha * z^2 + z / 2;  z <= 0: limit * (exp(z) - 1 - z) + z / 2
+// (results rounded to bf16: near zero the absolute error of the difference, 2e-7, is below half a step of
+// z / 2 wherever that exceeds 1e-4)
 __device__ __forceinline__ float xielu(float z, float alpha, float limit) {
+  const float a = z > 0.f ? alpha * z * z : limit * (__expf(z) - 1.f - z);
+  return fmaf(0.5f, z, a);
+}
+__device__ __forceinline__ float xielu_exact(float z, float alpha, float limit) {
   const float a = z > 0.f ? alpha * z * z : limit * (expm1f(z) - z);
   return fmaf(0.5f, z, a);
 }

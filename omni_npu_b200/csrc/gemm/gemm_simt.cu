@@ -97,7 +97,7 @@ __global__ void __launch_bounds__(simt::THREADS) gemm_simt_kernel(const SimtGemm
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int col = n0 + tx * 4 + j;
-        if (col < p.N) p.C[row * p.ldc + col] = p.act == kActXielu ? xielu(acc[i][j], p.act_alpha, p.act_limit) : acc[i][j];
+        if (col < p.N) p.C[row * p.ldc + col] = p.act == kActXielu ? xielu_exact(acc[i][j], p.act_alpha, p.act_limit) : acc[i][j];
       }
     }
     return;

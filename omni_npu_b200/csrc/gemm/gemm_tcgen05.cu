@@ -732,6 +732,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               }
               return;
             }
+            if (p.swiglu == kActXielu) {
+#pragma unroll
+              for (int i = 0; i < 4; ++i) v[i] = xielu(v[i], p.act_alpha, p.act_limit);
+            }
             for (int i = 0; i < ncols; ++i) {
               if (p.bias) v[i] += __bfloat162float(p.bias[col + i]);
               if (p.residual)
@@ -1555,7 +1559,8 @@ static int gemm_impl(const void* A, const void* W, void* C, const void* bias, co
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const int eb = dtype_fp8 ? 1 : 2;
   if (BN < 16 || BN > 256 || (BN % 16) != 0) return -10;
-  if (swiglu && ((act_is_gated(swiglu) && (N % 16) != 0) || splits != 1)) return -11;
+  if (act_is_gated(swiglu) && ((N % 16) != 0 || splits != 1)) return -11;
+  if (swiglu && splits != 1 && !cluster_split) return -11;
   if (splits <= 1) cluster_split = 0;
   if (cluster_split && (splits > 8 || BN > 128 || (kBM % splits) != 0)) return -14;
   if (splits > 1 && !cluster_split && (workspace == nullptr || counters == nullptr)) return -12;

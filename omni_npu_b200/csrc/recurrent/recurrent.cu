@@ -86,9 +86,48 @@ struct DeltaPrepParams {
 
 static constexpr int kPrepWarps = 8;
 
-// One warp = one unit (a head of q, k, v, or a head's decays) over a run of tokens; lane l has the
-// channels l + 32 i.  The convolution's window slides in registers.
-template <typename T, int CPL, int TAPS>
+// One warp = one unit (a head of q, k, v, or a head's decays) over a run of tokens.  PAIR: a lane has the
+// channels 2 lane + 64 i and the one after it, else lane + 32 i.  The convolution's window slides in
+// registers; the next token's inputs are requested before the current ones are worked off.
+template <typename T>
+__device__ __forceinline__ void load_pair(const T* p, float& a, float& b);
+template <>
+__device__ __forceinline__ void load_pair(const float* p, float& a, float& b) {
+  const float2 x = *reinterpret_cast<const float2*>(p);
+  a = x.x;
+  b = x.y;
+}
+template <>
+__device__ __forceinline__ void load_pair(const __nv_bfloat16* p, float& a, float& b) {
+  const uint32_t x = *reinterpret_cast<const uint32_t*>(p);
+  a = __uint_as_float(x << 16);
+  b = __uint_as_float(x & 0xffff0000u);
+}
+
+__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
+
+// CPL channels of a lane from a row; those at or beyond `width` are zero
+template <typename T, int CPL, bool PAIR>
+__device__ __forceinline__ void load_channels(const T* row, int lane, int width, float (&x)[CPL]) {
+  if constexpr (PAIR) {
+#pragma unroll
+    for (int i = 0; i < CPL; i += 2) {
+      const int c = lane * 2 + 32 * i;
+      x[i] = x[i + 1] = 0.f;
+      if (c < width) load_pair<T>(row + c, x[i], x[i + 1]);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < CPL; ++i) x[i] = lane + 32 * i < width ? as_float(row[lane + 32 * i]) : 0.f;
+  }
+}
+
+__device__ __forceinline__ float quick_sigmoid(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
+
+template <typename T, int CPL, int TAPS, bool PAIR>
 __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const DeltaPrepParams p) {
   pdl_trigger();
   pdl_wait();
@@ -98,15 +137,31 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const Delta
   const long long t1 = min(t0 + p.run, static_cast<long long>(p.T));
   const int n_qk = 2 * p.groups, n_v = p.heads * p.v_parts;
   if (unit >= n_qk + n_v + p.heads) return;
+  auto channel = [&](int i) { return PAIR ? lane * 2 + 32 * (i & ~1) + (i & 1) : lane + 32 * i; };
 
   if (unit >= n_qk + n_v) {                               // decays and step size of a head
     const int h = unit - n_qk - n_v;
     const float a = expf(p.a_log[h]);
+    float bias[CPL], x[CPL], nx[CPL];
+    load_channels<float, CPL, PAIR>(p.dt_bias + h * p.dim, lane, p.dim, bias);
+    const T* low = static_cast<const T*>(p.low) + static_cast<long long>(h) * p.dim;
+    load_channels<T, CPL, PAIR>(low + t0 * p.low_stride, lane, p.dim, nx);
     for (long long t = t0; t < t1; ++t) {
-      const T* low = static_cast<const T*>(p.low) + t * p.low_stride + static_cast<long long>(h) * p.dim;
+#pragma unroll
+      for (int i = 0; i < CPL; ++i) x[i] = nx[i];
+      if (t + 1 < t1) load_channels<T, CPL, PAIR>(low + (t + 1) * p.low_stride, lane, p.dim, nx);
       float* g = p.g + (t * p.heads + h) * p.DP;
-      for (int d = lane; d < p.DP; d += 32)
-        g[d] = d < p.dim ? expf(-a * softplus_f(as_float(low[d]) + p.dt_bias[h * p.dim + d])) : 0.f;
+#pragma unroll
+      for (int i = 0; i < CPL; ++i) x[i] = channel(i) < p.dim ? expf(-a * softplus_f(x[i] + bias[i])) : 0.f;
+#pragma unroll
+      for (int i = 0; i < CPL; i += 2) {
+        if constexpr (PAIR) {
+          if (channel(i) < p.DP) *reinterpret_cast<float2*>(g + channel(i)) = make_float2(x[i], x[i + 1]);
+        } else {
+          if (channel(i) < p.DP) g[channel(i)] = x[i];
+          if (channel(i + 1) < p.DP) g[channel(i + 1)] = x[i + 1];
+        }
+      }
       if (lane == 0)
         p.beta[t * p.heads + h] = sigmoid_f(as_float(static_cast<const T*>(p.proj)[t * p.stride + p.b_off + h]));
     }
@@ -125,19 +180,20 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const Delta
     col0 = (unit < p.groups ? p.q_off : p.k_off) + head * p.dim;
     width = p.dim;
   }
-  float w[CPL][TAPS], win[CPL][TAPS];
+  float w[CPL][TAPS], win[CPL][TAPS], next[CPL];
 #pragma unroll
   for (int i = 0; i < CPL; ++i)
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
       // the last register is the current token's; shorter convolutions leave the first ones idle
       const int tap = j - (TAPS - p.taps);
-      const int c = lane + 32 * i;
+      const int c = channel(i);
       w[i][j] = tap >= 0 && c < width
                     ? as_float(static_cast<const T*>(p.conv_w)[static_cast<long long>(col0 + c) * p.taps + tap]) : 0.f;
       win[i][j] = 0.f;
     }
-  const T* proj = static_cast<const T*>(p.proj);
+  const T* proj = static_cast<const T*>(p.proj) + col0;
+  load_channels<T, CPL, PAIR>(proj + t0 * p.stride, lane, width, next);
   long long begin = -1, end = -1;
   for (long long t = t0; t < t1; ++t) {
     if (t >= end) {                                       // first token of the run or of a portion
@@ -150,38 +206,46 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const Delta
       for (int j = 1; j < TAPS; ++j) {
         const long long rel = t - begin - (TAPS - j);
         const int row = static_cast<int>(rel) + p.taps - 1;         // of the stored inputs, when rel < 0
+        float x[CPL];
 #pragma unroll
-        for (int i = 0; i < CPL; ++i) {
-          const int c = lane + 32 * i;
-          float x = 0.f;
-          if (c < width) {
-            if (rel >= 0) x = as_float(proj[(begin + rel) * p.stride + col0 + c]);
-            else if (row >= 0 && slot >= 0)
-              x = as_float(static_cast<const T*>(p.conv_state)[(static_cast<long long>(slot) * (p.taps - 1) + row) *
-                                                                   p.channels + col0 + c]);
-          }
-          win[i][j] = x;
-        }
+        for (int i = 0; i < CPL; ++i) x[i] = 0.f;
+        if (rel >= 0)
+          load_channels<T, CPL, PAIR>(proj + (begin + rel) * p.stride, lane, width, x);
+        else if (row >= 0 && slot >= 0)
+          load_channels<T, CPL, PAIR>(static_cast<const T*>(p.conv_state) +
+                                          (static_cast<long long>(slot) * (p.taps - 1) + row) * p.channels + col0,
+                                      lane, width, x);
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) win[i][j] = x[i];
       }
     }
     float y[CPL], ss = 0.f;
 #pragma unroll
     for (int i = 0; i < CPL; ++i) {
-      const int c = lane + 32 * i;
 #pragma unroll
       for (int j = 0; j + 1 < TAPS; ++j) win[i][j] = win[i][j + 1];
-      win[i][TAPS - 1] = c < width ? as_float(proj[t * p.stride + col0 + c]) : 0.f;
+      win[i][TAPS - 1] = next[i];
+    }
+    if (t + 1 < t1) load_channels<T, CPL, PAIR>(proj + (t + 1) * p.stride, lane, width, next);
+#pragma unroll
+    for (int i = 0; i < CPL; ++i) {
       float acc = 0.f;
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) acc = fmaf(w[i][j], win[i][j], acc);
-      y[i] = silu_f(acc);
+      y[i] = acc * quick_sigmoid(acc);
       ss = fmaf(y[i], y[i], ss);
     }
     if (is_v) {
       T* v = static_cast<T*>(p.v) + (t * p.heads + head) * p.vdim + part * 32 * CPL;
 #pragma unroll
-      for (int i = 0; i < CPL; ++i)
-        if (lane + 32 * i < width) v[lane + 32 * i] = from_float<T>(y[i]);
+      for (int i = 0; i < CPL; i += 2) {
+        if constexpr (PAIR) {
+          if (channel(i) < width) store_pair(v + channel(i), y[i], y[i + 1]);
+        } else {
+          if (channel(i) < width) v[channel(i)] = from_float<T>(y[i]);
+          if (channel(i + 1) < width) v[channel(i + 1)] = from_float<T>(y[i + 1]);
+        }
+      }
       continue;
     }
 #pragma unroll
@@ -189,16 +253,24 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const Delta
     const float inv = (unit < p.groups ? p.q_scale : 1.f) / sqrtf(ss + p.unit_eps);
     float* dst = (unit < p.groups ? p.q : p.k) + (t * p.groups + head) * p.DP;
 #pragma unroll
-    for (int i = 0; i < CPL; ++i)
-      if (lane + 32 * i < p.DP) dst[lane + 32 * i] = lane + 32 * i < width ? y[i] * inv : 0.f;
+    for (int i = 0; i < CPL; i += 2) {
+      // (channels beyond the head have no weights and are zero)
+      if constexpr (PAIR) {
+        if (channel(i) < p.DP) *reinterpret_cast<float2*>(dst + channel(i)) = make_float2(y[i] * inv, y[i + 1] * inv);
+      } else {
+        if (channel(i) < p.DP) dst[channel(i)] = y[i] * inv;
+        if (channel(i + 1) < p.DP) dst[channel(i + 1)] = y[i + 1] * inv;
+      }
+    }
   }
 }
 
 // ------------------------------------------------------------- the scan
 // One CTA = 32 columns (of the value axis) of one (sequence, head); a warp has 8 of them and all rows:
-// lane = 16 * (column half) + row group, a thread 4 columns x RPT rows.  The column sums (S^T k, S^T q) are
-// folded inside the warp, so that no block barrier stands between tokens.  q, k, g are staged CH tokens
-// at a time through shared memory, the next ones on their way while these are worked off.
+// lane = 8 * (column pair) + row group, a thread two columns x RPT rows, rows in pairs for the packed fp32
+// instructions.  The column sums (S^T k, and S^T q of four tokens at a time) are folded inside the warp, so
+// that no block barrier stands between tokens.  q, k, g and v are staged CH tokens at a time through shared
+// memory, the next ones on their way while these are worked off.
 struct ScanParams {
   const float* q;              // [T, G, DP]
   const float* k;              // [T, G, DP]
@@ -219,11 +291,11 @@ struct ScanParams {
 };
 
 namespace scan {
-constexpr int WARPS = 4, THREADS = WARPS * 32, COLS = 32;
+constexpr int WARPS = 4, THREADS = WARPS * 32, COLS = 32, GROUP = 4;
 template <int RPT, bool DELTA>
 struct Cfg {
-  static constexpr int ROWS = 16 * RPT;
-  static constexpr int CH = RPT <= 8 ? 16 : RPT <= 16 ? 8 : 4;
+  static constexpr int ROWS = 8 * RPT;
+  static constexpr int CH = RPT <= 16 ? 16 : RPT <= 32 ? 8 : 4;
   static constexpr int ARR = DELTA ? 3 : 2;
   static constexpr int STAGE = ARR * CH * ROWS;                     // floats
   static constexpr int SMEM = (2 * STAGE + 2 * CH * (COLS + 1)) * 4;
@@ -234,18 +306,32 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))),
                "l"(src) : "memory");
 }
+__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))),
+               "l"(src) : "memory");
+}
 
-// Sums of four columns over the 16 row groups; every lane ends with the one of column
-// 2 * (bit 3 of the lane) + (bit 2).
-__device__ __forceinline__ float fold_columns(const float (&a)[4], int lane) {
-  const bool hi = lane & 8, odd = lane & 4;
-  float k0 = hi ? a[2] : a[0], k1 = hi ? a[3] : a[1];
-  k0 += __shfl_xor_sync(0xffffffffu, hi ? a[0] : a[2], 8);
-  k1 += __shfl_xor_sync(0xffffffffu, hi ? a[1] : a[3], 8);
-  float c = (odd ? k1 : k0) + __shfl_xor_sync(0xffffffffu, odd ? k0 : k1, 4);
-  c += __shfl_xor_sync(0xffffffffu, c, 2);
-  c += __shfl_xor_sync(0xffffffffu, c, 1);
-  return c;
+// two fp32 numbers in a 64-bit register
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float sum2(f32x2 x) {
+  float lo, hi;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(x));
+  return lo + hi;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
 }
 
 template <typename T, int RPT, bool DELTA>
@@ -253,15 +339,16 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
   using namespace scan;
   using C = Cfg<RPT, DELTA>;
   constexpr int CH = C::CH, ROWS = C::ROWS, Q4 = RPT / 4;
+  constexpr bool KEEP_K = RPT <= 32;                      // k of a token in registers between its two uses
   extern __shared__ __align__(16) float smem[];
-  float* s_v = smem + 2 * C::STAGE;                       // [2][CH][COLS]
-  float* s_b = s_v + 2 * CH * COLS;                       // [2][CH]
+  T* s_v = reinterpret_cast<T*>(smem + 2 * C::STAGE);     // [2][CH][COLS]
+  float* s_b = smem + 2 * C::STAGE + 2 * CH * COLS;       // [2][CH]
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int rg = lane & 15;
+  const int rg = lane & 7;
   const int b = blockIdx.z, h = blockIdx.y, c_base = blockIdx.x * COLS;
   const int grp = h / (p.H / p.G);
-  const int col0 = warp * 8 + (lane >> 4) * 4;            // first of this thread's columns, within the CTA
+  const int col0 = warp * 8 + (lane >> 3) * 2;            // first of this thread's columns, within the CTA
 
   if (p.DP < ROWS) {                                      // rows beyond the head's size stay zero
     for (int i = tid; i < 2 * C::STAGE; i += THREADS) smem[i] = 0.f;
@@ -277,123 +364,172 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
   const bool fresh = p.seq_lens[b] <= n || slot < 0;
 
   const int quads = p.DP >> 2;
+  const T* v_src = static_cast<const T*>(p.v) + begin * p.v_stride + static_cast<long long>(h) * p.E + c_base;
+  constexpr int VPIECES = COLS * static_cast<int>(sizeof(T)) / 16;          // 16-byte pieces of a token's columns
+  const bool v_vec = c_base + COLS <= p.E && (reinterpret_cast<uintptr_t>(v_src) & 15) == 0 &&
+                     (p.v_stride * sizeof(T)) % 16 == 0;
   auto stage = [&](int c) {                               // start copying chunk c
     const int t0 = c * CH, m = min(CH, n - t0);
     float* dst = smem + (c & 1) * C::STAGE;
-    for (int i = tid; i < C::ARR * m * quads; i += THREADS) {
-      const int quad = i % quads, r = i / quads;
-      const int arr = r / m, j = r - arr * m;
-      const long long t = begin + t0 + j;
-      const float* src = arr == 0 ? p.q + (t * p.G + grp) * p.DP
-                                  : arr == 1 ? p.k + (t * p.G + grp) * p.DP : p.g + (t * p.H + h) * p.DP;
-      cp_async16(dst + (arr * CH + j) * ROWS + quad * 4, src + quad * 4);
+#pragma unroll
+    for (int arr = 0; arr < C::ARR; ++arr) {
+      const float* src = (arr == 0 ? p.q : arr == 1 ? p.k : p.g) +
+                         ((begin + t0) * (arr == 2 ? p.H : p.G) + (arr == 2 ? h : grp)) * p.DP;
+      const long long pitch = static_cast<long long>(arr == 2 ? p.H : p.G) * p.DP;
+      for (int j = warp; j < m; j += WARPS)
+        for (int quad = lane; quad < quads; quad += 32)
+          cp_async16(dst + (arr * CH + j) * ROWS + quad * 4, src + j * pitch + quad * 4);
     }
+    T* dv = s_v + (c & 1) * CH * COLS;
+    if (v_vec) {
+      for (int i = tid; i < m * VPIECES; i += THREADS) {
+        const int j = i / VPIECES, piece = i % VPIECES;
+        cp_async16(reinterpret_cast<char*>(dv + j * COLS) + piece * 16,
+                   reinterpret_cast<const char*>(v_src + (t0 + j) * p.v_stride) + piece * 16);
+      }
+    } else {
+      for (int i = tid; i < m * COLS; i += THREADS) {
+        const int j = i / COLS, col = i % COLS;
+        dv[i] = c_base + col < p.E ? v_src[(t0 + j) * p.v_stride + col] : from_float<T>(0.f);
+      }
+    }
+    if (DELTA && tid < m) cp_async4(s_b + (c & 1) * CH + tid, p.beta + (begin + t0 + tid) * p.H + h);
     asm volatile("cp.async.commit_group;" ::: "memory");
-    for (int i = tid; i < m * COLS; i += THREADS) {
-      const int j = i / COLS, col = i % COLS;
-      const long long t = begin + t0 + j;
-      s_v[((c & 1) * CH + j) * COLS + col] =
-          c_base + col < p.E ? as_float(static_cast<const T*>(p.v)[t * p.v_stride + static_cast<long long>(h) * p.E +
-                                                                   c_base + col]) : 0.f;
-    }
-    if (DELTA && tid < m) s_b[(c & 1) * CH + tid] = p.beta[(begin + t0 + tid) * p.H + h];
   };
   stage(0);
 
-  float s[4][RPT];
+  f32x2 s[2][RPT / 2];
   float* st = p.state + ((static_cast<long long>(slot < 0 ? 0 : slot) * p.H + h) * p.E + c_base + col0) * p.DP;
 #pragma unroll
-  for (int c = 0; c < 4; ++c)
+  for (int c = 0; c < 2; ++c)
 #pragma unroll
     for (int i = 0; i < Q4; ++i) {
-      const int r = i * 64 + rg * 4;
+      const int r = i * 32 + rg * 4;
       float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
       if (!fresh && r < p.DP && c_base + col0 + c < p.E)
         x = *reinterpret_cast<const float4*>(st + static_cast<long long>(c) * p.DP + r);
-      s[c][4 * i] = x.x;
-      s[c][4 * i + 1] = x.y;
-      s[c][4 * i + 2] = x.z;
-      s[c][4 * i + 3] = x.w;
+      s[c][2 * i] = pack2(x.x, x.y);
+      s[c][2 * i + 1] = pack2(x.z, x.w);
     }
 
-  const int my_col = col0 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);     // the column this lane has after a fold
-  const bool writes = (lane & 3) == 0 && c_base + my_col < p.E;
+  const int my_col = col0 + (lane & 1);                   // the column this lane has after a fold
+  const bool writes = c_base + my_col < p.E;
   float* o = p.o + (begin * p.H + h) * p.E + c_base + my_col;
   const long long o_step = static_cast<long long>(p.H) * p.E;
+  const f32x2 one = pack2(1.f, 1.f), minus = pack2(-1.f, -1.f), zero = pack2(0.f, 0.f);
 
   const int chunks = (n + CH - 1) / CH;
   for (int c = 0; c < chunks; ++c) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                      // chunk c is there; the buffer of c + 1 is free
     if (c + 1 < chunks) stage(c + 1);
-    const float* sq = smem + (c & 1) * C::STAGE;
+    const float* sq = smem + (c & 1) * C::STAGE + rg * 4;
     const float* sk = sq + CH * ROWS;
     const float* sg = sk + CH * ROWS;
-    const float* vv = s_v + (c & 1) * CH * COLS;
+    const T* vv = s_v + (c & 1) * CH * COLS;
     const float* bb = s_b + (c & 1) * CH;
     const int m = min(CH, n - c * CH);
-    for (int j = 0; j < m; ++j) {
-      float k[RPT];
+    for (int j0 = 0; j0 < m; j0 += GROUP) {
+      float acc_o[GROUP][2];
 #pragma unroll
-      for (int i = 0; i < Q4; ++i) {
-        const float4 x = *reinterpret_cast<const float4*>(sk + j * ROWS + i * 64 + rg * 4);
-        k[4 * i] = x.x; k[4 * i + 1] = x.y; k[4 * i + 2] = x.z; k[4 * i + 3] = x.w;
-      }
-      if (DELTA) {
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int jj = 0; jj < GROUP; ++jj) {
+        const int j = j0 + jj;
+        acc_o[jj][0] = acc_o[jj][1] = 0.f;
+        if (j < m) {
+          auto load = [&](const float* base, int i) {
+            return *reinterpret_cast<const ulonglong2*>(base + j * ROWS + i * 32);
+          };
+          f32x2 k[KEEP_K ? RPT / 2 : 1];
+          if constexpr (KEEP_K) {
 #pragma unroll
-        for (int i = 0; i < Q4; ++i) {
-          const float4 x = *reinterpret_cast<const float4*>(sg + j * ROWS + i * 64 + rg * 4);
-          const float g[4] = {x.x, x.y, x.z, x.w};
-#pragma unroll
-          for (int e = 0; e < 4; ++e)
-#pragma unroll
-            for (int cc = 0; cc < 4; ++cc) {
-              s[cc][4 * i + e] *= g[e];
-              acc[cc] = fmaf(s[cc][4 * i + e], k[4 * i + e], acc[cc]);
+            for (int i = 0; i < Q4; ++i) {
+              const ulonglong2 x = load(sk, i);
+              k[2 * i] = x.x;
+              k[2 * i + 1] = x.y;
             }
-        }
-        const float u = bb[j] * (vv[j * COLS + my_col] - fold_columns(acc, lane));
+          }
+          auto k_pair = [&](int i) {                      // rows 4 i .. 4 i + 3 of this thread
+            if constexpr (KEEP_K) return make_ulonglong2(k[2 * i], k[2 * i + 1]);
+            else return load(sk, i);
+          };
+          float u0, u1;
+          if constexpr (DELTA) {
+            f32x2 a0 = zero, a1 = zero, b0 = zero, b1 = zero;
 #pragma unroll
-        for (int cc = 0; cc < 4; ++cc) {
-          const float uc = __shfl_sync(0xffffffffu, u, (lane & 16) | (cc << 2));
+            for (int i = 0; i < Q4; ++i) {
+              const ulonglong2 g = load(sg, i), kk = k_pair(i);
+              s[0][2 * i] = mul2(s[0][2 * i], g.x);
+              s[1][2 * i] = mul2(s[1][2 * i], g.x);
+              s[0][2 * i + 1] = mul2(s[0][2 * i + 1], g.y);
+              s[1][2 * i + 1] = mul2(s[1][2 * i + 1], g.y);
+              a0 = fma2(s[0][2 * i], kk.x, a0);
+              a1 = fma2(s[1][2 * i], kk.x, a1);
+              b0 = fma2(s[0][2 * i + 1], kk.y, b0);
+              b1 = fma2(s[1][2 * i + 1], kk.y, b1);
+            }
+            const float f0 = sum2(a0) + sum2(b0), f1 = sum2(a1) + sum2(b1);
+            float f = (lane & 1 ? f1 : f0) + __shfl_xor_sync(0xffffffffu, lane & 1 ? f0 : f1, 1);
+            f += __shfl_xor_sync(0xffffffffu, f, 2);
+            f += __shfl_xor_sync(0xffffffffu, f, 4);
+            const float u = bb[j] * (as_float(vv[j * COLS + my_col]) - f);
+            const float other = __shfl_xor_sync(0xffffffffu, u, 1);
+            u0 = lane & 1 ? other : u;
+            u1 = lane & 1 ? u : other;
+          } else {
+            u0 = as_float(vv[j * COLS + col0]);
+            u1 = as_float(vv[j * COLS + col0 + 1]);
+          }
+          const f32x2 w0 = pack2(u0, u0), w1 = pack2(u1, u1);
+          f32x2 o0 = zero, o1 = zero;
 #pragma unroll
-          for (int r = 0; r < RPT; ++r) s[cc][r] = fmaf(k[r], uc, s[cc][r]);
-        }
-      } else {
-        const float4 x = *reinterpret_cast<const float4*>(vv + j * COLS + col0);
-        const float u[4] = {x.x, x.y, x.z, x.w};
-#pragma unroll
-        for (int r = 0; r < RPT; ++r) {
-          const float g = 1.f - k[r];
-#pragma unroll
-          for (int cc = 0; cc < 4; ++cc) s[cc][r] = fmaf(s[cc][r], g, k[r] * u[cc]);
+          for (int i = 0; i < Q4; ++i) {
+            const ulonglong2 q = load(sq, i), kk = k_pair(i);
+            if constexpr (DELTA) {
+              s[0][2 * i] = fma2(kk.x, w0, s[0][2 * i]);
+              s[1][2 * i] = fma2(kk.x, w1, s[1][2 * i]);
+              s[0][2 * i + 1] = fma2(kk.y, w0, s[0][2 * i + 1]);
+              s[1][2 * i + 1] = fma2(kk.y, w1, s[1][2 * i + 1]);
+            } else {
+              const f32x2 gx = fma2(kk.x, minus, one), gy = fma2(kk.y, minus, one);
+              s[0][2 * i] = fma2(s[0][2 * i], gx, mul2(kk.x, w0));
+              s[1][2 * i] = fma2(s[1][2 * i], gx, mul2(kk.x, w1));
+              s[0][2 * i + 1] = fma2(s[0][2 * i + 1], gy, mul2(kk.y, w0));
+              s[1][2 * i + 1] = fma2(s[1][2 * i + 1], gy, mul2(kk.y, w1));
+            }
+            o0 = fma2(s[0][2 * i], q.x, o0);
+            o1 = fma2(s[1][2 * i], q.x, o1);
+            o0 = fma2(s[0][2 * i + 1], q.y, o0);
+            o1 = fma2(s[1][2 * i + 1], q.y, o1);
+          }
+          acc_o[jj][0] = sum2(o0);
+          acc_o[jj][1] = sum2(o1);
         }
       }
-      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      // eight sums over eight lanes: lane bits 2, 1 end up choosing the token, bit 0 the column
+      float x[2][2], y[2];
 #pragma unroll
-      for (int i = 0; i < Q4; ++i) {
-        const float4 x = *reinterpret_cast<const float4*>(sq + j * ROWS + i * 64 + rg * 4);
-        const float q[4] = {x.x, x.y, x.z, x.w};
+      for (int e = 0; e < 2; ++e)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
+        for (int cc = 0; cc < 2; ++cc)
+          x[e][cc] = (lane & 4 ? acc_o[2 + e][cc] : acc_o[e][cc]) +
+                     __shfl_xor_sync(0xffffffffu, lane & 4 ? acc_o[e][cc] : acc_o[2 + e][cc], 4);
 #pragma unroll
-          for (int cc = 0; cc < 4; ++cc) acc[cc] = fmaf(s[cc][4 * i + e], q[e], acc[cc]);
-      }
-      const float r = fold_columns(acc, lane);
-      if (writes) *o = r;
-      o += o_step;
+      for (int cc = 0; cc < 2; ++cc)
+        y[cc] = (lane & 2 ? x[1][cc] : x[0][cc]) + __shfl_xor_sync(0xffffffffu, lane & 2 ? x[0][cc] : x[1][cc], 2);
+      const float r = (lane & 1 ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, lane & 1 ? y[0] : y[1], 1);
+      const int jt = (lane >> 1) & 3;
+      if (writes && j0 + jt < m) o[(c * CH + j0 + jt) * o_step] = r;
     }
   }
   if (slot < 0) return;
 #pragma unroll
-  for (int c = 0; c < 4; ++c)
+  for (int c = 0; c < 2; ++c)
 #pragma unroll
     for (int i = 0; i < Q4; ++i) {
-      const int r = i * 64 + rg * 4;
+      const int r = i * 32 + rg * 4;
       if (r < p.DP && c_base + col0 + c < p.E)
-        *reinterpret_cast<float4*>(st + static_cast<long long>(c) * p.DP + r) =
-            make_float4(s[c][4 * i], s[c][4 * i + 1], s[c][4 * i + 2], s[c][4 * i + 3]);
+        *reinterpret_cast<ulonglong2*>(st + static_cast<long long>(c) * p.DP + r) =
+            make_ulonglong2(s[c][2 * i], s[c][2 * i + 1]);
     }
   if (p.proj && p.keep > 0) {
     // the newest `keep` inputs of the convolution, channels dealt out over this sequence's CTAs; a channel
@@ -428,10 +564,10 @@ static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
 
 template <typename T, bool DELTA>
 static int pick_scan(const ScanParams& p, int B, cudaStream_t stream) {
-  if (p.DP <= 64) return launch_scan<T, 4, DELTA>(p, B, stream);
-  if (p.DP <= 128) return launch_scan<T, 8, DELTA>(p, B, stream);
-  if (p.DP <= 256) return launch_scan<T, 16, DELTA>(p, B, stream);
-  if (p.DP <= 512) return launch_scan<T, 32, DELTA>(p, B, stream);
+  if (p.DP <= 64) return launch_scan<T, 8, DELTA>(p, B, stream);
+  if (p.DP <= 128) return launch_scan<T, 16, DELTA>(p, B, stream);
+  if (p.DP <= 256) return launch_scan<T, 32, DELTA>(p, B, stream);
+  if (p.DP <= 512) return launch_scan<T, 64, DELTA>(p, B, stream);
   return -2;
 }
 
@@ -444,6 +580,7 @@ struct HeadNormParams {
   void* out;                   // [T, out_width]
   int out_width, T, H, E;
   float eps;
+  int vec;                     // rows are whole four-element pieces
 };
 
 static constexpr int kHeadNormWarps = 8;
@@ -458,18 +595,49 @@ __global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_kernel(const He
   const long long t = unit / p.H;
   const int h = static_cast<int>(unit - t * p.H);
   const float* o = p.o + unit * p.E;
-  float ss = 0.f;
-  for (int d = lane; d < p.E; d += 32) ss = fmaf(o[d], o[d], ss);
-#pragma unroll
-  for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
-  const float inv = 1.f / sqrtf(ss / static_cast<float>(p.E) + p.eps);
   const T* w = static_cast<const T*>(p.w);
   const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_stride + static_cast<long long>(h) * p.E : nullptr;
   T* dst = static_cast<T*>(p.out) + t * p.out_width;
-  for (int d = lane; d < p.E; d += 32) {
-    float y = o[d] * inv * as_float(w[d]);
-    if (gate) y *= sigmoid_f(as_float(gate[d]));
-    dst[h * p.E + d] = from_float<T>(y);
+  float ss = 0.f;
+  if (p.vec) {                                            // up to 512 columns, four at a time in registers
+    float x[4][4], g[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int v = lane + 32 * i;
+      if (v * 4 < p.E) {
+        Row4<float>::load(o, v, x[i]);
+        if (gate) Row4<T>::load(gate, v, g[i]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss = fmaf(x[i][j], x[i][j], ss);
+      }
+    }
+#pragma unroll
+    for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
+    const float inv = 1.f / sqrtf(ss / static_cast<float>(p.E) + p.eps);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int v = lane + 32 * i;
+      if (v * 4 < p.E) {
+        float ww[4];
+        Row4<T>::load(w, v, ww);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          x[i][j] *= inv * ww[j];
+          if (gate) x[i][j] *= quick_sigmoid(g[i][j]);
+        }
+        Row4<T>::store(dst + h * p.E, v, x[i]);
+      }
+    }
+  } else {
+    for (int d = lane; d < p.E; d += 32) ss = fmaf(o[d], o[d], ss);
+#pragma unroll
+    for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
+    const float inv = 1.f / sqrtf(ss / static_cast<float>(p.E) + p.eps);
+    for (int d = lane; d < p.E; d += 32) {
+      float y = o[d] * inv * as_float(w[d]);
+      if (gate) y *= quick_sigmoid(as_float(gate[d]));
+      dst[h * p.E + d] = from_float<T>(y);
+    }
   }
   if (h == p.H - 1)
     for (int d = p.H * p.E + lane; d < p.out_width; d += 32) dst[d] = from_float<T>(0.f);
@@ -478,8 +646,16 @@ __global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_kernel(const He
 template <typename T, int CPL>
 static cudaError_t launch_delta_prep(const DeltaPrepParams& p, dim3 grid, cudaStream_t stream) {
   const dim3 block(kPrepWarps * 32);
-  if (p.taps <= 4) return launch_pdl(delta_prep_kernel<T, CPL, 4>, grid, block, 0, stream, 1, p);
-  return launch_pdl(delta_prep_kernel<T, CPL, 8>, grid, block, 0, stream, 1, p);
+  const int W = 2;                                       // pairs: everything a pair touches starts at an even channel
+  const bool pair = p.dim % W == 0 && p.vdim % W == 0 && p.stride % W == 0 && p.low_stride % W == 0 &&
+                    p.channels % W == 0 && p.q_off % W == 0 && p.k_off % W == 0 && p.v_off % W == 0 &&
+                    (reinterpret_cast<uintptr_t>(p.proj) & 7) == 0 && (reinterpret_cast<uintptr_t>(p.low) & 7) == 0;
+  if (pair) {
+    if (p.taps <= 4) return launch_pdl(delta_prep_kernel<T, CPL, 4, true>, grid, block, 0, stream, 1, p);
+    return launch_pdl(delta_prep_kernel<T, CPL, 8, true>, grid, block, 0, stream, 1, p);
+  }
+  if (p.taps <= 4) return launch_pdl(delta_prep_kernel<T, CPL, 4, false>, grid, block, 0, stream, 1, p);
+  return launch_pdl(delta_prep_kernel<T, CPL, 8, false>, grid, block, 0, stream, 1, p);
 }
 
 template <typename T>
@@ -547,7 +723,11 @@ extern "C" int b200_recurrent_scan(const float* q, const float* k, const float* 
 extern "C" int b200_head_norm_gate(const float* o, const void* w, const void* gate, long long gate_stride, void* out,
                                    int out_width, int T, int H, int E, float eps, int is_fp32, cudaStream_t stream) {
   if (T <= 0) return 0;
-  HeadNormParams p{o, w, gate, gate_stride, out, out_width, T, H, E, eps};
+  const uintptr_t align = is_fp32 ? 15 : 7;
+  const bool vec = E % 4 == 0 && E <= 512 && out_width % 4 == 0 && gate_stride % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(gate) & align) == 0 && (reinterpret_cast<uintptr_t>(out) & align) == 0 &&
+                   (reinterpret_cast<uintptr_t>(w) & align) == 0;
+  HeadNormParams p{o, w, gate, gate_stride, out, out_width, T, H, E, eps, vec ? 1 : 0};
   const long long units = static_cast<long long>(T) * H;
   const dim3 grid(static_cast<unsigned>((units + kHeadNormWarps - 1) / kHeadNormWarps)), block(kHeadNormWarps * 32);
   const cudaError_t e = is_fp32 ? launch_pdl(head_norm_kernel<float>, grid, block, 0, stream, 1, p)

@@ -248,11 +248,11 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         _count(1)
         return C.gemm_pair(a, w, bias, residual, out_dtype == torch.float32, kind[0], pbn, st.status, max_ctas,
                            kind[1], kind[2])
-    fused = kind[0] != 0
-    key = (m, n, k, a.dtype.itemsize, fused, bn, splits)
+    fused, gated = kind[0] != 0, kind[0] in (1, 2)
+    key = (m, n, k, a.dtype.itemsize, kind[0], bn, splits)
     plan = st.plans.get(key)
     if plan is None:
-        plan = C.gemm_plan(m, n, k, a.dtype.itemsize, fused, bn, 1 if fused else splits)
+        plan = C.gemm_plan(m, n, k, a.dtype.itemsize, gated, bn, 1 if gated else max(0, splits) if fused else splits)
         st.plans[key] = plan
     pbn, psplits, ws_bytes, ncnt, cluster = plan
     if library_small_m(m, bool(cluster), bias is None and residual is None and not fused and bn == 0

@@ -267,10 +267,12 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const Delta
 
 // ------------------------------------------------------------- the scan
 // One CTA = 32 columns (of the value axis) of one (sequence, head); a warp has 8 of them and all rows:
-// lane = 8 * (column pair) + row group, a thread two columns x RPT rows, rows in pairs for the packed fp32
-// instructions.  The column sums (S^T k, and S^T q of four tokens at a time) are folded inside the warp, so
-// that no block barrier stands between tokens.  q, k, g and v are staged CH tokens at a time through shared
-// memory, the next ones on their way while these are worked off.
+// lane = 16 * (column half) + row group, a thread four columns x RPT rows, rows in pairs for the packed fp32
+// instructions.  (Every thread reads RPT elements of q, k and g per token: with more rows and fewer columns
+// per thread shared memory, 128 bytes per clock and SM, would have as much to do as the arithmetic.)  The
+// column sums (S^T k, and S^T q of four tokens at a time) are folded inside the warp, so that no block
+// barrier stands between tokens.  q, k, g and v are staged CH tokens at a time through shared memory, the
+// next ones on their way while these are worked off.
 struct ScanParams {
   const float* q;              // [T, G, DP]
   const float* k;              // [T, G, DP]
@@ -294,8 +296,8 @@ namespace scan {
 constexpr int WARPS = 4, THREADS = WARPS * 32, COLS = 32, GROUP = 4;
 template <int RPT, bool DELTA>
 struct Cfg {
-  static constexpr int ROWS = 8 * RPT;
-  static constexpr int CH = RPT <= 16 ? 16 : RPT <= 32 ? 8 : 4;
+  static constexpr int ROWS = 16 * RPT;
+  static constexpr int CH = RPT <= 8 ? 16 : RPT <= 16 ? 8 : 4;
   static constexpr int ARR = DELTA ? 3 : 2;
   static constexpr int STAGE = ARR * CH * ROWS;                     // floats
   static constexpr int SMEM = (2 * STAGE + 2 * CH * (COLS + 1)) * 4;
@@ -339,16 +341,16 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
   using namespace scan;
   using C = Cfg<RPT, DELTA>;
   constexpr int CH = C::CH, ROWS = C::ROWS, Q4 = RPT / 4;
-  constexpr bool KEEP_K = RPT <= 32;                      // k of a token in registers between its two uses
+  constexpr bool KEEP_K = RPT <= 16;                      // k of a token in registers between its two uses
   extern __shared__ __align__(16) float smem[];
   T* s_v = reinterpret_cast<T*>(smem + 2 * C::STAGE);     // [2][CH][COLS]
   float* s_b = smem + 2 * C::STAGE + 2 * CH * COLS;       // [2][CH]
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int rg = lane & 7;
+  const int rg = lane & 15;
   const int b = blockIdx.z, h = blockIdx.y, c_base = blockIdx.x * COLS;
   const int grp = h / (p.H / p.G);
-  const int col0 = warp * 8 + (lane >> 3) * 2;            // first of this thread's columns, within the CTA
+  const int col0 = warp * 8 + (lane >> 4) * 4;            // first of this thread's columns, within the CTA
 
   if (p.DP < ROWS) {                                      // rows beyond the head's size stay zero
     for (int i = tid; i < 2 * C::STAGE; i += THREADS) smem[i] = 0.f;
@@ -398,13 +400,13 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
   };
   stage(0);
 
-  f32x2 s[2][RPT / 2];
+  f32x2 s[4][RPT / 2];
   float* st = p.state + ((static_cast<long long>(slot < 0 ? 0 : slot) * p.H + h) * p.E + c_base + col0) * p.DP;
 #pragma unroll
-  for (int c = 0; c < 2; ++c)
+  for (int c = 0; c < 4; ++c)
 #pragma unroll
     for (int i = 0; i < Q4; ++i) {
-      const int r = i * 32 + rg * 4;
+      const int r = i * 64 + rg * 4;
       float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
       if (!fresh && r < p.DP && c_base + col0 + c < p.E)
         x = *reinterpret_cast<const float4*>(st + static_cast<long long>(c) * p.DP + r);
@@ -412,7 +414,7 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
       s[c][2 * i + 1] = pack2(x.z, x.w);
     }
 
-  const int my_col = col0 + (lane & 1);                   // the column this lane has after a fold
+  const int my_col = col0 + (lane & 3);                   // the column this lane has after a fold
   const bool writes = c_base + my_col < p.E;
   float* o = p.o + (begin * p.H + h) * p.E + c_base + my_col;
   const long long o_step = static_cast<long long>(p.H) * p.E;
@@ -430,103 +432,118 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
     const float* bb = s_b + (c & 1) * CH;
     const int m = min(CH, n - c * CH);
     for (int j0 = 0; j0 < m; j0 += GROUP) {
-      float acc_o[GROUP][2];
-#pragma unroll
-      for (int jj = 0; jj < GROUP; ++jj) {
-        const int j = j0 + jj;
-        acc_o[jj][0] = acc_o[jj][1] = 0.f;
-        if (j < m) {
-          auto load = [&](const float* base, int i) {
-            return *reinterpret_cast<const ulonglong2*>(base + j * ROWS + i * 32);
-          };
-          f32x2 k[KEEP_K ? RPT / 2 : 1];
-          if constexpr (KEEP_K) {
-#pragma unroll
-            for (int i = 0; i < Q4; ++i) {
-              const ulonglong2 x = load(sk, i);
-              k[2 * i] = x.x;
-              k[2 * i + 1] = x.y;
-            }
-          }
-          auto k_pair = [&](int i) {                      // rows 4 i .. 4 i + 3 of this thread
-            if constexpr (KEEP_K) return make_ulonglong2(k[2 * i], k[2 * i + 1]);
-            else return load(sk, i);
-          };
-          float u0, u1;
-          if constexpr (DELTA) {
-            f32x2 a0 = zero, a1 = zero, b0 = zero, b1 = zero;
-#pragma unroll
-            for (int i = 0; i < Q4; ++i) {
-              const ulonglong2 g = load(sg, i), kk = k_pair(i);
-              s[0][2 * i] = mul2(s[0][2 * i], g.x);
-              s[1][2 * i] = mul2(s[1][2 * i], g.x);
-              s[0][2 * i + 1] = mul2(s[0][2 * i + 1], g.y);
-              s[1][2 * i + 1] = mul2(s[1][2 * i + 1], g.y);
-              a0 = fma2(s[0][2 * i], kk.x, a0);
-              a1 = fma2(s[1][2 * i], kk.x, a1);
-              b0 = fma2(s[0][2 * i + 1], kk.y, b0);
-              b1 = fma2(s[1][2 * i + 1], kk.y, b1);
-            }
-            const float f0 = sum2(a0) + sum2(b0), f1 = sum2(a1) + sum2(b1);
-            float f = (lane & 1 ? f1 : f0) + __shfl_xor_sync(0xffffffffu, lane & 1 ? f0 : f1, 1);
-            f += __shfl_xor_sync(0xffffffffu, f, 2);
-            f += __shfl_xor_sync(0xffffffffu, f, 4);
-            const float u = bb[j] * (as_float(vv[j * COLS + my_col]) - f);
-            const float other = __shfl_xor_sync(0xffffffffu, u, 1);
-            u0 = lane & 1 ? other : u;
-            u1 = lane & 1 ? u : other;
-          } else {
-            u0 = as_float(vv[j * COLS + col0]);
-            u1 = as_float(vv[j * COLS + col0 + 1]);
-          }
-          const f32x2 w0 = pack2(u0, u0), w1 = pack2(u1, u1);
-          f32x2 o0 = zero, o1 = zero;
+      const float *qj = sq + j0 * ROWS, *kj = sk + j0 * ROWS, *gj = sg + j0 * ROWS, *bj = bb + j0;
+      const T* vj = vv + j0 * COLS;
+      float acc_o[GROUP][4];
+      auto token = [&](int jj) {
+        auto load = [&](const float* base, int i) {
+          return *reinterpret_cast<const ulonglong2*>(base + jj * ROWS + i * 64);
+        };
+        f32x2 k[KEEP_K ? RPT / 2 : 1];
+        if constexpr (KEEP_K) {
 #pragma unroll
           for (int i = 0; i < Q4; ++i) {
-            const ulonglong2 q = load(sq, i), kk = k_pair(i);
-            if constexpr (DELTA) {
-              s[0][2 * i] = fma2(kk.x, w0, s[0][2 * i]);
-              s[1][2 * i] = fma2(kk.x, w1, s[1][2 * i]);
-              s[0][2 * i + 1] = fma2(kk.y, w0, s[0][2 * i + 1]);
-              s[1][2 * i + 1] = fma2(kk.y, w1, s[1][2 * i + 1]);
-            } else {
-              const f32x2 gx = fma2(kk.x, minus, one), gy = fma2(kk.y, minus, one);
-              s[0][2 * i] = fma2(s[0][2 * i], gx, mul2(kk.x, w0));
-              s[1][2 * i] = fma2(s[1][2 * i], gx, mul2(kk.x, w1));
-              s[0][2 * i + 1] = fma2(s[0][2 * i + 1], gy, mul2(kk.y, w0));
-              s[1][2 * i + 1] = fma2(s[1][2 * i + 1], gy, mul2(kk.y, w1));
-            }
-            o0 = fma2(s[0][2 * i], q.x, o0);
-            o1 = fma2(s[1][2 * i], q.x, o1);
-            o0 = fma2(s[0][2 * i + 1], q.y, o0);
-            o1 = fma2(s[1][2 * i + 1], q.y, o1);
+            const ulonglong2 x = load(kj, i);
+            k[2 * i] = x.x;
+            k[2 * i + 1] = x.y;
           }
-          acc_o[jj][0] = sum2(o0);
-          acc_o[jj][1] = sum2(o1);
+        }
+        auto k_pair = [&](int i) {                        // rows 4 i .. 4 i + 3 of this thread
+          if constexpr (KEEP_K) return make_ulonglong2(k[2 * i], k[2 * i + 1]);
+          else return load(kj, i);
+        };
+        f32x2 u[4];                                       // of the four columns, in both halves
+        if constexpr (DELTA) {
+          f32x2 acc[4] = {zero, zero, zero, zero};
+#pragma unroll
+          for (int i = 0; i < Q4; ++i) {
+            const ulonglong2 g = load(gj, i), kk = k_pair(i);
+#pragma unroll
+            for (int cc = 0; cc < 4; ++cc) {
+              s[cc][2 * i] = mul2(s[cc][2 * i], g.x);
+              s[cc][2 * i + 1] = mul2(s[cc][2 * i + 1], g.y);
+              acc[cc] = fma2(s[cc][2 * i], kk.x, acc[cc]);
+              acc[cc] = fma2(s[cc][2 * i + 1], kk.y, acc[cc]);
+            }
+          }
+          // four sums over sixteen lanes: lane bits 1, 0 end up choosing the column
+          float f[4];
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc) f[cc] = sum2(acc[cc]);
+          const bool hi = lane & 2, odd = lane & 1;
+          const float f0 = (hi ? f[2] : f[0]) + __shfl_xor_sync(0xffffffffu, hi ? f[0] : f[2], 2);
+          const float f1 = (hi ? f[3] : f[1]) + __shfl_xor_sync(0xffffffffu, hi ? f[1] : f[3], 2);
+          float fc = (odd ? f1 : f0) + __shfl_xor_sync(0xffffffffu, odd ? f0 : f1, 1);
+          fc += __shfl_xor_sync(0xffffffffu, fc, 4);
+          fc += __shfl_xor_sync(0xffffffffu, fc, 8);
+          const float mine = bj[jj] * (as_float(vj[jj * COLS + my_col]) - fc);
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc) {
+            const float x = __shfl_sync(0xffffffffu, mine, (lane & 16) | cc);
+            u[cc] = pack2(x, x);
+          }
+        } else {
+          float x[4];
+          Row4<T>::load(vj + jj * COLS + col0, 0, x);
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc) u[cc] = pack2(x[cc], x[cc]);
+        }
+        f32x2 oo[4] = {zero, zero, zero, zero};
+#pragma unroll
+        for (int i = 0; i < Q4; ++i) {
+          const ulonglong2 q = load(qj, i), kk = k_pair(i);
+          const f32x2 gx = fma2(kk.x, minus, one), gy = fma2(kk.y, minus, one);       // (not used by the delta rule)
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc) {
+            if constexpr (DELTA) {
+              s[cc][2 * i] = fma2(kk.x, u[cc], s[cc][2 * i]);
+              s[cc][2 * i + 1] = fma2(kk.y, u[cc], s[cc][2 * i + 1]);
+            } else {
+              s[cc][2 * i] = fma2(s[cc][2 * i], gx, mul2(kk.x, u[cc]));
+              s[cc][2 * i + 1] = fma2(s[cc][2 * i + 1], gy, mul2(kk.y, u[cc]));
+            }
+            oo[cc] = fma2(s[cc][2 * i], q.x, oo[cc]);
+            oo[cc] = fma2(s[cc][2 * i + 1], q.y, oo[cc]);
+          }
+        }
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) acc_o[jj][cc] = sum2(oo[cc]);
+      };
+      if (j0 + GROUP <= m) {
+#pragma unroll
+        for (int jj = 0; jj < GROUP; ++jj) token(jj);
+      } else {
+#pragma unroll
+        for (int jj = 0; jj < GROUP; ++jj) {
+          acc_o[jj][0] = acc_o[jj][1] = acc_o[jj][2] = acc_o[jj][3] = 0.f;
+          if (j0 + jj < m) token(jj);
         }
       }
-      // eight sums over eight lanes: lane bits 2, 1 end up choosing the token, bit 0 the column
-      float x[2][2], y[2];
+      // sixteen sums over sixteen lanes: lane bits 3, 2 end up choosing the token, bits 1, 0 the column
+      float x[2][4], y[4], z[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e)
 #pragma unroll
-        for (int cc = 0; cc < 2; ++cc)
-          x[e][cc] = (lane & 4 ? acc_o[2 + e][cc] : acc_o[e][cc]) +
-                     __shfl_xor_sync(0xffffffffu, lane & 4 ? acc_o[e][cc] : acc_o[2 + e][cc], 4);
+        for (int cc = 0; cc < 4; ++cc)
+          x[e][cc] = (lane & 8 ? acc_o[2 + e][cc] : acc_o[e][cc]) +
+                     __shfl_xor_sync(0xffffffffu, lane & 8 ? acc_o[e][cc] : acc_o[2 + e][cc], 8);
 #pragma unroll
-      for (int cc = 0; cc < 2; ++cc)
-        y[cc] = (lane & 2 ? x[1][cc] : x[0][cc]) + __shfl_xor_sync(0xffffffffu, lane & 2 ? x[0][cc] : x[1][cc], 2);
-      const float r = (lane & 1 ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, lane & 1 ? y[0] : y[1], 1);
-      const int jt = (lane >> 1) & 3;
+      for (int cc = 0; cc < 4; ++cc)
+        y[cc] = (lane & 4 ? x[1][cc] : x[0][cc]) + __shfl_xor_sync(0xffffffffu, lane & 4 ? x[0][cc] : x[1][cc], 4);
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        z[e] = (lane & 2 ? y[2 + e] : y[e]) + __shfl_xor_sync(0xffffffffu, lane & 2 ? y[e] : y[2 + e], 2);
+      const float r = (lane & 1 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, lane & 1 ? z[0] : z[1], 1);
+      const int jt = (lane >> 2) & 3;
       if (writes && j0 + jt < m) o[(c * CH + j0 + jt) * o_step] = r;
     }
   }
   if (slot < 0) return;
 #pragma unroll
-  for (int c = 0; c < 2; ++c)
+  for (int c = 0; c < 4; ++c)
 #pragma unroll
     for (int i = 0; i < Q4; ++i) {
-      const int r = i * 32 + rg * 4;
+      const int r = i * 64 + rg * 4;
       if (r < p.DP && c_base + col0 + c < p.E)
         *reinterpret_cast<ulonglong2*>(st + static_cast<long long>(c) * p.DP + r) =
             make_ulonglong2(s[c][2 * i], s[c][2 * i + 1]);
@@ -564,10 +581,10 @@ static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
 
 template <typename T, bool DELTA>
 static int pick_scan(const ScanParams& p, int B, cudaStream_t stream) {
-  if (p.DP <= 64) return launch_scan<T, 8, DELTA>(p, B, stream);
-  if (p.DP <= 128) return launch_scan<T, 16, DELTA>(p, B, stream);
-  if (p.DP <= 256) return launch_scan<T, 32, DELTA>(p, B, stream);
-  if (p.DP <= 512) return launch_scan<T, 64, DELTA>(p, B, stream);
+  if (p.DP <= 64) return launch_scan<T, 4, DELTA>(p, B, stream);
+  if (p.DP <= 128) return launch_scan<T, 8, DELTA>(p, B, stream);
+  if (p.DP <= 256) return launch_scan<T, 16, DELTA>(p, B, stream);
+  if (p.DP <= 512) return launch_scan<T, 32, DELTA>(p, B, stream);
   return -2;
 }
 

@@ -354,11 +354,16 @@ class FuviraxForCausalLM(nn.Module):
     # ---------------------------------------------------------------- weights
     def load_weights(self, weights: Iterable[Tuple[str, torch.Tensor]]) -> set:
         """Place the checkpoint's tensors (padded with zeros where the parameters are wider).  Unknown
-        names, wrong shapes and missing tensors are errors."""
+        names, wrong shapes and missing tensors are errors; what a checkpoint holds for the feed-forward
+        place of a layer without one is not used."""
         want = self._expected()
+        idle = tuple(f"l{i}.{x}" for i, layer in enumerate(self.layers) if layer.mlp is None
+                     for x in ("norm2", "ls2", "hc2."))
         loaded = set()
         for name, t in weights:
             if name not in want:
+                if idle and name.startswith(idle):
+                    continue
                 raise ValueError(f"Fuvirax: unknown tensor {name!r}")
             shape, place = want[name]
             if tuple(t.shape) != shape:

@@ -118,6 +118,9 @@ def test_wrong_checkpoints_are_refused(tmp_path):
     from omni_npu_b200.engine.trace_replay import TraceReplay
     good = cases.write_model(tmp_path, cases.VARIED)
     file = str(tmp_path / "model.safetensors")
+    # (l0 has no feed-forward: tensors in its place are idle)
+    save_file({**good, "l0.norm2": torch.ones(96), "l0.hc2.in": torch.ones(3)}, file)
+    TraceReplay(str(tmp_path), "float32", 64, device="cpu")
     for change, text in ((lambda w: w.pop("l1.mix.g2"), "missing"),
                          (lambda w: w.__setitem__("l2.mix.dt_bias", torch.zeros(2)), "unknown"),
                          (lambda w: w.__setitem__("l3.mlp.down", torch.zeros(96, 71)), "expected")):

@@ -143,8 +143,14 @@ class GatedGQAAttention(torch.nn.Module):
         k_cache, v_cache = ctx.kv_caches[self.layer_idx]
         ops.gated_rope_cache_(q, k, v, k_cache, v_cache, md.positions, md.slot_mapping, cos_sin, self.head_dim,
                               self.head_dim_v, self.rot_dim, self.neox)
+        return self._attend(q, gate, md, k_cache, v_cache, out_width)
+
+    def _attend(self, q: torch.Tensor, gate: Optional[torch.Tensor], md: AttentionMetadata, k_cache: torch.Tensor,
+                v_cache: torch.Tensor, out_width: int = 0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Attention of this step's rotated queries over the cache (into the rows ``out`` when given)."""
         t, used = q.shape[0], self.num_heads * self.head_dim_v
-        out = q.new_zeros(t, out_width) if out_width > used else q.new_empty(t, used)
+        if out is None:
+            out = q.new_zeros(t, out_width) if out_width > used else q.new_empty(t, used)
 
         def run(rows: slice, seqs: slice, cu_q, n: int, max_q: int):
             ops.gated_attention(q[rows], None if gate is None else gate[rows], k_cache, v_cache, out[rows],
@@ -163,3 +169,37 @@ class GatedGQAAttention(torch.nn.Module):
         else:
             run(slice(None), slice(None), md.cu_q, md.num_seqs, md.max_q_len)
         return out
+
+
+class NormedGQAAttention(GatedGQAAttention):
+    """The same with a norm on q and k (``ops.qk_norm_rope_cache``) and, optionally, values blended with those of
+    another layer before they are cached.  ``norm`` "projection" has weights over this rank's rows and counts
+    the rows of all ranks; ``value_mix`` is the other layer's share."""
+
+    def __init__(self, layer_idx: int, num_heads: int, num_kv_heads: int, head_dim: int, head_dim_v: int, scale: float,
+                 rot_dim: int, norm: Optional[str], eps: float, dtype, device, sliding_window: int = 0, group=None) -> None:
+        super().__init__(layer_idx, num_heads, num_kv_heads, head_dim, head_dim_v, scale, rot_dim, True, sliding_window)
+        self.norm, self.eps, self.group = norm, eps, group
+        self.q_norm = self.k_norm = None
+        if norm == "projection":
+            self.q_norm, self.k_norm = (torch.nn.Parameter(torch.ones(n * head_dim, dtype=dtype, device=device),
+                                                           requires_grad=False) for n in (num_heads, num_kv_heads))
+        self.value_mix = 0.0
+
+    def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cos_sin: torch.Tensor, out_width: int = 0,
+                v_first: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """q [T, Hq*D], k [T, Hk*D], v and ``v_first`` [T, Hk*Dv]: views into fused projections.  Returns
+        [T, max(Hq*Dv, out_width)], zero beyond the heads, or writes the rows ``out``."""
+        ctx = get_forward_context()
+        md: AttentionMetadata = ctx.attn_metadata
+        k_cache, v_cache = ctx.kv_caches[self.layer_idx]
+        sums = None
+        if self.norm == "projection" and self.group is not None and self.group.world_size > 1:
+            s = torch.stack([x.float().pow(2).sum(-1) for x in (q, k)], 1)
+            world = self.group.world_size
+            sums = self.group.all_reduce(s), q.shape[1] * world, k.shape[1] * world
+        weights = (self.q_norm, self.k_norm) if self.norm == "projection" else None
+        q = ops.qk_norm_rope_cache(q, k, v, k_cache, v_cache, md.positions, md.slot_mapping, cos_sin, self.head_dim,
+                                   self.head_dim_v, self.rot_dim, self.norm, self.eps, weights, sums, v_first,
+                                   self.value_mix)
+        return self._attend(q, None, md, k_cache, v_cache, out_width, out)

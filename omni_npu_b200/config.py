@@ -44,13 +44,17 @@ class AttentionSpec:
     sliding_window: int = 0               # 0 = every earlier key
     sink: Optional[float] = None          # score of a key without a value in every softmax
     output_gate: bool = False             # result times the sigmoid of its own projection
+    qk_norm: Optional[str] = None         # "projection": over all of q / of k before the rotation; "head": after it
+    bias: bool = False                    # of all four projections
+    value_mix: bool = False               # values blended with those of the first such layer
 
 
 @dataclass(frozen=True)
 class ExpertSpec:
-    """A gated feed-forward: width and activation ((0, 0) = silu, else slope and limit of the clamped form)."""
+    """A feed-forward: width and activation; gated for a pair of numbers ((0, 0) = silu, else slope and limit of
+    the clamped form), without a gate for a name ("relu2")."""
     intermediate_size: int
-    act: Tuple[float, float] = (0.0, 0.0)
+    act: Union[Tuple[float, float], str] = (0.0, 0.0)
 
 
 @dataclass(frozen=True)
@@ -64,6 +68,7 @@ class MoESpec:
     scale: float = 1.0
     n_group: int = 1
     topk_group: int = 1
+    correction: bool = False              # a bias per expert that takes part in the choice only
 
 
 @dataclass(frozen=True)
@@ -102,21 +107,50 @@ class DeltaRuleSpec:
 
 
 @dataclass(frozen=True)
+class DecayLinearSpec:
+    """Linear attention with a decay per head and key channel, sigmoid(low-rank projection + bias)^(1 / tau)."""
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+    tau: float
+    decay_rank: int
+
+
+@dataclass(frozen=True)
+class TimeMixSpec:
+    """Linear attention on blends with the previous token's input, with a low-rank decay per head and key
+    channel and a weight of its own for the current token."""
+    num_heads: int
+    head_dim: int
+    decay_rank: int
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Attention and time mixing side by side on one input, added with weights."""
+    left: AttentionSpec
+    right: TimeMixSpec
+    left_scale: float
+    right_scale: float
+
+
+@dataclass(frozen=True)
 class DenseSpec:
-    """A feed-forward without experts: down(act(up(h)))."""
+    """A feed-forward without experts: down(act(up(h))) ("xielu") or down(act(gate(h)) * up(h)) ("gelu_tanh")."""
     intermediate_size: int
     act: str = "xielu"
+    bias: bool = False
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    attention: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, DeltaRuleSpec]
+    attention: Union[AttentionSpec, LatentAttentionSpec, GatedLinearSpec, DeltaRuleSpec, DecayLinearSpec, ParallelSpec]
     mlp: Union[MoESpec, DenseSpec, None] = None
 
     @property
     def kv_elems(self) -> int:
         """Cached elements per token (recurrent layers keep a state per sequence instead)."""
-        a = self.attention
+        a = self.attention.left if isinstance(self.attention, ParallelSpec) else self.attention
         if isinstance(a, AttentionSpec):
             return a.num_kv_heads * (a.head_dim + a.v_head_dim)
         return a.kv_rank + a.rope_dim if isinstance(a, LatentAttentionSpec) else 0
@@ -186,6 +220,7 @@ class ModelConfig:
     embedding_scale: float = 1.0
     norm_weight_offset: float = 0.0       # 1: norm weights are stored around zero
     layer_loop: Optional[LoopSpec] = None
+    residual_mult: float = 1.0            # of what a sublayer adds to the residual
     residual_streams: int = 1             # parallel residual streams joined by hyper-connections
     logit_scale: float = 1.0
     # --- misc

@@ -31,12 +31,12 @@ int b200_argmax(const void* logits, int* out, int B, int V, long long stride, in
 int b200_sample(const void* logits, int* out, const float* temperature, const int* top_k,
                 const float* top_p, const long long* seeds, const long long* step_offset, int B,
                 int V, long long stride, int is_fp32, cudaStream_t stream);
-int b200_gemm_simt(const float* A, const float* W, float* C, int M, int N, int K, long long lda, long long ldw,
+int b200_gemm_simt(const float* A, const float* W, float* C, const float* bias, int M, int N, int K, long long lda, long long ldw,
                    long long ldc, const int* expert_offsets, int num_experts, int act, float act_alpha,
                    float act_limit, cudaStream_t stream);
 int b200_residual_norm(float* residual, long long res_stride, const int* ids, const void* table, int table_rows,
                        float table_scale, const void* a, long long a_stride, const void* b, long long b_stride,
-                       const void* y, const int* slots, const float* w, int k, const void* norm_w, float eps,
+                       const void* y, const int* slots, const float* w, int k, float mult, const void* norm_w, float eps,
                        float w_offset, void* out, long long out_stride, long long rows, int H, int n_true,
                        int is_fp32, cudaStream_t stream);
 int b200_gated_rope_cache(void* q, const void* k, const void* v, void* k_cache, void* v_cache, const int* positions,
@@ -66,10 +66,24 @@ int b200_delta_prep(const void* proj, long long stride, const void* low, long lo
 int b200_recurrent_scan(const float* q, const float* k, const float* g, const void* v, long long v_stride,
                         const float* beta, float* state, float* o, const int* state_slots, const int* cu_q,
                         const int* seq_lens, int B, int H, int G, int E, int DP, const void* proj,
-                        long long proj_stride, void* conv_state, int keep, int channels, int is_fp32,
+                        long long proj_stride, void* conv_state, int keep, int channels, int mode, int is_fp32,
                         cudaStream_t stream);
-int b200_head_norm_gate(const float* o, const void* w, const void* gate, long long gate_stride, void* out,
-                        int out_width, int T, int H, int E, float eps, int is_fp32, cudaStream_t stream);
+int b200_head_norm_gate(const float* o, const void* w, int w_step, const void* gate, long long gate_stride,
+                        int gate_silu, void* out, long long out_stride, int out_width, int T, int H, int E, float eps,
+                        float scale, int is_fp32, cudaStream_t stream);
+int b200_token_mix(const void* h, long long h_stride, const void* mu, int n, float* state, const int* seq_idx,
+                   const int* state_slots, const int* cu_q, const int* seq_lens, void* out, int* offsets, int T, int W,
+                   int is_fp32, cudaStream_t stream);
+int b200_decay_prep(const void* q, long long q_stride, const void* k, long long k_stride, const float* z,
+                    long long z_stride, const float* bias, const float* u, float* q_out, float* k_out, float* g_out,
+                    float* bonus, int T, int heads, int dim, float q_scale, float inv_tau, int is_fp32,
+                    cudaStream_t stream);
+int b200_qk_norm_rope(const void* q, const void* k, const void* v, const void* v_first, void* q_out, void* k_cache,
+                      void* v_cache, const int* positions, const int* slots, const float* cos_sin, int max_pos, int norm,
+                      const void* q_w, const void* k_w, const float* sums, int n_q, int n_k, float eps, float lambda,
+                      int T, int Hq, int Hk, int D, int DV, int DP, int DVP, int rot, long long q_stride,
+                      long long k_stride, long long v_stride, long long f_stride, int block_size, int is_fp32,
+                      cudaStream_t stream);
 int b200_latent_prep(void* q, long long q_stride, const void* kv, long long kv_stride, const void* norm_w, float eps,
                      void* cache, const int* positions, const int* slots, const float* cos_sin, int max_pos, int T,
                      int H, int dim, int rot, int rank, int row, int neox, void* q_latent, int num_latent, int is_fp32,
@@ -87,8 +101,8 @@ int b200_latent_decode(const void* q, const void* cache, void* out, const int* b
 
 namespace {
 
-// Activation kinds of the GEMM epilogues are those of gemm/gated_act.cuh; 1 and 2 join pairs of columns.
-inline bool gated(int64_t act) { return act == 1 || act == 2; }
+// Activation kinds of the GEMM epilogues are those of gemm/gated_act.cuh; 1, 2 and 4 join pairs of columns.
+inline bool gated(int64_t act) { return act == 1 || act == 2 || act == 4; }
 
 // (BN, splits, workspace bytes, counters, cluster flag) for a problem.
 std::tuple<int64_t, int64_t, int64_t, int64_t, int64_t> gemm_plan(int64_t M, int64_t N, int64_t K,
@@ -268,7 +282,7 @@ inline bool is_f32(const Tensor& t) {
 
 // fp32 A [M,K] @ W [N,K]^T; with expert_offsets W is [E,N,K] and rows belong to experts in order.
 Tensor gemm_simt(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& expert_offsets, int64_t act,
-                 double act_alpha, double act_limit) {
+                 double act_alpha, double act_limit, const c10::optional<Tensor>& bias) {
   CHECK_ROWS(a, at::kFloat);
   TORCH_CHECK(w.is_cuda() && w.scalar_type() == at::kFloat && w.is_contiguous(), "gemm_simt: fp32 weights");
   const bool grouped = expert_offsets.has_value();
@@ -279,10 +293,16 @@ Tensor gemm_simt(const Tensor& a, const Tensor& w, const c10::optional<Tensor>& 
     TORCH_CHECK(expert_offsets->numel() == E + 1, "gemm_simt: offsets [E + 1]");
   }
   const int M = a.size(0), N = w.size(-2), K = a.size(1);
+  const float* bias_p = nullptr;
+  if (bias.has_value()) {
+    TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == at::kFloat && bias->is_contiguous() && bias->numel() == N,
+                "gemm_simt: bias [N] fp32");
+    bias_p = bias->data_ptr<float>();
+  }
   c10::cuda::CUDAGuard guard(a.device());
   const int n_out = gated(act) ? N / 2 : N;
   Tensor c = torch::empty({M, n_out}, a.options());
-  check(b200_gemm_simt(a.data_ptr<float>(), w.data_ptr<float>(), c.data_ptr<float>(), M, N, K, a.stride(0), K, n_out,
+  check(b200_gemm_simt(a.data_ptr<float>(), w.data_ptr<float>(), c.data_ptr<float>(), bias_p, M, N, K, a.stride(0), K, n_out,
                        grouped ? expert_offsets->data_ptr<int>() : nullptr, E, (int)act,
                        (float)act_alpha, (float)act_limit, cur_stream()),
         "gemm_simt");
@@ -295,7 +315,7 @@ Tensor residual_norm(Tensor residual, const c10::optional<Tensor>& ids, const c1
                      double table_scale, const c10::optional<Tensor>& a, const c10::optional<Tensor>& b,
                      const c10::optional<Tensor>& y, const c10::optional<Tensor>& slots,
                      const c10::optional<Tensor>& weights, const c10::optional<Tensor>& norm_w, double eps,
-                     double w_offset, int64_t n_true, bool out_fp32) {
+                     double w_offset, int64_t n_true, bool out_fp32, double mult) {
   CHECK_ROWS(residual, at::kFloat);
   const int64_t T = residual.size(0), H = residual.size(1);
   const auto dt = out_fp32 ? at::kFloat : at::kBFloat16;
@@ -353,7 +373,7 @@ Tensor residual_norm(Tensor residual, const c10::optional<Tensor>& ids, const c1
     out = torch::empty({0, H}, residual.options().dtype(dt));
   }
   check(b200_residual_norm(residual.data_ptr<float>(), residual.stride(0), ids_p, table_p, table_rows,
-                           (float)table_scale, ap, as, bp, bs, yp, sp, wp, k, nw, (float)eps, (float)w_offset,
+                           (float)table_scale, ap, as, bp, bs, yp, sp, wp, k, (float)mult, nw, (float)eps, (float)w_offset,
                            nw ? out.data_ptr() : nullptr, H, T, (int)H, (int)n_true, out_fp32 ? 1 : 0, cur_stream()),
         "residual_norm");
   return out;
@@ -582,7 +602,7 @@ std::tuple<Tensor, Tensor, Tensor, Tensor, Tensor> delta_prep(
 Tensor recurrent_scan(const Tensor& q, const Tensor& k, const c10::optional<Tensor>& g, const Tensor& v,
                       const c10::optional<Tensor>& beta, Tensor state, int64_t heads, int64_t vdim,
                       const Tensor& state_slots, const Tensor& cu_q, const Tensor& seq_lens, int64_t num_seqs,
-                      const c10::optional<Tensor>& proj, const c10::optional<Tensor>& conv_state) {
+                      const c10::optional<Tensor>& proj, const c10::optional<Tensor>& conv_state, bool bonus) {
   CHECK_F32(q);
   CHECK_F32(k);
   CHECK_F32(state);
@@ -596,12 +616,17 @@ Tensor recurrent_scan(const Tensor& q, const Tensor& k, const c10::optional<Tens
   TORCH_CHECK(v.size(0) == T && v.size(1) == heads * vdim && state.dim() == 4 && state.size(1) == heads &&
                   state.size(2) == vdim && state.size(3) == DP && heads % G == 0 && state_slots.numel() >= num_seqs &&
                   cu_q.numel() >= num_seqs + 1 && seq_lens.numel() >= num_seqs, "recurrent_scan: shapes");
-  TORCH_CHECK(g.has_value() == beta.has_value(), "recurrent_scan: decays and step sizes come together");
+  TORCH_CHECK(g.has_value() || !beta.has_value(), "recurrent_scan: beta without decays");
+  TORCH_CHECK(!bonus || beta.has_value(), "recurrent_scan: the bonus comes in beta");
   if (g.has_value()) {
     CHECK_F32(*g);
-    CHECK_F32(*beta);
-    TORCH_CHECK(g->numel() == T * heads * DP && beta->numel() == T * heads, "recurrent_scan: g [T, H, d], beta [T, H]");
+    TORCH_CHECK(g->numel() == T * heads * DP, "recurrent_scan: g [T, H, d]");
   }
+  if (beta.has_value()) {
+    CHECK_F32(*beta);
+    TORCH_CHECK(beta->numel() == T * heads, "recurrent_scan: beta [T, H]");
+  }
+  const int mode = !g.has_value() ? 0 : !beta.has_value() ? 2 : bonus ? 3 : 1;
   const void* proj_p = nullptr;
   void* cs = nullptr;
   long long ps = 0;
@@ -623,18 +648,20 @@ Tensor recurrent_scan(const Tensor& q, const Tensor& k, const c10::optional<Tens
                             v.data_ptr(), v.stride(0), beta.has_value() ? beta->data_ptr<float>() : nullptr,
                             state.data_ptr<float>(), o.data_ptr<float>(), state_slots.data_ptr<int>(),
                             cu_q.data_ptr<int>(), seq_lens.data_ptr<int>(), (int)num_seqs, (int)heads, (int)G,
-                            (int)vdim, (int)DP, proj_p, ps, cs, keep, channels, f32 ? 1 : 0, cur_stream()),
+                            (int)vdim, (int)DP, proj_p, ps, cs, keep, channels, mode, f32 ? 1 : 0, cur_stream()),
         "recurrent_scan");
   return o;
 }
 
+// weight [E] for all heads or [H, E]; out (rows [T, >= H * E], any pitch) is written when given
 Tensor head_norm_gate(const Tensor& o, const Tensor& weight, double eps, const c10::optional<Tensor>& gate,
-                      int64_t out_width) {
+                      int64_t out_width, bool gate_silu, double scale, const c10::optional<Tensor>& out_rows) {
   CHECK_F32(o);
   const auto dt = weight.scalar_type();
   const bool f32 = is_f32(weight);
-  TORCH_CHECK(o.dim() == 3 && out_width >= o.size(1) * o.size(2), "head_norm_gate: o [T, H, E]");
-  CHECK_VEC(weight, dt, o.size(2));
+  TORCH_CHECK(o.dim() == 3, "head_norm_gate: o [T, H, E]");
+  const bool per_head = weight.dim() == 2;
+  CHECK_VEC(weight, dt, per_head ? o.size(1) * o.size(2) : o.size(2));
   const void* gp = nullptr;
   long long gs = 0;
   if (gate.has_value()) {
@@ -644,10 +671,118 @@ Tensor head_norm_gate(const Tensor& o, const Tensor& weight, double eps, const c
     gs = gate->stride(0);
   }
   c10::cuda::CUDAGuard guard(o.device());
-  Tensor out = torch::empty({o.size(0), out_width}, weight.options());
-  check(b200_head_norm_gate(o.data_ptr<float>(), weight.data_ptr(), gp, gs, out.data_ptr(), (int)out_width,
-                            (int)o.size(0), (int)o.size(1), (int)o.size(2), (float)eps, f32 ? 1 : 0, cur_stream()),
+  Tensor out = out_rows.has_value() ? *out_rows : torch::empty({o.size(0), out_width}, weight.options());
+  CHECK_ROWS(out, dt);
+  TORCH_CHECK(out.size(0) == o.size(0) && out.size(1) >= o.size(1) * o.size(2), "head_norm_gate: out [T, >= H * E]");
+  check(b200_head_norm_gate(o.data_ptr<float>(), weight.data_ptr(), per_head ? (int)o.size(2) : 0, gp, gs,
+                            gate_silu ? 1 : 0, out.data_ptr(), out.stride(0), (int)out.size(1), (int)o.size(0),
+                            (int)o.size(1), (int)o.size(2), (float)eps, (float)scale, f32 ? 1 : 0, cur_stream()),
         "head_norm_gate");
+  return out;
+}
+
+// Rows h_t + (h_(t-1) - h_t) mu_s, one blend after another: (rows [n * T, W], offsets [n + 1]).
+std::tuple<Tensor, Tensor> token_mix(const Tensor& h, const Tensor& mu, Tensor state, const Tensor& seq_idx,
+                                     const Tensor& state_slots, const Tensor& cu_q, const Tensor& seq_lens) {
+  const auto dt = h.scalar_type();
+  const bool f32 = is_f32(h);
+  CHECK_ROWS(h, dt);
+  CHECK_F32(state);
+  CHECK_I32(seq_idx);
+  CHECK_I32(state_slots);
+  CHECK_I32(cu_q);
+  CHECK_I32(seq_lens);
+  const int64_t T = h.size(0), W = h.size(1), n = mu.size(0);
+  TORCH_CHECK(mu.is_cuda() && mu.scalar_type() == dt && mu.is_contiguous() && mu.dim() == 2 && mu.size(1) == W &&
+                  state.dim() == 2 && state.size(1) == W && seq_idx.numel() >= T, "token_mix: shapes");
+  c10::cuda::CUDAGuard guard(h.device());
+  Tensor out = torch::empty({n * T, W}, h.options()), offsets = torch::empty({n + 1}, cu_q.options());
+  check(b200_token_mix(h.data_ptr(), h.stride(0), mu.data_ptr(), (int)n, state.data_ptr<float>(),
+                       seq_idx.data_ptr<int>(), state_slots.data_ptr<int>(), cu_q.data_ptr<int>(),
+                       seq_lens.data_ptr<int>(), out.data_ptr(), offsets.data_ptr<int>(), (int)T, (int)W, f32 ? 1 : 0,
+                       cur_stream()),
+        "token_mix");
+  return {out, offsets};
+}
+
+// u given: time mixing (q, k, decays, bonus); else (q * q_scale, k, decays, empty).
+std::tuple<Tensor, Tensor, Tensor, Tensor> decay_prep(const Tensor& q, const Tensor& k, const Tensor& z,
+                                                      const Tensor& bias, const c10::optional<Tensor>& u, int64_t heads,
+                                                      int64_t dim, double q_scale, double inv_tau) {
+  const auto dt = q.scalar_type();
+  const bool f32 = is_f32(q);
+  CHECK_ROWS(q, dt);
+  CHECK_ROWS(k, dt);
+  CHECK_ROWS(z, at::kFloat);
+  CHECK_F32(bias);
+  const int64_t T = q.size(0), n = heads * dim, DP = (dim + 3) / 4 * 4;
+  TORCH_CHECK(q.size(1) >= n && k.size(0) == T && k.size(1) >= n && z.size(0) == T && z.size(1) >= n &&
+                  bias.numel() == n, "decay_prep: shapes");
+  if (u.has_value()) {
+    CHECK_F32(*u);
+    TORCH_CHECK(u->numel() == n, "decay_prep: u [heads, dim]");
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor qo = torch::empty({T, heads, DP}, bias.options()), ko = torch::empty_like(qo), go = torch::empty_like(qo);
+  Tensor bonus = torch::empty({u.has_value() ? T : 0, heads}, bias.options());
+  check(b200_decay_prep(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), z.data_ptr<float>(), z.stride(0),
+                        bias.data_ptr<float>(), u.has_value() ? u->data_ptr<float>() : nullptr, qo.data_ptr<float>(),
+                        ko.data_ptr<float>(), go.data_ptr<float>(), bonus.data_ptr<float>(), (int)T, (int)heads,
+                        (int)dim, (float)q_scale, (float)inv_tau, f32 ? 1 : 0, cur_stream()),
+        "decay_prep");
+  return {qo, ko, go, bonus};
+}
+
+// norm: 0 none, 1 over the whole projections (weights; sums of squares [T, 2] over n_q / n_k elements when they
+// were taken elsewhere), 2 per head.  Returns the queries [T, Hq * D].
+Tensor qk_norm_rope(const Tensor& q, const Tensor& k, const Tensor& v, const c10::optional<Tensor>& v_first,
+                    double lambda, Tensor k_cache, Tensor v_cache, const Tensor& positions, const Tensor& slots,
+                    const Tensor& cos_sin, int64_t head_dim, int64_t head_dim_v, int64_t rot, int64_t norm,
+                    const c10::optional<Tensor>& q_w, const c10::optional<Tensor>& k_w,
+                    const c10::optional<Tensor>& sums, int64_t n_q, int64_t n_k, double eps) {
+  const auto dt = q.scalar_type();
+  const bool f32 = is_f32(q);
+  CHECK_ROWS(q, dt);
+  CHECK_ROWS(k, dt);
+  CHECK_ROWS(v, dt);
+  CHECK_I32(positions);
+  CHECK_I32(slots);
+  check_gated_caches(k_cache, v_cache, dt, head_dim, head_dim_v);
+  const int T = q.size(0), Hk = k_cache.size(1);
+  TORCH_CHECK(positions.numel() >= T && slots.numel() >= T && q.size(1) % head_dim == 0 && k.size(0) == T &&
+                  v.size(0) == T && k.size(1) == Hk * head_dim && v.size(1) == Hk * head_dim_v, "qk_norm_rope: shapes");
+  TORCH_CHECK(cos_sin.is_cuda() && cos_sin.scalar_type() == at::kFloat && cos_sin.is_contiguous() &&
+                  cos_sin.dim() == 2 && cos_sin.size(1) == rot, "qk_norm_rope: cos_sin [max_pos, rot] fp32");
+  const void *qw = nullptr, *kw = nullptr, *vf = nullptr;
+  const float* sp = nullptr;
+  long long fs = 0;
+  if (norm == 1) {
+    TORCH_CHECK(q_w.has_value() && k_w.has_value(), "qk_norm_rope: norm weights");
+    CHECK_VEC(*q_w, dt, q.size(1));
+    CHECK_VEC(*k_w, dt, k.size(1));
+    qw = q_w->data_ptr();
+    kw = k_w->data_ptr();
+    if (sums.has_value()) {
+      CHECK_F32(*sums);
+      TORCH_CHECK(sums->numel() == 2 * T, "qk_norm_rope: sums [T, 2]");
+      sp = sums->data_ptr<float>();
+    }
+  }
+  if (v_first.has_value()) {
+    CHECK_ROWS(*v_first, dt);
+    TORCH_CHECK(v_first->size(0) == T && v_first->size(1) == v.size(1), "qk_norm_rope: v_first like v");
+    vf = v_first->data_ptr();
+    fs = v_first->stride(0);
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = torch::empty({T, q.size(1)}, q.options());
+  check(b200_qk_norm_rope(q.data_ptr(), k.data_ptr(), v.data_ptr(), vf, out.data_ptr(), k_cache.data_ptr(),
+                          v_cache.data_ptr(), positions.data_ptr<int>(), slots.data_ptr<int>(), cos_sin.data_ptr<float>(),
+                          (int)cos_sin.size(0), (int)norm, qw, kw, sp, (int)n_q, (int)n_k, (float)eps, (float)lambda, T,
+                          (int)(q.size(1) / head_dim), Hk, (int)head_dim, (int)head_dim_v, (int)k_cache.size(3),
+                          (int)v_cache.size(3), (int)rot, q.stride(0), k.stride(0), v.stride(0), fs,
+                          (int)k_cache.size(2), f32 ? 1 : 0, cur_stream()),
+        "qk_norm_rope");
   return out;
 }
 
@@ -763,6 +898,9 @@ TORCH_LIBRARY(omni_b200, m) {
   m.def("delta_prep", &delta_prep);
   m.def("recurrent_scan", &recurrent_scan);
   m.def("head_norm_gate", &head_norm_gate);
+  m.def("token_mix", &token_mix);
+  m.def("decay_prep", &decay_prep);
+  m.def("qk_norm_rope", &qk_norm_rope);
   m.def("latent_prep", &latent_prep);
   m.def("head_gemm", &head_gemm);
   m.def("latent_gather", &latent_gather);

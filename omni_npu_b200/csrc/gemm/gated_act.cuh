@@ -4,17 +4,30 @@
 
 namespace b200 {
 
-enum : int { kActNone = 0, kActSilu = 1, kActClampedGlu = 2, kActXielu = 3 };
+enum : int { kActNone = 0, kActSilu = 1, kActClampedGlu = 2, kActXielu = 3, kActGeluTanh = 4, kActRelu2 = 5, kActTanh = 6 };
 
 //   kActSilu        silu(g) * u
 //   kActClampedGlu  g' * sigmoid(alpha * g') * (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+//   kActGeluTanh    g / 2 * (1 + tanh(z)) * u = g * sigmoid(2 z) * u with z = sqrt(2 / pi) (g + 0.044715 g^3)
+__device__ __forceinline__ float gelu_exponent(float g) {
+  return -1.5957691216057308f * fmaf(0.044715f * g * g, g, g);       // -2 z
+}
 __device__ __forceinline__ float gated_act(int kind, float g, float u, float alpha, float limit) {
   if (kind == kActClampedGlu) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + __expf(-alpha * g)) * (u + 1.f);
   }
-  return (g / (1.f + __expf(-g))) * u;
+  return g / (1.f + __expf(kind == kActGeluTanh ? gelu_exponent(g) : -g)) * u;
+}
+// the same with the exact fp32 functions, for products that are not rounded to bf16
+__device__ __forceinline__ float gated_act_exact(int kind, float g, float u, float alpha, float limit) {
+  if (kind == kActClampedGlu) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+  }
+  return g / (1.f + expf(kind == kActGeluTanh ? gelu_exponent(g) : -g)) * u;
 }
 
 //   kActXielu       z > 0: alpha * z^2 + z / 2;  z <= 0: limit * (exp(z) - 1 - z) + z / 2
@@ -29,7 +42,31 @@ __device__ __forceinline__ float xielu_exact(float z, float alpha, float limit) 
   return fmaf(0.5f, z, a);
 }
 
-// Whether a kind joins pairs of columns (half as many come out).
-__host__ __device__ __forceinline__ bool act_is_gated(int kind) { return kind == kActSilu || kind == kActClampedGlu; }
+// Activations of single columns:
+//   kActRelu2       max(z, 0)^2
+//   kActTanh        tanh(z) = 1 - 2 / (exp(2 z) + 1) (absolute error 2e-7)
+__device__ __forceinline__ float unary_act(int kind, float z, float alpha, float limit) {
+  if (kind == kActRelu2) {
+    z = fmaxf(z, 0.f);
+    return z * z;
+  }
+  if (kind == kActTanh) return 1.f - 2.f / (__expf(2.f * fminf(z, 40.f)) + 1.f);
+  return xielu(z, alpha, limit);
+}
+__device__ __forceinline__ float unary_act_exact(int kind, float z, float alpha, float limit) {
+  if (kind == kActRelu2) {
+    z = fmaxf(z, 0.f);
+    return z * z;
+  }
+  return kind == kActTanh ? tanhf(z) : xielu_exact(z, alpha, limit);
+}
+
+// Whether a kind joins pairs of columns (half as many come out), or works on single ones.
+__host__ __device__ __forceinline__ bool act_is_gated(int kind) {
+  return kind == kActSilu || kind == kActClampedGlu || kind == kActGeluTanh;
+}
+__host__ __device__ __forceinline__ bool act_is_unary(int kind) {
+  return kind == kActXielu || kind == kActRelu2 || kind == kActTanh;
+}
 
 }  // namespace b200

@@ -24,7 +24,8 @@ struct SimtGemmParams {
   long long lda, ldw, ldc;
   const int* expert_offsets;   // grouped: [E + 1] row offsets into A / C, W is [E, N, K]; null = dense
   int num_experts;
-  int act;                     // gated activation (gate / up columns interleaved in groups of eight)
+  const float* bias;           // [N] or null: added before a gated activation, after a unary one
+  int act;                     // activation (gated: gate / up columns interleaved in groups of eight)
   float act_alpha, act_limit;
 };
 
@@ -97,7 +98,10 @@ __global__ void __launch_bounds__(simt::THREADS) gemm_simt_kernel(const SimtGemm
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int col = n0 + tx * 4 + j;
-        if (col < p.N) p.C[row * p.ldc + col] = p.act == kActXielu ? xielu_exact(acc[i][j], p.act_alpha, p.act_limit) : acc[i][j];
+        if (col >= p.N) continue;
+        float x = acc[i][j];
+        if (act_is_unary(p.act)) x = unary_act_exact(p.act, x, p.act_alpha, p.act_limit);
+        p.C[row * p.ldc + col] = p.bias ? x + p.bias[col] : x;
       }
     }
     return;
@@ -110,8 +114,14 @@ __global__ void __launch_bounds__(simt::THREADS) gemm_simt_kernel(const SimtGemm
   for (int idx = tid; idx < BM * BN / 2; idx += THREADS) {
     const int r = idx / (BN / 2), o = idx % (BN / 2);
     const int c = (o >> 3) * 16 + (o & 7);              // gate column of output column o
-    if (m0 + r < m1 && n0 + c + 8 < p.N)
-      p.C[(m0 + r) * p.ldc + n0 / 2 + o] = gated_act(p.act, sC[r][c], sC[r][c + 8], p.act_alpha, p.act_limit);
+    if (m0 + r < m1 && n0 + c + 8 < p.N) {
+      float g = sC[r][c], u = sC[r][c + 8];
+      if (p.bias) {
+        g += p.bias[n0 + c];
+        u += p.bias[n0 + c + 8];
+      }
+      p.C[(m0 + r) * p.ldc + n0 / 2 + o] = gated_act_exact(p.act, g, u, p.act_alpha, p.act_limit);
+    }
   }
 }
 
@@ -119,12 +129,12 @@ __global__ void __launch_bounds__(simt::THREADS) gemm_simt_kernel(const SimtGemm
 
 using namespace b200;
 
-extern "C" int b200_gemm_simt(const float* A, const float* W, float* C, int M, int N, int K, long long lda,
+extern "C" int b200_gemm_simt(const float* A, const float* W, float* C, const float* bias, int M, int N, int K, long long lda,
                               long long ldw, long long ldc, const int* expert_offsets, int num_experts, int act,
                               float act_alpha, float act_limit, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (act_is_gated(act) && (N % 16) != 0) return -11;
-  SimtGemmParams p{A, W, C, M, N, K, lda, ldw, ldc, expert_offsets, num_experts, act, act_alpha, act_limit};
+  SimtGemmParams p{A, W, C, M, N, K, lda, ldw, ldc, expert_offsets, num_experts, bias, act, act_alpha, act_limit};
   // grouped: every expert may end in a partly filled tile
   const long long tiles = (M + simt::BM - 1) / simt::BM + (expert_offsets ? num_experts : 0);
   if (tiles > 65535) return -12;

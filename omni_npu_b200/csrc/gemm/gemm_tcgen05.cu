@@ -732,9 +732,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               }
               return;
             }
-            if (p.swiglu == kActXielu) {
+            if (act_is_unary(p.swiglu)) {
 #pragma unroll
-              for (int i = 0; i < 4; ++i) v[i] = xielu(v[i], p.act_alpha, p.act_limit);
+              for (int i = 0; i < 4; ++i) v[i] = unary_act(p.swiglu, v[i], p.act_alpha, p.act_limit);
             }
             for (int i = 0; i < ncols; ++i) {
               if (p.bias) v[i] += __bfloat162float(p.bias[col + i]);
@@ -913,12 +913,16 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
           }
           continue;
         }
-        if (p.swiglu == kActXielu) {
+        if (act_is_unary(p.swiglu)) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) v[i] = xielu(v[i], p.act_alpha, p.act_limit);
+          for (int i = 0; i < 16; ++i) v[i] = unary_act(p.swiglu, v[i], p.act_alpha, p.act_limit);
         } else if (p.swiglu) {
-          // Columns [c, c+8) hold gate values, [c+8, c+16) the matching up values.
+          // Columns [c, c+8) hold gate values, [c+8, c+16) the matching up values (N is a multiple of 16).
           const int ocol = col >> 1;
+          if (p.bias) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) v[i] += __bfloat162float(p.bias[col + i]);
+          }
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {

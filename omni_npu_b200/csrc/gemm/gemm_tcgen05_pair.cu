@@ -319,11 +319,15 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
         for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
         const int col = n0 + c;
         if (!row_ok || col >= p.N) continue;
-        if (p.swiglu == kActXielu) {
+        if (act_is_unary(p.swiglu)) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) v[i] = xielu(v[i], p.act_alpha, p.act_limit);
+          for (int i = 0; i < 16; ++i) v[i] = unary_act(p.swiglu, v[i], p.act_alpha, p.act_limit);
         } else if (p.swiglu) {
           const int ocol = col >> 1;
+          if (p.bias) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) v[i] += __bfloat162float(p.bias[col + i]);
+          }
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {

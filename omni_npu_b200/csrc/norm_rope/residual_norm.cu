@@ -1,7 +1,7 @@
 // The end of one layer and the start of the next on a 32-bit residual stream, in one pass per token:
 //
 //   residual  = scale * table[id]                       (start of the model), or
-//   residual += a + b + sum_j w_j * y[slot_j]           (end of a layer)
+//   residual += mult * (a + b + sum_j w_j * y[slot_j])  (end of a sublayer)
 //   out       = residual / sqrt(mean(residual^2) + eps) * (w_offset + norm_w)
 //
 // a, b: dense sublayer outputs (either may be absent); y, slots, w: the rows that a mixture of
@@ -37,6 +37,7 @@ struct ResidualNormParams {
   const int* slots;            // [T, k] row of y per chosen expert (< 0: none)
   const float* w;              // [T, k]
   int k;
+  float mult;                  // of everything that is added
   const void* norm_w;
   float eps;
   float w_offset;
@@ -104,7 +105,7 @@ __global__ void __launch_bounds__(kResThreads) residual_norm_kernel(const Residu
       }
       Row8<float>::load(res, v, x[i]);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) x[i][j] += add[j];
+      for (int j = 0; j < 8; ++j) x[i][j] = fmaf(p.mult, add[j], x[i][j]);
     }
     Row8<float>::store(res, v, x[i]);
 #pragma unroll
@@ -153,7 +154,7 @@ using namespace b200;
 extern "C" int b200_residual_norm(float* residual, long long res_stride, const int* ids, const void* table,
                                   int table_rows, float table_scale, const void* a, long long a_stride,
                                   const void* b, long long b_stride, const void* y, const int* slots,
-                                  const float* w, int k, const void* norm_w, float eps, float w_offset, void* out,
+                                  const float* w, int k, float mult, const void* norm_w, float eps, float w_offset, void* out,
                                   long long out_stride, long long rows, int H, int n_true, int is_fp32,
                                   cudaStream_t stream) {
   if (rows <= 0) return 0;
@@ -173,6 +174,7 @@ extern "C" int b200_residual_norm(float* residual, long long res_stride, const i
   p.slots = slots;
   p.w = w;
   p.k = k;
+  p.mult = mult;
   p.norm_w = norm_w;
   p.eps = eps;
   p.w_offset = w_offset;

@@ -1,10 +1,13 @@
 // Recurrent layers: a matrix S per sequence and head, fp32, carried from token to token.
 //
 //   S <- diag(g) S;  S <- S + k u^T;  o = S^T q
-//   gated linear attention:  u = v,                   k = 1 - g
-//   delta rule:              u = beta (v - S^T k)     (after the decay)
+//   tied:    u = v,                   k = 1 - g
+//   delta:   u = beta (v - S^T k)     (after the decay)
+//   decay:   u = v,                   g free
+//   bonus:   as decay, but o = S^T q + beta v of the S before this token (beta: the current token's weight)
 //
-// One elementwise kernel per kind prepares q, k, g and beta in fp32 from the projections, the scan runs
+// One elementwise kernel per kind prepares q, k, g and beta in fp32 from the projections (here and in
+// decay_prep.cu), the scan runs
 // the recurrence over a step's tokens (any mixture of prompt portions and single tokens), a last kernel
 // norms each head's result and applies the output gate.  This file is compiled without the fast-math
 // flag: what enters a recurrence keeps the accuracy of the fp32 functions.
@@ -16,12 +19,9 @@
 #include "../common/device_once.h"
 #include "../common/pdl.cuh"
 #include "../common/rows.cuh"
+#include "recurrent_common.cuh"
 
 namespace b200 {
-
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // ------------------------------------------------------------- gated linear attention: q and keys
 struct GatedPrepParams {
@@ -276,10 +276,10 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const Delta
 struct ScanParams {
   const float* q;              // [T, G, DP]
   const float* k;              // [T, G, DP]
-  const float* g;              // [T, H, DP] (delta rule)
+  const float* g;              // [T, H, DP] (not tied)
   const void* v;               // [T, H * E], row pitch v_stride
   long long v_stride;
-  const float* beta;           // [T, H] (delta rule)
+  const float* beta;           // [T, H] (delta, bonus)
   float* state;                // [slots, H, E, DP]
   float* o;                    // [T, H, E]
   const int* state_slots;
@@ -294,11 +294,12 @@ struct ScanParams {
 
 namespace scan {
 constexpr int WARPS = 4, THREADS = WARPS * 32, COLS = 32, GROUP = 4;
-template <int RPT, bool DELTA>
+enum : int { TIED = 0, DELTA = 1, DECAY = 2, BONUS = 3 };
+template <int RPT, int MODE>
 struct Cfg {
   static constexpr int ROWS = 16 * RPT;
   static constexpr int CH = RPT <= 8 ? 16 : RPT <= 16 ? 8 : 4;
-  static constexpr int ARR = DELTA ? 3 : 2;
+  static constexpr int ARR = MODE == TIED ? 2 : 3;
   static constexpr int STAGE = ARR * CH * ROWS;                     // floats
   static constexpr int SMEM = (2 * STAGE + 2 * CH * (COLS + 1)) * 4;
 };
@@ -336,10 +337,10 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
   return d;
 }
 
-template <typename T, int RPT, bool DELTA>
+template <typename T, int RPT, int MODE>
 __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const ScanParams p) {
   using namespace scan;
-  using C = Cfg<RPT, DELTA>;
+  using C = Cfg<RPT, MODE>;
   constexpr int CH = C::CH, ROWS = C::ROWS, Q4 = RPT / 4;
   constexpr bool KEEP_K = RPT <= 16;                      // k of a token in registers between its two uses
   extern __shared__ __align__(16) float smem[];
@@ -395,7 +396,7 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
         dv[i] = c_base + col < p.E ? v_src[(t0 + j) * p.v_stride + col] : from_float<T>(0.f);
       }
     }
-    if (DELTA && tid < m) cp_async4(s_b + (c & 1) * CH + tid, p.beta + (begin + t0 + tid) * p.H + h);
+    if ((MODE == DELTA || MODE == BONUS) && tid < m) cp_async4(s_b + (c & 1) * CH + tid, p.beta + (begin + t0 + tid) * p.H + h);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   stage(0);
@@ -453,7 +454,7 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
           else return load(kj, i);
         };
         f32x2 u[4];                                       // of the four columns, in both halves
-        if constexpr (DELTA) {
+        if constexpr (MODE == DELTA) {
           f32x2 acc[4] = {zero, zero, zero, zero};
 #pragma unroll
           for (int i = 0; i < Q4; ++i) {
@@ -492,18 +493,32 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
 #pragma unroll
         for (int i = 0; i < Q4; ++i) {
           const ulonglong2 q = load(qj, i), kk = k_pair(i);
-          const f32x2 gx = fma2(kk.x, minus, one), gy = fma2(kk.y, minus, one);       // (not used by the delta rule)
+          f32x2 gx = zero, gy = zero;
+          if constexpr (MODE == TIED) {
+            gx = fma2(kk.x, minus, one);
+            gy = fma2(kk.y, minus, one);
+          } else if constexpr (MODE != DELTA) {
+            const ulonglong2 g = load(gj, i);
+            gx = g.x;
+            gy = g.y;
+          }
 #pragma unroll
           for (int cc = 0; cc < 4; ++cc) {
-            if constexpr (DELTA) {
+            if constexpr (MODE == BONUS) {                // the state before this token is read
+              oo[cc] = fma2(s[cc][2 * i], q.x, oo[cc]);
+              oo[cc] = fma2(s[cc][2 * i + 1], q.y, oo[cc]);
+            }
+            if constexpr (MODE == DELTA) {
               s[cc][2 * i] = fma2(kk.x, u[cc], s[cc][2 * i]);
               s[cc][2 * i + 1] = fma2(kk.y, u[cc], s[cc][2 * i + 1]);
             } else {
               s[cc][2 * i] = fma2(s[cc][2 * i], gx, mul2(kk.x, u[cc]));
               s[cc][2 * i + 1] = fma2(s[cc][2 * i + 1], gy, mul2(kk.y, u[cc]));
             }
-            oo[cc] = fma2(s[cc][2 * i], q.x, oo[cc]);
-            oo[cc] = fma2(s[cc][2 * i + 1], q.y, oo[cc]);
+            if constexpr (MODE != BONUS) {
+              oo[cc] = fma2(s[cc][2 * i], q.x, oo[cc]);
+              oo[cc] = fma2(s[cc][2 * i + 1], q.y, oo[cc]);
+            }
           }
         }
 #pragma unroll
@@ -533,8 +548,9 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
 #pragma unroll
       for (int e = 0; e < 2; ++e)
         z[e] = (lane & 2 ? y[2 + e] : y[e]) + __shfl_xor_sync(0xffffffffu, lane & 2 ? y[e] : y[2 + e], 2);
-      const float r = (lane & 1 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, lane & 1 ? z[0] : z[1], 1);
+      float r = (lane & 1 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, lane & 1 ? z[0] : z[1], 1);
       const int jt = (lane >> 2) & 3;
+      if constexpr (MODE == BONUS) r = fmaf(bj[jt], as_float(vj[jt * COLS + my_col]), r);
       if (writes && j0 + jt < m) o[(c * CH + j0 + jt) * o_step] = r;
     }
   }
@@ -565,10 +581,10 @@ __global__ void __launch_bounds__(scan::THREADS) recurrent_scan_kernel(const Sca
   }
 }
 
-template <typename T, int RPT, bool DELTA>
+template <typename T, int RPT, int MODE>
 static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
-  auto kern = recurrent_scan_kernel<T, RPT, DELTA>;
-  constexpr int smem = scan::Cfg<RPT, DELTA>::SMEM;
+  auto kern = recurrent_scan_kernel<T, RPT, MODE>;
+  constexpr int smem = scan::Cfg<RPT, MODE>::SMEM;
   static DeviceOnce once;
   int dev = 0;
   if (once.needed(&dev)) {
@@ -579,24 +595,38 @@ static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
   return launch_pdl(kern, grid, dim3(scan::THREADS), smem, stream, 1, p) == cudaSuccess ? 0 : -21;
 }
 
-template <typename T, bool DELTA>
+template <typename T, int MODE>
 static int pick_scan(const ScanParams& p, int B, cudaStream_t stream) {
-  if (p.DP <= 64) return launch_scan<T, 4, DELTA>(p, B, stream);
-  if (p.DP <= 128) return launch_scan<T, 8, DELTA>(p, B, stream);
-  if (p.DP <= 256) return launch_scan<T, 16, DELTA>(p, B, stream);
-  if (p.DP <= 512) return launch_scan<T, 32, DELTA>(p, B, stream);
+  if (p.DP <= 64) return launch_scan<T, 4, MODE>(p, B, stream);
+  if (p.DP <= 128) return launch_scan<T, 8, MODE>(p, B, stream);
+  if (p.DP <= 256) return launch_scan<T, 16, MODE>(p, B, stream);
+  if (p.DP <= 512) return launch_scan<T, 32, MODE>(p, B, stream);
+  return -2;
+}
+
+template <typename T>
+static int scan_mode(const ScanParams& p, int mode, int B, cudaStream_t stream) {
+  switch (mode) {
+    case scan::TIED: return pick_scan<T, scan::TIED>(p, B, stream);
+    case scan::DELTA: return pick_scan<T, scan::DELTA>(p, B, stream);
+    case scan::DECAY: return pick_scan<T, scan::DECAY>(p, B, stream);
+    case scan::BONUS: return pick_scan<T, scan::BONUS>(p, B, stream);
+  }
   return -2;
 }
 
 // ------------------------------------------------------------- norm and gate of a head's result
 struct HeadNormParams {
   const float* o;              // [T, H, E]
-  const void* w;               // [E]
-  const void* gate;            // [T, H * E] before the sigmoid, or null
+  const void* w;               // [E], or [H, E] (w_step = E)
+  int w_step;
+  const void* gate;            // [T, H * E] before its activation, or null
   long long gate_stride;
-  void* out;                   // [T, out_width]
+  int gate_silu;               // silu instead of sigmoid
+  void* out;                   // [T, out_width], row pitch out_stride
+  long long out_stride;
   int out_width, T, H, E;
-  float eps;
+  float eps, scale;
   int vec;                     // rows are whole four-element pieces
 };
 
@@ -612,9 +642,10 @@ __global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_kernel(const He
   const long long t = unit / p.H;
   const int h = static_cast<int>(unit - t * p.H);
   const float* o = p.o + unit * p.E;
-  const T* w = static_cast<const T*>(p.w);
+  const T* w = static_cast<const T*>(p.w) + h * p.w_step;
   const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_stride + static_cast<long long>(h) * p.E : nullptr;
-  T* dst = static_cast<T*>(p.out) + t * p.out_width;
+  T* dst = static_cast<T*>(p.out) + t * p.out_stride;
+  const bool silu = p.gate_silu != 0;
   float ss = 0.f;
   if (p.vec) {                                            // up to 512 columns, four at a time in registers
     float x[4][4], g[4][4];
@@ -630,7 +661,7 @@ __global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_kernel(const He
     }
 #pragma unroll
     for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
-    const float inv = 1.f / sqrtf(ss / static_cast<float>(p.E) + p.eps);
+    const float inv = p.scale / sqrtf(ss / static_cast<float>(p.E) + p.eps);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int v = lane + 32 * i;
@@ -640,7 +671,7 @@ __global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_kernel(const He
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           x[i][j] *= inv * ww[j];
-          if (gate) x[i][j] *= quick_sigmoid(g[i][j]);
+          if (gate) x[i][j] *= quick_sigmoid(g[i][j]) * (silu ? g[i][j] : 1.f);
         }
         Row4<T>::store(dst + h * p.E, v, x[i]);
       }
@@ -649,10 +680,10 @@ __global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_kernel(const He
     for (int d = lane; d < p.E; d += 32) ss = fmaf(o[d], o[d], ss);
 #pragma unroll
     for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
-    const float inv = 1.f / sqrtf(ss / static_cast<float>(p.E) + p.eps);
+    const float inv = p.scale / sqrtf(ss / static_cast<float>(p.E) + p.eps);
     for (int d = lane; d < p.E; d += 32) {
       float y = o[d] * inv * as_float(w[d]);
-      if (gate) y *= quick_sigmoid(as_float(gate[d]));
+      if (gate) y *= quick_sigmoid(as_float(gate[d])) * (silu ? as_float(gate[d]) : 1.f);
       dst[h * p.E + d] = from_float<T>(y);
     }
   }
@@ -723,28 +754,29 @@ extern "C" int b200_delta_prep(const void* proj, long long stride, const void* l
   return e == cudaSuccess ? 0 : -3;
 }
 
-// g and beta null: gated linear attention.  Head sizes (rows) up to 512.
+// mode: 0 tied (g and beta null), 1 delta, 2 decay (beta null), 3 bonus.  Head sizes (rows) up to 512.
 extern "C" int b200_recurrent_scan(const float* q, const float* k, const float* g, const void* v, long long v_stride,
                                    const float* beta, float* state, float* o, const int* state_slots, const int* cu_q,
                                    const int* seq_lens, int B, int H, int G, int E, int DP, const void* proj,
-                                   long long proj_stride, void* conv_state, int keep, int channels, int is_fp32,
-                                   cudaStream_t stream) {
+                                   long long proj_stride, void* conv_state, int keep, int channels, int mode,
+                                   int is_fp32, cudaStream_t stream) {
   if (B <= 0) return 0;
   if ((DP & 3) || G <= 0 || H % G) return -1;
   ScanParams p{q, k, g, v, v_stride, beta, state, o, state_slots, cu_q, seq_lens, H, G, E, DP, proj, proj_stride,
                conv_state, keep, channels};
-  if (g) return is_fp32 ? pick_scan<float, true>(p, B, stream) : pick_scan<__nv_bfloat16, true>(p, B, stream);
-  return is_fp32 ? pick_scan<float, false>(p, B, stream) : pick_scan<__nv_bfloat16, false>(p, B, stream);
+  if ((mode != scan::TIED && !g) || ((mode == scan::DELTA || mode == scan::BONUS) && !beta)) return -1;
+  return is_fp32 ? scan_mode<float>(p, mode, B, stream) : scan_mode<__nv_bfloat16>(p, mode, B, stream);
 }
 
-extern "C" int b200_head_norm_gate(const float* o, const void* w, const void* gate, long long gate_stride, void* out,
-                                   int out_width, int T, int H, int E, float eps, int is_fp32, cudaStream_t stream) {
+extern "C" int b200_head_norm_gate(const float* o, const void* w, int w_step, const void* gate, long long gate_stride,
+                                   int gate_silu, void* out, long long out_stride, int out_width, int T, int H, int E,
+                                   float eps, float scale, int is_fp32, cudaStream_t stream) {
   if (T <= 0) return 0;
   const uintptr_t align = is_fp32 ? 15 : 7;
-  const bool vec = E % 4 == 0 && E <= 512 && out_width % 4 == 0 && gate_stride % 4 == 0 &&
+  const bool vec = E % 4 == 0 && E <= 512 && out_stride % 4 == 0 && gate_stride % 4 == 0 &&
                    (reinterpret_cast<uintptr_t>(gate) & align) == 0 && (reinterpret_cast<uintptr_t>(out) & align) == 0 &&
                    (reinterpret_cast<uintptr_t>(w) & align) == 0;
-  HeadNormParams p{o, w, gate, gate_stride, out, out_width, T, H, E, eps, vec ? 1 : 0};
+  HeadNormParams p{o, w, w_step, gate, gate_stride, gate_silu, out, out_stride, out_width, T, H, E, eps, scale, vec ? 1 : 0};
   const long long units = static_cast<long long>(T) * H;
   const dim3 grid(static_cast<unsigned>((units + kHeadNormWarps - 1) / kHeadNormWarps)), block(kHeadNormWarps * 32);
   const cudaError_t e = is_fp32 ? launch_pdl(head_norm_kernel<float>, grid, block, 0, stream, 1, p)

@@ -348,10 +348,11 @@ class GatedQKVParallelLinear(QKVParallelLinear):
 class SegmentedLinear(LinearBase):
     """Several projections of one input as one product, each with its own rows: ``segments`` = name ->
     (rows, sharded).  Sharded segments are split over the group, the others are whole on every rank.  A
-    segment starts at a whole 16-byte column of the result (``offsets``); the rows between are zero."""
+    segment starts at a whole 16-byte column of the result (``offsets``); the rows between are zero, and so is
+    the bias there."""
 
-    def __init__(self, in_features: int, segments, dtype=torch.bfloat16, device=None, **kw) -> None:
-        super().__init__(in_features, sum(n for n, _ in segments.values()), False, dtype, device, **kw)
+    def __init__(self, in_features: int, segments, bias: bool = False, dtype=torch.bfloat16, device=None, **kw) -> None:
+        super().__init__(in_features, sum(n for n, _ in segments.values()), bias, dtype, device, **kw)
         self.sharded = {k: sh for k, (_, sh) in segments.items()}
         self.rows = {}
         self.offsets = {}
@@ -365,8 +366,8 @@ class SegmentedLinear(LinearBase):
         self._create(in_features, off, device)
         self.weight.data.zero_()
 
-    def forward(self, x: torch.Tensor) -> torch.Tensor:
-        return self.quant_method.apply(self, x, None)
+    def forward(self, x: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        return self.quant_method.apply(self, x, self.bias, out_dtype=out_dtype)
 
     def segment(self, y: torch.Tensor, name: str) -> torch.Tensor:
         return y[:, self.offsets[name]: self.offsets[name] + self.rows[name]]
@@ -381,7 +382,8 @@ class SegmentedLinear(LinearBase):
     def weight_loader(self, param: nn.Parameter, loaded: torch.Tensor, shard_id=None) -> None:
         n, off = self.rows[shard_id], self.offsets[shard_id]
         src = loaded.narrow(0, self.tp_rank * n, n) if self.sharded[shard_id] else loaded
-        param.data[off: off + n, : src.shape[1]] = src.to(param.dtype).to(param.device)
+        rows = param.data[off: off + n]
+        (rows if param.dim() == 1 else rows[:, : src.shape[1]]).copy_(src)
 
 
 class RowParallelLinear(LinearBase):

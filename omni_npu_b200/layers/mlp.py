@@ -20,17 +20,17 @@ from .linear import ColumnParallelLinear, MergedColumnParallelLinear, RowParalle
 class FusedMLP(nn.Module):
     def __init__(self, hidden_size: int, intermediate_size: int, dtype=torch.bfloat16, device=None,
                  quant_method_factory=None, prefix: str = "", group=None,
-                 reduce_results: bool = True, fuse_swiglu: bool = True, act=None) -> None:
+                 reduce_results: bool = True, fuse_swiglu: bool = True, act=None, bias: bool = False) -> None:
         super().__init__()
         qm = quant_method_factory or (lambda: None)
         self.fuse_swiglu = fuse_swiglu
         self.gate_up_proj = MergedColumnParallelLinear(
-            hidden_size, [intermediate_size, intermediate_size], dtype=dtype, device=device,
+            hidden_size, [intermediate_size, intermediate_size], bias=bias, dtype=dtype, device=device,
             swiglu_interleave=fuse_swiglu, quant_method=qm(), prefix=f"{prefix}.gate_up_proj",
             group=group)
         if act is not None:
             self.gate_up_proj.gated_act = act        # applied in the GEMM epilogue (needs fuse_swiglu)
-        self.down_proj = RowParallelLinear(intermediate_size, hidden_size, dtype=dtype, device=device,
+        self.down_proj = RowParallelLinear(intermediate_size, hidden_size, bias=bias, dtype=dtype, device=device,
                                            quant_method=qm(), prefix=f"{prefix}.down_proj",
                                            group=group, reduce_results=reduce_results)
         self.act = SiluAndMul()
@@ -52,6 +52,22 @@ class FusedMLP(nn.Module):
         else:
             h = self.act(self.gate_up_proj(x))
         return row_parallel_add_rms_norm(self.down_proj, h, norm, residual)
+
+
+class UnaryMLP(nn.Module):
+    """down(act(up(x))): one up projection, the activation (a name of ``ops.UNARY``) in its epilogue."""
+
+    def __init__(self, hidden_size: int, intermediate_size: int, act: str, dtype=torch.bfloat16, device=None,
+                 prefix: str = "", group=None, reduce_results: bool = True) -> None:
+        super().__init__()
+        self.act = act
+        self.up_proj = ColumnParallelLinear(hidden_size, intermediate_size, dtype=dtype, device=device,
+                                            prefix=f"{prefix}.up_proj", group=group)
+        self.down_proj = RowParallelLinear(intermediate_size, hidden_size, dtype=dtype, device=device,
+                                           prefix=f"{prefix}.down_proj", group=group, reduce_results=reduce_results)
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return self.down_proj(ops.gemm(x, self.up_proj.weight, unary=self.act))
 
 
 class XieluMLP(nn.Module):

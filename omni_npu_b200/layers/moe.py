@@ -16,7 +16,8 @@ all-gathered afterwards when the residual stream is replicated
 (omni_npu/v1/layers/fused_moe/layer.py:46-56,89-90).
 
 Expert weights: ``w13`` [E_local, 2I, H] with gate / up rows interleaved in
-groups of eight (SwiGLU epilogue layout), ``w2`` [E_local, H, I].
+groups of eight (SwiGLU epilogue layout), or [E_local, I, H] for experts without a
+gate (``unary``); ``w2`` [E_local, H, I].
 """
 from __future__ import annotations
 
@@ -29,7 +30,7 @@ from .. import ops
 from ..ops import ref
 from ..parallel import state as pstate
 from .linear import ReplicatedLinear
-from .mlp import FusedMLP
+from .mlp import FusedMLP, UnaryMLP
 from .moe_dispatch import EpBuffers, ep_combine, ep_dispatch
 
 
@@ -64,7 +65,7 @@ class FusedMoE(nn.Module):
                  shared_intermediate_size: Optional[int] = None, enable_expert_parallel: bool = True,
                  prefix: str = "", max_tokens: int = 8192, quant: Optional[str] = None,
                  num_redundant_experts: int = 0, shared_quant_factory=None,
-                 act: Tuple[float, float] = ops.SILU, shared_act: Optional[Tuple[float, float]] = None) -> None:
+                 act=ops.SILU, shared_act=None, unary: Optional[str] = None) -> None:
         super().__init__()
         self.num_experts, self.top_k = num_experts, top_k
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
@@ -74,6 +75,11 @@ class FusedMoE(nn.Module):
         self.max_tokens = max_tokens
         self.dtype = dtype
         self.act = act               # gated activation of the routed experts (ops.gemm); shared_act: of the shared one
+        # experts without a gate: activation (a name of ops.UNARY) of all of them
+        self.unary = unary
+        if unary is not None and quant is not None:
+            raise ValueError("experts without a gate have no quantised form")
+        up_rows = intermediate_size * (2 if unary is None else 1)
         self.tp_group = pstate.get_tp_group()
         self.ep_group = pstate.get_ep_group() if enable_expert_parallel else None
         self.ep_size = self.ep_group.world_size if self.ep_group is not None else 1
@@ -96,7 +102,7 @@ class FusedMoE(nn.Module):
             self.e_score_correction_bias = None
         wdt = torch.float8_e4m3fn if quant == "fp8" else dtype
         self.quant = quant
-        self.w13 = nn.Parameter(torch.empty(self.local_experts, 2 * intermediate_size, hidden_size,
+        self.w13 = nn.Parameter(torch.empty(self.local_experts, up_rows, hidden_size,
                                             dtype=wdt, device=device), requires_grad=False)
         self.w2 = nn.Parameter(torch.empty(self.local_experts, hidden_size, intermediate_size,
                                            dtype=wdt, device=device), requires_grad=False)
@@ -112,11 +118,14 @@ class FusedMoE(nn.Module):
             inter = (shared_intermediate_size or intermediate_size) * num_shared_experts
             # shared experts are replicated when tokens are de-duplicated across TP ranks
             # quantised checkpoints quantise the shared experts like every other linear
-            self.shared_experts = FusedMLP(hidden_size, inter, dtype, device, prefix=f"{prefix}.shared_experts",
-                                           quant_method_factory=shared_quant_factory,
-                                           group=_solo_group() if self.ep_size > 1 else None,
-                                           reduce_results=False, fuse_swiglu=shared_quant_factory is None,
-                                           act=shared_act)
+            where = dict(prefix=f"{prefix}.shared_experts", group=_solo_group() if self.ep_size > 1 else None,
+                         reduce_results=False)
+            if unary is not None:
+                self.shared_experts = UnaryMLP(hidden_size, inter, unary, dtype, device, **where)
+            else:
+                self.shared_experts = FusedMLP(hidden_size, inter, dtype, device,
+                                               quant_method_factory=shared_quant_factory,
+                                               fuse_swiglu=shared_quant_factory is None, act=shared_act, **where)
         self.buffers: Optional[EpBuffers] = None
         self._side_stream: Optional[torch.cuda.Stream] = None
         self.expert_load: Optional[torch.Tensor] = None   # per-expert token counts (EPLB statistics)
@@ -162,7 +171,7 @@ class FusedMoE(nn.Module):
 
     def _load_slot(self, param: nn.Parameter, loaded: torch.Tensor, local: int, shard: Optional[str]) -> None:
         i = self.intermediate_size
-        if shard in ("gate", "up"):
+        if shard in ("gate", "up") and self.unary is None:
             j = torch.arange(i, device=param.device)
             rows = (j // 8) * 16 + (0 if shard == "gate" else 8) + (j % 8)
             if param.dim() == 3 and param.shape[1] == 2 * i:
@@ -219,6 +228,10 @@ class FusedMoE(nn.Module):
         return moved
 
     # ----------------------------------------------------------------- forward
+    def _expert_rows(self, rows: torch.Tensor, offsets: torch.Tensor) -> torch.Tensor:
+        h = ops.grouped_gemm(rows, self.w13, offsets, swiglu=self.unary is None, act=self.act, unary=self.unary)
+        return ops.grouped_gemm(h, self.w2, offsets)
+
     def forward(self, hidden: torch.Tensor) -> torch.Tensor:
         """hidden [T,H] (replicated across TP ranks) -> [T,H]."""
         tp = self.tp_group.world_size
@@ -269,7 +282,7 @@ class FusedMoE(nn.Module):
             with torch.cuda.stream(self._side_stream):
                 shared_out = self.shared_experts(hidden)
         rows, offsets, handle = ep_dispatch(None, hidden, ids, w, self.num_physical, self.buffers)
-        y = ops.grouped_gemm(ops.grouped_gemm(rows, self.w13, offsets, swiglu=True, act=self.act), self.w2, offsets)
+        y = self._expert_rows(rows, offsets)
         if shared_out is not None:
             cur.wait_stream(self._side_stream)
         return RoutedRows(y, handle.slots, w), shared_out
@@ -300,8 +313,7 @@ class FusedMoE(nn.Module):
                 hq, hs = ops.quant_fp8_1x128(h1)
                 y = ops.grouped_gemm_fp8_block(hq, hs, self.w2, self.w2_scale, offsets)
             else:
-                h1 = ops.grouped_gemm(rows, self.w13, offsets, swiglu=True, act=self.act)
-                y = ops.grouped_gemm(h1, self.w2, offsets)
+                y = self._expert_rows(rows, offsets)
             self.buffers.expert_y[: y.shape[0]].copy_(y)
             if shared_out is not None:
                 torch.cuda.current_stream(x.device).wait_stream(self._side_stream)
@@ -310,8 +322,7 @@ class FusedMoE(nn.Module):
         if self.shared_experts is not None:
             shared_out = self.shared_experts(x)
         rows, offsets, handle = ep_dispatch(comm, x, ids, w, self.num_physical)
-        h1 = ops.grouped_gemm(rows, self.w13, offsets, swiglu=True, act=self.act)
-        y = ops.grouped_gemm(h1, self.w2, offsets)
+        y = self._expert_rows(rows, offsets)
         return ep_combine(comm, y, handle, shared_out)
 
 

@@ -26,6 +26,7 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "OpenPanguVLForConditionalGeneration": ("omni_npu_b200.models.openpangu_vl", "OpenPanguVLForConditionalGeneration"),
     "Rivudra": ("omni_npu_b200.models.rivudra", "RivudraForCausalLM"),
     "Fuvirax": ("omni_npu_b200.models.fuvirax", "FuviraxForCausalLM"),
+    "Gatosun": ("omni_npu_b200.models.gatosun", "GatosunForCausalLM"),
     "MockModel": ("omni_npu_b200.models.mock", "MockModelForCausalLM"),
 }
 
@@ -34,11 +35,12 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
 _CONFIG_READERS: Dict[str, Tuple[str, str]] = {
     "Rivudra": ("omni_npu_b200.models.rivudra", "read_config"),
     "Fuvirax": ("omni_npu_b200.models.fuvirax", "read_config"),
+    "Gatosun": ("omni_npu_b200.models.gatosun", "read_config"),
 }
 
 
 # architectures whose kernels are all in the core library (_build.CORE_SOURCES)
-_CORE_LIBRARY_ONLY = {"Rivudra", "Fuvirax"}
+_CORE_LIBRARY_ONLY = {"Rivudra", "Fuvirax", "Gatosun"}
 
 
 def runs_on_core_library(arch: str) -> bool:

@@ -197,11 +197,20 @@ PAIR_MIN_M = int(os.environ.get("OMNI_B200_GEMM_PAIR_MIN_M", "1024"))
 SMALL_M_GEMM = os.environ.get("OMNI_B200_SMALL_M_GEMM", "library")
 SMALL_M_LIBRARY_ROWS = (64, 256)
 
-def _act_kind(swiglu: bool, act: Tuple[float, float], xielu: Optional[Tuple[float, float]]) -> Tuple[int, float, float]:
+GELU_TANH = "gelu_tanh"    # gated activation gelu(gate) * up, gelu in its tanh form
+UNARY = {"relu2": 5, "tanh": 6}
+
+
+def _act_kind(swiglu: bool, act, xielu: Optional[Tuple[float, float]] = None,
+              unary: Optional[str] = None) -> Tuple[int, float, float]:
     """(kind, constants) of a GEMM epilogue's activation as csrc/gemm/gated_act.cuh numbers them."""
     if xielu is not None:
         return (3, *xielu)
-    return (0, *act) if not swiglu else (2 if act[0] != 0.0 else 1, *act)
+    if unary is not None:
+        return (UNARY[unary], 0.0, 0.0)
+    if not swiglu:
+        return (0, 0.0, 0.0)
+    return (4, 0.0, 0.0) if act == GELU_TANH else (2 if act[0] != 0.0 else 1, *act)
 
 
 def library_small_m(m: int, cluster_split_plan: bool, plain_bf16: bool) -> bool:
@@ -215,27 +224,26 @@ def library_small_m(m: int, cluster_split_plan: bool, plain_bf16: bool) -> bool:
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
          swiglu: bool = False, bn: int = 0, splits: int = 0, max_ctas: int = 0,
-         pair: Optional[bool] = None, act: Tuple[float, float] = SILU,
-         xielu: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+         pair: Optional[bool] = None, act=SILU, xielu: Optional[Tuple[float, float]] = None,
+         unary: Optional[str] = None) -> torch.Tensor:
     """``a[M,K] @ w[N,K].T`` (+bias, +residual).  bf16 or float8_e4m3fn inputs,
     fp32 accumulation, bf16 (default) or fp32 output.  ``swiglu`` fuses
     silu(gate)*up for weights laid out by :func:`ref.interleave_gate_up`; ``act`` = (slope, limit)
-    with a non-zero slope selects the clamped form of it (:func:`ref.gated_act`).  ``xielu`` = (a, b)
-    applies :func:`ref.xielu` to every output.  fp32 inputs run on the CUDA cores, with no
+    with a non-zero slope selects the clamped form of it, ``GELU_TANH`` gelu (:func:`ref.gated_act`); the
+    bias is added before a gated activation.  ``xielu`` = (a, b) applies :func:`ref.xielu` to every output,
+    ``unary`` the named :func:`ref.unary_act`.  fp32 inputs run on the CUDA cores, with no
     reduced-precision mode.
     ``splits`` > 1 forces split-K (as a thread-block cluster when it fits), a
     negative value forces the workspace variant with |splits| slices.
     ``pair`` selects the CTA-pair kernel (256-row tiles over two SMs); by default
     it runs for M >= PAIR_MIN_M when no split-K was asked for."""
     if not a.is_cuda:
-        return ref.gemm(a, w, bias, residual, out_dtype, swiglu, act, xielu)
+        return ref.gemm(a, w, bias, residual, out_dtype, swiglu, act, xielu, unary)
     C = _core()
-    kind = _act_kind(swiglu, act, xielu)
+    kind = _act_kind(swiglu, act, xielu, unary)
     if a.dtype == torch.float32:
         _count(1)
-        y = C.gemm_simt(a, w, None, *kind)
-        if bias is not None:
-            y = y + bias
+        y = C.gemm_simt(a, w, None, *kind, bias)
         return y if residual is None else y + residual
     st = device_state(a.device)
     m, k = a.shape
@@ -248,7 +256,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         _count(1)
         return C.gemm_pair(a, w, bias, residual, out_dtype == torch.float32, kind[0], pbn, st.status, max_ctas,
                            kind[1], kind[2])
-    fused, gated = kind[0] != 0, kind[0] in (1, 2)
+    fused, gated = kind[0] != 0, kind[0] in (1, 2, 4)
     key = (m, n, k, a.dtype.itemsize, kind[0], bn, splits)
     plan = st.plans.get(key)
     if plan is None:
@@ -368,21 +376,21 @@ def gemm_scaled(a_q: torch.Tensor, w_q: torch.Tensor, a_scale: torch.Tensor, w_s
 
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
                  swiglu: bool = False, bn: int = 0, max_ctas: int = 0,
-                 act: Tuple[float, float] = SILU) -> torch.Tensor:
+                 act=SILU, unary: Optional[str] = None) -> torch.Tensor:
     """Per-expert GEMM: rows expert_offsets[e]:expert_offsets[e+1] of ``a`` times ``w[e].T``
-    (``swiglu`` / ``act`` as in :func:`gemm`)."""
+    (``swiglu`` / ``act`` / ``unary`` as in :func:`gemm`)."""
     if not a.is_cuda:
-        return ref.grouped_gemm(a, w, expert_offsets, swiglu, act)
+        return ref.grouped_gemm(a, w, expert_offsets, swiglu, act, unary)
+    kind = _act_kind(swiglu, act, None, unary)
     if a.dtype == torch.float32:
         _count(1)
-        return _core().gemm_simt(a, w, expert_offsets, *_act_kind(swiglu, act, None))
+        return _core().gemm_simt(a, w, expert_offsets, *kind, None)
     if bn <= 0:
         n = w.shape[1]
         bn = 256 if n % 256 == 0 else (128 if n % 128 == 0 else (64 if n % 64 == 0 else 32))
     st = device_state(a.device)
     _count(1)
-    kind, c0, c1 = _act_kind(swiglu, act, None)
-    return _core().grouped_gemm(a, w, expert_offsets, kind, bn, st.status, max_ctas, c0, c1)
+    return _core().grouped_gemm(a, w, expert_offsets, kind[0], bn, st.status, max_ctas, kind[1], kind[2])
 
 
 # ------------------------------------------------------------- norm/activation
@@ -675,6 +683,25 @@ def gated_rope_cache_(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache
                              rot_dim, neox)
 
 
+def qk_norm_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                       positions: torch.Tensor, slot_mapping: torch.Tensor, cos_sin: torch.Tensor, head_dim: int,
+                       head_dim_v: int, rot_dim: int, norm: Optional[str], eps: float, weights=None, sums=None,
+                       v_first: Optional[torch.Tensor] = None, mix: float = 0.0) -> torch.Tensor:
+    """Norm and rotation (rotate-half pairs) of q and k, k / v into the paged cache, whose rows may be wider than
+    the heads; returns the queries [T, Hq * head_dim].  ``norm``: "projection" = RMS norm over all of q (and of
+    k) with ``weights`` = (q, k) before the rotation, "head" = every head divided by its root mean square
+    after it, None.  ``sums`` = (sums of squares of q and k [T, 2], elements of q, of k): taken over more than
+    these rows.  ``v_first``: what is stored is (1 - mix) v + mix v_first."""
+    if not q.is_cuda:
+        return ref.qk_norm_rope_cache(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim, head_dim_v,
+                                      rot_dim, norm, eps, weights, sums, v_first, mix)
+    qw, kw = weights if weights is not None else (None, None)
+    s, nq, nk = sums if sums is not None else (None, q.shape[1], k.shape[1])
+    _count(1)
+    return _core().qk_norm_rope(q, k, v, v_first, mix, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim,
+                                head_dim_v, rot_dim, {None: 0, "projection": 1, "head": 2}[norm], qw, kw, s, nq, nk, eps)
+
+
 def gated_decode_splits(num_seqs: int, num_kv_heads: int, keys: int, sms: int = 148) -> int:
     """CTAs (of one cluster) that share the visible keys of a (sequence, key/value head): as many as
     are resident at once (two per SM), at least 128 keys each."""
@@ -716,21 +743,21 @@ def embed_residual_norm(residual: torch.Tensor, ids: torch.Tensor, table: torch.
         return ref.embed_residual_norm(residual, ids, table, scale, weight, eps, weight_offset, true_width)
     _count(1)
     return _core().residual_norm(residual, ids, table, scale, None, None, None, None, None, weight, eps,
-                                 weight_offset, true_width, weight.dtype == torch.float32)
+                                 weight_offset, true_width, weight.dtype == torch.float32, 1.0)
 
 
 def residual_add_norm(residual: torch.Tensor, a: Optional[torch.Tensor], b: Optional[torch.Tensor], routed,
-                      weight: Optional[torch.Tensor], eps: float, weight_offset: float, true_width: int):
-    """residual += a + b + routed (in place, fp32); returns its RMS norm times (weight_offset + weight),
+                      weight: Optional[torch.Tensor], eps: float, weight_offset: float, true_width: int, mult: float = 1.0):
+    """residual += mult * (a + b + routed) (in place, fp32); returns its RMS norm times (weight_offset + weight),
     or None without a weight.  ``routed`` = (y, slots, weights): expert outputs in expert order that are
     brought back to their tokens here (layers/moe.py:RoutedRows), or None."""
     if not residual.is_cuda:
-        return ref.residual_add_norm(residual, a, b, routed, weight, eps, weight_offset, true_width)
+        return ref.residual_add_norm(residual, a, b, routed, weight, eps, weight_offset, true_width, mult)
     y, slots, w = routed if routed is not None else (None, None, None)
     like = next(x for x in (weight, a, b, y) if x is not None)
     _count(1)
     out = _core().residual_norm(residual, None, None, 1.0, a, b, y, slots, w, weight, eps, weight_offset, true_width,
-                                like.dtype == torch.float32)
+                                like.dtype == torch.float32, mult)
     return out if weight is not None else None
 
 
@@ -781,23 +808,56 @@ def delta_prep(proj: torch.Tensor, low: torch.Tensor, offs, heads: int, kv_heads
 
 def recurrent_scan(q: torch.Tensor, k: torch.Tensor, g: Optional[torch.Tensor], v: torch.Tensor,
                    beta: Optional[torch.Tensor], state: torch.Tensor, heads: int, vdim: int, state_slots: torch.Tensor,
-                   cu_q: torch.Tensor, seq_lens: torch.Tensor, num_seqs: int, conv=None) -> torch.Tensor:
+                   cu_q: torch.Tensor, seq_lens: torch.Tensor, num_seqs: int, conv=None,
+                   bonus: bool = False) -> torch.Tensor:
     """Carry the state of every sequence over its tokens of this step (:func:`ref.recurrent_scan`);
     o [T, heads, vdim] fp32."""
     if not q.is_cuda:
-        return ref.recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, conv)
+        return ref.recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, conv, bonus)
     proj, cs = conv if conv is not None else (None, None)
     _count(1)
-    return _core().recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, proj, cs)
+    return _core().recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, proj, cs,
+                                  bonus)
 
 
 def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[torch.Tensor],
-                   out_width: int) -> torch.Tensor:
-    """RMS norm per head, times the sigmoid of ``gate``: [T, out_width], zero beyond the heads."""
+                   out_width: int = 0, silu: bool = False, scale: float = 1.0,
+                   out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """RMS norm per head (``weight`` [E] for all heads or [H, E]), times ``scale`` and the sigmoid (or ``silu``) of
+    ``gate``: [T, out_width] or the rows ``out``, zero beyond the heads."""
     if not o.is_cuda:
-        return ref.head_norm_gate(o, weight, eps, gate, out_width)
+        return ref.head_norm_gate(o, weight, eps, gate, out_width, silu, scale, out)
     _count(1)
-    return _core().head_norm_gate(o, weight, eps, gate, out_width)
+    y = _core().head_norm_gate(o, weight, eps, gate, out_width, silu, scale, out)
+    return y if out is None else out
+
+
+def token_mix(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, seq_idx: torch.Tensor, state_slots: torch.Tensor,
+              cu_q: torch.Tensor, seq_lens: torch.Tensor, num_seqs: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Rows h_t + (h_(t-1) - h_t) mu_s for the rows s of ``mu`` [n, W], one blend after another: ([n * T, W],
+    offsets [n + 1] of the blends).  ``state`` [slots, W] fp32 keeps every sequence's newest row."""
+    if not h.is_cuda:
+        return ref.token_mix(h, mu, state, cu_q, seq_lens, state_slots, num_seqs)
+    _count(1)
+    return _core().token_mix(h, mu, state, seq_idx, state_slots, cu_q, seq_lens)
+
+
+def decay_prep(q: torch.Tensor, k: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, heads: int, dim: int,
+               q_scale: float, tau: float):
+    """(q * q_scale, k, sigmoid(z + bias)^(1 / tau)), fp32 [T, heads, dim rounded up to 4]; z fp32."""
+    if not q.is_cuda:
+        return ref.decay_prep(q, k, z, bias, heads, dim, q_scale, tau)
+    _count(1)
+    return _core().decay_prep(q, k, z, bias, None, heads, dim, q_scale, 1.0 / tau)[:3]
+
+
+def time_mix_prep(r: torch.Tensor, k: torch.Tensor, z: torch.Tensor, w0: torch.Tensor, u: torch.Tensor, heads: int,
+                  dim: int):
+    """(r, k, exp(-exp(z + w0)), sum over a head of r u k), fp32 [T, heads, dim rounded up to 4] and [T, heads]."""
+    if not r.is_cuda:
+        return ref.time_mix_prep(r, k, z, w0, u, heads, dim)
+    _count(1)
+    return _core().decay_prep(r, k, z, w0, u, heads, dim, 1.0, 1.0)
 
 
 # ------------------------------------------------------- latent attention with run-time sizes

@@ -16,12 +16,16 @@ import torch.nn.functional as F
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
          swiglu: bool = False, act: Tuple[float, float] = (0.0, 0.0),
-         xielu_ab: Optional[Tuple[float, float]] = None) -> torch.Tensor:
+         xielu_ab: Optional[Tuple[float, float]] = None, unary: Optional[str] = None) -> torch.Tensor:
     """``a @ w.T`` with fp32 accumulation.  With ``swiglu`` the N columns are
-    interpreted as interleaved groups of 8 gate / 8 up columns, joined by :func:`gated_act`;
-    ``xielu_ab`` applies :func:`xielu`."""
+    interpreted as interleaved groups of 8 gate / 8 up columns, joined by :func:`gated_act` (the bias comes
+    first); ``xielu_ab`` applies :func:`xielu`, ``unary`` :func:`unary_act`."""
     out = a.float() @ w.float().t()
+    if unary is not None:
+        out = unary_act(out, unary)
     if swiglu:
+        if bias is not None:
+            out, bias = out + bias.float(), None
         n = out.shape[-1]
         g = out.view(*out.shape[:-1], n // 16, 2, 8)
         out = gated_act(g[..., 0, :], g[..., 1, :], act).reshape(*out.shape[:-1], n // 2)
@@ -42,9 +46,15 @@ def xielu(z: torch.Tensor, ab: Tuple[float, float]) -> torch.Tensor:
     return torch.where(z > 0, ab[0] * z * z, ab[1] * (torch.expm1(neg) - neg)) + z / 2
 
 
-def gated_act(gate: torch.Tensor, up: torch.Tensor, act: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
-    """silu(gate) * up; with ``act`` = (slope, limit), slope non-zero:
+def unary_act(z: torch.Tensor, kind: str) -> torch.Tensor:
+    return torch.tanh(z) if kind == "tanh" else {"relu2": F.relu}[kind](z).square()
+
+
+def gated_act(gate: torch.Tensor, up: torch.Tensor, act=(0.0, 0.0)) -> torch.Tensor:
+    """silu(gate) * up, or gelu (tanh form) for ``act`` "gelu_tanh"; with ``act`` = (slope, limit), slope non-zero:
     g * sigmoid(slope * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    if act == "gelu_tanh":
+        return F.gelu(gate, approximate="tanh") * up
     slope, limit = act
     if slope == 0.0:
         return F.silu(gate) * up
@@ -63,7 +73,7 @@ def interleave_gate_up(w_gate: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor
 
 
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
-                 swiglu: bool = False, act: Tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
+                 swiglu: bool = False, act=(0.0, 0.0), unary: Optional[str] = None) -> torch.Tensor:
     e = w.shape[0]
     offs = expert_offsets.tolist()
     n_out = w.shape[1] // 2 if swiglu else w.shape[1]
@@ -72,7 +82,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
     for i in range(e):
         lo, hi = offs[i], offs[i + 1]
         if hi > lo:
-            out[lo:hi] = gemm(a[lo:hi], w[i], swiglu=swiglu, out_dtype=out.dtype, act=act)
+            out[lo:hi] = gemm(a[lo:hi], w[i], swiglu=swiglu, out_dtype=out.dtype, act=act, unary=unary)
     return out
 
 
@@ -249,6 +259,26 @@ def gated_rope_cache_(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_si
     gqa_cache_write(ko, v, k_cache[..., :head_dim], v_cache[..., :head_dim_v], slot_mapping)
 
 
+def qk_norm_rope_cache(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim, head_dim_v, rot_dim, norm,
+                       eps, weights, sums, v_first, mix):
+    """Norm, rotation, value mixing, cache write; returns the queries."""
+    qf, kf, vf = q.float(), k.float(), v.float()
+    if norm == "projection":
+        if sums is None:
+            sums = torch.stack([qf.pow(2).sum(-1), kf.pow(2).sum(-1)], 1), q.shape[1], k.shape[1]
+        s, nq, nk = sums
+        qf = qf * torch.rsqrt(s[:, :1] / nq + eps) * weights[0].float()
+        kf = kf * torch.rsqrt(s[:, 1:] / nk + eps) * weights[1].float()
+    qf, kf = rope_qk(qf, kf, positions, cos_sin, head_dim, rot_dim, True)
+    if norm == "head":
+        qf, kf = (x.reshape(x.shape[0], -1, head_dim) for x in (qf, kf))
+        qf, kf = ((x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) for x in (qf, kf))
+    if v_first is not None:
+        vf = (1 - mix) * vf + mix * v_first.float()
+    gqa_cache_write(kf.to(k.dtype), vf.to(v.dtype), k_cache[..., :head_dim], v_cache[..., :head_dim_v], slot_mapping)
+    return qf.to(q.dtype)
+
+
 def gated_attention(q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len, num_q_heads,
                     head_dim, head_dim_v, scale, window=0, sink=None) -> None:
     """Windowed paged attention; a sink of score ``sink`` scales a row's plain result by
@@ -271,7 +301,7 @@ def embed_residual_norm(residual, ids, table, scale, weight, eps, weight_offset,
     return _unit_norm(residual, weight, eps, weight_offset, true_width)
 
 
-def residual_add_norm(residual, a, b, routed, weight, eps, weight_offset, true_width):
+def residual_add_norm(residual, a, b, routed, weight, eps, weight_offset, true_width, mult=1.0):
     add = torch.zeros_like(residual)
     if routed is not None:
         y, slots, w = routed
@@ -282,7 +312,7 @@ def residual_add_norm(residual, a, b, routed, weight, eps, weight_offset, true_w
     for x in (b, a):
         if x is not None:
             add += x.float()
-    residual += add
+    residual += mult * add
     return _unit_norm(residual, weight, eps, weight_offset, true_width) if weight is not None else None
 
 
@@ -358,7 +388,7 @@ def moe_topk(logits: torch.Tensor, bias: Optional[torch.Tensor], k: int, sigmoid
     t, e = scores.shape
     if n_group > 1:
         grp = choice.view(t, n_group, e // n_group)
-        gscore = grp.topk(2, dim=-1).values.sum(-1) if bias is not None else grp.max(-1).values
+        gscore = grp.topk(min(2, grp.shape[-1]), dim=-1).values.sum(-1) if bias is not None else grp.max(-1).values
         gi = _stable_topk(gscore, topk_group)
         gmask = torch.zeros_like(gscore, dtype=torch.bool).scatter_(1, gi, True)
         choice = choice.masked_fill(~gmask.unsqueeze(-1).expand(t, n_group, e // n_group).reshape(t, e),
@@ -660,9 +690,38 @@ def delta_prep(proj, low, offs, heads, kv_heads, dim, vdim, conv_w, conv_state, 
     return F.pad(q, pad), F.pad(k, pad), F.pad(g, pad), v, beta
 
 
-def recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, conv=None):
+def token_mix(h, mu, state, cu_q, seq_lens, state_slots, num_seqs):
+    t, n = h.shape[0], mu.shape[0]
+    x = h.float()
+    before = torch.zeros_like(x)
+    before[1:] = x[:-1]
+    for lo, hi, start, slot in _portions(cu_q, seq_lens, state_slots, num_seqs):
+        before[lo] = state[slot] if start > 0 and slot >= 0 else 0
+        if slot >= 0:
+            state[slot] = x[hi - 1]
+    out = x[None] + (before - x)[None] * mu.float()[:, None]
+    return out.reshape(n * t, -1).to(h.dtype), torch.arange(0, (n + 1) * t, t, dtype=torch.int32)[: n + 1]
+
+
+def _head_rows(x, heads, dim):
+    return F.pad(x[:, : heads * dim].float().reshape(-1, heads, dim), (0, -dim % 4))
+
+
+def decay_prep(q, k, z, bias, heads, dim, q_scale, tau):
+    g = torch.exp(F.logsigmoid(z[:, : heads * dim] + bias) / tau)
+    return _head_rows(q, heads, dim) * q_scale, _head_rows(k, heads, dim), _head_rows(g, heads, dim)
+
+
+def time_mix_prep(r, k, z, w0, u, heads, dim):
+    g = _head_rows(torch.exp(-torch.exp(z[:, : heads * dim] + w0)), heads, dim)
+    rr, kk = _head_rows(r, heads, dim), _head_rows(k, heads, dim)
+    return rr, kk, g, (rr * kk)[..., :dim].mul(u.view(heads, dim)).sum(-1)
+
+
+def recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_lens, num_seqs, conv=None, bonus=False):
     """Token by token, per head: S <- g S (g None: 1 - k), then S <- S + k u^T with u = v, or with ``beta``
-    u = beta (v - S^T k); o = S^T q.  q, k [T, G, d], v [T, heads * vdim] -> o [T, heads, vdim] fp32.
+    u = beta (v - S^T k); o = S^T q.  ``bonus``: u = v, and o = S^T q + beta v of the S before the token.
+    q, k [T, G, d], v [T, heads * vdim] -> o [T, heads, vdim] fp32.
     ``state`` [slots, heads, vdim, d] holds S^T; ``conv`` = (proj, conv_state): the newest convolution
     inputs are stored too."""
     per = heads // q.shape[1]
@@ -672,12 +731,15 @@ def recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_
     for lo, hi, start, slot in _portions(cu_q, seq_lens, state_slots, num_seqs):
         s = state[slot].clone() if start > 0 and slot >= 0 else torch.zeros(heads, vdim, q.shape[-1])
         for t in range(lo, hi):
+            if bonus:
+                o[t] = torch.einsum("hed,hd->he", s, qq[t]) + beta[t][:, None] * vv[t]
             s = s * (g[t] if g is not None else 1 - kk[t])[:, None, :]
             u = vv[t]
-            if beta is not None:
+            if beta is not None and not bonus:
                 u = beta[t][:, None] * (u - torch.einsum("hed,hd->he", s, kk[t]))
             s = s + u[:, :, None] * kk[t][:, None, :]
-            o[t] = torch.einsum("hed,hd->he", s, qq[t])
+            if not bonus:
+                o[t] = torch.einsum("hed,hd->he", s, qq[t])
         if slot < 0:
             continue
         state[slot] = s
@@ -690,14 +752,16 @@ def recurrent_scan(q, k, g, v, beta, state, heads, vdim, state_slots, cu_q, seq_
     return o
 
 
-def head_norm_gate(o, weight, eps, gate, out_width):
-    """Per-head RMS norm (plain weight), times the sigmoid of ``gate``; [T, out_width] in the weight's type."""
+def head_norm_gate(o, weight, eps, gate, out_width, silu=False, scale=1.0, out=None):
+    """Per-head RMS norm (plain weight), times ``scale`` and the sigmoid or silu of ``gate``; [T, out_width] in
+    the weight's type."""
     t, heads, d = o.shape
-    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+    y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float() * scale
     y = y.reshape(t, heads * d)
     if gate is not None:
-        y = y * torch.sigmoid(gate.float())
-    return F.pad(y, (0, out_width - heads * d)).to(weight.dtype)
+        y = y * (F.silu(gate.float()) if silu else torch.sigmoid(gate.float()))
+    y = F.pad(y, (0, (out_width if out is None else out.shape[1]) - heads * d)).to(weight.dtype)
+    return y if out is None else out.copy_(y)
 
 
 # ------------------------------------------------------------- latent attention of any size

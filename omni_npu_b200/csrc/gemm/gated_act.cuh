@@ -2,6 +2,9 @@
 // single columns.
 #pragma once
 
+#include <cuda_bf16.h>
+#include <stdint.h>
+
 namespace b200 {
 
 enum : int { kActNone = 0, kActSilu = 1, kActClampedGlu = 2, kActXielu = 3, kActGeluTanh = 4, kActRelu2 = 5, kActTanh = 6 };
@@ -59,6 +62,28 @@ __device__ __forceinline__ float unary_act_exact(int kind, float z, float alpha,
     return z * z;
   }
   return kind == kActTanh ? tanhf(z) : xielu_exact(z, alpha, limit);
+}
+
+// v[i] += bias[col + i] for the columns below N.  Whole, aligned groups are two 16-byte loads, the same address
+// in every lane.
+__device__ __forceinline__ void add_bias16(float (&v)[16], const __nv_bfloat16* bias, int col, int N) {
+  const __nv_bfloat16* b = bias + col;
+  if (col + 16 <= N && (reinterpret_cast<uintptr_t>(b) & 15) == 0) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const uint4 u = __ldg(reinterpret_cast<const uint4*>(b) + h);
+      const uint32_t r[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        v[8 * h + 2 * i] += __uint_as_float(r[i] << 16);
+        v[8 * h + 2 * i + 1] += __uint_as_float(r[i] & 0xffff0000u);
+      }
+    }
+    return;
+  }
+#pragma unroll
+  for (int i = 0; i < 16; ++i)
+    if (col + i < N) v[i] += __bfloat162float(b[i]);
 }
 
 // Whether a kind joins pairs of columns (half as many come out), or works on single ones.

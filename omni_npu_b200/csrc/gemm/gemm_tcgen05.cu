@@ -919,10 +919,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
         } else if (p.swiglu) {
           // Columns [c, c+8) hold gate values, [c+8, c+16) the matching up values (N is a multiple of 16).
           const int ocol = col >> 1;
-          if (p.bias) {
-#pragma unroll
-            for (int i = 0; i < 16; ++i) v[i] += __bfloat162float(p.bias[col + i]);
-          }
+          if (p.bias) add_bias16(v, p.bias, col, p.N);
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
@@ -939,11 +936,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
           continue;
         }
         const int ncols = min(16, p.N - col);
-        if (p.bias) {
-#pragma unroll
-          for (int i = 0; i < 16; ++i)
-            if (i < ncols) v[i] += __bfloat162float(p.bias[col + i]);
-        }
+        if (p.bias) add_bias16(v, p.bias, col, p.N);
         if (p.residual) {
           const __nv_bfloat16* rsd = p.residual + static_cast<size_t>(row) * p.ldc + col;
 #pragma unroll

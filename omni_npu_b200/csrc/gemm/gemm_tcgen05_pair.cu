@@ -324,10 +324,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
           for (int i = 0; i < 16; ++i) v[i] = unary_act(p.swiglu, v[i], p.act_alpha, p.act_limit);
         } else if (p.swiglu) {
           const int ocol = col >> 1;
-          if (p.bias) {
-#pragma unroll
-            for (int i = 0; i < 16; ++i) v[i] += __bfloat162float(p.bias[col + i]);
-          }
+          if (p.bias) add_bias16(v, p.bias, col, p.N);
           float o[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
@@ -343,11 +340,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
           continue;
         }
         const int ncols = min(16, p.N - col);
-        if (p.bias) {
-#pragma unroll
-          for (int i = 0; i < 16; ++i)
-            if (i < ncols) v[i] += __bfloat162float(p.bias[col + i]);
-        }
+        if (p.bias) add_bias16(v, p.bias, col, p.N);
         if (p.residual) {
           const __nv_bfloat16* rsd = p.residual + static_cast<size_t>(row) * p.ldc + col;
 #pragma unroll

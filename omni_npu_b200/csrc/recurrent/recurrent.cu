@@ -627,68 +627,72 @@ struct HeadNormParams {
   long long out_stride;
   int out_width, T, H, E;
   float eps, scale;
-  int vec;                     // rows are whole four-element pieces
+  int vec;                     // rows are whole eight-element pieces
+  int lanes;                   // of a warp that share a head
 };
 
 static constexpr int kHeadNormWarps = 8;
 
+// `lanes` (a power of two) of a warp share a head; rows of whole eight-element pieces, up to 512 columns, stay in
+// registers.
 template <typename T>
 __global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_kernel(const HeadNormParams p) {
   pdl_trigger();
   pdl_wait();
-  const long long unit = static_cast<long long>(blockIdx.x) * kHeadNormWarps + (threadIdx.x >> 5);
-  if (unit >= static_cast<long long>(p.T) * p.H) return;
-  const int lane = threadIdx.x & 31;
-  const long long t = unit / p.H;
-  const int h = static_cast<int>(unit - t * p.H);
-  const float* o = p.o + unit * p.E;
+  const int lane = threadIdx.x & 31, per_warp = 32 / p.lanes, li = lane & (p.lanes - 1);
+  const long long unit =
+      (static_cast<long long>(blockIdx.x) * kHeadNormWarps + (threadIdx.x >> 5)) * per_warp + lane / p.lanes;
+  const bool live = unit < static_cast<long long>(p.T) * p.H;
+  const long long t = live ? unit / p.H : 0;
+  const int h = live ? static_cast<int>(unit - t * p.H) : 0;
+  const int E = live ? p.E : 0;
+  const float* o = p.o + (live ? unit * p.E : 0);
   const T* w = static_cast<const T*>(p.w) + h * p.w_step;
   const T* gate = p.gate ? static_cast<const T*>(p.gate) + t * p.gate_stride + static_cast<long long>(h) * p.E : nullptr;
-  T* dst = static_cast<T*>(p.out) + t * p.out_stride;
+  T* dst = static_cast<T*>(p.out) + t * p.out_stride + static_cast<long long>(h) * p.E;
   const bool silu = p.gate_silu != 0;
-  float ss = 0.f;
-  if (p.vec) {                                            // up to 512 columns, four at a time in registers
-    float x[4][4], g[4][4];
+  float ss = 0.f, x[2][8], g[2][8];
+  if (p.vec) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int v = lane + 32 * i;
-      if (v * 4 < p.E) {
-        Row4<float>::load(o, v, x[i]);
-        if (gate) Row4<T>::load(gate, v, g[i]);
+    for (int i = 0; i < 2; ++i) {
+      const int v = li + p.lanes * i;
+      if (v * 8 < E) {
+        Row8<float>::load(o, v, x[i]);
+        if (gate) Row8<T>::load(gate, v, g[i]);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) ss = fmaf(x[i][j], x[i][j], ss);
-      }
-    }
-#pragma unroll
-    for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
-    const float inv = p.scale / sqrtf(ss / static_cast<float>(p.E) + p.eps);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int v = lane + 32 * i;
-      if (v * 4 < p.E) {
-        float ww[4];
-        Row4<T>::load(w, v, ww);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          x[i][j] *= inv * ww[j];
-          if (gate) x[i][j] *= quick_sigmoid(g[i][j]) * (silu ? g[i][j] : 1.f);
-        }
-        Row4<T>::store(dst + h * p.E, v, x[i]);
+        for (int j = 0; j < 8; ++j) ss = fmaf(x[i][j], x[i][j], ss);
       }
     }
   } else {
-    for (int d = lane; d < p.E; d += 32) ss = fmaf(o[d], o[d], ss);
+    for (int d = li; d < E; d += p.lanes) ss = fmaf(o[d], o[d], ss);
+  }
+  for (int i = p.lanes >> 1; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
+  if (!live) return;
+  const float inv = p.scale / sqrtf(ss / static_cast<float>(p.E) + p.eps);
+  if (p.vec) {
 #pragma unroll
-    for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
-    const float inv = p.scale / sqrtf(ss / static_cast<float>(p.E) + p.eps);
-    for (int d = lane; d < p.E; d += 32) {
+    for (int i = 0; i < 2; ++i) {
+      const int v = li + p.lanes * i;
+      if (v * 8 < E) {
+        float ww[8];
+        Row8<T>::load(w, v, ww);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          x[i][j] *= inv * ww[j];
+          if (gate) x[i][j] *= quick_sigmoid(g[i][j]) * (silu ? g[i][j] : 1.f);
+        }
+        Row8<T>::store(dst, v, x[i]);
+      }
+    }
+  } else {
+    for (int d = li; d < E; d += p.lanes) {
       float y = o[d] * inv * as_float(w[d]);
       if (gate) y *= quick_sigmoid(as_float(gate[d])) * (silu ? as_float(gate[d]) : 1.f);
-      dst[h * p.E + d] = from_float<T>(y);
+      dst[d] = from_float<T>(y);
     }
   }
   if (h == p.H - 1)
-    for (int d = p.H * p.E + lane; d < p.out_width; d += 32) dst[d] = from_float<T>(0.f);
+    for (int d = p.E + li; d < p.out_width - h * p.E; d += p.lanes) dst[d] = from_float<T>(0.f);
 }
 
 template <typename T, int CPL>
@@ -772,13 +776,14 @@ extern "C" int b200_head_norm_gate(const float* o, const void* w, int w_step, co
                                    int gate_silu, void* out, long long out_stride, int out_width, int T, int H, int E,
                                    float eps, float scale, int is_fp32, cudaStream_t stream) {
   if (T <= 0) return 0;
-  const uintptr_t align = is_fp32 ? 15 : 7;
-  const bool vec = E % 4 == 0 && E <= 512 && out_stride % 4 == 0 && gate_stride % 4 == 0 &&
-                   (reinterpret_cast<uintptr_t>(gate) & align) == 0 && (reinterpret_cast<uintptr_t>(out) & align) == 0 &&
-                   (reinterpret_cast<uintptr_t>(w) & align) == 0;
-  HeadNormParams p{o, w, w_step, gate, gate_stride, gate_silu, out, out_stride, out_width, T, H, E, eps, scale, vec ? 1 : 0};
-  const long long units = static_cast<long long>(T) * H;
-  const dim3 grid(static_cast<unsigned>((units + kHeadNormWarps - 1) / kHeadNormWarps)), block(kHeadNormWarps * 32);
+  const bool vec = E % 8 == 0 && E <= 512 && out_stride % 8 == 0 && gate_stride % 8 == 0 &&
+                   (reinterpret_cast<uintptr_t>(gate) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 &&
+                   (reinterpret_cast<uintptr_t>(w) & 15) == 0;
+  int lanes = 1;
+  while (lanes < 32 && lanes * (vec ? 8 : 1) < E) lanes <<= 1;
+  HeadNormParams p{o, w, w_step, gate, gate_stride, gate_silu, out, out_stride, out_width, T, H, E, eps, scale, vec ? 1 : 0, lanes};
+  const long long units = static_cast<long long>(T) * H, per_cta = static_cast<long long>(kHeadNormWarps) * (32 / lanes);
+  const dim3 grid(static_cast<unsigned>((units + per_cta - 1) / per_cta)), block(kHeadNormWarps * 32);
   const cudaError_t e = is_fp32 ? launch_pdl(head_norm_kernel<float>, grid, block, 0, stream, 1, p)
                                 : launch_pdl(head_norm_kernel<__nv_bfloat16>, grid, block, 0, stream, 1, p);
   return e == cudaSuccess ? 0 : -3;

@@ -287,7 +287,10 @@ class ParallelMixer(_Mixer):
     def _right(self, h: torch.Tensor, run: int, out: torch.Tensor) -> None:
         t, n = h.shape[0], self.mix_rows
         rows, offsets = self.time.blend(h, run)
-        r, k, v, g = ops.grouped_gemm(rows[: 4 * t], self.rkvg, offsets[:5])[:, :n].split(t)
+        if h.is_cuda and t >= ops.PAIR_MIN_M > 0 and h.dtype == torch.bfloat16:      # large enough for CTA pairs
+            r, k, v, g = (ops.gemm(rows[i * t: (i + 1) * t], self.rkvg[i])[:, :n] for i in range(4))
+        else:
+            r, k, v, g = ops.grouped_gemm(rows[: 4 * t], self.rkvg, offsets[:5])[:, :n].split(t)
         z = self.low_proj(ops.gemm(rows[4 * t:], self.w1, unary="tanh"), out_dtype=torch.float32)
         self.time(r, k, v, z, g, run, self.right, out)
 

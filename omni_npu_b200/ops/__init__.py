@@ -11,6 +11,7 @@ launched (graph replays add the number of kernels captured in the graph).
 """
 from __future__ import annotations
 
+import functools
 import os
 import threading
 from pathlib import Path
@@ -186,7 +187,7 @@ def check_status(device: Optional[torch.device] = None) -> None:
 SILU = (0.0, 0.0)          # gated activation silu(gate) * up: no slope, no limit
 # smallest M routed to the CTA-pair GEMM (0 = never); prefill-sized problems only
 PAIR_MIN_M = int(os.environ.get("OMNI_B200_GEMM_PAIR_MIN_M", "1024"))
-# Plain bf16 products (no bias, residual, SwiGLU, scales or fused collective) of a decode-sized batch
+# Plain bf16 products (no residual, SwiGLU, scales or fused collective) of a decode-sized batch
 # whose plan here is a cluster split-K: "library" hands them to cuBLAS, "own" keeps them on
 # gemm_tcgen05_kernel.  Measured at M = 128 inside a CUDA graph (us, own / cuBLAS): 4096 x 4096
 # 19.0 / 10.6, 6144 x 4096 20.2 / 12.6, 4096 x 14336 37.4 / 26.3: every CTA of the own kernel re-reads
@@ -263,9 +264,9 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         plan = C.gemm_plan(m, n, k, a.dtype.itemsize, gated, bn, 1 if gated else max(0, splits) if fused else splits)
         st.plans[key] = plan
     pbn, psplits, ws_bytes, ncnt, cluster = plan
-    if library_small_m(m, bool(cluster), bias is None and residual is None and not fused and bn == 0
+    if library_small_m(m, bool(cluster), residual is None and not fused and bn == 0
                        and splits == 0 and a.dtype == torch.bfloat16 and out_dtype in (None, torch.bfloat16)):
-        return torch.nn.functional.linear(a, w)          # a library kernel: not counted as a launch of ours
+        return torch.nn.functional.linear(a, w, bias)    # a library kernel: not counted as a launch of ours
     ws = cnt = None
     if psplits > 1 and not cluster:
         ws, cnt = st.gemm_workspace(torch.cuda.current_stream(a.device).cuda_stream, ws_bytes, ncnt)
@@ -374,6 +375,25 @@ def gemm_scaled(a_q: torch.Tensor, w_q: torch.Tensor, a_scale: torch.Tensor, w_s
                             out_dtype == torch.float32, bn, st.status, max_ctas)
 
 
+@functools.lru_cache(maxsize=4096)
+def grouped_tile(rows: int, groups: int, n: int, k: int, sms: int = 148) -> int:
+    """Tile width of a grouped bf16 product whose ``rows`` rows spread evenly over the groups: 256, or the largest
+    power of two from 32 that divides n, unless another width is clearly better under the cost model of the
+    dense plan (csrc/gemm/gemm_tcgen05.cu): fewer idle SMs in a decode step, less padding of n in a prompt."""
+    live = max(1, min(groups, rows))
+    per = -(-rows // live)
+    m_tiles = live * -(-per // 128)
+
+    def cost(bn: int) -> float:
+        tiles = m_tiles * -(-n // bn)
+        cta = max((min(per, 128) + bn) * k * 2 / 90e9, 2.0 * 128 * bn * k * sms / 1.4e15) + 1.5e-6
+        return max(-(-tiles // sms) * cta, (live * n + rows) * k * 2 / 6.5e12)
+
+    first = next(bn for bn in (256, 128, 64, 32) if n % bn == 0 or bn == 32)
+    best = min(range(256, 31, -16), key=cost)
+    return best if cost(best) < 0.95 * cost(first) else first
+
+
 def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
                  swiglu: bool = False, bn: int = 0, max_ctas: int = 0,
                  act=SILU, unary: Optional[str] = None) -> torch.Tensor:
@@ -386,8 +406,7 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
         _count(1)
         return _core().gemm_simt(a, w, expert_offsets, *kind, None)
     if bn <= 0:
-        n = w.shape[1]
-        bn = 256 if n % 256 == 0 else (128 if n % 128 == 0 else (64 if n % 64 == 0 else 32))
+        bn = grouped_tile(a.shape[0], w.shape[0], w.shape[1], w.shape[2])
     st = device_state(a.device)
     _count(1)
     return _core().grouped_gemm(a, w, expert_offsets, kind[0], bn, st.status, max_ctas, kind[1], kind[2])

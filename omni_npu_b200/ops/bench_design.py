@@ -1,11 +1,12 @@
 """Throughput of a design beside the framework's closest existing model at equal size (random weights).
 
-``bench.py --design rivudra`` or ``--design fuvirax`` runs this on one GPU.  Per size it prints one JSON line
-with
+``bench.py --design rivudra``, ``--design fuvirax`` or ``--design gatosun`` runs this on one GPU.  Per size it
+prints one JSON line with
 
 * whole steps through the engine (device time of prompt and decode steps, CUDA events): Rivudra and a
-  Qwen3-MoE of the same width, heads, experts and window, or Fuvirax and a dense DeepSeek-V2 of the same
-  width, heads, latent sizes and feed-forward;
+  Qwen3-MoE of the same width, heads, experts and window, Fuvirax and a dense DeepSeek-V2 of the same
+  width, heads, latent sizes and feed-forward, or Gatosun and a Qwen3-MoE of the same width, heads and
+  experts (every layer full attention);
 * single kernels: time, the fraction of the measured roofline (the slower of bytes / copy bandwidth and
   FLOPs / library bf16 GEMM throughput) and the same for the like kernel of the other model.  Between
   iterations a 256 MB buffer is written, so inputs come from HBM.
@@ -20,8 +21,8 @@ from typing import Callable, Dict, List, Optional, Tuple
 import torch
 
 from .. import ops
-from ..config import (AttentionSpec, DeltaRuleSpec, DenseSpec, ExpertSpec, GatedLinearSpec, LatentAttentionSpec, LayerSpec,
-                      ModelConfig, MoESpec)
+from ..config import (AttentionSpec, DecayLinearSpec, DeltaRuleSpec, DenseSpec, ExpertSpec, GatedLinearSpec,
+                      LatentAttentionSpec, LayerSpec, ModelConfig, MoESpec, ParallelSpec, TimeMixSpec)
 
 LAYERS = 4
 CLAMPED = (1.702, 7.0)
@@ -431,9 +432,230 @@ def fuvirax_kernels(size) -> List[dict]:
     return out
 
 
+# ----------------------------------------------------------------------------- Gatosun
+# width, q heads, kv heads, head size, window, time-mixing heads and size, linear-attention heads, row and column
+# size, experts, top-k, expert width
+GATOSUN_SIZES: Dict[str, Tuple[int, ...]] = {
+    "2048x16h/4kv/128 w1024 t32x64 g4x256/512 e64k6 ff1024": (2048, 16, 4, 128, 1024, 32, 64, 4, 256, 512, 64, 6, 1024),
+    "4096x32h/8kv/128 w512 t64x64 g32x128/128 e32k4 ff2048": (4096, 32, 8, 128, 512, 64, 64, 32, 128, 128, 32, 4, 2048),
+    "2880x64h/8kv/64 w128 t45x64 g15x96/192 e32k4 ff2880": (2880, 64, 8, 64, 128, 45, 64, 15, 96, 192, 32, 4, 2880),
+}
+GATOSUN_LAYERS = 6           # two of each mixer
+DECAY_RANK = 64
+
+
+def gatosun(size) -> ModelConfig:
+    w, hq, hk, d, win, th, td, gh, gd, ge, e, k, ff = size
+    ex = ExpertSpec(ff, "relu2")
+    mlp = MoESpec(e, k, ex, ex, "sigmoid", renormalize=False, n_group=4, topk_group=2, correction=True)
+    full = AttentionSpec(hq, hk, d, d, d, 1e6, d ** -0.5, True, 0, qk_norm="projection", bias=True, value_mix=True)
+    left = AttentionSpec(hq, hk, d, d, d, 1e6, d ** -0.5, True, win, qk_norm="head")
+    specs = (LayerSpec(full, mlp), LayerSpec(ParallelSpec(left, TimeMixSpec(th, td, DECAY_RANK), 0.6, 0.5), mlp),
+             LayerSpec(DecayLinearSpec(gh, gd, ge, 16.0, DECAY_RANK), mlp))
+    return ModelConfig(architecture="Gatosun", model_type="gatosun", hidden_size=w, num_layers=GATOSUN_LAYERS, num_heads=hq,
+                       num_kv_heads=hk, head_dim=d, vocab_size=VOCAB, max_position_embeddings=1 << 16,
+                       layer_specs=specs * (GATOSUN_LAYERS // 3), residual_mult=0.3, num_experts=e, num_experts_per_tok=k)
+
+
+def qwen3_moe_full(size) -> ModelConfig:
+    w, hq, hk, d, *_, e, k, ff = size
+    mc = qwen3_moe((w, hq, hk, d, 0, e, k, ff))
+    mc.num_layers = GATOSUN_LAYERS
+    return mc
+
+
+def gatosun_kernels(size) -> List[dict]:
+    w, hq, hk, d, win, th, td, gh, gd, ge, e, k, ff = size
+    bw, fl = _peaks()
+    out: List[dict] = []
+    bf, f32, i32 = (dict(dtype=t, device="cuda") for t in (torch.bfloat16, torch.float32, torch.int32))
+
+    def entry(name: str, fn, nbytes: float, flops: float = 0.0, like: Optional[Tuple] = None, peak: float = fl):
+        """``like``: (call, bytes, FLOPs[, FLOP rate]) of the like kernel."""
+        ms = _time(fn)
+        bound = max(nbytes / bw, flops / peak) * 1e3
+        r = {"kernel": f"{name}, {kind}", "ms": round(ms, 4), "roofline": round(bound / ms, 3)}
+        if like is not None:
+            lms = _time(like[0])
+            lb = max(like[1] / bw, like[2] / (like[3] if len(like) > 3 else fl)) * 1e3
+            r.update(like_ms=round(lms, 4), like_roofline=round(lb / lms, 3),
+                     distance=round((lb / lms) / (bound / ms), 2))
+        out.append(r)
+
+    def gemm_cost(rows, weight, live=None):
+        n, c = weight.shape[-2:]
+        return (rows * (n + c) + (live or 1) * n * c) * 2, 2.0 * rows * n * c
+
+    bs, group = 64, 4
+    for kind, n, rows in (("prefill", 8, 1024), ("decode b1", 1, 1), ("decode b16", 16, 1), ("decode b128", 128, 1)):
+        t, pre = n * rows, kind == "prefill"
+        ctx = rows if pre else CONTEXT
+        x = torch.randn(t, w, **bf)
+        cu, lens = torch.arange(0, (n + 1) * rows, rows, **i32), torch.full((n,), ctx, **i32)
+        slots, idx = torch.arange(n, **i32), torch.arange(n, **i32).repeat_interleave(rows)
+        states = (slots, cu, lens, n)
+        gain = torch.randn(w, **bf)
+        res16 = torch.randn(t, w, **bf)
+        add_norm = (lambda: ops.fused_add_rms_norm(x, res16, gain, 1e-6), t * w * 8, 0.0)
+
+        def product(name, cols, like_cols, bias=False, act=None, like_act=None, pairs=False):
+            a, b = torch.randn(cols, w, **bf), torch.randn(like_cols, w, **bf)
+            bb = torch.randn(cols, **bf) if bias else None
+            halve = lambda c, cols: (c[0] - t * cols, c[1])                              # noqa: E731
+            own, other = gemm_cost(t, a), gemm_cost(t, b)
+            entry(name, lambda: ops.gemm(x, a, bb, **(act or {})), *(halve(own, cols) if pairs else own),
+                  like=(lambda: ops.gemm(x, b, **(like_act or {})), *(halve(other, like_cols) if like_act else other)))
+
+        # ---- attention: full with projection norms, and windowed with unit heads
+        qkv_cols = (hq + 2 * hk) * d
+        product("q / k / v with bias (like: q / k / v)", qkv_cols, qkv_cols, bias=True)
+        per = (ctx + bs - 1) // bs
+        kc, vc = (torch.randn(n * per, hk, bs, d, **bf) for _ in range(2))
+        bt = torch.randperm(n * per, device="cuda").int().view(n, per)
+        pos = torch.arange(ctx - rows, ctx, **i32).repeat(n)
+        slot = (bt.long().gather(1, (pos.view(n, rows) // bs).long()) * bs + pos.view(n, rows) % bs).int().view(-1)
+        cs = torch.randn(CONTEXT + 128, d, **f32)
+        qkv = torch.randn(t, qkv_cols, **bf)
+        q, kk, vv = qkv.split([hq * d, hk * d, hk * d], 1)
+        first = torch.randn(t, hk * d, **bf)
+        qn, kn, hn = torch.randn(hq * d, **bf), torch.randn(hk * d, **bf), torch.randn(d, **bf)
+        moved = t * (2 * hq + 4 * hk) * d * 2
+
+        def like_prep():
+            a = ops.rms_norm(q.reshape(-1, d), hn, 1e-6).view(t, -1)
+            b = ops.rms_norm(kk.reshape(-1, d), hn, 1e-6).view(t, -1)
+            ops.rope_cache_gqa_(a, b, vv, kc, vc, pos, slot, cs, d, d, True)
+
+        prep = lambda norm, wts, vf: ops.qk_norm_rope_cache(q, kk, vv, kc, vc, pos, slot, cs, d, d, d, norm, 1e-6, wts,  # noqa: E731
+                                                            None, vf, 0.4)
+        entry("projection norm + rotation + values + cache (like: head norms + rotation + cache)",
+              lambda: prep("projection", (qn, kn), first), moved + t * hk * d * 2, 0, (like_prep, moved, 0.0))
+        entry("rotation + unit heads + cache (like: head norms + rotation + cache)", lambda: prep("head", None, None), moved,
+              0, (like_prep, moved, 0.0))
+        o = torch.empty(t, hq * d, **bf)
+        for name, window in (("full", 0), ("windowed", win)):
+            pairs = sum(min(window or ctx, p + 1) for p in range(ctx - rows, ctx))
+            cost = (n * hk * 4 * d * min(ctx, (window or ctx) + rows - 1) + t * hq * d * 4, 4.0 * n * hq * d * pairs)
+
+            def own_attn(window=window):
+                ops.gated_attention(q, None, kc, vc, o, bt, cu if pre else None, lens, n, rows, hq, d, d, d ** -0.5, window,
+                                    None, max_seq_len=ctx)
+
+            def like_attn(window=window):
+                if pre:
+                    return ops.gqa_prefill(q, kc, vc, bt, cu, lens, n, rows, hq, d ** -0.5, True, window)
+                return ops.gqa_decode(q, kc, vc, bt, lens, n, hq, d ** -0.5, 1, window, max_seq_len=ctx)
+            entry(f"attention, {name} (like: the same)", own_attn, *cost, like=(like_attn, *cost))
+        del kc, vc, qkv, q, kk, vv
+        # ---- time mixing
+        mu, shift = torch.rand(5, w, **bf), torch.zeros(n, w, **f32)
+        entry("blends with the previous token (like: add + norm)", lambda: ops.token_mix(x, mu, shift, idx, *states),
+              t * w * 2 * 6 + n * w * 8, 0, add_norm)
+        mixed, offs = ops.token_mix(x, mu, shift, idx, *states)
+        tm = th * td
+        rkvg = torch.randn(4, tm, w, **bf)
+        flat = rkvg.view(4 * tm, w)
+
+        def four():
+            if pre:
+                return [ops.gemm(mixed[i * t: (i + 1) * t], rkvg[i]) for i in range(4)]
+            return ops.grouped_gemm(mixed[: 4 * t], rkvg, offs[:5])
+        entry("r / k / v / gate of four blends (like: one product)", four,
+              (4 * t * (w + tm) + 4 * tm * w) * 2, 8.0 * t * tm * w, (lambda: ops.gemm(x, flat), *gemm_cost(t, flat)))
+        w1, w2 = torch.randn(DECAY_RANK, w, **bf), torch.randn(tm, DECAY_RANK, **bf)
+        entry("low rank + tanh", lambda: ops.gemm(mixed[4 * t:], w1, unary="tanh"), *gemm_cost(t, w1))
+        low = ops.gemm(mixed[4 * t:], w1, unary="tanh")
+        entry("decays from the low rank, fp32", lambda: ops.gemm(low, w2, out_dtype=torch.float32),
+              gemm_cost(t, w2)[0] + t * tm * 2, gemm_cost(t, w2)[1])
+        y4 = torch.randn(4 * t, tm, **bf)
+        r, kt, vt, gt = y4.split(t)
+        z, w0, u = torch.randn(t, tm, **f32), torch.randn(tm, **f32), torch.randn(th, td, **f32)
+        like_lin = torch.randn(t, 2 * tm, **bf)
+        entry("time mixing: r, k, decays, bonus (like: q and keys of gated linear attention)",
+              lambda: ops.time_mix_prep(r, kt, z, w0, u, th, td), t * tm * (4 + 4 + 12), 0,
+              (lambda: ops.gated_linear_prep(like_lin, 0, tm, th, td, w0, w0), t * tm * (4 + 8), 0.0))
+        rf, kf, gf, beta = ops.time_mix_prep(r, kt, z, w0, u, th, td)
+        state = torch.zeros(n, th, td, td, **f32)
+        cost = (t * th * 18 * td + n * th * td * td * 8, 5.0 * t * th * td * td)
+        like_cost = (t * th * 14 * td + n * th * td * td * 8, cost[1], FP32_FLOPS)
+        entry("time mixing: scan (like: scan of gated linear attention)",
+              lambda: ops.recurrent_scan(rf, kf, gf, vt, beta, state, th, td, *states, bonus=True), *cost,
+              like=(lambda: ops.recurrent_scan(rf, kf, None, vt, None, state, th, td, *states), *like_cost), peak=FP32_FLOPS)
+        of, nw, sw = torch.randn(t, th, td, **f32), torch.randn(th, td, **bf), torch.randn(td, **bf)
+        wide = torch.empty(t, hq * d + tm, **bf)
+        entry("time mixing: head norm + silu gate (like: head norm + gate)",
+              lambda: ops.head_norm_gate(of, nw, 1e-5, gt, silu=True, scale=0.8, out=wide[:, hq * d:]), t * tm * 8, 0,
+              (lambda: ops.head_norm_gate(of, sw, 1e-5, gt, tm), t * tm * 8, 0.0))
+        both, wo = torch.randn(w, hq * d + tm, **bf), torch.randn(w, hq * d, **bf)
+        entry("output of both halves (like: output projection)", lambda: ops.gemm(wide, both), *gemm_cost(t, both),
+              like=(lambda: ops.gemm(o, wo), *gemm_cost(t, wo)))
+        del mixed, rkvg, flat, y4, rf, kf, gf, of, wide, both
+        # ---- decayed linear attention
+        gn, gm = gh * gd, gh * ge
+        product("projection, decayed linear attention (like: q / k / v)", 2 * gn + 2 * gm + DECAY_RANK, qkv_cols)
+        proj = torch.randn(t, 2 * gn + 2 * gm + DECAY_RANK, **bf)
+        q2, k2, v2, g2 = proj[:, : 2 * gn + 2 * gm].split([gn, gn, gm, gm], 1)
+        z2, b2 = torch.randn(t, gn, **f32), torch.randn(gn, **f32)
+        entry("decayed linear: q, k, decays (like: q and keys of gated linear attention)",
+              lambda: ops.decay_prep(q2, k2, z2, b2, gh, gd, gd ** -0.5, 16.0), t * gn * (4 + 4 + 12), 0,
+              (lambda: ops.gated_linear_prep(proj, 0, gn, gh, gd, b2, b2), t * gn * (4 + 8), 0.0))
+        qf, kf, gf = ops.decay_prep(q2, k2, z2, b2, gh, gd, gd ** -0.5, 16.0)
+        state = torch.zeros(n, gh, ge, gd, **f32)
+        cost = (t * gh * (12 * gd + 6 * ge) + n * gh * gd * ge * 8, 5.0 * t * gh * gd * ge)
+        like_cost = (t * gh * (8 * gd + 6 * ge) + n * gh * gd * ge * 8, cost[1], FP32_FLOPS)
+        entry("decayed linear: scan (like: scan of gated linear attention)",
+              lambda: ops.recurrent_scan(qf, kf, gf, v2, None, state, gh, ge, *states), *cost,
+              like=(lambda: ops.recurrent_scan(qf, kf, None, v2, None, state, gh, ge, *states), *like_cost), peak=FP32_FLOPS)
+        of, nw = torch.randn(t, gh, ge, **f32), torch.randn(ge, **bf)
+        entry("decayed linear: head norm + silu gate (like: head norm + gate)",
+              lambda: ops.head_norm_gate(of, nw, 1e-5, g2, gm, silu=True), t * gm * 8, 0,
+              (lambda: ops.head_norm_gate(of, nw, 1e-5, g2, gm), t * gm * 8, 0.0))
+        del proj, q2, k2, v2, g2, qf, kf, gf, of, state
+        # ---- feed-forwards and the residual
+        product("gate/up + bias + gelu (like: gate/up + silu)", 4 * ff, 4 * ff, bias=True,
+                act=dict(swiglu=True, act=ops.GELU_TANH), like_act=dict(swiglu=True), pairs=True)
+        ids = torch.stack([torch.randperm(e, device="cuda")[:k] for _ in range(min(t, 512))]).repeat(
+            (t + 511) // 512, 1)[:t].int()
+        counts = torch.bincount(ids.view(-1).long(), minlength=e)
+        offs = torch.zeros(e + 1, **i32)
+        offs[1:] = counts.cumsum(0)
+        live = int((counts > 0).sum())
+        xr, w13 = torch.randn(t * k, w, **bf), torch.randn(e, 2 * ff, w, **bf)
+        up = w13[:, :ff].contiguous()
+        nb, nf = gemm_cost(t * k, w13, live)
+        entry("experts up + squared relu (like: experts gate/up + silu)",
+              lambda: ops.grouped_gemm(xr, up, offs, unary="relu2"), *gemm_cost(t * k, up, live),
+              like=(lambda: ops.grouped_gemm(xr, w13, offs, swiglu=True), nb - t * k * 2 * ff, nf))
+        del w13, up
+        res = torch.randn(t, w, **f32)
+        entry("residual + norm (like: add + norm)",
+              lambda: ops.residual_add_norm(res, x, None, None, gain, 1e-6, 0.0, w, mult=0.3), t * w * 12, 0, add_norm)
+        wt, rslots = torch.rand(t, k, **f32), torch.randperm(t * k, device="cuda").int()
+        from ..layers.moe import _solo_group
+        from ..layers.moe_dispatch import DispatchHandle, EpBuffers, ep_combine
+        buf = EpBuffers(_solo_group(), torch.device("cuda", torch.cuda.current_device()), e, w, t, k)
+        handle = DispatchHandle(ids, wt, rslots, t, t * k, offs)
+
+        def like_end():
+            ops.fused_add_rms_norm(ep_combine(None, buf.expert_y, handle, x, buf), res16, gain, 1e-6)
+        entry("experts' rows + shared + residual + norm (like: combine, add + norm)",
+              lambda: ops.residual_add_norm(res, None, x, (xr, rslots, wt), gain, 1e-6, 0.0, w, mult=0.3),
+              t * w * (2 * k + 2 + 8 + 2), 0, (like_end, t * w * (2 * k + 2 + 8), 0.0))
+        logits, corr = torch.randn(t, e, **f32), torch.randn(e, **f32)
+        entry("routing, sigmoid + correction + groups (like: softmax)",
+              lambda: ops.moe_topk(logits, corr, k, True, group, 2, False, 1.0), t * (e + 2 * k) * 4, 0,
+              (lambda: ops.moe_topk(logits, None, k, False, 1, 1, True, 1.0), t * (e + 2 * k) * 4, 0.0))
+        del x, xr, buf, res, res16
+        gc.collect()
+        torch.cuda.empty_cache()
+    ops.check_status()
+    return out
+
+
 DESIGNS = {
     "rivudra": (SIZES, LAYERS, kernels, {"rivudra": rivudra, "qwen3-moe": qwen3_moe}),
     "fuvirax": (FUVIRAX_SIZES, FUVIRAX_LAYERS, fuvirax_kernels, {"fuvirax": fuvirax, "deepseek-v2 dense": deepseek_dense}),
+    "gatosun": (GATOSUN_SIZES, GATOSUN_LAYERS, gatosun_kernels, {"gatosun": gatosun, "qwen3-moe": qwen3_moe_full}),
 }
 
 

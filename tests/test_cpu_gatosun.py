@@ -217,3 +217,13 @@ def test_two_ranks(tmp_path):
             logits = oracle.forward(seq, w, cfg)[-1]
             assert float(logits.max() - logits[t]) < 1e-3 * float(logits.std())
             seq.append(t)
+
+
+@pytest.mark.parametrize("layer", [cases.attention(2, 1, 16, 8, 8), cases.gla(2, 8, 12, mlp=cases.dense(16)),
+                                   cases.parallel(cases.heads(2, 2, 16, 8, 8, window=5), (2, 8), 0.3, 0.0)])
+def test_models_of_one_mixer(tmp_path, layer):
+    """A model without a cache, one without a recurrent layer, one whose right half counts for nothing."""
+    cfg = cases.model(32, 40, [layer] * 2)
+    w = cases.write_model(tmp_path, cfg, seed=3)
+    cases.check_mixed(cases.Driver(tmp_path, cfg, w, "cpu", "float32", max_tokens=192), rounds=1)
+    cases.check_generate(tmp_path, cfg, w, "cpu", num_gpu_blocks=24)

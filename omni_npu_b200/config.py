@@ -44,9 +44,16 @@ class AttentionSpec:
     sliding_window: int = 0               # 0 = every earlier key
     sink: Optional[float] = None          # score of a key without a value in every softmax
     output_gate: bool = False             # result times the sigmoid of its own projection
-    qk_norm: Optional[str] = None         # "projection": over all of q / of k before the rotation; "head": after it
-    bias: bool = False                    # of all four projections
+    # "projection": over all of q / of k before the rotation; "head": per head after it; "head_weight": per head with
+    # one weight for all heads, before it
+    qk_norm: Optional[str] = None
+    bias: bool = False                    # of the projections
     value_mix: bool = False               # values blended with those of the first such layer
+    query_temperature: Optional[Tuple[float, int]] = None    # (c, n): q times 1 + c ln(floor((p + 1) / n) + 1)
+    softcap: float = 0.0                  # scores <- softcap tanh(score / softcap)
+    distance_bias: bool = False           # learned per head: r1 ln(1 + r2 distance) off the score
+    score_mix: bool = False               # learned mixture of the heads' scores before the softmax
+    head_sink: bool = False               # learned per head: score of a key without a value
 
 
 @dataclass(frozen=True)
@@ -73,7 +80,9 @@ class MoESpec:
 
 @dataclass(frozen=True)
 class LatentAttentionSpec:
-    """Attention over a cached latent (``kv_rank``, normed) and one rotated key part that all heads share."""
+    """Attention over a cached latent (``kv_rank``, normed) and one rotated key part that all heads share.
+    ``q_rank``: queries go through a normed latent of their own; ``kv_from``: the rows cached by that layer are
+    read instead of own ones."""
     num_heads: int
     nope_dim: int
     rope_dim: int
@@ -82,6 +91,8 @@ class LatentAttentionSpec:
     rope_theta: float
     scale: float
     rope_neox: bool = True
+    q_rank: int = 0
+    kv_from: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -136,7 +147,7 @@ class ParallelSpec:
 
 @dataclass(frozen=True)
 class DenseSpec:
-    """A feed-forward without experts: down(act(up(h))) ("xielu") or down(act(gate(h)) * up(h)) ("gelu_tanh")."""
+    """A feed-forward without experts: down(act(up(h))) ("xielu") or down(act(gate(h)) * up(h)) ("gelu_tanh", "relu")."""
     intermediate_size: int
     act: str = "xielu"
     bias: bool = False
@@ -153,7 +164,7 @@ class LayerSpec:
         a = self.attention.left if isinstance(self.attention, ParallelSpec) else self.attention
         if isinstance(a, AttentionSpec):
             return a.num_kv_heads * (a.head_dim + a.v_head_dim)
-        return a.kv_rank + a.rope_dim if isinstance(a, LatentAttentionSpec) else 0
+        return a.kv_rank + a.rope_dim if isinstance(a, LatentAttentionSpec) and a.kv_from is None else 0
 
 
 @dataclass(frozen=True)
@@ -223,6 +234,8 @@ class ModelConfig:
     residual_mult: float = 1.0            # of what a sublayer adds to the residual
     residual_streams: int = 1             # parallel residual streams joined by hyper-connections
     logit_scale: float = 1.0
+    norm_groups: int = 1                  # equal parts of a row that the norms treat one by one
+    token_side_dim: int = 0               # per-layer token input: width of a layer's part
     # --- misc
     eos_token_id: Optional[int] = None
     hf_config: Dict[str, Any] = field(default_factory=dict)

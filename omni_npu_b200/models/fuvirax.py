@@ -21,7 +21,7 @@ divide by the true width.
 """
 from __future__ import annotations
 
-from typing import Any, Callable, Dict, Iterable, List, Optional, Tuple
+from typing import Any, Dict, Iterable, List, Optional, Tuple
 
 import torch
 from torch import nn
@@ -38,6 +38,7 @@ from ..layers.linear import RowParallelLinear, SegmentedLinear
 from ..layers.mlp import XieluMLP
 from ..layers.rope import get_rope
 from ..parallel import state as pstate
+from .layered import Want, fit, pad8, place_tensors
 
 UNIT_EPS = 1e-6          # of the unit norm of the delta rule's q and k
 
@@ -90,22 +91,6 @@ def read_config(d: Dict[str, Any], dtype=None, path: Optional[str] = None) -> Mo
         residual_streams=int(d.get("streams") or 1), logit_scale=float(d.get("logit_scale", 1.0)), hf_config=d)
 
 
-def _pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
-def _fit(t: torch.Tensor, *shape: int) -> torch.Tensor:
-    """``t`` with zeros appended up to ``shape``."""
-    if tuple(t.shape) == shape:
-        return t
-    out = t.new_zeros(shape)
-    out[tuple(slice(0, n) for n in t.shape)] = t
-    return out
-
-
-Want = Dict[str, Tuple[Tuple[int, ...], Callable[[torch.Tensor], Any]]]     # tensor -> (shape, how it is placed)
-
-
 # --------------------------------------------------------------------- mixers
 class FuviraxMixer(nn.Module):
     """Projections around a mixer's core: one product in, one out."""
@@ -113,13 +98,13 @@ class FuviraxMixer(nn.Module):
     def __init__(self, cfg: ModelConfig, segments: Dict[str, Tuple[int, bool]], out_features: int, device,
                  prefix: str) -> None:
         super().__init__()
-        self.width, wp = cfg.hidden_size, _pad8(cfg.hidden_size)
+        self.width, wp = cfg.hidden_size, pad8(cfg.hidden_size)
         self.in_proj = SegmentedLinear(wp, segments, dtype=cfg.dtype, device=device, prefix=f"{prefix}.in_proj")
         self.tp, self.rank = self.in_proj.tp_size, self.in_proj.tp_rank
         self.true_out = out_features
         if self.tp > 1 and out_features // self.tp % 8:
             raise ValueError(f"Fuvirax: {out_features // self.tp} value columns per rank are not whole 16-byte rows")
-        self.o_proj = RowParallelLinear(out_features if self.tp > 1 else _pad8(out_features), wp, dtype=cfg.dtype,
+        self.o_proj = RowParallelLinear(out_features if self.tp > 1 else pad8(out_features), wp, dtype=cfg.dtype,
                                         device=device, prefix=f"{prefix}.o_proj")
 
     def heads(self, n: int) -> int:
@@ -139,7 +124,7 @@ class FuviraxMixer(nn.Module):
             rows = n * self.tp if proj.sharded[name] else n
             want[p + name] = (rows, self.width), lambda t, name=name: proj.weight_loader(proj.weight, t, name)
         want[p + "o"] = (self.width, self.true_out), lambda t: o.weight_loader(
-            o.weight, _fit(t, o.out_features, o.in_features))
+            o.weight, fit(t, o.out_features, o.in_features))
 
     def expect_vector(self, want: Want, name: str, param: nn.Parameter, split: bool) -> None:
         shape = (param.shape[0] * (self.tp if split else 1), *param.shape[1:])
@@ -207,7 +192,7 @@ class DeltaMixer(FuviraxMixer):
         super().__init__(cfg, {"q": (s.num_kv_heads * s.head_dim, True), "k": (s.num_kv_heads * s.head_dim, True),
                                "v": (e, True), "b": (s.num_heads, True), "a1": (s.decay_rank, False),
                                "g1": (s.gate_rank, False)}, e, device, prefix)
-        self.low_cols = _pad8(s.decay_rank), _pad8(s.gate_rank)
+        self.low_cols = pad8(s.decay_rank), pad8(s.gate_rank)
         self.low_proj = SegmentedLinear(sum(self.low_cols), {"a2": (n, True), "g2": (e, True)}, dtype=cfg.dtype,
                                         device=device, prefix=f"{prefix}.low_proj")
         self.attn = DeltaRuleAttention(self.heads(s.num_heads), self.heads(s.num_kv_heads), s.head_dim, s.v_head_dim,
@@ -253,7 +238,7 @@ class FuviraxLayer(nn.Module):
         super().__init__()
         cfg, spec = engine.model, engine.model.layer_specs[idx]
         self.spec = spec
-        wp, prefix = _pad8(cfg.hidden_size), f"layers.{idx}"
+        wp, prefix = pad8(cfg.hidden_size), f"layers.{idx}"
         args = (wp, cfg.hidden_size, cfg.residual_streams, cfg.rms_norm_eps, cfg.dtype, device)
         self.hc1 = HyperSublayer(*args, shift=True)
         a = spec.attention
@@ -281,7 +266,7 @@ class FuviraxForCausalLM(nn.Module):
     def __init__(self, engine_config: EngineConfig, device=None) -> None:
         super().__init__()
         cfg = self.config = engine_config.model
-        self.width, self.padded_width = cfg.hidden_size, _pad8(cfg.hidden_size)
+        self.width, self.padded_width = cfg.hidden_size, pad8(cfg.hidden_size)
         self.embed = ParallelLMHead(cfg.vocab_size, self.padded_width, cfg.dtype, device)     # the head as well
         self.layers = nn.ModuleList([FuviraxLayer(engine_config, i, device) for i in range(cfg.num_layers)])
         self.end = HyperSublayer(self.padded_width, self.width, cfg.residual_streams, cfg.rms_norm_eps, cfg.dtype, device,
@@ -356,32 +341,17 @@ class FuviraxForCausalLM(nn.Module):
         """Place the checkpoint's tensors (padded with zeros where the parameters are wider).  Unknown
         names, wrong shapes and missing tensors are errors; what a checkpoint holds for the feed-forward
         place of a layer without one is not used."""
-        want = self._expected()
         idle = tuple(f"l{i}.{x}" for i, layer in enumerate(self.layers) if layer.mlp is None
                      for x in ("norm2", "ls2", "hc2."))
-        loaded = set()
-        for name, t in weights:
-            if name not in want:
-                if idle and name.startswith(idle):
-                    continue
-                raise ValueError(f"Fuvirax: unknown tensor {name!r}")
-            shape, place = want[name]
-            if tuple(t.shape) != shape:
-                raise ValueError(f"Fuvirax: tensor {name!r} is {tuple(t.shape)}, expected {shape}")
-            place(t)
-            loaded.add(name)
-        missing = sorted(set(want) - loaded)
-        if missing:
-            raise ValueError(f"Fuvirax: {len(missing)} tensors missing, first {missing[:3]}")
-        return loaded
+        return place_tensors(weights, self._expected(), "Fuvirax", lambda name: name.startswith(idle))
 
     def _expected(self) -> Want:
         w, wp = self.width, self.padded_width
         want: Want = {"embed": ((self.config.vocab_size, w), lambda t: self.embed.weight_loader(
-            self.embed.weight, _fit(t, t.shape[0], wp)))}
+            self.embed.weight, fit(t, t.shape[0], wp)))}
 
         def row(name: str, param: nn.Parameter) -> None:
-            want[name] = (w,), lambda t: param.data.copy_(_fit(t, wp))
+            want[name] = (w,), lambda t: param.data.copy_(fit(t, wp))
 
         def norm(name: str, sub: HyperSublayer) -> None:
             row(name, sub.norm_weight)
@@ -402,9 +372,9 @@ class FuviraxForCausalLM(nn.Module):
             if layer.mlp is not None:
                 ff, up, down = layer.spec.mlp.intermediate_size, layer.mlp.up_proj, layer.mlp.down_proj
                 want[p + "mlp.up"] = (ff, w), lambda t, up=up: up.weight_loader(
-                    up.weight, _fit(t, up.out_features, wp))
+                    up.weight, fit(t, up.out_features, wp))
                 want[p + "mlp.down"] = (w, ff), lambda t, down=down: down.weight_loader(
-                    down.weight, _fit(t, wp, down.in_features))
+                    down.weight, fit(t, wp, down.in_features))
                 want[p + "mlp.act"] = (2,), lambda t, m=layer.mlp: m.act_params.data.copy_(t)
         return want
 

@@ -36,11 +36,11 @@ from ..attention.recurrent import DecayLinearAttention, TimeMixAttention
 from ..config import (AttentionSpec, DecayLinearSpec, DenseSpec, EngineConfig, ExpertSpec, LayerSpec, ModelConfig, MoESpec,
                       ParallelSpec, TimeMixSpec, to_dtype)
 from ..layers.embedding import ParallelLMHead, VocabParallelEmbedding
-from ..layers.linear import RowParallelLinear, SegmentedLinear
+from ..layers.linear import SegmentedLinear
 from ..layers.mlp import FusedMLP
 from ..layers.moe import FusedMoE
 from ..layers.rope import get_rope
-from ..parallel import state as pstate
+from .layered import Mixer, Want, fit, pad8, place_tensors
 
 # Steps of at most this many rows run the two halves of a parallel mixer on two streams.
 OVERLAP_ROWS = int(os.environ.get("OMNI_B200_PARALLEL_SUBLAYER_ROWS", "256"))
@@ -118,97 +118,8 @@ def read_config(d: Dict[str, Any], dtype=None, path: Optional[str] = None) -> Mo
         num_experts_per_tok=max((m.top_k for m in moes), default=0), hf_config=d)
 
 
-def _pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
-def _fit(t: torch.Tensor, *shape: int) -> torch.Tensor:
-    """``t`` with zeros appended up to ``shape``."""
-    if tuple(t.shape) == shape:
-        return t
-    out = t.new_zeros(shape)
-    out[tuple(slice(0, n) for n in t.shape)] = t
-    return out
-
-
-Want = Dict[str, Tuple[Tuple[int, ...], Callable[[torch.Tensor], Any]]]     # tensor -> (shape, how it is placed)
-
-
 # --------------------------------------------------------------------- mixers
-class _Mixer(nn.Module):
-    """What the mixers share: this rank's part of heads and rows, and the output projection."""
-
-    def __init__(self, cfg: ModelConfig) -> None:
-        super().__init__()
-        self.width, self.padded_width, self.eps = cfg.hidden_size, _pad8(cfg.hidden_size), cfg.rms_norm_eps
-        group = self.group = pstate.get_tp_group()
-        self.tp, self.rank = group.world_size, group.rank_in_group
-        self.out_scale = 1.0                     # of the mixer's result, for the residual kernel
-
-    def share(self, n: int, what: str = "heads") -> int:
-        if n % self.tp:
-            raise ValueError(f"Gatosun: {n} {what} do not split over {self.tp} ranks")
-        return n // self.tp
-
-    def own(self, t: torch.Tensor, dim: int = 0) -> torch.Tensor:
-        """This rank's part of a tensor that is split by heads."""
-        n = t.shape[dim] // self.tp
-        return t.narrow(dim, self.rank * n, n)
-
-    def output_proj(self, cfg: ModelConfig, parts: List[int], device, prefix: str, bias: bool = False) -> None:
-        """One product for the mixer's parts, each ``parts[i]`` columns of this rank at a whole 16-byte place."""
-        self.parts, self.starts, at = parts, [], 0
-        for n in parts:
-            self.starts.append(at)
-            at += _pad8(n)
-        self.o_proj = RowParallelLinear(at * self.tp, self.padded_width, bias=bias, dtype=cfg.dtype, device=device,
-                                        prefix=f"{prefix}.o_proj")
-        self.o_proj.weight.data.zero_()
-
-    def expect_rows(self, want: Want, p: str, proj: SegmentedLinear) -> None:
-        for name, n in proj.rows.items():
-            rows = n * self.tp if proj.sharded[name] else n
-            want[p + name] = (rows, self.width), lambda t, name=name: proj.weight_loader(proj.weight, t, name)
-            if proj.bias is not None:
-                want[f"{p}{name}.b"] = (rows,), lambda t, name=name: proj.weight_loader(proj.bias, t, name)
-
-    def expect_output(self, want: Want, name: str, part: int) -> None:
-        n, at = self.parts[part], self.starts[part]
-        want[name] = (self.width, n * self.tp), lambda t: self.o_proj.weight.data[: self.width, at: at + n].copy_(
-            self.own(t, 1))
-
-    def expect_vector(self, want: Want, name: str, param: nn.Parameter, split: bool, shape=None) -> None:
-        full = (param.shape[0] * (self.tp if split else 1), *param.shape[1:])
-        want[name] = shape or full, lambda t: param.data.copy_((self.own(t) if split else t).view(param.shape))
-
-    def expect_low(self, want: Want, name: str, low: SegmentedLinear, rank: int) -> None:
-        want[name] = (low.rows["z"] * self.tp, rank), lambda t: low.weight_loader(
-            low.weight, _fit(t, t.shape[0], low.in_features), "z")
-
-    @torch.no_grad()
-    def clear(self, proj: SegmentedLinear, columns: int) -> None:
-        """Zeros in the padding of a projection whose input has ``columns`` true columns."""
-        w = proj.weight.data
-        rows = proj.padding_rows().to(w.device)
-        w[rows] = 0
-        w[:, columns:] = 0
-        if proj.bias is not None:
-            proj.bias.data[rows] = 0
-
-    @torch.no_grad()
-    def clear_output(self) -> None:
-        w = self.o_proj.weight.data
-        w[self.width:] = 0
-        for n, at in zip(self.parts, self.starts):
-            w[:, at + n: at + _pad8(n)] = 0
-        if self.o_proj.bias is not None:
-            self.o_proj.bias.data[self.width:] = 0
-
-    def clear_padding(self) -> None:
-        self.clear_output()
-
-
-def _attention_core(self: _Mixer, cfg: ModelConfig, s: AttentionSpec, cache_idx: int, device, max_position: int):
+def _attention_core(self: Mixer, cfg: ModelConfig, s: AttentionSpec, cache_idx: int, device, max_position: int):
     heads, kv = self.share(s.num_heads), self.share(s.num_kv_heads, "key/value heads")
     self.rotary = get_rope(s.head_dim, s.rotary_dim, max_position, s.rope_theta, s.rope_neox, None, device,
                            exact_angles=True)
@@ -218,7 +129,7 @@ def _attention_core(self: _Mixer, cfg: ModelConfig, s: AttentionSpec, cache_idx:
             "v": (s.num_kv_heads * s.v_head_dim, True)}
 
 
-class AttentionMixer(_Mixer):
+class AttentionMixer(Mixer):
     """``first_values``: whether other layers blend their values with this one's; ``blends``: whether this one does."""
 
     def __init__(self, cfg: ModelConfig, s: AttentionSpec, cache_idx: int, device, prefix: str, max_position: int,
@@ -243,7 +154,7 @@ class AttentionMixer(_Mixer):
         self.expect_rows(want, p, self.in_proj)
         self.expect_output(want, p + "o", 0)
         if self.o_proj.bias is not None:
-            want[p + "o.b"] = (self.width,), lambda t: self.o_proj.bias.data.copy_(_fit(t, self.padded_width))
+            want[p + "o.b"] = (self.width,), lambda t: self.o_proj.bias.data.copy_(fit(t, self.padded_width))
         if self.attn.norm == "projection":
             self.expect_vector(want, p + "q.norm", self.attn.q_norm, True)
             self.expect_vector(want, p + "k.norm", self.attn.k_norm, True)
@@ -256,7 +167,7 @@ class AttentionMixer(_Mixer):
         self.attn.value_mix = float(self.vmix)
 
 
-class ParallelMixer(_Mixer):
+class ParallelMixer(Mixer):
     def __init__(self, cfg: ModelConfig, s: ParallelSpec, cache_idx: int, device, prefix: str, max_position: int) -> None:
         super().__init__(cfg)
         self.spec = s
@@ -271,9 +182,9 @@ class ParallelMixer(_Mixer):
             return nn.Parameter(torch.zeros(*shape, dtype=cfg.dtype, device=device), requires_grad=False)
 
         # r, k, v and the gate read different blends: one grouped product
-        self.rkvg = param(4, _pad8(self.mix_rows), self.padded_width)
-        self.w1 = param(_pad8(s.right.decay_rank), self.padded_width)
-        self.low_proj = SegmentedLinear(_pad8(s.right.decay_rank), {"z": (s.right.num_heads * d, True)}, dtype=cfg.dtype,
+        self.rkvg = param(4, pad8(self.mix_rows), self.padded_width)
+        self.w1 = param(pad8(s.right.decay_rank), self.padded_width)
+        self.low_proj = SegmentedLinear(pad8(s.right.decay_rank), {"z": (s.right.num_heads * d, True)}, dtype=cfg.dtype,
                                         device=device, prefix=f"{prefix}.low_proj")
         self.output_proj(cfg, [self.attn.num_heads * s.left.v_head_dim, self.mix_rows], device, prefix)
         # left_scale * L + right_scale * R = out_scale * (L + right * R); without a left half R alone
@@ -320,7 +231,7 @@ class ParallelMixer(_Mixer):
         p += "right."
         self.expect_output(want, p + "o", 1)
         for i, s in enumerate(a.BLENDS):
-            want[f"{p}mu.{s}"] = (w,), lambda t, i=i: a.mu.data[i].copy_(_fit(t, self.padded_width))
+            want[f"{p}mu.{s}"] = (w,), lambda t, i=i: a.mu.data[i].copy_(fit(t, self.padded_width))
             if i < 4:
                 want[p + s] = (n, w), lambda t, i=i: self.rkvg.data[i, : self.mix_rows, :w].copy_(self.own(t))
         rank = self.spec.right.decay_rank
@@ -345,7 +256,7 @@ class ParallelMixer(_Mixer):
             self.o_proj.weight.data[:, : self.starts[1]] = 0
 
 
-class DecayLinearMixer(_Mixer):
+class DecayLinearMixer(Mixer):
     def __init__(self, cfg: ModelConfig, s: DecayLinearSpec, device, prefix: str) -> None:
         super().__init__(cfg)
         self.spec = s
@@ -354,7 +265,7 @@ class DecayLinearMixer(_Mixer):
         self.in_proj = SegmentedLinear(self.padded_width, {"q": (n, True), "k": (n, True), "v": (e, True), "g": (e, True),
                                                            "a1": (s.decay_rank, False)},
                                        dtype=cfg.dtype, device=device, prefix=f"{prefix}.in_proj")
-        self.low_proj = SegmentedLinear(_pad8(s.decay_rank), {"z": (n, True)}, dtype=cfg.dtype, device=device,
+        self.low_proj = SegmentedLinear(pad8(s.decay_rank), {"z": (n, True)}, dtype=cfg.dtype, device=device,
                                         prefix=f"{prefix}.low_proj")
         self.attn = DecayLinearAttention(heads, s.head_dim, s.v_head_dim, s.tau, cfg.rms_norm_eps, cfg.dtype, device)
         self.output_proj(cfg, [heads * s.v_head_dim], device, prefix)
@@ -394,7 +305,7 @@ class GatosunLayer(nn.Module):
         super().__init__()
         cfg, spec = engine.model, engine.model.layer_specs[idx]
         self.spec = spec
-        w, prefix, positions = _pad8(cfg.hidden_size), f"layers.{idx}", engine.scheduler.max_model_len
+        w, prefix, positions = pad8(cfg.hidden_size), f"layers.{idx}", engine.scheduler.max_model_len
 
         def gain():
             return nn.Parameter(torch.zeros(w, dtype=cfg.dtype, device=device), requires_grad=False)
@@ -417,10 +328,10 @@ class GatosunLayer(nn.Module):
         elif m is not None:
             par = engine.parallel
             self.mlp = FusedMoE(
-                m.num_experts, m.top_k, w, _pad8(m.expert.intermediate_size), cfg.dtype, device, m.scoring_func,
+                m.num_experts, m.top_k, w, pad8(m.expert.intermediate_size), cfg.dtype, device, m.scoring_func,
                 m.renormalize, m.scale, m.n_group, m.topk_group, router_bias=m.correction,
                 num_shared_experts=1 if m.shared else 0,
-                shared_intermediate_size=_pad8(m.shared.intermediate_size) if m.shared else None,
+                shared_intermediate_size=pad8(m.shared.intermediate_size) if m.shared else None,
                 enable_expert_parallel=par.enable_expert_parallel or par.tensor_parallel_size > 1,
                 prefix=f"{prefix}.mlp", unary=m.expert.act,
                 max_tokens=max(engine.scheduler.max_num_batched_tokens, engine.scheduler.max_num_seqs),
@@ -440,7 +351,7 @@ class GatosunForCausalLM(nn.Module):
     def __init__(self, engine_config: EngineConfig, device=None) -> None:
         super().__init__()
         cfg = self.config = engine_config.model
-        self.width, self.padded_width = cfg.hidden_size, _pad8(cfg.hidden_size)
+        self.width, self.padded_width = cfg.hidden_size, pad8(cfg.hidden_size)
         self.embed = VocabParallelEmbedding(cfg.vocab_size, self.padded_width, cfg.dtype, device)
         self.head = ParallelLMHead(cfg.vocab_size, self.padded_width, cfg.dtype, device)
         mixing = [i for i, s in enumerate(cfg.layer_specs)
@@ -519,34 +430,19 @@ class GatosunForCausalLM(nn.Module):
         """Place the checkpoint's tensors (padded with zeros where the parameters are wider).  Unknown names,
         wrong shapes and missing tensors are errors; a norm of a feed-forward that a layer does not have,
         and a blend factor of one that does not blend, are not used."""
-        want = self._expected()
         idle = {f"l{i}.norm2" for i, layer in enumerate(self.layers) if layer.mlp is None}
         idle |= {f"l{i}.mix.vmix" for i, layer in enumerate(self.layers) if isinstance(layer.mix, AttentionMixer)}
-        loaded = set()
-        for name, t in weights:
-            if name not in want:
-                if name in idle:
-                    continue
-                raise ValueError(f"Gatosun: unknown tensor {name!r}")
-            shape, place = want[name]
-            if tuple(t.shape) != shape:
-                raise ValueError(f"Gatosun: tensor {name!r} is {tuple(t.shape)}, expected {shape}")
-            place(t)
-            loaded.add(name)
-        missing = sorted(set(want) - loaded)
-        if missing:
-            raise ValueError(f"Gatosun: {len(missing)} tensors missing, first {missing[:3]}")
-        return loaded
+        return place_tensors(weights, self._expected(), "Gatosun", idle.__contains__)
 
     def _expected(self) -> Want:
         w, wp, vocab = self.width, self.padded_width, self.config.vocab_size
         want: Want = {}
 
         def rows(module, n: int, shard=None):
-            return (n, w), lambda t: module.weight_loader(module.weight, _fit(t, n, wp), shard)
+            return (n, w), lambda t: module.weight_loader(module.weight, fit(t, n, wp), shard)
 
         def norm(name: str, param: nn.Parameter) -> None:
-            want[name] = (w,), lambda t: param.data.copy_(_fit(t, wp))
+            want[name] = (w,), lambda t: param.data.copy_(fit(t, wp))
 
         want["embed"], want["head"] = rows(self.embed, vocab), rows(self.head, vocab)
         norm("final.norm", self.final_norm)
@@ -565,22 +461,22 @@ class GatosunForCausalLM(nn.Module):
         w, wp, ff, gu, down = self.width, self.padded_width, m.intermediate_size, mlp.gate_up_proj, mlp.down_proj
         full = gu.output_sizes[0]
         for j, name in enumerate(("gate", "up")):
-            want[p + name] = (ff, w), lambda t, j=j: gu.weight_loader(gu.weight, _fit(t, full, wp), j)
+            want[p + name] = (ff, w), lambda t, j=j: gu.weight_loader(gu.weight, fit(t, full, wp), j)
             if m.bias:
-                want[f"{p}{name}.b"] = (ff,), lambda t, j=j: gu.weight_loader(gu.bias, _fit(t, full), j)
-        want[p + "down"] = (w, ff), lambda t: down.weight_loader(down.weight, _fit(t, wp, full))
+                want[f"{p}{name}.b"] = (ff,), lambda t, j=j: gu.weight_loader(gu.bias, fit(t, full), j)
+        want[p + "down"] = (w, ff), lambda t: down.weight_loader(down.weight, fit(t, wp, full))
         if m.bias:
-            want[p + "down.b"] = (w,), lambda t: down.weight_loader(down.bias, _fit(t, wp))
+            want[p + "down.b"] = (w,), lambda t: down.weight_loader(down.bias, fit(t, wp))
 
     def _expect_moe(self, want: Want, p: str, moe: FusedMoE, m: MoESpec) -> None:
         w, wp = self.width, self.padded_width
-        want[p + "router"] = (m.num_experts, w), lambda t: moe.gate.weight_loader(moe.gate.weight, _fit(t, t.shape[0], wp))
+        want[p + "router"] = (m.num_experts, w), lambda t: moe.gate.weight_loader(moe.gate.weight, fit(t, t.shape[0], wp))
         want[p + "correction"] = (m.num_experts,), lambda t: moe.e_score_correction_bias.data.copy_(t)
 
         def expert(prefix: str, ff: int, up, down) -> None:
-            fp = _pad8(ff)
-            want[prefix + "up"] = (ff, w), lambda t: up(_fit(t, fp, wp))
-            want[prefix + "down"] = (w, ff), lambda t: down(_fit(t, wp, fp))
+            fp = pad8(ff)
+            want[prefix + "up"] = (ff, w), lambda t: up(fit(t, fp, wp))
+            want[prefix + "down"] = (w, ff), lambda t: down(fit(t, wp, fp))
 
         for e in range(m.num_experts):
             expert(f"{p}e{e}.", m.expert.intermediate_size, lambda t, e=e: moe.weight_loader(moe.w13, t, e, "up"),

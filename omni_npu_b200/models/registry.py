@@ -27,6 +27,7 @@ _REGISTRY: Dict[str, Tuple[str, str]] = {
     "Rivudra": ("omni_npu_b200.models.rivudra", "RivudraForCausalLM"),
     "Fuvirax": ("omni_npu_b200.models.fuvirax", "FuviraxForCausalLM"),
     "Gatosun": ("omni_npu_b200.models.gatosun", "GatosunForCausalLM"),
+    "Dalavik": ("omni_npu_b200.models.dalavik", "DalavikForCausalLM"),
     "MockModel": ("omni_npu_b200.models.mock", "MockModelForCausalLM"),
 }
 
@@ -36,11 +37,12 @@ _CONFIG_READERS: Dict[str, Tuple[str, str]] = {
     "Rivudra": ("omni_npu_b200.models.rivudra", "read_config"),
     "Fuvirax": ("omni_npu_b200.models.fuvirax", "read_config"),
     "Gatosun": ("omni_npu_b200.models.gatosun", "read_config"),
+    "Dalavik": ("omni_npu_b200.models.dalavik", "read_config"),
 }
 
 
 # architectures whose kernels are all in the core library (_build.CORE_SOURCES)
-_CORE_LIBRARY_ONLY = {"Rivudra", "Fuvirax", "Gatosun"}
+_CORE_LIBRARY_ONLY = {"Rivudra", "Fuvirax", "Gatosun", "Dalavik"}
 
 
 def runs_on_core_library(arch: str) -> bool:

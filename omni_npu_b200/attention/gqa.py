@@ -153,10 +153,8 @@ class GatedGQAAttention(torch.nn.Module):
             out = q.new_zeros(t, out_width) if out_width > used else q.new_empty(t, used)
 
         def run(rows: slice, seqs: slice, cu_q, n: int, max_q: int):
-            ops.gated_attention(q[rows], None if gate is None else gate[rows], k_cache, v_cache, out[rows],
-                                md.block_tables[seqs], cu_q, md.seq_lens[seqs], n, max_q, self.num_heads,
-                                self.head_dim, self.head_dim_v, self.scale, self.window, self.sink,
-                                max_seq_len=md.max_seq_len)
+            self._run(q[rows], None if gate is None else gate[rows], k_cache, v_cache, out[rows], md.block_tables[seqs],
+                      cu_q, md.seq_lens[seqs], n, max_q, md.max_seq_len)
 
         if not md.is_prefill:
             run(slice(None), slice(None), None, md.num_seqs, md.q_len)
@@ -169,6 +167,10 @@ class GatedGQAAttention(torch.nn.Module):
         else:
             run(slice(None), slice(None), md.cu_q, md.num_seqs, md.max_q_len)
         return out
+
+    def _run(self, q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, n: int, max_q: int, max_seq: int) -> None:
+        ops.gated_attention(q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, n, max_q, self.num_heads,
+                            self.head_dim, self.head_dim_v, self.scale, self.window, self.sink, max_seq_len=max_seq)
 
 
 class NormedGQAAttention(GatedGQAAttention):
@@ -203,3 +205,44 @@ class NormedGQAAttention(GatedGQAAttention):
                                    self.head_dim_v, self.rot_dim, self.norm, self.eps, weights, sums, v_first,
                                    self.value_mix)
         return self._attend(q, None, md, k_cache, v_cache, out_width, out)
+
+
+class MixedScoreAttention(GatedGQAAttention):
+    """Attention without rotation whose heads mix their scores before the softmax (``ops.mixed_attention``): q and k
+    normed per head with a weight, queries with a temperature that grows with the position, scores capped and lowered
+    by a learned distance bias, a learned sink per head.
+
+    ``num_heads`` score heads over ``num_kv_heads`` key heads, whole on every rank; ``out_heads`` output heads over
+    ``v_heads`` value heads of this rank.  The constants that multiply scores are kept in fp32."""
+
+    def __init__(self, layer_idx: int, num_heads: int, num_kv_heads: int, out_heads: int, v_heads: int, head_dim: int,
+                 head_dim_v: int, scale: float, softcap: float, temperature: Optional[Tuple[float, int]], eps: float, dtype,
+                 device) -> None:
+        super().__init__(layer_idx, num_heads, num_kv_heads, head_dim, head_dim_v, scale, 0)
+        self.out_heads, self.v_heads = out_heads, v_heads
+        self.softcap, self.temperature, self.eps = softcap, temperature, eps
+
+        def param(*shape, fill=0.0, dt=torch.float32):
+            return torch.nn.Parameter(torch.full(shape, fill, dtype=dt, device=device), requires_grad=False)
+
+        self.q_norm, self.k_norm = param(head_dim, fill=1.0, dt=dtype), param(head_dim, fill=1.0, dt=dtype)
+        self.r1, self.r2, self.sink = param(num_heads), param(num_heads), param(out_heads)
+        self.talk = param(out_heads, num_heads)
+
+    def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out_width: int = 0) -> torch.Tensor:
+        """q [T, Hs*D], k [T, Hk*D], v [T, Hv*Dv]: views into the fused projection.  Returns
+        [T, max(Ho*Dv, out_width)], zero beyond the heads."""
+        ctx = get_forward_context()
+        md: AttentionMetadata = ctx.attn_metadata
+        k_cache, v_cache = ctx.kv_caches[self.layer_idx]
+        q = ops.qk_norm_rope_cache(q, k, v, k_cache, v_cache, md.positions, md.slot_mapping, None, self.head_dim,
+                                   self.head_dim_v, 0, "head_weight", self.eps, (self.q_norm, self.k_norm),
+                                   temperature=self.temperature)
+        t, used = q.shape[0], self.out_heads * self.head_dim_v
+        out = q.new_zeros(t, out_width) if out_width > used else q.new_empty(t, used)
+        self._attend(q, None, md, k_cache, v_cache, out=out)
+        return out
+
+    def _run(self, q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, n: int, max_q: int, max_seq: int) -> None:
+        ops.mixed_attention(q, k_cache, v_cache, out, block_tables, cu_q, seq_lens, n, max_q, self.head_dim, self.head_dim_v,
+                            self.scale, self.softcap, (self.r1, self.r2), self.talk, self.sink, max_seq_len=max_seq)

@@ -9,6 +9,9 @@ or take them from here) there are two paths:
   copies the rotated part, so that the product yields whole keys;
 * single new tokens: queries are folded into the latent space, attend over the rows themselves, and the
   result is brought back per head.
+
+Queries may come from a latent of their own (``q_rank``); its norm runs with the cache row's (``store``).  A layer
+that reads another layer's rows stores none; what that layer gathered for a prompt step is used again.
 """
 from __future__ import annotations
 
@@ -26,8 +29,10 @@ class LatentAttention(nn.Module):
     set before ``build_absorbed``."""
 
     def __init__(self, num_heads: int, nope_dim: int, rope_dim: int, v_head_dim: int, kv_rank: int, scale: float,
-                 neox: bool, eps: float, dtype: torch.dtype, device) -> None:
+                 neox: bool, eps: float, dtype: torch.dtype, device, q_rank: int = 0, own_rows: bool = True,
+                 rows_shared: bool = False) -> None:
         super().__init__()
+        self.q_rank, self.own_rows, self.rows_shared = q_rank, own_rows, rows_shared
         self.num_heads, self.nope, self.rot, self.v_dim, self.rank = num_heads, nope_dim, rope_dim, v_head_dim, kv_rank
         self.scale, self.neox, self.eps, self.dtype = scale, neox, eps, dtype
         self.qk_dim = nope_dim + rope_dim
@@ -37,7 +42,8 @@ class LatentAttention(nn.Module):
         def param(*shape, fill=0.0):
             return nn.Parameter(torch.full(shape, fill, dtype=dtype, device=device), requires_grad=False)
 
-        self.latent_norm = param(kv_rank, fill=1.0)
+        self.latent_norm = param(kv_rank, fill=1.0) if own_rows else None
+        self.query_norm = param(q_rank, fill=1.0) if q_rank else None
         self.w_uk = param(num_heads * nope_dim, kv_rank)
         self.w_uv = param(num_heads * v_head_dim, kv_rank)
         # products of the two paths, derived from the two above
@@ -60,10 +66,21 @@ class LatentAttention(nn.Module):
         self.w_fold.copy_(uk.transpose(1, 2))
 
     # ------------------------------------------------------------------ forward
-    def forward(self, q: torch.Tensor, kv_a: torch.Tensor, cos_sin: torch.Tensor, cache_idx: int,
+    def store(self, z: torch.Tensor, kv_a: Optional[torch.Tensor], cos_sin: torch.Tensor, cache_idx: int) -> torch.Tensor:
+        """The queries' latent z [T, q_rank] normed (with zeros up to whole 16-byte rows), and the cache row when the
+        layer has its own: views into the projection."""
+        ctx = get_forward_context()
+        md: AttentionMetadata = ctx.attn_metadata
+        c_q = z.new_empty(z.shape[0], (self.q_rank + 7) // 8 * 8)
+        ops.latent_prep_(None, kv_a, self.latent_norm, self.eps, ctx.kv_caches[cache_idx], md.positions, md.slot_mapping,
+                         cos_sin, self.num_heads, self.nope, self.rot, self.rank, self.neox,
+                         low=(z, self.query_norm, c_q))
+        return c_q
+
+    def forward(self, q: torch.Tensor, kv_a: Optional[torch.Tensor], cos_sin: torch.Tensor, cache_idx: int,
                 out_width: int = 0) -> torch.Tensor:
-        """q [T, heads * (nope + rot)] (rotated in place), kv_a [T, rank + rot]: views into the
-        projection.  Returns [T, max(heads * v, out_width)], zero beyond the heads."""
+        """q [T, heads * (nope + rot)] (rotated in place), kv_a [T, rank + rot] or None (the rows are stored
+        already): views into the projection.  Returns [T, max(heads * v, out_width)], zero beyond the heads."""
         ctx = get_forward_context()
         md: AttentionMetadata = ctx.attn_metadata
         cache = ctx.kv_caches[cache_idx]
@@ -77,7 +94,7 @@ class LatentAttention(nn.Module):
         if nd:
             self._decode(q[:nd], q_latent[:nd], cache, md, nd, out[:nd])
         if nd < t:
-            self._prompt(q[nd:], cache, md, nd, out[nd:])
+            self._prompt(q[nd:], cache, cache_idx, md, nd, out[nd:])
         return out
 
     def _decode(self, q, q_latent, cache, md: AttentionMetadata, n: int, out) -> None:
@@ -89,7 +106,7 @@ class LatentAttention(nn.Module):
         uv = self.w_uv.view(self.num_heads, self.v_dim, self.rank)
         ops.head_gemm(o, uv, out[:, : self.num_heads * self.v_dim].unflatten(1, (self.num_heads, self.v_dim)))
 
-    def _prompt(self, q, cache, md: AttentionMetadata, nd: int, out) -> None:
+    def _prompt(self, q, cache, cache_idx: int, md: AttentionMetadata, nd: int, out) -> None:
         n = md.num_seqs - nd
         bt, lens = md.block_tables[nd: md.num_seqs], md.seq_lens[nd: md.num_seqs]
         shared = md.extra.setdefault("latent_prompt", {})           # same for every layer of the step
@@ -97,7 +114,11 @@ class LatentAttention(nn.Module):
             host = md.extra.get("seq_lens_host")
             total = sum((lens.tolist() if host is None else host[nd:]))
             shared.update(total=total, start=(torch.cumsum(lens, 0, dtype=torch.int32) - lens).contiguous())
-        rows = ops.latent_gather(cache, bt, lens, shared["start"], n, shared["total"], md.max_seq_len)
+        rows = shared.get(cache_idx) if not self.own_rows else None
+        if rows is None:
+            rows = ops.latent_gather(cache, bt, lens, shared["start"], n, shared["total"], md.max_seq_len)
+            if self.rows_shared:
+                shared[cache_idx] = rows
         k = ops.gemm(rows, self.w_key).view(-1, self.num_heads, 1, self.k_pad)
         v = ops.gemm(rows, self.w_value).view(-1, self.num_heads, 1, self.v_pad)
         cu_q = md.extra["cu_q_prefill"] if nd else md.cu_q

@@ -199,7 +199,9 @@ SMALL_M_GEMM = os.environ.get("OMNI_B200_SMALL_M_GEMM", "library")
 SMALL_M_LIBRARY_ROWS = (64, 256)
 
 GELU_TANH = "gelu_tanh"    # gated activation gelu(gate) * up, gelu in its tanh form
+RELU = "relu"              # gated activation max(gate, 0) * up
 UNARY = {"relu2": 5, "tanh": 6}
+_GATED = {GELU_TANH: 4, RELU: 7}
 
 
 def _act_kind(swiglu: bool, act, xielu: Optional[Tuple[float, float]] = None,
@@ -211,7 +213,7 @@ def _act_kind(swiglu: bool, act, xielu: Optional[Tuple[float, float]] = None,
         return (UNARY[unary], 0.0, 0.0)
     if not swiglu:
         return (0, 0.0, 0.0)
-    return (4, 0.0, 0.0) if act == GELU_TANH else (2 if act[0] != 0.0 else 1, *act)
+    return (_GATED[act], 0.0, 0.0) if isinstance(act, str) else (2 if act[0] != 0.0 else 1, *act)
 
 
 def library_small_m(m: int, cluster_split_plan: bool, plain_bf16: bool) -> bool:
@@ -230,7 +232,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
     """``a[M,K] @ w[N,K].T`` (+bias, +residual).  bf16 or float8_e4m3fn inputs,
     fp32 accumulation, bf16 (default) or fp32 output.  ``swiglu`` fuses
     silu(gate)*up for weights laid out by :func:`ref.interleave_gate_up`; ``act`` = (slope, limit)
-    with a non-zero slope selects the clamped form of it, ``GELU_TANH`` gelu (:func:`ref.gated_act`); the
+    with a non-zero slope selects the clamped form of it, ``GELU_TANH`` gelu, ``RELU`` relu (:func:`ref.gated_act`); the
     bias is added before a gated activation.  ``xielu`` = (a, b) applies :func:`ref.xielu` to every output,
     ``unary`` the named :func:`ref.unary_act`.  fp32 inputs run on the CUDA cores, with no
     reduced-precision mode.
@@ -257,7 +259,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         _count(1)
         return C.gemm_pair(a, w, bias, residual, out_dtype == torch.float32, kind[0], pbn, st.status, max_ctas,
                            kind[1], kind[2])
-    fused, gated = kind[0] != 0, kind[0] in (1, 2, 4)
+    fused, gated = kind[0] != 0, kind[0] in (1, 2, 4, 7)
     key = (m, n, k, a.dtype.itemsize, kind[0], bn, splits)
     plan = st.plans.get(key)
     if plan is None:
@@ -702,23 +704,30 @@ def gated_rope_cache_(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache
                              rot_dim, neox)
 
 
+QK_NORMS = {None: 0, "projection": 1, "head": 2, "head_weight": 3}
+
+
 def qk_norm_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
-                       positions: torch.Tensor, slot_mapping: torch.Tensor, cos_sin: torch.Tensor, head_dim: int,
+                       positions: torch.Tensor, slot_mapping: torch.Tensor, cos_sin: Optional[torch.Tensor], head_dim: int,
                        head_dim_v: int, rot_dim: int, norm: Optional[str], eps: float, weights=None, sums=None,
-                       v_first: Optional[torch.Tensor] = None, mix: float = 0.0) -> torch.Tensor:
+                       v_first: Optional[torch.Tensor] = None, mix: float = 0.0,
+                       temperature: Optional[Tuple[float, int]] = None) -> torch.Tensor:
     """Norm and rotation (rotate-half pairs) of q and k, k / v into the paged cache, whose rows may be wider than
     the heads; returns the queries [T, Hq * head_dim].  ``norm``: "projection" = RMS norm over all of q (and of
-    k) with ``weights`` = (q, k) before the rotation, "head" = every head divided by its root mean square
-    after it, None.  ``sums`` = (sums of squares of q and k [T, 2], elements of q, of k): taken over more than
-    these rows.  ``v_first``: what is stored is (1 - mix) v + mix v_first."""
+    k) with ``weights`` = (q, k) before the rotation, "head_weight" = per head with ``weights`` [head_dim] for all
+    heads before it, "head" = every head divided by its root mean square after it, None.  ``sums`` = (sums of
+    squares of q and k [T, 2], elements of q, of k): taken over more than these rows.  ``v_first``: what is
+    stored is (1 - mix) v + mix v_first.  ``temperature`` = (c, n): queries at position p times
+    1 + c ln(floor((p + 1) / n) + 1)."""
     if not q.is_cuda:
         return ref.qk_norm_rope_cache(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim, head_dim_v,
-                                      rot_dim, norm, eps, weights, sums, v_first, mix)
+                                      rot_dim, norm, eps, weights, sums, v_first, mix, temperature)
     qw, kw = weights if weights is not None else (None, None)
     s, nq, nk = sums if sums is not None else (None, q.shape[1], k.shape[1])
+    c, n = temperature if temperature is not None else (0.0, 0)
     _count(1)
     return _core().qk_norm_rope(q, k, v, v_first, mix, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim,
-                                head_dim_v, rot_dim, {None: 0, "projection": 1, "head": 2}[norm], qw, kw, s, nq, nk, eps)
+                                head_dim_v, rot_dim, QK_NORMS[norm], qw, kw, s, nq, nk, eps, c, n)
 
 
 def gated_decode_splits(num_seqs: int, num_kv_heads: int, keys: int, sms: int = 148) -> int:
@@ -753,6 +762,59 @@ def gated_attention(q: torch.Tensor, gate: Optional[torch.Tensor], k_cache: torc
                             device_state(q.device).status, False)
 
 
+# --------------------------------------------------- attention whose heads share their scores
+MIXED_SCORE_BYTES = int(os.environ.get("OMNI_B200_MIXED_SCORE_MB", "512")) << 20
+
+
+def mixed_decode_splits(num_rows: int, keys: int, sms: int = 148) -> int:
+    """CTAs that share the keys of a decode row: at least 64 keys each, the GPU filled once."""
+    return max(1, min(32, sms // max(1, num_rows), (keys + 63) // 64))
+
+
+def mixed_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
+                    block_tables: torch.Tensor, cu_q: Optional[torch.Tensor], seq_lens: torch.Tensor, num_seqs: int,
+                    max_q_len: int, head_dim: int, head_dim_v: int, scale: float, softcap: float, bias,
+                    talk: torch.Tensor, sink: Optional[torch.Tensor], max_seq_len: int = 0, splits: int = 0,
+                    variant: int = 0) -> None:
+    """Attention over the paged cache whose heads mix their scores before the softmax (csrc/attn/mixed_attn.cuh),
+    written into ``out`` [T, >= Ho * Dv].  q [T, Hs * Dk]; ``softcap`` 0: none; ``bias`` = (r1, r2) fp32 [Hs] or
+    None: r1 ln(1 + r2 distance) is taken off; ``talk`` fp32 [Ho, Hs]; ``sink`` fp32 [Ho] or None: score of a key
+    without a value.  Score head h reads key head h / (Hs / Hk), output head h value head h / (Ho / Hv).
+    ``cu_q``: query offsets of prompt portions; None = decode step with ``max_q_len`` rows per sequence.
+    ``variant``: 0 = by shape, 1 = the tensor-core kernels or an error, 2 = the plain kernel."""
+    if not q.is_cuda:
+        return ref.mixed_attention(q, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len, head_dim,
+                                   head_dim_v, scale, softcap, bias, talk, sink)
+    core, rows = _core(), q.shape[0]
+    keys = max_seq_len or block_tables.shape[1] * k_cache.shape[2]
+    r1, r2 = bias if bias is not None else (None, None)
+    args = (q, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len, keys, head_dim, head_dim_v, scale,
+            softcap, r1, r2, talk, sink)
+    kind = core.mixed_attention_kind(q, k_cache, v_cache, talk, cu_q is not None, variant)     # 0 plain, 1 tensor cores
+    if kind == 0:
+        _count(1)
+        core.mixed_attention(*args, 0, 1, None, 0, 0)
+        return
+    st = device_state(q.device)
+    if cu_q is None:
+        if splits <= 0:
+            splits = mixed_decode_splits(rows, keys)
+        scratch = None
+        if splits > 1:
+            nbytes = rows * splits * talk.shape[0] * (v_cache.shape[3] + 2) * 4
+            scratch = st.decode_scratch(torch.cuda.current_stream(q.device).cuda_stream, nbytes)
+        _count(2 if splits > 1 else 1)
+        core.mixed_attention(*args, 1, splits, scratch, 0, 0)
+        return
+    # prompt portions: the mixed scores of a run of query tiles go through memory
+    tile, tiles, pitch = 16, (max_q_len + 15) // 16, (keys + 63) // 64 * 64
+    run = max(1, min(tiles, MIXED_SCORE_BYTES // (num_seqs * tile * talk.shape[0] * pitch * 4)))
+    scores = torch.empty(num_seqs * run * tile * talk.shape[0] * pitch, dtype=torch.float32, device=q.device)
+    for t0 in range(0, tiles, run):
+        _count(2)
+        core.mixed_attention(*args, 1, 1, scores, t0, min(run, tiles - t0))
+
+
 # ----------------------------------------------------------- 32-bit residual stream
 def embed_residual_norm(residual: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, scale: float,
                         weight: torch.Tensor, eps: float, weight_offset: float, true_width: int) -> torch.Tensor:
@@ -778,6 +840,28 @@ def residual_add_norm(residual: torch.Tensor, a: Optional[torch.Tensor], b: Opti
     out = _core().residual_norm(residual, None, None, 1.0, a, b, y, slots, w, weight, eps, weight_offset, true_width,
                                 like.dtype == torch.float32, mult)
     return out if weight is not None else None
+
+
+def post_norm_residual(residual: torch.Tensor, y: Optional[torch.Tensor], weight: Optional[torch.Tensor], groups: int,
+                       eps: float, true_width: int, ids: Optional[torch.Tensor] = None,
+                       table: Optional[torch.Tensor] = None, out_norm=None) -> torch.Tensor:
+    """residual [T, W] fp32 += norm(y) * weight, every one of ``groups`` equal parts of the row by its own root mean
+    square (or, with ``ids``, residual <- table[ids]).  Returns the residual in y's type, or with ``out_norm`` =
+    (weight, groups) its norm of the same kind."""
+    if not residual.is_cuda:
+        return ref.post_norm_residual(residual, y, weight, groups, eps, true_width, ids, table, out_norm)
+    ow, og = out_norm if out_norm is not None else (None, 1)
+    _count(1)
+    return _core().post_norm_residual(residual, y, weight, groups, eps, true_width, ids, table, ow, og)
+
+
+def gelu_rows(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, offset: int, dim: int) -> torch.Tensor:
+    """gelu(z) (tanh form) times the columns ``offset`` .. ``offset + dim`` of the rows ``table[ids]``; like z, zero
+    beyond ``dim``."""
+    if not z.is_cuda:
+        return ref.gelu_rows(z, ids, table, offset, dim)
+    _count(1)
+    return _core().gelu_rows(z, ids, table, offset, dim)
 
 
 # ------------------------------------ several residual streams, layer norm and token shift in one pass
@@ -880,20 +964,25 @@ def time_mix_prep(r: torch.Tensor, k: torch.Tensor, z: torch.Tensor, w0: torch.T
 
 
 # ------------------------------------------------------- latent attention with run-time sizes
-def latent_prep_(q: torch.Tensor, kv_a: torch.Tensor, norm_w: torch.Tensor, eps: float, cache: torch.Tensor,
-                 positions: torch.Tensor, slot_mapping: torch.Tensor, cos_sin: torch.Tensor, heads: int, dim: int,
-                 rot: int, rank: int, neox: bool, q_latent: Optional[torch.Tensor] = None, num_latent: int = 0) -> None:
+def latent_prep_(q: Optional[torch.Tensor], kv_a: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], eps: float,
+                 cache: torch.Tensor, positions: torch.Tensor, slot_mapping: torch.Tensor, cos_sin: torch.Tensor, heads: int,
+                 dim: int, rot: int, rank: int, neox: bool, q_latent: Optional[torch.Tensor] = None, num_latent: int = 0,
+                 low=None) -> None:
     """RMS norm of the latent and rotation of the shared key part into the cache row
     [latent | rotated | zeros]; rotation of the queries: in place, but for the first ``num_latent`` rows into
-    columns ``rank`` .. of ``q_latent`` [num_latent.., heads, row]."""
-    if not q.is_cuda:
-        for rows, lat in ((slice(0, num_latent), q_latent), (slice(num_latent, q.shape[0]), None)):
-            ref.latent_prep_(q[rows], kv_a[rows], norm_w, eps, cache, positions[: q.shape[0]][rows],
-                             slot_mapping[: q.shape[0]][rows], cos_sin, heads, dim, rot, rank, neox, lat)
+    columns ``rank`` .. of ``q_latent`` [num_latent.., heads, row].  Either part may be absent.  ``low`` = (z, weight
+    [n], out [T, >= n]): RMS norm of the queries' own latent, zeros behind it."""
+    some = next(x for x in (q, kv_a, low[0] if low else None) if x is not None)
+    if not some.is_cuda:
+        t = some.shape[0]
+        for rows, lat in ((slice(0, num_latent), q_latent), (slice(num_latent, t), None)):
+            ref.latent_prep_(None if q is None else q[rows], None if kv_a is None else kv_a[rows], norm_w, eps, cache,
+                             positions[:t][rows], slot_mapping[:t][rows], cos_sin, heads, dim, rot, rank, neox, lat,
+                             None if low is None else (low[0][rows], low[1], low[2][rows]))
         return
     _count(1)
     _core().latent_prep(q, kv_a, norm_w, eps, cache, positions, slot_mapping, cos_sin, heads, dim, rot, rank, neox,
-                        q_latent, num_latent)
+                        q_latent, num_latent, *(low or (None, None, None)))
 
 
 def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:

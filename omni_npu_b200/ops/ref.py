@@ -51,10 +51,12 @@ def unary_act(z: torch.Tensor, kind: str) -> torch.Tensor:
 
 
 def gated_act(gate: torch.Tensor, up: torch.Tensor, act=(0.0, 0.0)) -> torch.Tensor:
-    """silu(gate) * up, or gelu (tanh form) for ``act`` "gelu_tanh"; with ``act`` = (slope, limit), slope non-zero:
+    """silu(gate) * up, gelu (tanh form) for ``act`` "gelu_tanh", max(gate, 0) for "relu"; with ``act`` = (slope, limit), slope non-zero:
     g * sigmoid(slope * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
     if act == "gelu_tanh":
         return F.gelu(gate, approximate="tanh") * up
+    if act == "relu":
+        return F.relu(gate) * up
     slope, limit = act
     if slope == 0.0:
         return F.silu(gate) * up
@@ -259,20 +261,30 @@ def gated_rope_cache_(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_si
     gqa_cache_write(ko, v, k_cache[..., :head_dim], v_cache[..., :head_dim_v], slot_mapping)
 
 
+def _head_rms(x, head_dim, eps):
+    x = x.reshape(x.shape[0], -1, head_dim)
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
 def qk_norm_rope_cache(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_sin, head_dim, head_dim_v, rot_dim, norm,
-                       eps, weights, sums, v_first, mix):
+                       eps, weights, sums, v_first, mix, temperature=None):
     """Norm, rotation, value mixing, cache write; returns the queries."""
     qf, kf, vf = q.float(), k.float(), v.float()
+    if norm == "head_weight":
+        qf, kf = ((_head_rms(x, head_dim, eps) * w.float()).flatten(1) for x, w in zip((qf, kf), weights))
     if norm == "projection":
         if sums is None:
             sums = torch.stack([qf.pow(2).sum(-1), kf.pow(2).sum(-1)], 1), q.shape[1], k.shape[1]
         s, nq, nk = sums
         qf = qf * torch.rsqrt(s[:, :1] / nq + eps) * weights[0].float()
         kf = kf * torch.rsqrt(s[:, 1:] / nk + eps) * weights[1].float()
-    qf, kf = rope_qk(qf, kf, positions, cos_sin, head_dim, rot_dim, True)
+    if rot_dim:
+        qf, kf = rope_qk(qf, kf, positions, cos_sin, head_dim, rot_dim, True)
     if norm == "head":
-        qf, kf = (x.reshape(x.shape[0], -1, head_dim) for x in (qf, kf))
-        qf, kf = ((x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) for x in (qf, kf))
+        qf, kf = (_head_rms(x, head_dim, eps).flatten(1) for x in (qf, kf))
+    if temperature is not None:
+        c, n = temperature
+        qf = qf * (1 + c * torch.log(((positions.long() + 1) // n).float() + 1)).unsqueeze(1)
     if v_first is not None:
         vf = (1 - mix) * vf + mix * v_first.float()
     gqa_cache_write(kf.to(k.dtype), vf.to(v.dtype), k_cache[..., :head_dim], v_cache[..., :head_dim_v], slot_mapping)
@@ -294,6 +306,52 @@ def gated_attention(q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens
     if gate is not None:
         y = y * torch.sigmoid(gate.float())
     out[:, : y.shape[1]].copy_(y)
+
+
+def mixed_attention(q, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len, head_dim, head_dim_v, scale,
+                    softcap, bias, talk, sink) -> None:
+    """Paged attention whose heads' scores are capped, lowered by a distance bias and mixed before the softmax."""
+    if cu_q is None:
+        cu_q = torch.arange(0, (num_seqs + 1) * max_q_len, max_q_len, dtype=torch.int32)
+    cu, heads, ho = cu_q.tolist(), talk.shape[1], talk.shape[0]
+    for b in range(num_seqs):
+        qs, qe, n = cu[b], cu[b + 1], int(seq_lens[b])
+        if qs == qe:
+            continue
+        k = _gather_kv(k_cache[..., :head_dim], block_tables[b], n).float().repeat_interleave(heads // k_cache.shape[1], 1)
+        v = _gather_kv(v_cache[..., :head_dim_v], block_tables[b], n).float().repeat_interleave(ho // v_cache.shape[1], 1)
+        s = torch.einsum("qhd,khd->hqk", q[qs:qe].float().view(qe - qs, heads, head_dim), k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        dist = torch.arange(n - (qe - qs), n)[:, None] - torch.arange(n)[None, :]
+        if bias is not None:
+            s = s - bias[0][:, None, None] * torch.log1p(bias[1][:, None, None] * dist.clamp(min=0))
+        s = torch.einsum("hg,gqk->hqk", talk, s).masked_fill(dist < 0, float("-inf"))
+        if sink is not None:
+            s = torch.cat([s, sink[:, None, None].expand(-1, qe - qs, 1)], -1)
+        p = torch.softmax(s, -1)[..., :n]
+        out[qs:qe, : ho * head_dim_v] = torch.einsum("hqk,khd->qhd", p, v).flatten(1).to(out.dtype)
+
+
+def _grouped_norm(x, weight, groups, true_width, eps):
+    g = x[:, :true_width].unflatten(1, (groups, true_width // groups))
+    g = (g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) * weight[:true_width].float()
+    return F.pad(g, (0, x.shape[1] - true_width))
+
+
+def post_norm_residual(residual, y, weight, groups, eps, true_width, ids, table, out_norm):
+    if ids is not None:
+        residual.copy_(table[ids.long()].float())
+    else:
+        residual += _grouped_norm(y.float(), weight, groups, true_width, eps)
+    like = table if ids is not None else y
+    return (residual if out_norm is None else _grouped_norm(residual, *out_norm, true_width, eps)).to(like.dtype)
+
+
+def gelu_rows(z, ids, table, offset, dim):
+    out = torch.zeros_like(z)
+    out[:, :dim] = F.gelu(z[:, :dim].float(), approximate="tanh") * table[ids.long(), offset: offset + dim].float()
+    return out
 
 
 def embed_residual_norm(residual, ids, table, scale, weight, eps, weight_offset, true_width):
@@ -765,23 +823,30 @@ def head_norm_gate(o, weight, eps, gate, out_width, silu=False, scale=1.0, out=N
 
 
 # ------------------------------------------------------------- latent attention of any size
-def latent_prep_(q, kv_a, norm_w, eps, cache, positions, slot_mapping, cos_sin, heads, dim, rot, rank, neox, q_latent):
-    t = q.shape[0]
+def latent_prep_(q, kv_a, norm_w, eps, cache, positions, slot_mapping, cos_sin, heads, dim, rot, rank, neox, q_latent,
+                 low=None):
     half = rot // 2
     cs = cos_sin[positions.long()]
     cos, sin = cs[:, :half], cs[:, half:]
-    qv = q[:, : heads * (dim + rot)].unflatten(1, (heads, dim + rot))
-    q_rot = _rope_one(qv[..., dim:].contiguous(), cos, sin, rot, neox)
-    if q_latent is None:
-        qv[..., dim:] = q_rot
-    else:
-        q_latent[:t, :, rank: rank + rot] = q_rot
-        q_latent[:t, :, rank + rot:] = 0
-    c = kv_a[:, :rank].float()
-    c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
-    pe = _rope_one(kv_a[:, rank: rank + rot].reshape(t, 1, rot), cos, sin, rot, neox).view(t, rot)
-    row = F.pad(torch.cat([c.to(cache.dtype), pe.to(cache.dtype)], -1), (0, cache.shape[-1] - rank - rot))
-    paged_scatter_rows(cache, row, slot_mapping)
+    if q is not None:
+        qv = q[:, : heads * (dim + rot)].unflatten(1, (heads, dim + rot))
+        q_rot = _rope_one(qv[..., dim:].contiguous(), cos, sin, rot, neox)
+        if q_latent is None:
+            qv[..., dim:] = q_rot
+        else:
+            q_latent[: q.shape[0], :, rank: rank + rot] = q_rot
+            q_latent[: q.shape[0], :, rank + rot:] = 0
+    if low is not None:
+        z, w, out = low
+        n = w.shape[0]
+        out[:, :n] = rms_norm(z[:, :n], w, eps)
+        out[:, n:] = 0
+    if kv_a is not None:
+        t = kv_a.shape[0]
+        c = rms_norm(kv_a[:, :rank].float(), norm_w, eps)
+        pe = _rope_one(kv_a[:, rank: rank + rot].reshape(t, 1, rot), cos, sin, rot, neox).view(t, rot)
+        row = F.pad(torch.cat([c.to(cache.dtype), pe.to(cache.dtype)], -1), (0, cache.shape[-1] - rank - rot))
+        paged_scatter_rows(cache, row, slot_mapping)
 
 
 def head_gemm(a, w, out):

@@ -39,15 +39,16 @@ CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function"]
 # sources of the core library, relative to csrc/
 CORE_SOURCES = [
     "attn/gqa_gated.cu", "attn/gqa_gated_decode.cu", "attn/gqa_gated_prefill.cu", "attn/gqa_prefill_tcgen05.cu",
-    "attn/latent_attn.cu", "attn/mla_decode.cu", "attn/qk_norm_rope.cu",
+    "attn/latent_attn.cu", "attn/mixed_attn.cu", "attn/mixed_attn_decode.cu", "attn/mixed_attn_prefill.cu",
+    "attn/mla_decode.cu", "attn/qk_norm_rope.cu",
     "gemm/gemm_simt.cu", "gemm/gemm_tcgen05.cu", "gemm/gemm_tcgen05_pair.cu", "moe/moe_ep.cu",
-    "norm_rope/hyper_norm.cu", "norm_rope/residual_norm.cu", "recurrent/decay_prep.cu", "recurrent/recurrent.cu",
+    "norm_rope/hyper_norm.cu", "norm_rope/post_norm.cu", "norm_rope/residual_norm.cu", "recurrent/decay_prep.cu", "recurrent/recurrent.cu",
     "sample/sampling.cu",
 ]
 
 # sources whose fp32 functions and divisions keep their full accuracy
-PRECISE_SOURCES = ["attn/latent_attn.cu", "attn/qk_norm_rope.cu", "gemm/gemm_simt.cu", "norm_rope/hyper_norm.cu",
-                   "recurrent/decay_prep.cu", "recurrent/recurrent.cu"]
+PRECISE_SOURCES = ["attn/latent_attn.cu", "attn/mixed_attn.cu", "attn/qk_norm_rope.cu", "gemm/gemm_simt.cu",
+                   "norm_rope/hyper_norm.cu", "norm_rope/post_norm.cu", "recurrent/decay_prep.cu", "recurrent/recurrent.cu"]
 
 
 def _nvcc() -> str:

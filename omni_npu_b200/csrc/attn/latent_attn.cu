@@ -1,6 +1,7 @@
 // Latent attention with run-time sizes: what stands around its attention kernels.
 //
-//   latent_prep     RMS norm of the latent, rotation of the shared key part and of the queries, cache row
+//   latent_prep     RMS norm of the latent, rotation of the shared key part and of the queries, cache row; RMS norm
+//                   of the queries' own latent
 //   head_gemm       out[t, h] = W[h] a[t, h] for few tokens (folding queries into the latent space and back)
 //   latent_gather   cached rows of all sequences of a step, one after another
 
@@ -14,9 +15,9 @@ namespace b200 {
 
 // ------------------------------------------------------------- norm, rotation, cache row
 struct LatentPrepParams {
-  void* q;                     // [T, H * (dim + rot)], rotated in place from row num_latent on
+  void* q;                     // [T, H * (dim + rot)], rotated in place from row num_latent on; or null
   long long q_stride;
-  const void* kv;              // [T, rank + rot]
+  const void* kv;              // [T, rank + rot], or null
   long long kv_stride;
   const void* norm_w;          // [rank]
   float eps;
@@ -26,6 +27,11 @@ struct LatentPrepParams {
   const float* cos_sin;        // [max_pos, rot]: cosines then sines
   int max_pos, H, dim, rot, rank, row, neox, num_latent;
   void* q_latent;              // [num_latent, H, row]: columns rank .. of a row take the rotated part
+  const void* low;             // [T, low_rank], normed into low_out [T, low_width] (zeros behind), or null
+  long long low_stride;
+  const void* low_w;
+  void* low_out;
+  int low_rank, low_width;
 };
 
 static constexpr int kLatentThreads = 256;
@@ -38,9 +44,27 @@ __device__ __forceinline__ void rotate_pair(const T* src, T* dst, int i, int hal
   dst[b] = from_float<T>(v * c + u * s);
 }
 
+// 1 / root mean square of a row, the same in every thread
+template <typename T>
+__device__ __forceinline__ float row_inv_rms(const T* x, int n, float eps, float* red) {
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < n; d += kLatentThreads) {
+    const float v = as_float(x[d]);
+    ss = fmaf(v, v, ss);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < kLatentThreads / 32; ++w) tot += red[w];
+  return 1.f / sqrtf(tot / static_cast<float>(n) + eps);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kLatentThreads) latent_prep_kernel(const LatentPrepParams p) {
-  __shared__ float red[kLatentThreads / 32];
+  __shared__ float red[2][kLatentThreads / 32];
   pdl_trigger();
   pdl_wait();
   const long long t = blockIdx.x;
@@ -49,27 +73,24 @@ __global__ void __launch_bounds__(kLatentThreads) latent_prep_kernel(const Laten
   const float* cs = p.cos_sin + static_cast<long long>(pos) * p.rot;
   const int half = p.rot >> 1, tid = threadIdx.x;
   const int slot = p.slots[t];
-  if (blockIdx.y == 0 && slot >= 0) {
+  if (p.kv && blockIdx.y == 0 && slot >= 0) {
     const T* kv = static_cast<const T*>(p.kv) + t * p.kv_stride;
-    float ss = 0.f;
-    for (int d = tid; d < p.rank; d += kLatentThreads) {
-      const float x = as_float(kv[d]);
-      ss = fmaf(x, x, ss);
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float tot = 0.f;
-#pragma unroll
-    for (int w = 0; w < kLatentThreads / 32; ++w) tot += red[w];
-    const float inv = 1.f / sqrtf(tot / static_cast<float>(p.rank) + p.eps);
+    const float inv = row_inv_rms(kv, p.rank, p.eps, red[0]);
     T* dst = static_cast<T*>(p.cache) + static_cast<long long>(slot) * p.row;
     const T* w = static_cast<const T*>(p.norm_w);
     for (int d = tid; d < p.rank; d += kLatentThreads) dst[d] = from_float<T>(as_float(kv[d]) * inv * as_float(w[d]));
     for (int i = tid; i < half; i += kLatentThreads) rotate_pair<T>(kv + p.rank, dst + p.rank, i, half, p.neox, cs);
     for (int d = p.rank + p.rot + tid; d < p.row; d += kLatentThreads) dst[d] = from_float<T>(0.f);
   }
+  if (p.low && blockIdx.y == gridDim.y - 1) {
+    const T* z = static_cast<const T*>(p.low) + t * p.low_stride;
+    const float inv = row_inv_rms(z, p.low_rank, p.eps, red[1]);
+    T* dst = static_cast<T*>(p.low_out) + t * p.low_width;
+    const T* w = static_cast<const T*>(p.low_w);
+    for (int d = tid; d < p.low_width; d += kLatentThreads)
+      dst[d] = from_float<T>(d < p.low_rank ? as_float(z[d]) * inv * as_float(w[d]) : 0.f);
+  }
+  if (p.q == nullptr) return;
   const bool fold = t < p.num_latent;
   const int total = p.H * half;
   for (int i = blockIdx.y * kLatentThreads + tid; i < total; i += gridDim.y * kLatentThreads) {
@@ -247,12 +268,16 @@ using namespace b200;
 extern "C" int b200_latent_prep(void* q, long long q_stride, const void* kv, long long kv_stride, const void* norm_w,
                                 float eps, void* cache, const int* positions, const int* slots, const float* cos_sin,
                                 int max_pos, int T, int H, int dim, int rot, int rank, int row, int neox,
-                                void* q_latent, int num_latent, int is_fp32, cudaStream_t stream) {
+                                void* q_latent, int num_latent, const void* low, long long low_stride,
+                                const void* low_w, void* low_out, int low_rank, int low_width, int is_fp32,
+                                cudaStream_t stream) {
   if (T <= 0) return 0;
   if ((rot & 1) || row < rank + rot || (num_latent > 0 && q_latent == nullptr)) return -1;
+  if (low != nullptr && (low_rank <= 0 || low_width < low_rank)) return -1;
   LatentPrepParams p{q, q_stride, kv, kv_stride, norm_w, eps, cache, positions, slots, cos_sin, max_pos,
-                     H, dim, rot, rank, row, neox, num_latent, q_latent};
-  int ny = (H * rot / 2 + 4 * kLatentThreads - 1) / (4 * kLatentThreads);
+                     H, dim, rot, rank, row, neox, num_latent, q_latent, low, low_stride, low_w, low_out, low_rank,
+                     low_width};
+  int ny = q ? (H * rot / 2 + 4 * kLatentThreads - 1) / (4 * kLatentThreads) : (kv && low ? 2 : 1);
   if (T >= 1024 || ny < 1) ny = 1;
   const dim3 grid(T, ny), block(kLatentThreads);
   const cudaError_t e = is_fp32 ? launch_pdl(latent_prep_kernel<float>, grid, block, 0, stream, 1, p)

@@ -1,0 +1,63 @@
+// Attention over the paged cache whose heads mix their scores before the softmax: the arguments its kernels share.
+//
+//   a_g  = scale * (q_g . k)                         of score head g and a key `dist` tokens back
+//   a_g <- softcap * tanh(a_g / softcap)             (softcap 0: none)
+//   a_g <- a_g - r1_g * ln(1 + r2_g * dist)          (r1 null: none)
+//   s_h  = sum_g talk[h, g] a_g                      for every output head h
+//   p_h  = exp(s_h) / (exp(sink_h) + sum exp(s_h))   over the keys at or before the query (sink null: plain softmax)
+//   out  = sum p_h v
+//
+// Score head g reads key head g / (Hs / Hk), output head h value head h / (Ho / Hv).  All of it is fp32 but the
+// products, whose operands may be bf16.  The cache rows are padded to DP / DVP elements; the padding holds zeros.
+#pragma once
+
+#include <cuda_bf16.h>
+#include <stdint.h>
+
+namespace b200 {
+
+struct MixedAttnParams {
+  const void* q;               // [T, Hs * D], row pitch q_stride
+  const void* k_cache;         // [blocks, Hk, block_size, DP]
+  const void* v_cache;         // [blocks, Hv, block_size, DVP]
+  void* out;                   // [T, >= Ho * DV], row pitch out_stride
+  const int* block_tables;     // [B, max_blocks]
+  const int* cu_q;             // [B + 1]; null: every sequence has q_len rows
+  const int* seq_lens;         // [B] keys including this step's
+  const float* r1;             // [Hs] or null
+  const float* r2;
+  const float* talk;           // [Ho, Hs]
+  const float* sink;           // [Ho] or null
+  int B, rows, q_len, max_blocks, block_size;
+  int bs_shift;                // log2(block_size), -1 when it is not a power of two
+  int Hs, Hk, Ho, Hv, D, DV, DP, DVP;
+  long long q_stride, out_stride;
+  float scale, softcap;
+  int splits;                  // decode: CTAs that share a row's keys
+  float* scratch;              // decode: [rows, splits, Ho, DVP + 2]; prompts: mixed scores, see pitch
+  // prompts: the query tiles of 16 rows tile0 .. tile0 + tiles - 1 of every sequence; their mixed scores (times
+  // log2 e) are [B, tiles, 16, Ho, pitch]
+  int tile0, tiles, max_q_len, max_keys;
+  long long pitch;
+};
+
+// Index of the key's row in a cache with `heads` heads.
+__device__ __forceinline__ long long cache_row(const MixedAttnParams& p, const int* bt, int key, int head, int heads) {
+  const int blk = p.bs_shift >= 0 ? key >> p.bs_shift : key / p.block_size;
+  const int off = p.bs_shift >= 0 ? key & (p.block_size - 1) : key - blk * p.block_size;
+  return (static_cast<long long>(bt[blk]) * heads + head) * p.block_size + off;
+}
+
+// The score of one head before the mixture, from the raw product; hardware exponentials and logarithms (absolute
+// errors of a few 1e-7 times softcap and r1).
+__device__ __forceinline__ float head_score(const MixedAttnParams& p, float x, float dist, float r1, float r2) {
+  if (p.softcap > 0.f) {
+    const float z = x * (p.scale / p.softcap);
+    x = p.softcap - __fdividef(2.f * p.softcap, __expf(2.f * z) + 1.f);
+  } else {
+    x *= p.scale;
+  }
+  return p.r1 ? x - r1 * __logf(fmaf(r2, dist, 1.f)) : x;
+}
+
+}  // namespace b200

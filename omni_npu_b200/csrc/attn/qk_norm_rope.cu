@@ -2,7 +2,9 @@
 //
 //   norm over the projection:  x <- x / sqrt(mean(x^2) + eps) * w over all rows of q (and of k) at once, then rotation
 //   norm per head:             rotation, then every head of q and k / sqrt(mean over the head + eps)
+//   weighted norm per head:    every head / sqrt(mean over the head + eps) * w, w shared by the heads, then rotation
 //   rotation:                  of the first `rot` dimensions of a head, i paired with i + rot / 2
+//   query temperature:         q at position p times 1 + c ln(floor((p + 1) / n) + 1)
 //   values:                    v, or (1 - lambda) v + lambda v_first with v_first those of another layer
 //
 // q goes to rows of its own, k and v into the paged cache (rows padded to DP / DVP, the padding is never
@@ -15,7 +17,7 @@
 
 namespace b200 {
 
-enum : int { kNormNone = 0, kNormProjection = 1, kNormHead = 2 };
+enum : int { kNormNone = 0, kNormProjection = 1, kNormHead = 2, kNormHeadWeight = 3 };
 
 struct QkNormParams {
   const void* q;
@@ -28,7 +30,7 @@ struct QkNormParams {
   const int* positions;
   const int* slots;            // < 0: nothing is stored
   const float* cos_sin;        // [max_pos, rot]: cosines then sines
-  const void* q_w;             // norm weights of the whole projections
+  const void* q_w;             // norm weights of the whole projections, or of a head
   const void* k_w;
   const float* sums;           // [T, 2] sums of squares of q and k over all ranks, or null: computed here
   int n_q, n_k;                // elements they stand for
@@ -36,6 +38,8 @@ struct QkNormParams {
   int lanes;                   // of a warp that share a head: a power of two
   long long q_stride, k_stride, v_stride, f_stride;
   float eps, lambda;
+  float temp;                  // c of the query temperature
+  int temp_every;              // n, 0: none
 };
 
 static constexpr int kQkThreads = 256, kQkWarps = kQkThreads / 32;
@@ -78,6 +82,9 @@ __global__ void __launch_bounds__(kQkThreads) qk_norm_rope_kernel(const QkNormPa
   int pos = p.positions[t];
   pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
   const float* cs = p.cos_sin + static_cast<long long>(pos) * p.rot;
+  constexpr bool WEIGHTS = NORM == kNormProjection || NORM == kNormHeadWeight;
+  const float heat =
+      p.temp_every > 0 ? 1.f + p.temp * logf(static_cast<float>((p.positions[t] + 1) / p.temp_every) + 1.f) : 1.f;
   float inv_q = 1.f, inv_k = 1.f;
   if constexpr (NORM == kNormProjection) {
     float sq, sk;
@@ -139,8 +146,9 @@ __global__ void __launch_bounds__(kQkThreads) qk_norm_rope_kernel(const QkNormPa
     T* dst = is_q ? static_cast<T*>(p.q_out) + (t * p.Hq + h) * p.D
                   : static_cast<T*>(p.k_cache) + ((blk * p.Hk + h) * p.block_size + off) * p.DP;
     float inv = is_q ? inv_q : inv_k;
-    const T* w = NORM == kNormProjection ? static_cast<const T*>(is_q ? p.q_w : p.k_w) + (head ? h * p.D : 0) : nullptr;
-    if constexpr (NORM == kNormHead) {                     // (a rotation leaves the sum of squares as it is)
+    const T* w = static_cast<const T*>(is_q ? p.q_w : p.k_w);
+    if (NORM == kNormProjection && head) w += h * p.D;
+    if constexpr (NORM == kNormHead || NORM == kNormHeadWeight) {    // (a rotation leaves the sum of squares as it is)
       float ss = 0.f;
       if (head)
         for (int d = li * W; d < p.D; d += p.lanes * W) {
@@ -153,10 +161,11 @@ __global__ void __launch_bounds__(kQkThreads) qk_norm_rope_kernel(const QkNormPa
       inv = 1.f / sqrtf(ss / static_cast<float>(p.D) + p.eps);
     }
     if (!head) continue;
+    if (is_q) inv *= heat;
     for (int d = li * W; d < p.D; d += p.lanes * W) {
       float x[W];
       load_w<T, W>(src, d, x);
-      if constexpr (NORM == kNormProjection) {
+      if constexpr (WEIGHTS) {
         float g[W];
         load_w<T, W>(w, d, g);
 #pragma unroll
@@ -169,7 +178,7 @@ __global__ void __launch_bounds__(kQkThreads) qk_norm_rope_kernel(const QkNormPa
         load_w<T, W>(src, lo ? d + half : a, y);
         load_w<float, W>(cs, a, c);
         load_w<float, W>(cs + half, a, s);
-        if constexpr (NORM == kNormProjection) {
+        if constexpr (WEIGHTS) {
           float g[W];
           load_w<T, W>(w, lo ? d + half : a, g);
 #pragma unroll
@@ -178,10 +187,8 @@ __global__ void __launch_bounds__(kQkThreads) qk_norm_rope_kernel(const QkNormPa
 #pragma unroll
         for (int j = 0; j < W; ++j) x[j] = x[j] * c[j] + (lo ? -y[j] : y[j]) * s[j];
       }
-      if constexpr (NORM != kNormNone) {
 #pragma unroll
-        for (int j = 0; j < W; ++j) x[j] *= inv;
-      }
+      for (int j = 0; j < W; ++j) x[j] *= inv;
       store_w<T, W>(dst, d, x);
     }
   }
@@ -192,6 +199,7 @@ static cudaError_t launch_qk(const QkNormParams& p, int norm, dim3 grid, cudaStr
   const dim3 block(kQkThreads);
   if (norm == kNormProjection) return launch_pdl(qk_norm_rope_kernel<T, W, kNormProjection>, grid, block, 0, stream, 1, p);
   if (norm == kNormHead) return launch_pdl(qk_norm_rope_kernel<T, W, kNormHead>, grid, block, 0, stream, 1, p);
+  if (norm == kNormHeadWeight) return launch_pdl(qk_norm_rope_kernel<T, W, kNormHeadWeight>, grid, block, 0, stream, 1, p);
   return launch_pdl(qk_norm_rope_kernel<T, W, kNormNone>, grid, block, 0, stream, 1, p);
 }
 
@@ -204,10 +212,11 @@ extern "C" int b200_qk_norm_rope(const void* q, const void* k, const void* v, co
                                  const float* cos_sin, int max_pos, int norm, const void* q_w, const void* k_w,
                                  const float* sums, int n_q, int n_k, float eps, float lambda, int T, int Hq, int Hk,
                                  int D, int DV, int DP, int DVP, int rot, long long q_stride, long long k_stride,
-                                 long long v_stride, long long f_stride, int block_size, int is_fp32,
-                                 cudaStream_t stream) {
+                                 long long v_stride, long long f_stride, int block_size, float temp, int temp_every,
+                                 int is_fp32, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (rot < 0 || rot > D || (rot & 1) || DP < D || DVP < DV || norm < 0 || norm > 2) return -1;
+  if (rot < 0 || rot > D || (rot & 1) || DP < D || DVP < DV || norm < 0 || norm > 3 || temp_every < 0) return -1;
+  if (rot > 0 && cos_sin == nullptr) return -1;
   const uintptr_t align = is_fp32 ? 15 : 7;
   const auto ok = [&](const void* ptr, long long stride) {
     return (reinterpret_cast<uintptr_t>(ptr) & align) == 0 && stride % 4 == 0;
@@ -218,7 +227,7 @@ extern "C" int b200_qk_norm_rope(const void* q, const void* k, const void* v, co
   int lanes = 1;
   while (lanes < 32 && lanes * (vec ? 4 : 1) < D) lanes <<= 1;
   QkNormParams p{q, k, v, v_first, q_out, k_cache, v_cache, positions, slots, cos_sin, q_w, k_w, sums, n_q, n_k, Hq, Hk,
-                 D, DV, DP, DVP, rot, block_size, max_pos, lanes, q_stride, k_stride, v_stride, f_stride, eps, lambda};
+                 D, DV, DP, DVP, rot, block_size, max_pos, lanes, q_stride, k_stride, v_stride, f_stride, eps, lambda, temp, temp_every};
   const int per_cta = kQkWarps * (32 / lanes);
   int ny = (Hq + 2 * Hk + per_cta - 1) / per_cta;
   if (T >= 256) ny = 1;                                   // enough tokens: longer CTAs

@@ -82,12 +82,27 @@ int b200_qk_norm_rope(const void* q, const void* k, const void* v, const void* v
                       void* v_cache, const int* positions, const int* slots, const float* cos_sin, int max_pos, int norm,
                       const void* q_w, const void* k_w, const float* sums, int n_q, int n_k, float eps, float lambda,
                       int T, int Hq, int Hk, int D, int DV, int DP, int DVP, int rot, long long q_stride,
-                      long long k_stride, long long v_stride, long long f_stride, int block_size, int is_fp32,
-                      cudaStream_t stream);
+                      long long k_stride, long long v_stride, long long f_stride, int block_size, float temp, int temp_every,
+                      int is_fp32, cudaStream_t stream);
 int b200_latent_prep(void* q, long long q_stride, const void* kv, long long kv_stride, const void* norm_w, float eps,
                      void* cache, const int* positions, const int* slots, const float* cos_sin, int max_pos, int T,
-                     int H, int dim, int rot, int rank, int row, int neox, void* q_latent, int num_latent, int is_fp32,
+                     int H, int dim, int rot, int rank, int row, int neox, void* q_latent, int num_latent, const void* low,
+                     long long low_stride, const void* low_w, void* low_out, int low_rank, int low_width, int is_fp32,
                      cudaStream_t stream);
+int b200_mixed_attention_kind(int Hs, int Hk, int Ho, int Hv, int DP, int DVP, int prompt, int is_fp32);
+int b200_mixed_attention(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_tables,
+                         const int* cu_q, const int* seq_lens, const float* r1, const float* r2, const float* talk,
+                         const float* sink, int B, int rows, int q_len, int max_keys, int max_blocks, int block_size,
+                         int Hs, int Hk, int Ho, int Hv, int D, int DV, int DP, int DVP, long long q_stride,
+                         long long out_stride, float scale, float softcap, int kind, int splits, float* scratch, int tile0,
+                         int tiles, long long pitch, int is_fp32, cudaStream_t stream);
+int b200_post_norm_residual(float* residual, long long res_stride, const int* ids, const void* table, int table_rows,
+                            const void* y, long long y_stride, const void* w, int groups, const void* out_w,
+                            int out_groups, void* out, long long out_stride, float eps, long long rows, int W, int n_true,
+                            int is_fp32, cudaStream_t stream);
+int b200_gelu_rows(const void* z, long long z_stride, const int* ids, const void* table, int table_rows,
+                   long long table_stride, int offset, int dim, int width, void* out, int T, int is_fp32,
+                   cudaStream_t stream);
 int b200_head_gemm(const void* a, long long a_t, long long a_h, const void* w, void* out, long long o_t, long long o_h,
                    int T, int H, int N, int K, int is_fp32, cudaStream_t stream);
 int b200_latent_gather(const void* cache, void* out, const int* block_tables, const int* seq_lens, const int* start,
@@ -101,8 +116,8 @@ int b200_latent_decode(const void* q, const void* cache, void* out, const int* b
 
 namespace {
 
-// Activation kinds of the GEMM epilogues are those of gemm/gated_act.cuh; 1, 2 and 4 join pairs of columns.
-inline bool gated(int64_t act) { return act == 1 || act == 2 || act == 4; }
+// Activation kinds of the GEMM epilogues are those of gemm/gated_act.cuh; 1, 2, 4 and 7 join pairs of columns.
+inline bool gated(int64_t act) { return act == 1 || act == 2 || act == 4 || act == 7; }
 
 // (BN, splits, workspace bytes, counters, cluster flag) for a problem.
 std::tuple<int64_t, int64_t, int64_t, int64_t, int64_t> gemm_plan(int64_t M, int64_t N, int64_t K,
@@ -737,9 +752,10 @@ std::tuple<Tensor, Tensor, Tensor, Tensor> decay_prep(const Tensor& q, const Ten
 // were taken elsewhere), 2 per head.  Returns the queries [T, Hq * D].
 Tensor qk_norm_rope(const Tensor& q, const Tensor& k, const Tensor& v, const c10::optional<Tensor>& v_first,
                     double lambda, Tensor k_cache, Tensor v_cache, const Tensor& positions, const Tensor& slots,
-                    const Tensor& cos_sin, int64_t head_dim, int64_t head_dim_v, int64_t rot, int64_t norm,
+                    const c10::optional<Tensor>& cos_sin, int64_t head_dim, int64_t head_dim_v, int64_t rot, int64_t norm,
                     const c10::optional<Tensor>& q_w, const c10::optional<Tensor>& k_w,
-                    const c10::optional<Tensor>& sums, int64_t n_q, int64_t n_k, double eps) {
+                    const c10::optional<Tensor>& sums, int64_t n_q, int64_t n_k, double eps,
+                    double temp, int64_t temp_every) {
   const auto dt = q.scalar_type();
   const bool f32 = is_f32(q);
   CHECK_ROWS(q, dt);
@@ -751,18 +767,25 @@ Tensor qk_norm_rope(const Tensor& q, const Tensor& k, const Tensor& v, const c10
   const int T = q.size(0), Hk = k_cache.size(1);
   TORCH_CHECK(positions.numel() >= T && slots.numel() >= T && q.size(1) % head_dim == 0 && k.size(0) == T &&
                   v.size(0) == T && k.size(1) == Hk * head_dim && v.size(1) == Hk * head_dim_v, "qk_norm_rope: shapes");
-  TORCH_CHECK(cos_sin.is_cuda() && cos_sin.scalar_type() == at::kFloat && cos_sin.is_contiguous() &&
-                  cos_sin.dim() == 2 && cos_sin.size(1) == rot, "qk_norm_rope: cos_sin [max_pos, rot] fp32");
+  const float* cs = nullptr;
+  int max_pos = 1 << 30;
+  if (cos_sin.has_value()) {
+    TORCH_CHECK(cos_sin->is_cuda() && cos_sin->scalar_type() == at::kFloat && cos_sin->is_contiguous() &&
+                    cos_sin->dim() == 2 && cos_sin->size(1) == rot, "qk_norm_rope: cos_sin [max_pos, rot] fp32");
+    cs = cos_sin->data_ptr<float>();
+    max_pos = (int)cos_sin->size(0);
+  }
+  TORCH_CHECK(cs || rot == 0, "qk_norm_rope: a rotation needs cos_sin");
   const void *qw = nullptr, *kw = nullptr, *vf = nullptr;
   const float* sp = nullptr;
   long long fs = 0;
-  if (norm == 1) {
+  if (norm == 1 || norm == 3) {
     TORCH_CHECK(q_w.has_value() && k_w.has_value(), "qk_norm_rope: norm weights");
-    CHECK_VEC(*q_w, dt, q.size(1));
-    CHECK_VEC(*k_w, dt, k.size(1));
+    CHECK_VEC(*q_w, dt, norm == 1 ? q.size(1) : head_dim);
+    CHECK_VEC(*k_w, dt, norm == 1 ? k.size(1) : head_dim);
     qw = q_w->data_ptr();
     kw = k_w->data_ptr();
-    if (sums.has_value()) {
+    if (norm == 1 && sums.has_value()) {
       CHECK_F32(*sums);
       TORCH_CHECK(sums->numel() == 2 * T, "qk_norm_rope: sums [T, 2]");
       sp = sums->data_ptr<float>();
@@ -777,45 +800,199 @@ Tensor qk_norm_rope(const Tensor& q, const Tensor& k, const Tensor& v, const c10
   c10::cuda::CUDAGuard guard(q.device());
   Tensor out = torch::empty({T, q.size(1)}, q.options());
   check(b200_qk_norm_rope(q.data_ptr(), k.data_ptr(), v.data_ptr(), vf, out.data_ptr(), k_cache.data_ptr(),
-                          v_cache.data_ptr(), positions.data_ptr<int>(), slots.data_ptr<int>(), cos_sin.data_ptr<float>(),
-                          (int)cos_sin.size(0), (int)norm, qw, kw, sp, (int)n_q, (int)n_k, (float)eps, (float)lambda, T,
+                          v_cache.data_ptr(), positions.data_ptr<int>(), slots.data_ptr<int>(), cs, max_pos, (int)norm, qw, kw, sp, (int)n_q, (int)n_k, (float)eps, (float)lambda, T,
                           (int)(q.size(1) / head_dim), Hk, (int)head_dim, (int)head_dim_v, (int)k_cache.size(3),
                           (int)v_cache.size(3), (int)rot, q.stride(0), k.stride(0), v.stride(0), fs,
-                          (int)k_cache.size(2), f32 ? 1 : 0, cur_stream()),
+                          (int)k_cache.size(2), (float)temp, (int)temp_every, f32 ? 1 : 0, cur_stream()),
         "qk_norm_rope");
   return out;
 }
 
-void latent_prep(Tensor q, const Tensor& kv, const Tensor& norm_w, double eps, Tensor cache, const Tensor& positions,
-                 const Tensor& slots, const Tensor& cos_sin, int64_t heads, int64_t dim, int64_t rot, int64_t rank,
-                 bool neox, const c10::optional<Tensor>& q_latent, int64_t num_latent) {
-  const auto dt = q.scalar_type();
-  const bool f32 = is_f32(q);
-  CHECK_ROWS(q, dt);
-  CHECK_ROWS(kv, dt);
-  CHECK_VEC(norm_w, dt, rank);
+void latent_prep(const c10::optional<Tensor>& q, const c10::optional<Tensor>& kv, const c10::optional<Tensor>& norm_w,
+                 double eps, Tensor cache, const Tensor& positions, const Tensor& slots, const Tensor& cos_sin,
+                 int64_t heads, int64_t dim, int64_t rot, int64_t rank, bool neox, const c10::optional<Tensor>& q_latent,
+                 int64_t num_latent, const c10::optional<Tensor>& low, const c10::optional<Tensor>& low_w,
+                 const c10::optional<Tensor>& low_out) {
+  const auto dt = cache.scalar_type();
+  const bool f32 = is_f32(cache);
   CHECK_I32(positions);
   CHECK_I32(slots);
-  const int64_t T = q.size(0);
-  TORCH_CHECK(cache.is_cuda() && cache.scalar_type() == dt && cache.is_contiguous() && cache.dim() == 3,
+  TORCH_CHECK(q.has_value() || kv.has_value() || low.has_value(), "latent_prep: nothing to do");
+  const int64_t T = q.has_value() ? q->size(0) : kv.has_value() ? kv->size(0) : low->size(0);
+  TORCH_CHECK(cache.is_cuda() && cache.is_contiguous() && cache.dim() == 3 && cache.size(2) >= rank + rot,
               "latent_prep: cache [blocks, block_size, row]");
-  TORCH_CHECK(q.size(1) >= heads * (dim + rot) && kv.size(0) == T && kv.size(1) >= rank + rot &&
-                  cache.size(2) >= rank + rot && positions.numel() >= T && slots.numel() >= T, "latent_prep: shapes");
+  TORCH_CHECK(positions.numel() >= T && slots.numel() >= T, "latent_prep: positions, slots [T]");
   TORCH_CHECK(cos_sin.is_cuda() && cos_sin.scalar_type() == at::kFloat && cos_sin.is_contiguous() &&
                   cos_sin.dim() == 2 && cos_sin.size(1) == rot, "latent_prep: cos_sin [max_pos, rot] fp32");
-  void* ql = nullptr;
-  if (num_latent > 0) {
+  void *qp = nullptr, *ql = nullptr, *lo = nullptr;
+  const void *kvp = nullptr, *nw = nullptr, *lp = nullptr, *lw = nullptr;
+  long long qs = 0, kvs = 0, ls = 0;
+  int low_rank = 0, low_width = 0;
+  if (q.has_value()) {
+    CHECK_ROWS(*q, dt);
+    TORCH_CHECK(q->size(1) >= heads * (dim + rot), "latent_prep: q [T, heads * (dim + rot)]");
+    qp = q->data_ptr();
+    qs = q->stride(0);
+  }
+  if (kv.has_value()) {
+    CHECK_ROWS(*kv, dt);
+    TORCH_CHECK(kv->size(0) == T && kv->size(1) >= rank + rot && norm_w.has_value(), "latent_prep: kv [T, rank + rot]");
+    CHECK_VEC(*norm_w, dt, rank);
+    kvp = kv->data_ptr();
+    nw = norm_w->data_ptr();
+    kvs = kv->stride(0);
+  }
+  if (low.has_value()) {
+    CHECK_ROWS(*low, dt);
+    TORCH_CHECK(low_w.has_value() && low_out.has_value(), "latent_prep: weight and result of the queries' latent");
+    low_rank = (int)low_w->numel();
+    CHECK_VEC(*low_w, dt, low_rank);
+    TORCH_CHECK(low_out->is_cuda() && low_out->scalar_type() == dt && low_out->is_contiguous() && low_out->dim() == 2 &&
+                    low_out->size(0) == T && low_out->size(1) >= low_rank && low->size(0) == T &&
+                    low->size(1) >= low_rank, "latent_prep: queries' latent [T, n]");
+    low_width = (int)low_out->size(1);
+    lp = low->data_ptr();
+    lw = low_w->data_ptr();
+    lo = low_out->data_ptr();
+    ls = low->stride(0);
+  }
+  if (num_latent > 0 && q.has_value()) {
     TORCH_CHECK(q_latent.has_value() && q_latent->is_cuda() && q_latent->scalar_type() == dt &&
                     q_latent->is_contiguous() && q_latent->dim() == 3 && q_latent->size(0) >= num_latent &&
                     q_latent->size(1) == heads && q_latent->size(2) == cache.size(2), "latent_prep: q_latent");
     ql = q_latent->data_ptr();
+  } else {
+    num_latent = 0;
+  }
+  c10::cuda::CUDAGuard guard(cache.device());
+  check(b200_latent_prep(qp, qs, kvp, kvs, nw, (float)eps, cache.data_ptr(), positions.data_ptr<int>(),
+                         slots.data_ptr<int>(), cos_sin.data_ptr<float>(), (int)cos_sin.size(0), (int)T, (int)heads,
+                         (int)dim, (int)rot, (int)rank, (int)cache.size(2), neox ? 1 : 0, ql, (int)num_latent, lp, ls, lw,
+                         lo, low_rank, low_width, f32 ? 1 : 0, cur_stream()),
+        "latent_prep");
+}
+
+// 0: the plain kernel, 1: the tensor-core kernels; variant 2 asks for the plain one, 1 for an error instead of it
+int64_t mixed_attention_kind(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& talk, bool prompt,
+                             int64_t variant) {
+  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && talk.dim() == 2, "mixed_attention: shapes");
+  const int kind = variant == 2 ? 0
+                                : b200_mixed_attention_kind((int)talk.size(1), (int)k_cache.size(1), (int)talk.size(0),
+                                                            (int)v_cache.size(1), (int)k_cache.size(3),
+                                                            (int)v_cache.size(3), prompt ? 1 : 0, is_f32(q) ? 1 : 0);
+  TORCH_CHECK(kind || variant != 1, "mixed_attention: these sizes are beyond the tensor-core kernels");
+  return kind;
+}
+
+// out [T, >= Ho * Dv].  kind 1: `scratch` holds the partial results of a split decode row, or the mixed scores of the
+// query tiles tile0 .. tile0 + tiles - 1 of every portion.
+void mixed_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, Tensor out, const Tensor& block_tables,
+                     const c10::optional<Tensor>& cu_q, const Tensor& seq_lens, int64_t num_seqs, int64_t q_len,
+                     int64_t max_keys, int64_t head_dim, int64_t head_dim_v, double scale, double softcap,
+                     const c10::optional<Tensor>& r1, const c10::optional<Tensor>& r2, const Tensor& talk,
+                     const c10::optional<Tensor>& sink, int64_t kind, int64_t splits, const c10::optional<Tensor>& scratch,
+                     int64_t tile0, int64_t tiles) {
+  const auto dt = q.scalar_type();
+  const bool f32 = is_f32(q);
+  CHECK_ROWS(q, dt);
+  CHECK_ROWS(out, dt);
+  for (const Tensor& c : {k_cache, v_cache})
+    TORCH_CHECK(c.is_cuda() && c.scalar_type() == dt && c.dim() == 4 && c.is_contiguous() &&
+                    c.size(0) == k_cache.size(0) && c.size(2) == k_cache.size(2),
+                "mixed_attention: caches [blocks, heads, block_size, width]");
+  const int64_t T = q.size(0), Hs = talk.size(1), Ho = talk.size(0);
+  TORCH_CHECK(k_cache.size(3) >= head_dim && v_cache.size(3) >= head_dim_v && q.size(1) == Hs * head_dim &&
+                  out.size(0) == T && out.size(1) >= Ho * head_dim_v, "mixed_attention: shapes");
+  TORCH_CHECK(block_tables.is_cuda() && block_tables.scalar_type() == at::kInt && block_tables.dim() == 2 &&
+                  block_tables.stride(1) == 1 && block_tables.size(0) >= num_seqs, "mixed_attention: block tables");
+  CHECK_I32(seq_lens);
+  TORCH_CHECK(seq_lens.numel() >= num_seqs, "mixed_attention: sequences");
+  const auto vec = [&](const c10::optional<Tensor>& t, int64_t n) -> const float* {
+    if (!t.has_value()) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kFloat && t->is_contiguous() && t->numel() == n,
+                "mixed_attention: fp32 constants per head");
+    return t->data_ptr<float>();
+  };
+  const float *p1 = vec(r1, Hs), *p2 = vec(r2, Hs), *ps = vec(sink, Ho), *pt = vec(talk, Ho * Hs);
+  TORCH_CHECK((p1 == nullptr) == (p2 == nullptr), "mixed_attention: r1 and r2 go together");
+  const int* cu = nullptr;
+  if (cu_q.has_value()) {
+    CHECK_I32(*cu_q);
+    TORCH_CHECK(cu_q->numel() >= num_seqs + 1, "mixed_attention: cu_q [B + 1]");
+    cu = cu_q->data_ptr<int>();
+  } else {
+    TORCH_CHECK(T == num_seqs * q_len, "mixed_attention: rows");
+  }
+  const int64_t pitch = (max_keys + 63) / 64 * 64;
+  float* sp = nullptr;
+  if (scratch.has_value()) {
+    const int64_t need = cu ? num_seqs * tiles * 16 * Ho * pitch : T * splits * Ho * (v_cache.size(3) + 2);
+    TORCH_CHECK(scratch->is_cuda() && scratch->is_contiguous() && (int64_t)scratch->nbytes() >= need * 4,
+                "mixed_attention: scratch");
+    sp = static_cast<float*>(scratch->data_ptr());
   }
   c10::cuda::CUDAGuard guard(q.device());
-  check(b200_latent_prep(q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), norm_w.data_ptr(), (float)eps,
-                         cache.data_ptr(), positions.data_ptr<int>(), slots.data_ptr<int>(), cos_sin.data_ptr<float>(),
-                         (int)cos_sin.size(0), (int)T, (int)heads, (int)dim, (int)rot, (int)rank, (int)cache.size(2),
-                         neox ? 1 : 0, ql, (int)num_latent, f32 ? 1 : 0, cur_stream()),
-        "latent_prep");
+  check(b200_mixed_attention(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
+                             block_tables.data_ptr<int>(), cu, seq_lens.data_ptr<int>(), p1, p2, pt, ps, (int)num_seqs,
+                             (int)T, (int)q_len, (int)max_keys, (int)block_tables.stride(0), (int)k_cache.size(2), (int)Hs,
+                             (int)k_cache.size(1), (int)Ho, (int)v_cache.size(1), (int)head_dim, (int)head_dim_v,
+                             (int)k_cache.size(3), (int)v_cache.size(3), q.stride(0), out.stride(0), (float)scale,
+                             (float)softcap, (int)kind, (int)splits, sp, (int)tile0, (int)tiles, pitch, f32 ? 1 : 0,
+                             cur_stream()),
+        "mixed_attention");
+}
+
+Tensor post_norm_residual(Tensor residual, const c10::optional<Tensor>& y, const c10::optional<Tensor>& w, int64_t groups,
+                          double eps, int64_t true_width, const c10::optional<Tensor>& ids,
+                          const c10::optional<Tensor>& table, const c10::optional<Tensor>& out_w, int64_t out_groups) {
+  CHECK_ROWS(residual, at::kFloat);
+  const int64_t T = residual.size(0), W = residual.size(1);
+  const bool start = ids.has_value();
+  TORCH_CHECK(start ? table.has_value() : y.has_value() && w.has_value(), "post_norm_residual: ids and table, or y and w");
+  const Tensor& like = start ? *table : *y;
+  const auto dt = like.scalar_type();
+  const bool f32 = is_f32(like);
+  CHECK_ROWS(like, dt);
+  TORCH_CHECK(like.size(1) == W && (reinterpret_cast<uintptr_t>(like.data_ptr()) & 15) == 0, "post_norm_residual: rows [W]");
+  const int* idp = nullptr;
+  const void *wp = nullptr, *owp = nullptr;
+  if (start) {
+    CHECK_I32(*ids);
+    TORCH_CHECK(ids->numel() >= T && like.is_contiguous(), "post_norm_residual: ids [T], table [rows, W]");
+    idp = ids->data_ptr<int>();
+  } else {
+    TORCH_CHECK(like.size(0) == T, "post_norm_residual: y [T, W]");
+    CHECK_VEC(*w, dt, W);
+    wp = w->data_ptr();
+  }
+  if (out_w.has_value()) {
+    CHECK_VEC(*out_w, dt, W);
+    owp = out_w->data_ptr();
+  }
+  c10::cuda::CUDAGuard guard(residual.device());
+  Tensor out = torch::empty({T, W}, like.options());
+  check(b200_post_norm_residual(residual.data_ptr<float>(), residual.stride(0), idp, start ? like.data_ptr() : nullptr,
+                                start ? (int)like.size(0) : 0, start ? nullptr : like.data_ptr(),
+                                start ? 0 : like.stride(0), wp, (int)groups, owp, (int)out_groups, out.data_ptr(), W,
+                                (float)eps, T, (int)W, (int)true_width, f32 ? 1 : 0, cur_stream()),
+        "post_norm_residual");
+  return out;
+}
+
+Tensor gelu_rows(const Tensor& z, const Tensor& ids, const Tensor& table, int64_t offset, int64_t dim) {
+  const auto dt = z.scalar_type();
+  const bool f32 = is_f32(z);
+  CHECK_ROWS(z, dt);
+  CHECK_ROWS(table, dt);
+  CHECK_I32(ids);
+  TORCH_CHECK(ids.numel() >= z.size(0) && z.size(1) >= dim && table.is_contiguous() && offset >= 0 &&
+                  offset + dim <= table.size(1) && (reinterpret_cast<uintptr_t>(z.data_ptr()) & 15) == 0, "gelu_rows: shapes");
+  c10::cuda::CUDAGuard guard(z.device());
+  Tensor out = torch::empty({z.size(0), z.size(1)}, z.options());
+  check(b200_gelu_rows(z.data_ptr(), z.stride(0), ids.data_ptr<int>(), table.data_ptr(), (int)table.size(0), table.stride(0),
+                       (int)offset, (int)dim, (int)z.size(1), out.data_ptr(), (int)z.size(0), f32 ? 1 : 0, cur_stream()),
+        "gelu_rows");
+  return out;
 }
 
 void head_gemm(const Tensor& a, const Tensor& w, Tensor out) {
@@ -902,6 +1079,10 @@ TORCH_LIBRARY(omni_b200, m) {
   m.def("decay_prep", &decay_prep);
   m.def("qk_norm_rope", &qk_norm_rope);
   m.def("latent_prep", &latent_prep);
+  m.def("mixed_attention_kind", &mixed_attention_kind);
+  m.def("mixed_attention", &mixed_attention);
+  m.def("post_norm_residual", &post_norm_residual);
+  m.def("gelu_rows", &gelu_rows);
   m.def("head_gemm", &head_gemm);
   m.def("latent_gather", &latent_gather);
   m.def("latent_decode_scratch_bytes", &latent_decode_scratch_bytes);

@@ -7,11 +7,13 @@
 
 namespace b200 {
 
-enum : int { kActNone = 0, kActSilu = 1, kActClampedGlu = 2, kActXielu = 3, kActGeluTanh = 4, kActRelu2 = 5, kActTanh = 6 };
+enum : int { kActNone = 0, kActSilu = 1, kActClampedGlu = 2, kActXielu = 3, kActGeluTanh = 4, kActRelu2 = 5, kActTanh = 6,
+             kActReluGate = 7 };
 
 //   kActSilu        silu(g) * u
 //   kActClampedGlu  g' * sigmoid(alpha * g') * (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
 //   kActGeluTanh    g / 2 * (1 + tanh(z)) * u = g * sigmoid(2 z) * u with z = sqrt(2 / pi) (g + 0.044715 g^3)
+//   kActReluGate    max(g, 0) * u
 __device__ __forceinline__ float gelu_exponent(float g) {
   return -1.5957691216057308f * fmaf(0.044715f * g * g, g, g);       // -2 z
 }
@@ -21,6 +23,7 @@ __device__ __forceinline__ float gated_act(int kind, float g, float u, float alp
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + __expf(-alpha * g)) * (u + 1.f);
   }
+  if (kind == kActReluGate) return fmaxf(g, 0.f) * u;
   return g / (1.f + __expf(kind == kActGeluTanh ? gelu_exponent(g) : -g)) * u;
 }
 // the same with the exact fp32 functions, for products that are not rounded to bf16
@@ -30,6 +33,7 @@ __device__ __forceinline__ float gated_act_exact(int kind, float g, float u, flo
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + expf(-alpha * g)) * (u + 1.f);
   }
+  if (kind == kActReluGate) return fmaxf(g, 0.f) * u;
   return g / (1.f + expf(kind == kActGeluTanh ? gelu_exponent(g) : -g)) * u;
 }
 
@@ -88,7 +92,7 @@ __device__ __forceinline__ void add_bias16(float (&v)[16], const __nv_bfloat16* 
 
 // Whether a kind joins pairs of columns (half as many come out), or works on single ones.
 __host__ __device__ __forceinline__ bool act_is_gated(int kind) {
-  return kind == kActSilu || kind == kActClampedGlu || kind == kActGeluTanh;
+  return kind == kActSilu || kind == kActClampedGlu || kind == kActGeluTanh || kind == kActReluGate;
 }
 __host__ __device__ __forceinline__ bool act_is_unary(int kind) {
   return kind == kActXielu || kind == kActRelu2 || kind == kActTanh;

@@ -26,7 +26,7 @@ struct QkNormParams {
   const void* v_first;         // or null
   void* q_out;                 // [T, Hq * D]
   void* k_cache;               // [blocks, Hk, block_size, DP]
-  void* v_cache;               // [blocks, Hk, block_size, DVP]
+  void* v_cache;               // [blocks, Hv, block_size, DVP]
   const int* positions;
   const int* slots;            // < 0: nothing is stored
   const float* cos_sin;        // [max_pos, rot]: cosines then sines
@@ -34,7 +34,7 @@ struct QkNormParams {
   const void* k_w;
   const float* sums;           // [T, 2] sums of squares of q and k over all ranks, or null: computed here
   int n_q, n_k;                // elements they stand for
-  int Hq, Hk, D, DV, DP, DVP, rot, block_size, max_pos;
+  int Hq, Hk, Hv, D, DV, DP, DVP, rot, block_size, max_pos;
   int lanes;                   // of a warp that share a head: a power of two
   long long q_stride, k_stride, v_stride, f_stride;
   float eps, lambda;
@@ -116,7 +116,7 @@ __global__ void __launch_bounds__(kQkThreads) qk_norm_rope_kernel(const QkNormPa
   }
   const long long blk = slot < 0 ? 0 : slot / p.block_size, off = slot < 0 ? 0 : slot % p.block_size;
   const int half = p.rot >> 1, per_warp = 32 / p.lanes, li = lane & (p.lanes - 1);
-  const int units = slot < 0 ? p.Hq : p.Hq + 2 * p.Hk;
+  const int units = slot < 0 ? p.Hq : p.Hq + p.Hk + p.Hv;
   const int step = gridDim.y * kQkWarps * per_warp;
   const int base = (blockIdx.y * kQkWarps + warp) * per_warp;
   for (int u0 = base; u0 < units; u0 += step) {            // (warp-uniform)
@@ -124,7 +124,7 @@ __global__ void __launch_bounds__(kQkThreads) qk_norm_rope_kernel(const QkNormPa
     const bool live = unit < units;
     if (live && unit >= p.Hq + p.Hk) {                     // a value head
       const int h = unit - p.Hq - p.Hk;
-      T* dst = static_cast<T*>(p.v_cache) + ((blk * p.Hk + h) * p.block_size + off) * p.DVP;
+      T* dst = static_cast<T*>(p.v_cache) + ((blk * p.Hv + h) * p.block_size + off) * p.DVP;
       const T* src = v + h * p.DV;
       const T* first = p.v_first ? static_cast<const T*>(p.v_first) + t * p.f_stride + h * p.DV : nullptr;
       for (int d = li * W; d < p.DV; d += p.lanes * W) {
@@ -210,7 +210,7 @@ using namespace b200;
 extern "C" int b200_qk_norm_rope(const void* q, const void* k, const void* v, const void* v_first, void* q_out,
                                  void* k_cache, void* v_cache, const int* positions, const int* slots,
                                  const float* cos_sin, int max_pos, int norm, const void* q_w, const void* k_w,
-                                 const float* sums, int n_q, int n_k, float eps, float lambda, int T, int Hq, int Hk,
+                                 const float* sums, int n_q, int n_k, float eps, float lambda, int T, int Hq, int Hk, int Hv,
                                  int D, int DV, int DP, int DVP, int rot, long long q_stride, long long k_stride,
                                  long long v_stride, long long f_stride, int block_size, float temp, int temp_every,
                                  int is_fp32, cudaStream_t stream) {
@@ -226,10 +226,10 @@ extern "C" int b200_qk_norm_rope(const void* q, const void* k, const void* v, co
                    ok(k_w, 0) && (reinterpret_cast<uintptr_t>(cos_sin) & 15) == 0;
   int lanes = 1;
   while (lanes < 32 && lanes * (vec ? 4 : 1) < D) lanes <<= 1;
-  QkNormParams p{q, k, v, v_first, q_out, k_cache, v_cache, positions, slots, cos_sin, q_w, k_w, sums, n_q, n_k, Hq, Hk,
+  QkNormParams p{q, k, v, v_first, q_out, k_cache, v_cache, positions, slots, cos_sin, q_w, k_w, sums, n_q, n_k, Hq, Hk, Hv,
                  D, DV, DP, DVP, rot, block_size, max_pos, lanes, q_stride, k_stride, v_stride, f_stride, eps, lambda, temp, temp_every};
   const int per_cta = kQkWarps * (32 / lanes);
-  int ny = (Hq + 2 * Hk + per_cta - 1) / per_cta;
+  int ny = (Hq + Hk + Hv + per_cta - 1) / per_cta;
   if (T >= 256) ny = 1;                                   // enough tokens: longer CTAs
   const dim3 grid(T, ny);
   cudaError_t e;

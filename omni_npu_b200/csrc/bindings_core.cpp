@@ -81,7 +81,7 @@ int b200_decay_prep(const void* q, long long q_stride, const void* k, long long 
 int b200_qk_norm_rope(const void* q, const void* k, const void* v, const void* v_first, void* q_out, void* k_cache,
                       void* v_cache, const int* positions, const int* slots, const float* cos_sin, int max_pos, int norm,
                       const void* q_w, const void* k_w, const float* sums, int n_q, int n_k, float eps, float lambda,
-                      int T, int Hq, int Hk, int D, int DV, int DP, int DVP, int rot, long long q_stride,
+                      int T, int Hq, int Hk, int Hv, int D, int DV, int DP, int DVP, int rot, long long q_stride,
                       long long k_stride, long long v_stride, long long f_stride, int block_size, float temp, int temp_every,
                       int is_fp32, cudaStream_t stream);
 int b200_latent_prep(void* q, long long q_stride, const void* kv, long long kv_stride, const void* norm_w, float eps,
@@ -763,10 +763,14 @@ Tensor qk_norm_rope(const Tensor& q, const Tensor& k, const Tensor& v, const c10
   CHECK_ROWS(v, dt);
   CHECK_I32(positions);
   CHECK_I32(slots);
-  check_gated_caches(k_cache, v_cache, dt, head_dim, head_dim_v);
-  const int T = q.size(0), Hk = k_cache.size(1);
+  for (const Tensor& c : {k_cache, v_cache})
+    TORCH_CHECK(c.is_cuda() && c.scalar_type() == dt && c.dim() == 4 && c.is_contiguous() &&
+                    c.size(0) == k_cache.size(0) && c.size(2) == k_cache.size(2),
+                "qk_norm_rope: caches [blocks, heads, block_size, width]");
+  TORCH_CHECK(k_cache.size(3) >= head_dim && v_cache.size(3) >= head_dim_v, "qk_norm_rope: width of the cache rows");
+  const int T = q.size(0), Hk = k_cache.size(1), Hv = v_cache.size(1);
   TORCH_CHECK(positions.numel() >= T && slots.numel() >= T && q.size(1) % head_dim == 0 && k.size(0) == T &&
-                  v.size(0) == T && k.size(1) == Hk * head_dim && v.size(1) == Hk * head_dim_v, "qk_norm_rope: shapes");
+                  v.size(0) == T && k.size(1) == Hk * head_dim && v.size(1) == Hv * head_dim_v, "qk_norm_rope: shapes");
   const float* cs = nullptr;
   int max_pos = 1 << 30;
   if (cos_sin.has_value()) {
@@ -801,7 +805,7 @@ Tensor qk_norm_rope(const Tensor& q, const Tensor& k, const Tensor& v, const c10
   Tensor out = torch::empty({T, q.size(1)}, q.options());
   check(b200_qk_norm_rope(q.data_ptr(), k.data_ptr(), v.data_ptr(), vf, out.data_ptr(), k_cache.data_ptr(),
                           v_cache.data_ptr(), positions.data_ptr<int>(), slots.data_ptr<int>(), cs, max_pos, (int)norm, qw, kw, sp, (int)n_q, (int)n_k, (float)eps, (float)lambda, T,
-                          (int)(q.size(1) / head_dim), Hk, (int)head_dim, (int)head_dim_v, (int)k_cache.size(3),
+                          (int)(q.size(1) / head_dim), Hk, Hv, (int)head_dim, (int)head_dim_v, (int)k_cache.size(3),
                           (int)v_cache.size(3), (int)rot, q.stride(0), k.stride(0), v.stride(0), fs,
                           (int)k_cache.size(2), (float)temp, (int)temp_every, f32 ? 1 : 0, cur_stream()),
         "qk_norm_rope");

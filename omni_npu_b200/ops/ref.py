@@ -287,7 +287,9 @@ def qk_norm_rope_cache(q, k, v, k_cache, v_cache, positions, slot_mapping, cos_s
         qf = qf * (1 + c * torch.log(((positions.long() + 1) // n).float() + 1)).unsqueeze(1)
     if v_first is not None:
         vf = (1 - mix) * vf + mix * v_first.float()
-    gqa_cache_write(kf.to(k.dtype), vf.to(v.dtype), k_cache[..., :head_dim], v_cache[..., :head_dim_v], slot_mapping)
+    kc, vc = k_cache[..., :head_dim], v_cache[..., :head_dim_v]
+    gqa_cache_write(kf.to(k.dtype), kf.to(k.dtype), kc, kc, slot_mapping)       # (keys and values may differ in heads)
+    gqa_cache_write(vf.to(v.dtype), vf.to(v.dtype), vc, vc, slot_mapping)
     return qf.to(q.dtype)
 
 

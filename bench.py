@@ -53,7 +53,7 @@ def parse_args():
                     help="decoding requests ride along in prefill steps (default: prompts first)")
     ap.add_argument("--profile", default=None,
                     help="write a per-kernel time table (torch profiler, one extra untimed pass) to this file")
-    ap.add_argument("--design", default=None, choices=["rivudra", "fuvirax", "gatosun"],
+    ap.add_argument("--design", default=None, choices=["rivudra", "fuvirax", "gatosun", "dalavik"],
                     help="instead of the workload: steps and kernels of this design beside the closest existing "
                          "model at equal size, one JSON line per size (one GPU)")
     ap.add_argument("--design-size", default=None, help="with --design: only the sizes whose name contains this")

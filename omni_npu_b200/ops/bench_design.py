@@ -1,12 +1,13 @@
 """Throughput of a design beside the framework's closest existing model at equal size (random weights).
 
-``bench.py --design rivudra``, ``--design fuvirax`` or ``--design gatosun`` runs this on one GPU.  Per size it
-prints one JSON line with
+``bench.py --design rivudra`` (``fuvirax``, ``gatosun``, ``dalavik``) runs this on one GPU.  Per size it prints one JSON
+line with
 
 * whole steps through the engine (device time of prompt and decode steps, CUDA events): Rivudra and a
   Qwen3-MoE of the same width, heads, experts and window, Fuvirax and a dense DeepSeek-V2 of the same
-  width, heads, latent sizes and feed-forward, or Gatosun and a Qwen3-MoE of the same width, heads and
-  experts (every layer full attention);
+  width, heads, latent sizes and feed-forward, Gatosun and a Qwen3-MoE of the same width, heads and
+  experts (every layer full attention), or Dalavik and a dense DeepSeek-V2 of the same width, heads, latent
+  sizes and feed-forward (every layer latent attention);
 * single kernels: time, the fraction of the measured roofline (the slower of bytes / copy bandwidth and
   FLOPs / library bf16 GEMM throughput) and the same for the like kernel of the other model.  Between
   iterations a 256 MB buffer is written, so inputs come from HBM.
@@ -652,10 +653,242 @@ def gatosun_kernels(size) -> List[dict]:
     return out
 
 
+# ----------------------------------------------------------------------------- Dalavik
+# width, heads, rotated keys, latent, query latent (head and value size of the latent layers: 128), key/value heads, head
+# and value size of the mixed-score layers, feed-forward, token input, norm groups
+DALAVIK_SIZES: Dict[str, Tuple[int, ...]] = {
+    "2048x16h/128 q768 g4x128/128 ff8192 s128": (2048, 16, 64, 512, 768, 4, 128, 128, 8192, 128, 2),
+    "4096x32h/128 q1536 g8x128/128 ff12288 s256": (4096, 32, 64, 512, 1536, 8, 128, 128, 12288, 256, 4),
+    "3072x24h/128 q1024 g6x96/64 ff8192 s256": (3072, 24, 64, 512, 1024, 6, 96, 64, 8192, 256, 8),
+}
+DALAVIK_LAYERS = 6           # two of each: own latent rows, shared ones, mixed scores
+DALAVIK_HEAD = 128
+SOFTCAP, QUERY_TEMPERATURE = 30.0, (0.1, 512)
+
+
+def dalavik(size) -> ModelConfig:
+    w, h, rot, rank, qr, g, d, e, ff, side, groups = size
+    hd, mlp = DALAVIK_HEAD, DenseSpec(ff, ops.RELU)
+
+    def lat(source):
+        return LayerSpec(LatentAttentionSpec(h, hd, rot, hd, rank, 1e4, (hd + rot) ** -0.5, False, qr, source), mlp)
+    mixed = LayerSpec(AttentionSpec(h, g, d, e, 0, 0.0, d ** -0.5, qk_norm="head_weight", bias=True, softcap=SOFTCAP,
+                                    query_temperature=QUERY_TEMPERATURE, distance_bias=True, score_mix=True,
+                                    head_sink=True), mlp)
+    return ModelConfig(architecture="Dalavik", model_type="dalavik", hidden_size=w, num_layers=DALAVIK_LAYERS, num_heads=h,
+                       num_kv_heads=1, head_dim=hd, v_head_dim=hd, vocab_size=VOCAB, max_position_embeddings=1 << 16,
+                       layer_specs=(lat(None), mixed, lat(0), lat(None), mixed, lat(3)), tie_word_embeddings=True,
+                       norm_groups=groups, token_side_dim=side)
+
+
+def deepseek_query_latent(size) -> ModelConfig:
+    w, h, rot, rank, qr, _, _, _, ff, _, _ = size
+    hd = DALAVIK_HEAD
+    return ModelConfig(architecture="DeepseekV2ForCausalLM", model_type="deepseek_v2", hidden_size=w,
+                       num_layers=DALAVIK_LAYERS, num_heads=h, num_kv_heads=h, head_dim=hd + rot, intermediate_size=ff,
+                       vocab_size=VOCAB, max_position_embeddings=1 << 16, rope_neox=False, use_mla=True, q_lora_rank=qr,
+                       kv_lora_rank=rank, qk_nope_head_dim=hd, qk_rope_head_dim=rot, v_head_dim=hd)
+
+
+def dalavik_kernels(size) -> List[dict]:
+    from ..attention.latent import LatentAttention
+    w, h, rot, rank, qr, kvh, d, e, ff, side, groups = size
+    hd = DALAVIK_HEAD
+    bw, fl = _peaks()
+    out: List[dict] = []
+    bf = dict(dtype=torch.bfloat16, device="cuda")
+    f32 = dict(dtype=torch.float32, device="cuda")
+    i32 = dict(dtype=torch.int32, device="cuda")
+
+    def bound(nbytes: float, flops: float = 0.0, fp32: float = 0.0) -> float:
+        return max(nbytes / bw, flops / fl, fp32 / FP32_FLOPS) * 1e3
+
+    def entry(name: str, fn, cost, like=None, like_cost=None):
+        ms, b = _time(fn), bound(*cost)
+        r = {"kernel": f"{name}, {kind}", "ms": round(ms, 4), "roofline": round(b / ms, 3)}
+        if like is not None:
+            lms, lb = _time(like), bound(*(like_cost or cost))
+            r.update(like_ms=round(lms, 4), like_roofline=round(lb / lms, 3), distance=round((lb / lms) / (b / ms), 2))
+        out.append(r)
+
+    bs, qk, row = 64, hd + rot, rank + rot
+    for kind, n, rows in (("prefill", 8, 1024), ("decode b1", 1, 1), ("decode b16", 16, 1), ("decode b128", 128, 1)):
+        t, pre = n * rows, kind == "prefill"
+        ctx = rows if pre else CONTEXT
+        x, gain = torch.randn(t, w, **bf), torch.randn(w, **bf)
+        res, res16 = torch.randn(t, w, **f32), torch.randn(t, w, **bf)
+
+        def add_norm():
+            ops.fused_add_rms_norm(x, res16, gain, 1e-6)
+        entry("norm of the result + add (like: add + norm)",
+              lambda: ops.post_norm_residual(res, x, gain, groups, 1e-6, w), (t * w * 12,), add_norm, (t * w * 8,))
+        entry("the same + final norm (like: add + norm)",
+              lambda: ops.post_norm_residual(res, x, gain, 1, 1e-6, w, out_norm=(gain, groups)), (t * w * 12,), add_norm,
+              (t * w * 8,))
+
+        def cost(a, b, cols=None):
+            return (a.numel() + b.numel() + a.shape[0] * (cols or b.shape[0])) * 2, 2.0 * a.shape[0] * b.numel()
+
+        def product(name, a, cols, like_cols, like_a=None, bias=False, act=None, like_act=None):
+            la = a if like_a is None else like_a
+            wa, wb = torch.randn(cols, a.shape[1], **bf), torch.randn(like_cols, la.shape[1], **bf)
+            bb = torch.randn(cols, **bf) if bias else None
+            entry(name, lambda: ops.gemm(a, wa, bb, **(act or {})), cost(a, wa, cols // 2 if act else None),
+                  lambda: ops.gemm(la, wb, **(like_act or {})), cost(la, wb, like_cols // 2 if like_act else None))
+        qkv = (h + kvh) * d + kvh * e
+        product("query and key latents (like: the same of MLA)", x, qr + row, qr + row)
+        product("query latent alone (like: both latents of MLA)", x, qr, qr + row)
+        zq = torch.randn(t, qr, **bf)
+        product("queries from their latent (like: the same of MLA)", zq, h * qk, h * qk)
+        product("q / k / v with bias (like: q of MLA)", x, qkv, h * qk, zq, bias=True)
+        product("gate / up + relu (like: gate / up + silu)", x, 2 * ff, 2 * ff, act=dict(swiglu=True, act=ops.RELU),
+                like_act=dict(swiglu=True))
+        sp = (side + 7) // 8 * 8
+        product("token input: gate (like: both latents of MLA)", x, sp, qr + row)
+        z = torch.randn(t, sp, **bf)
+        product("token input: back (like: queries from their latent)", z, w, h * qk, zq)
+        ids, table = torch.randint(0, VOCAB, (t,), **i32), torch.randn(VOCAB, side * DALAVIK_LAYERS, **bf)
+        gu = torch.randn(t, 2 * sp, **bf)
+        entry("token input: gated rows (like: silu(gate) * up)", lambda: ops.gelu_rows(z, ids, table, side, side),
+              (t * side * 6,), lambda: ops.silu_and_mul(gu))
+        del gu, table
+
+        # ---- latent attention
+        cu, lens = torch.arange(0, (n + 1) * rows, rows, **i32), torch.full((n,), ctx, **i32)
+        per = (ctx + bs - 1) // bs
+        cache = torch.randn(n * per, bs, row, **bf)
+        bt = torch.randperm(n * per, device="cuda").int().view(n, per)
+        pos = torch.arange(ctx - rows, ctx, **i32).repeat(n)
+        slot = (bt.long().gather(1, (pos.view(n, rows) // bs).long()) * bs + pos.view(n, rows) % bs).int().view(-1)
+        cs = torch.randn(CONTEXT + 128, rot, device="cuda")
+        q, y = torch.randn(t, h * qk, **bf), torch.randn(t, qr + row, **bf)
+        low, kv_a, c_q = y[:, :qr], y[:, qr:], torch.empty(t, qr, **bf)
+        low_c = low.contiguous()
+        attn = LatentAttention(h, hd, rot, hd, rank, qk ** -0.5, False, 1e-5, torch.bfloat16, torch.device("cuda"), qr)
+        attn.w_uk.data.normal_(std=0.02)
+        attn.w_uv.data.normal_(std=0.02)
+        attn.build_absorbed()
+        q_lat = torch.empty(t, h, row, **bf)
+
+        def like_norms():
+            ops.rms_norm(low_c, attn.query_norm, 1e-5)
+            ops.mla_kv_rmsnorm_rope_cache(kv_a[:, :rank], kv_a[:, rank:], attn.latent_norm, cache, pos, slot, cs, 1e-5, False)
+
+        def like_rotate():
+            pe = q.view(t, h, qk)[:, :, hd:].reshape(t, h * rot).contiguous()
+            ops.rope_qk_(pe, pe.new_empty(t, 0), pos, cs, rot, rot, False)
+        prep = (attn.latent_norm, 1e-5, cache, pos, slot, cs, h, hd, rot, rank, False)
+        entry("norms of both latents + rotation + cache (like: norm; norm + rotation + cache)",
+              lambda: ops.latent_prep_(None, kv_a, *prep, low=(low, attn.query_norm, c_q)), (t * (2 * row + 2 * qr) * 2,),
+              like_norms)
+        entry("norm of the query latent (like: norm)",
+              lambda: ops.latent_prep_(None, None, *prep, low=(low, attn.query_norm, c_q)), (t * qr * 4,),
+              lambda: ops.rms_norm(low_c, attn.query_norm, 1e-5))
+        entry("rotation of the queries (like: the same)",
+              lambda: ops.latent_prep_(q, None, *prep, None if pre else q_lat, 0 if pre else t), (t * h * rot * 4,),
+              like_rotate)
+        pairs = n * h * sum(p + 1 for p in range(ctx - rows, ctx))
+        if pre:
+            start = (torch.cumsum(lens, 0) - lens).int()
+            gathered = ops.latent_gather(cache, bt, lens, start, n, t, ctx)
+
+            def own_keys():
+                r = ops.latent_gather(cache, bt, lens, start, n, t, ctx)
+                return ops.gemm(r, attn.w_key), ops.gemm(r, attn.w_value)
+            kvb = torch.randn(h * 2 * hd, rank, **bf)
+
+            def like_keys():
+                lat = cache.index_select(0, bt.view(-1).long())
+                kv = ops.gemm(lat[..., :rank].reshape(-1, rank).contiguous(), kvb).view(-1, bs, h, 2 * hd)
+                pe = lat[..., rank:].unsqueeze(2).expand(-1, bs, h, rot)
+                k = torch.cat([kv[..., :hd], pe], -1).permute(0, 2, 1, 3).contiguous()
+                return k, kv[..., hd:].permute(0, 2, 1, 3).contiguous()
+            kc_ = t * (row + h * (qk + hd)) * 2 + kvb.numel() * 2, 2.0 * t * kvb.numel()
+            entry("keys and values from the latents (like: the same)", own_keys, kc_, like_keys)
+            entry("keys and values from shared rows (like: with the gather)",
+                  lambda: (ops.gemm(gathered, attn.w_key), ops.gemm(gathered, attn.w_value)), kc_, like_keys)
+            k, v = own_keys()
+            o = torch.empty(t, h * hd, **bf)
+            lk, lv = like_keys()
+            lbt = torch.arange(n * per, **i32).view(n, per)
+            entry("latent attention (like: the same)",
+                  lambda: ops.contiguous_attention(q, k.view(-1, h, 1, qk), v.view(-1, h, 1, hd), o, cu, start, lens, n, rows,
+                                                   h, qk, hd, 0.07), (t * h * (2 * qk + 2 * hd) * 2, 2.0 * pairs * (qk + hd)),
+                  lambda: ops.gqa_prefill(q, lk, lv, lbt, cu, lens, n, rows, h, 0.07, True, 0))
+            del k, v, lk, lv, gathered
+        else:
+            lat_o, o = torch.empty(t, h, rank, **bf), torch.empty(t, h * hd, **bf)
+            heads, uv = q.view(t, h, qk), attn.w_uv.view(h, hd, rank)
+            offs = torch.arange(0, (h + 1) * t, t, **i32)
+
+            def like_fold():
+                qn = heads[..., :hd].transpose(0, 1).reshape(h * t, hd).contiguous()
+                ql = ops.grouped_gemm(qn, attn.w_fold, offs).view(h, t, rank).transpose(0, 1)
+                return torch.cat([ql, q_lat[..., rank:]], -1).reshape(t, h * row).contiguous()
+
+            def like_unfold():
+                a = lat_o.transpose(0, 1).reshape(h * t, rank).contiguous()
+                return ops.grouped_gemm(a, uv, offs).view(h, t, hd).transpose(0, 1).reshape(t, h * hd).contiguous()
+            fc = (h * hd * rank + t * h * (hd + rank)) * 2, 2.0 * t * h * hd * rank
+            entry("queries into the latent space (like: the same)",
+                  lambda: ops.head_gemm(heads[..., :hd], attn.w_fold, q_lat[..., :rank]), fc, like_fold)
+            entry("results out of the latent space (like: the same)", lambda: ops.head_gemm(lat_o, uv, o.view(t, h, hd)), fc,
+                  like_unfold)
+            q_flat = torch.randn(t, h * row, **bf)
+            entry("latent attention (like: the same)",
+                  lambda: ops.latent_decode(q_flat.view(t, h, row), cache, bt, lens, n, h, rank, 0.07, lat_o,
+                                            max_seq_len=CONTEXT),
+                  ((n * ctx * row + t * h * (row + rank)) * 2, 2.0 * pairs * (row + rank)),
+                  lambda: ops.mla_decode(q_flat, cache, bt, lens, n, h, 0.07, 1, max_seq_len=CONTEXT))
+        del cache, q, y, q_lat, attn
+        # ---- attention with mixed scores; the like kernels are those of grouped-query attention
+        kc, vc = torch.randn(n * per, kvh, bs, d, **bf), torch.randn(n * per, kvh, bs, e, **bf)
+        lvc = vc if e == d else torch.randn(n * per, kvh, bs, d, **bf)
+        y = torch.randn(t, qkv, **bf)
+        q, kk, vv = y.split([h * d, kvh * d, kvh * e], 1)
+        lv_ = torch.randn(t, kvh * d, **bf)
+        hn, cs = torch.randn(d, **bf), torch.randn(CONTEXT + 128, d, **f32)
+
+        def like_prep():
+            a = ops.rms_norm(q.reshape(-1, d), hn, 1e-6).view(t, -1)
+            b = ops.rms_norm(kk.reshape(-1, d), hn, 1e-6).view(t, -1)
+            ops.rope_cache_gqa_(a, b, lv_, kc, lvc, pos, slot, cs, d, d, True)
+        entry("head norms + query temperature + cache (like: head norms + rotation + cache)",
+              lambda: ops.qk_norm_rope_cache(q, kk, vv, kc, vc, pos, slot, None, d, e, 0, "head_weight", 1e-6, (hn, hn),
+                                             temperature=QUERY_TEMPERATURE), (t * (2 * (h + kvh) * d + 2 * kvh * e) * 2,),
+              like_prep, (t * (2 * h + 4 * kvh) * d * 2,))
+        o, lo = torch.empty(t, h * e, **bf), torch.empty(t, h * d, **bf)
+        r1, r2, sink = torch.rand(h, **f32), torch.rand(h, **f32) * 0.1, torch.randn(h, **f32)
+        talk = torch.eye(h, **f32) + 0.1 * torch.randn(h, h, **f32)
+        qc = q.contiguous()
+
+        def like_attn():
+            if not pre:
+                return ops.gqa_decode(qc, kc, lvc, bt, lens, n, h, d ** -0.5, 1, 0, max_seq_len=ctx)
+            if d == e and d in (64, 128):
+                return ops.gqa_prefill(qc, kc, vc, bt, cu, lens, n, rows, h, d ** -0.5, True, 0)
+            return ops.gated_attention(qc, None, kc, vc, o, bt, cu, lens, n, rows, h, d, e, d ** -0.5, 0, None,
+                                       max_seq_len=ctx)
+        kv = n * kvh * ctx * 2
+        le = e if pre else d
+        entry("attention with mixed scores (like: grouped-query attention)",
+              lambda: ops.mixed_attention(qc, kc, vc, o, bt, cu if pre else None, lens, n, rows, d, e, d ** -0.5, SOFTCAP,
+                                          (r1, r2), talk, sink, max_seq_len=ctx),
+              (kv * (d + e) + t * h * (d + e) * 2, 2.0 * pairs * (d + e), 2.0 * pairs * h), like_attn,
+              (kv * (d + le) + t * h * (d + le) * 2, 2.0 * pairs * (d + le)))
+        del kc, vc, lvc, y, q, kk, vv, qc, res
+        gc.collect()
+        torch.cuda.empty_cache()
+    ops.check_status()
+    return out
+
+
 DESIGNS = {
     "rivudra": (SIZES, LAYERS, kernels, {"rivudra": rivudra, "qwen3-moe": qwen3_moe}),
     "fuvirax": (FUVIRAX_SIZES, FUVIRAX_LAYERS, fuvirax_kernels, {"fuvirax": fuvirax, "deepseek-v2 dense": deepseek_dense}),
     "gatosun": (GATOSUN_SIZES, GATOSUN_LAYERS, gatosun_kernels, {"gatosun": gatosun, "qwen3-moe": qwen3_moe_full}),
+    "dalavik": (DALAVIK_SIZES, DALAVIK_LAYERS, dalavik_kernels,
+                {"dalavik": dalavik, "deepseek-v2 dense": deepseek_query_latent}),
 }
 
 

@@ -49,15 +49,38 @@ __device__ __forceinline__ long long cache_row(const MixedAttnParams& p, const i
 }
 
 // The score of one head before the mixture, from the raw product; hardware exponentials and logarithms (absolute
-// errors of a few 1e-7 times softcap and r1).
-__device__ __forceinline__ float head_score(const MixedAttnParams& p, float x, float dist, float r1, float r2) {
-  if (p.softcap > 0.f) {
-    const float z = x * (p.scale / p.softcap);
-    x = p.softcap - __fdividef(2.f * p.softcap, __expf(2.f * z) + 1.f);
-  } else {
-    x *= p.scale;
-  }
-  return p.r1 ? x - r1 * __logf(fmaf(r2, dist, 1.f)) : x;
+// errors of a few 1e-7 times softcap and r1).  tanh(z) = 1 - 2 / (exp(2 z) + 1).
+struct ScoreConst {
+  float in;                    // capped: 2 scale / softcap * log2 e, else the scale
+  float cap;                   // softcap
+};
+__device__ __forceinline__ ScoreConst score_const(const MixedAttnParams& p) {
+  return {p.softcap > 0.f ? 2.f * 1.4426950408889634f * p.scale / p.softcap : p.scale, p.softcap};
 }
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float lg2_approx(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+template <bool CAP>
+__device__ __forceinline__ float capped_score(const ScoreConst& c, float x) {
+  if constexpr (CAP) return fmaf(-2.f * c.cap, rcp_approx(ex2_approx(x * c.in) + 1.f), c.cap);
+  else return x * c.in;
+}
+// r1 ln(1 + r2 dist), with r1 already times ln 2
+__device__ __forceinline__ float distance_bias(float r1_ln2, float r2, float dist) {
+  return r1_ln2 * lg2_approx(fmaf(r2, dist, 1.f));
+}
+constexpr float kLn2 = 0.6931471805599453f;
 
 }  // namespace b200

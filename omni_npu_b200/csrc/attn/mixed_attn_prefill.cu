@@ -3,10 +3,13 @@
 //
 //   mixed_scores_kernel   16 queries x a range of keys, all heads: Q K^T on mma.sync with the queries of a warp's heads in
 //                         registers, capped and lowered into shared memory, then the mixture as fp32 outer products
-//                         (8 output heads x 4 keys per thread); mixed scores to memory in fp32
+//                         (8 output heads x 4 keys per thread); mixed scores to memory in fp32.  The distance bias of a
+//                         tile has 15 + keys values per head: a table, made while the tile before is mixed
 //   mixed_values_kernel   128 rows = tokens x heads of a value head: online softmax over the stored scores, sink, P V
 //
 // The scores of as many query tiles as fit into the given buffer are made per call.
+
+#include <type_traits>
 
 #include "../common/device_once.h"
 #include "../common/pdl.cuh"
@@ -25,19 +28,20 @@ __device__ __forceinline__ uint32_t piece(int row, int chunk, int width) {
 }
 
 struct Layout {
-  int dk, ho8, s_pitch, k_bytes, s_off, t_off, r_off, bytes;
+  int dk, ho8, s_pitch, d_pitch, k_bytes, s_off, t_off, d_off, bytes;
 };
-// ring of `stages` key tiles | scores [Hs][16][s_pitch] | talk^T [Hs][ho8] | r1, r2
+// ring of `stages` key tiles | scores [Hs][16][s_pitch] | talk^T [Hs][ho8] | distance bias [2][Hs][d_pitch]
 __host__ __device__ inline Layout layout(int Hs, int Hk, int Ho, int DP, int bk, int stages) {
   Layout l;
-  l.dk = (DP + 63) / 64 * 64;
+  l.dk = DP <= 64 ? 64 : DP <= 128 ? 128 : 256;            // 16 times the kernel's KS
   l.ho8 = (Ho + 7) / 8 * 8;
   l.s_pitch = bk + 8;
   l.k_bytes = Hk * bk * l.dk * 2;
   l.s_off = stages * l.k_bytes;
   l.t_off = l.s_off + Hs * BQ * l.s_pitch * 4;
-  l.r_off = l.t_off + Hs * l.ho8 * 4;
-  l.bytes = l.r_off + 2 * Hs * 4;
+  l.d_pitch = bk + BQ;
+  l.d_off = l.t_off + Hs * l.ho8 * 4;
+  l.bytes = l.d_off + 2 * Hs * l.d_pitch * 4;
   return l;
 }
 
@@ -61,14 +65,14 @@ bool mixed_prefill_fits(int Hs, int Hk, int Ho, int Hv, int DP, int DVP) {
 // ------------------------------------------------------------- scores
 // KS: steps of 16 along the head size; HPW: heads per warp and pass (16 registers of query per head and 4 steps)
 template <int WARPS, int KS, int HPW, int BK>
-__global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAttnParams p, const int stages) {
+__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_kernel(const MixedAttnParams p, const int stages) {
   using namespace mpre;
-  constexpr int THREADS = WARPS * 32;
+  constexpr int THREADS = WARPS * 32, DK = KS * 16;
   extern __shared__ __align__(128) uint8_t smem[];
   const Layout L = layout(p.Hs, p.Hk, p.Ho, p.DP, BK, stages);
   float* sS = reinterpret_cast<float*>(smem + L.s_off);
   float* sT = reinterpret_cast<float*>(smem + L.t_off);
-  float* sR = reinterpret_cast<float*>(smem + L.r_off);
+  float* sD = reinterpret_cast<float*>(smem + L.d_off);
   const uint32_t ring = smem_u32(smem);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
@@ -88,22 +92,29 @@ __global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAtt
   const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(p.k_cache);
   const int per = p.Hs / p.Hk;
 
+  // `1 << ll` threads share a row, a thread has the same keys of every tile and walks over the heads
+  const int chunks = p.DP >> 3;
+  int ll = 0;
+  while (ll < 5 && (1 << ll) < chunks) ++ll;
+  const int slots = THREADS >> ll, kstep = min(slots, BK), slot = tid >> ll, li = tid & ((1 << ll) - 1);
+  const int g0 = slots > BK ? slot / BK : 0, gstep = slots > BK ? slots / BK : 1;
   auto issue = [&](int i) {
     const int n0 = k_begin + i * BK;
     if (n0 < k_end) {
       const uint32_t dst = ring + (stages == 2 ? i & 1 : 0) * L.k_bytes;
-      const int chunks = p.DP >> 3;
-      int ll = 0;
-      while (ll < 5 && (1 << ll) < chunks) ++ll;
-      const int li = lane & ((1 << ll) - 1), rows_per = 32 >> ll;
-      for (int r = warp * rows_per + (lane >> ll); r < p.Hk * BK; r += WARPS * rows_per) {
-        const int g = r / BK, key = n0 + r % BK;
+      for (int j = slot & (kstep - 1); j < BK; j += kstep) {
+        const int key = n0 + j;
         const bool ok = key < k_end;
-        const __nv_bfloat16* src = ok ? kc + cache_row(p, bt, key, g, p.Hk) * p.DP : kc;
+        const __nv_bfloat16* row0 = ok ? kc + cache_row(p, bt, key, g0, p.Hk) * p.DP : kc;
+        const long long step = ok ? static_cast<long long>(gstep) * p.block_size * p.DP : 0;
         const int sz = ok ? 16 : 0;
-        for (int c = li; c < chunks; c += 1 << ll)
-          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + piece(r, c, L.dk)),
-                       "l"(ok ? src + c * 8 : src), "r"(sz) : "memory");
+        for (int c = li; c < chunks; c += 1 << ll) {
+          const __nv_bfloat16* src = ok ? row0 + c * 8 : row0;
+          uint32_t to = dst + piece(g0 * BK + j, c, DK);
+#pragma unroll 4
+          for (int g = g0; g < p.Hk; g += gstep, src += step, to += gstep * BK * DK * 2)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to), "l"(src), "r"(sz) : "memory");
+        }
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -113,31 +124,41 @@ __global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAtt
     const int g = i / L.ho8, h = i - g * L.ho8;
     sT[i] = h < p.Ho ? p.talk[h * p.Hs + g] * kLog2e : 0.f;
   }
-  for (int i = tid; i < p.Hs; i += THREADS) {
-    sR[i] = p.r1 ? p.r1[i] : 0.f;
-    sR[p.Hs + i] = p.r1 ? p.r2[i] : 0.f;
-  }
+  // distance bias of tile i: entry x of a head is for distance base + x, base = first query - last key
+  auto make_bias = [&](int i) {
+    if (k_begin + i * BK >= k_end) return;
+    const int base = ctx + tok0 - (k_begin + i * BK + BK - 1);
+    float* dst = sD + (i & 1) * p.Hs * L.d_pitch;
+    for (int e = tid; e < p.Hs * (BK + BQ); e += THREADS) {
+      const int g = e / (BK + BQ), x = e - g * (BK + BQ);
+      dst[e] = p.r1 ? distance_bias(__ldg(p.r1 + g) * kLn2, __ldg(p.r2 + g), fmaxf(static_cast<float>(base + x), 0.f)) : 0.f;
+    }
+  };
+  make_bias(0);
 
   // query fragments of the heads of a pass, straight from memory
   uint32_t qf[HPW][KS][4];
   const bool pairs = (p.D & 1) == 0 && (p.q_stride & 1) == 0 && (reinterpret_cast<uintptr_t>(q) & 3) == 0;
-  auto load_q = [&](int pass) {
+  const int tok_a = min(tok0 + (lane >> 2), q_len - 1), tok_b = min(tok0 + (lane >> 2) + 8, q_len - 1);
+  auto load_q = [&](int pass) {                            // (rows beyond the portion repeat its last one)
 #pragma unroll
     for (int j = 0; j < HPW; ++j) {
       const int g = (pass * WARPS + warp) * HPW + j;
+      if (g >= p.Hs) continue;
+      const __nv_bfloat16* at = q + static_cast<long long>(g) * p.D + (lane & 3) * 2;
+      const __nv_bfloat16* src[2] = {at + (q_begin + tok_a) * p.q_stride, at + (q_begin + tok_b) * p.q_stride};
 #pragma unroll
       for (int ks = 0; ks < KS; ++ks)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int tok = tok0 + (lane >> 2) + (e & 1) * 8, d = ks * 16 + (lane & 3) * 2 + (e >> 1) * 8;
+          const int d = ks * 16 + (e >> 1) * 8;
           uint32_t v = 0u;
-          if (g < p.Hs && tok < q_len && d < p.D) {
-            const __nv_bfloat16* src = q + (q_begin + tok) * p.q_stride + static_cast<long long>(g) * p.D + d;
+          if (d + (lane & 3) * 2 < p.D) {
             if (pairs) {
-              v = *reinterpret_cast<const uint32_t*>(src);
+              v = *reinterpret_cast<const uint32_t*>(src[e & 1] + d);
             } else {
-              v = __bfloat16_as_ushort(src[0]);
-              if (d + 1 < p.D) v |= static_cast<uint32_t>(__bfloat16_as_ushort(src[1])) << 16;
+              v = __bfloat16_as_ushort(src[e & 1][d]);
+              if (d + (lane & 3) * 2 + 1 < p.D) v |= static_cast<uint32_t>(__bfloat16_as_ushort(src[e & 1][d + 1])) << 16;
             }
           }
           qf[j][ks][e] = v;
@@ -147,8 +168,12 @@ __global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAtt
   const int passes = (p.Hs + WARPS * HPW - 1) / (WARPS * HPW);
   if (passes == 1) load_q(0);
 
+  const ScoreConst c = score_const(p);
   const int tiles = (k_end - k_begin + BK - 1) / BK;
   const int ks_used = p.DP >> 4;
+  uint32_t kx[4];                                          // swizzled chunk of a row, by step modulo 4
+#pragma unroll
+  for (int i = 0; i < 4; ++i) kx[i] = ((i * 2 + ((lane >> 3) & 1)) ^ (lane & 7)) << 4;
   for (int it = 0; it < tiles; ++it) {
     if (stages == 1) {
       if (it) __syncthreads();
@@ -166,7 +191,7 @@ __global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAtt
       for (int j = 0; j < HPW; ++j) {
         const int g = (pass * WARPS + warp) * HPW + j;
         if (g >= p.Hs) continue;
-        const int krow = (g / per) * BK;
+        const uint32_t k_at = kt + ((g / per) * BK + (lane & 7) + ((lane >> 4) << 3)) * DK * 2;
         float s[BK / 8][4];
 #pragma unroll
         for (int n = 0; n < BK / 8; ++n)
@@ -178,27 +203,29 @@ __global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAtt
 #pragma unroll
             for (int n = 0; n < BK / 16; ++n) {
               uint32_t kf[4];
-              ldmatrix_x4(kf, kt + piece(krow + n * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1), L.dk));
+              ldmatrix_x4(kf, k_at + n * 16 * DK * 2 + (ks >> 2) * 128 + kx[ks & 3]);
               mma_bf16_16816(s[2 * n], qf[j][ks], kf[0], kf[1]);
               mma_bf16_16816(s[2 * n + 1], qf[j][ks], kf[2], kf[3]);
             }
           }
         }
-        const float r1 = sR[g], r2 = sR[p.Hs + g];
-        float* dst = sS + g * BQ * L.s_pitch;
+        float* dst = sS + g * BQ * L.s_pitch + (lane >> 2) * L.s_pitch + (lane & 3) * 2;
+        const float* bias = sD + ((it & 1) * p.Hs + g) * L.d_pitch + BK - 1 + (lane >> 2) - (lane & 3) * 2;
+        auto put = [&](auto cap) {
 #pragma unroll
-        for (int n = 0; n < BK / 8; ++n)
+          for (int n = 0; n < BK / 8; ++n)
 #pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const int row = (lane >> 2) + r * 8, key = n * 8 + (lane & 3) * 2;
-            const int dist = ctx + tok0 + row - n0 - key;
-            *reinterpret_cast<float2*>(dst + row * L.s_pitch + key) =
-                make_float2(head_score(p, s[n][2 * r], static_cast<float>(max(0, dist)), r1, r2),
-                            head_score(p, s[n][2 * r + 1], static_cast<float>(max(0, dist - 1)), r1, r2));
-          }
+            for (int r = 0; r < 2; ++r)
+              *reinterpret_cast<float2*>(dst + r * 8 * L.s_pitch + n * 8) =
+                  make_float2(capped_score<decltype(cap)::value>(c, s[n][2 * r]) - bias[r * 8 - n * 8],
+                              capped_score<decltype(cap)::value>(c, s[n][2 * r + 1]) - bias[r * 8 - n * 8 - 1]);
+        };
+        if (c.cap > 0.f) put(std::true_type{});
+        else put(std::false_type{});
       }
     }
     __syncthreads();
+    make_bias(it + 1);
 
     // ---- mixture: an item = 8 output heads x 4 keys of a query
     constexpr int GROUPS = BQ * BK / 4;
@@ -235,7 +262,6 @@ __global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAtt
             *reinterpret_cast<float4*>(dst + h * p.pitch) = make_float4(o[h][0], o[h][1], o[h][2], o[h][3]);
       }
     }
-    if (stages == 2) __syncthreads();
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
@@ -243,6 +269,8 @@ __global__ void __launch_bounds__(WARPS * 32) mixed_scores_kernel(const MixedAtt
 // ------------------------------------------------------------- softmax and values
 namespace mval {
 constexpr int BM = 128, BN = 64, THREADS = 256;
+constexpr int S_PITCH = BN + 8;          // floats
+constexpr int S_BYTES = BM * S_PITCH * 4;
 }
 
 // DV: upper bound of the padded value size
@@ -252,7 +280,7 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
   using namespace mval;
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int V_BYTES = BN * DV * 2;
-  const uint32_t v0 = smem_u32(smem);
+  const uint32_t v0 = smem_u32(smem), s0 = v0 + 2 * V_BYTES;
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -273,6 +301,13 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
   const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(p.v_cache);
   const int tiles = (hi + BN - 1) / BN;
 
+  const int rows_live = (tok_end - m0) * hc;                       // rows: (token, head of the group)
+  const float* sbase = p.scratch + ((static_cast<long long>(b) * p.tiles * mpre::BQ + (m0 - first)) * p.Ho +
+                                    vh * per + head0) * p.pitch;
+  auto srow = [&](int r) {
+    const int tok = r / hc;
+    return sbase + (static_cast<long long>(tok) * p.Ho + (r - tok * hc)) * p.pitch;
+  };
   auto issue = [&](int it) {
     if (it < tiles) {
       // four threads per key row, 16-byte pieces dealt out in turn
@@ -284,6 +319,15 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
       for (int c = tid & 3; c < (p.DVP >> 3); c += 4)
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + tile_offset<DV>(r, c)),
                      "l"(ok ? src + c * 8 : src), "r"(sz) : "memory");
+      // 16 threads per row of scores (all within the row's pitch; what lies beyond a row's position is masked)
+      const uint32_t sdst = s0 + (it & 1) * S_BYTES + (tid & 15) * 16;
+#pragma unroll
+      for (int i = 0; i < BM / 16; ++i) {
+        const int rr = (tid >> 4) + i * 16;
+        if (rows_live > rr)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sdst + rr * S_PITCH * 4),
+                       "l"(srow(rr) + it * BN + (tid & 15) * 4) : "memory");
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -296,7 +340,6 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
     for (int j = 0; j < 4; ++j) o_acc[i][j] = 0.f;
   float row_max[2], row_sum[2];
   int pos[2];
-  const float* src[2];
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int row = warp * 16 + (lane >> 2) + r * 8;
@@ -306,8 +349,6 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
     // the sink is a key seen from the start: maximum = its score, sum = 1 (summed over the quad at the end)
     row_max[r] = ok && p.sink ? p.sink[h] * kLog2e : -INFINITY;
     row_sum[r] = ok && p.sink && (lane & 3) == 0 ? 1.f : 0.f;
-    src[r] = p.scratch + ((static_cast<long long>(b) * p.tiles * mpre::BQ + (ok ? tok - first : 0)) * p.Ho + (ok ? h : 0)) *
-                             p.pitch + (lane & 3) * 2;
   }
   const int w_hi = min(ctx + tok_end - 1, ctx + m0 + (warp * 16 + 15) / hc);       // last position of this warp's rows
 
@@ -315,22 +356,22 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
     issue(it + 1);
     const int n0 = it * BN;
     const bool seen = n0 <= w_hi;
-    float s[BN / 8][4];
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
     if (seen) {
+      float s[BN / 8][4];
+      const float* st = reinterpret_cast<const float*>(smem + 2 * V_BYTES + (it & 1) * S_BYTES) +
+                        (warp * 16 + (lane >> 2)) * S_PITCH + (lane & 3) * 2;
+      const bool interior = n0 + BN - 1 <= ctx + m0 && (warp * 16 + 15) < rows_live;
 #pragma unroll
       for (int i = 0; i < BN / 8; ++i)
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
+          const float2 x = *reinterpret_cast<const float2*>(st + r * 8 * S_PITCH + i * 8);
           const int key = n0 + i * 8 + (lane & 3) * 2;
-          float2 x = make_float2(-INFINITY, -INFINITY);
-          if (key <= pos[r]) x = *reinterpret_cast<const float2*>(src[r] + n0 + i * 8);
-          s[i][2 * r] = x.x;
-          s[i][2 * r + 1] = key + 1 <= pos[r] ? x.y : -INFINITY;
+          s[i][2 * r] = interior || key <= pos[r] ? x.x : -INFINITY;
+          s[i][2 * r + 1] = interior || key + 1 <= pos[r] ? x.y : -INFINITY;
         }
-    }
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();
-    if (seen) {
       const uint32_t vt = v0 + (it & 1) * V_BYTES;
       float corr[2], m_use[2];
 #pragma unroll
@@ -429,7 +470,7 @@ static int launch_values(const MixedAttnParams& p, cudaStream_t stream) {
   auto kern = mixed_values_kernel<DV>;
   static DeviceOnce once;
   int dev = 0;
-  constexpr int SMEM = 2 * mval::BN * DV * 2;
+  constexpr int SMEM = 2 * mval::BN * DV * 2 + 2 * mval::S_BYTES;
   if (once.needed(&dev)) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return -20;
     once.mark(dev);

@@ -767,8 +767,8 @@ MIXED_SCORE_BYTES = int(os.environ.get("OMNI_B200_MIXED_SCORE_MB", "512")) << 20
 
 
 def mixed_decode_splits(num_rows: int, keys: int, sms: int = 148) -> int:
-    """CTAs that share the keys of a decode row: at least 64 keys each, the GPU filled once."""
-    return max(1, min(32, sms // max(1, num_rows), (keys + 63) // 64))
+    """CTAs that share the keys of a decode row: at least 64 keys each, two CTAs per SM."""
+    return max(1, min(32, 2 * sms // max(1, num_rows), (keys + 63) // 64))
 
 
 def mixed_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,

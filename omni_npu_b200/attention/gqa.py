@@ -228,6 +228,7 @@ class MixedScoreAttention(GatedGQAAttention):
         self.q_norm, self.k_norm = param(head_dim, fill=1.0, dt=dtype), param(head_dim, fill=1.0, dt=dtype)
         self.r1, self.r2, self.sink = param(num_heads), param(num_heads), param(out_heads)
         self.talk = param(out_heads, num_heads)
+        self.talk_exact = False                  # whether bf16 holds it (set after loading)
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out_width: int = 0) -> torch.Tensor:
         """q [T, Hs*D], k [T, Hk*D], v [T, Hv*Dv]: views into the fused projection.  Returns
@@ -245,4 +246,5 @@ class MixedScoreAttention(GatedGQAAttention):
 
     def _run(self, q, gate, k_cache, v_cache, out, block_tables, cu_q, seq_lens, n: int, max_q: int, max_seq: int) -> None:
         ops.mixed_attention(q, k_cache, v_cache, out, block_tables, cu_q, seq_lens, n, max_q, self.head_dim, self.head_dim_v,
-                            self.scale, self.softcap, (self.r1, self.r2), self.talk, self.sink, max_seq_len=max_seq)
+                            self.scale, self.softcap, (self.r1, self.r2), self.talk, self.sink, max_seq_len=max_seq,
+                            talk_exact=self.talk_exact)

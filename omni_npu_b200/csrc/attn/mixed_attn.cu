@@ -158,8 +158,8 @@ extern "C" int b200_mixed_attention(const void* q, const void* k_cache, const vo
                                     const float* r2, const float* talk, const float* sink, int B, int rows, int q_len,
                                     int max_keys, int max_blocks, int block_size, int Hs, int Hk, int Ho, int Hv, int D,
                                     int DV, int DP, int DVP, long long q_stride, long long out_stride, float scale,
-                                    float softcap, int kind, int splits, float* scratch, int tile0, int tiles,
-                                    long long pitch, int is_fp32, cudaStream_t stream) {
+                                    float softcap, int kind, int talk_terms, int splits, float* scratch, int tile0,
+                                    int tiles, long long pitch, int is_fp32, cudaStream_t stream) {
   if (B <= 0 || rows <= 0) return 0;
   if (Hk <= 0 || Hv <= 0 || Hs % Hk || Ho % Hv || DP < D || DVP < DV || block_size <= 0) return -1;
   MixedAttnParams p{};
@@ -198,6 +198,7 @@ extern "C" int b200_mixed_attention(const void* q, const void* k_cache, const vo
   p.softcap = softcap;
   p.splits = splits < 1 ? 1 : splits;
   p.scratch = scratch;
+  p.talk_terms = talk_terms;
   p.tile0 = tile0;
   p.tiles = tiles;
   p.pitch = pitch;

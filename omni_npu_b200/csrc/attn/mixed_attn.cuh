@@ -34,10 +34,12 @@ struct MixedAttnParams {
   long long q_stride, out_stride;
   float scale, softcap;
   int splits;                  // decode: CTAs that share a row's keys
-  float* scratch;              // decode: [rows, splits, Ho, DVP + 2]; prompts: mixed scores, see pitch
+  float* scratch;              // decode: [rows, splits, Ho, DVP], then [rows, splits, Ho, 2]; prompts: see pitch
   // prompts: the query tiles of 16 rows tile0 .. tile0 + tiles - 1 of every sequence; their mixed scores (times
   // log2 e) are [B, tiles, 16, Ho, pitch]
   int tile0, tiles, max_q_len, max_keys;
+  int range;                   // keys of a score CTA
+  int talk_terms;              // 1: bf16 holds every element of talk exactly, 3: it does not
   long long pitch;
 };
 
@@ -76,6 +78,12 @@ template <bool CAP>
 __device__ __forceinline__ float capped_score(const ScoreConst& c, float x) {
   if constexpr (CAP) return fmaf(-2.f * c.cap, rcp_approx(ex2_approx(x * c.in) + 1.f), c.cap);
   else return x * c.in;
+}
+// the same less a bias, from `start` = cap - bias (without a cap: -bias)
+template <bool CAP>
+__device__ __forceinline__ float biased_score(const ScoreConst& c, float x, float start) {
+  if constexpr (CAP) return fmaf(-2.f * c.cap, rcp_approx(ex2_approx(x * c.in) + 1.f), start);
+  else return fmaf(x, c.in, start);
 }
 // r1 ln(1 + r2 dist), with r1 already times ln 2
 __device__ __forceinline__ float distance_bias(float r1_ln2, float r2, float dist) {

@@ -33,10 +33,13 @@ struct Layout {
   int hs4;                     // score heads rounded up to 4
   int s_pitch, p_pitch;        // floats per score head, bf16 per weight row
   int q_off, k_off, v_off, s_off, p_off, t_off, r_off, m_off, bytes;
+  int per_k, per_v;            // heads of a key head, of a value head
 };
 
-__host__ __device__ inline Layout layout(int Hs, int Hk, int Ho, int Hv, int DP, int DVP, int kt) {
-  Layout l;
+inline Layout layout(int Hs, int Hk, int Ho, int Hv, int DP, int DVP, int kt) {
+  Layout l{};
+  l.per_k = Hs / Hk;
+  l.per_v = Ho / Hv;
   l.dk = (DP + 63) / 64 * 64;
   l.dv = (DVP + 63) / 64 * 64;
   l.hs4 = (Hs + 3) / 4 * 4;
@@ -85,11 +88,11 @@ bool mixed_decode_fits(int Hs, int Hk, int Ho, int Hv, int DP, int DVP) {
 
 // UNITS: accumulator tiles (8 heads x 16 columns) per warp.  HB: output heads that a lane mixes at a time
 template <int UNITS, int WARPS, int KT, int HB>
-__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && UNITS <= 8 ? 2 : 1) mixed_decode_kernel(const MixedAttnParams p) {
+__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && UNITS <= 8 ? 2 : 1) mixed_decode_kernel(const MixedAttnParams p,
+                                                                                                       const mdec::Layout L) {
   using namespace mdec;
   constexpr int THREADS = WARPS * 32, SUB = 32 / KT;
   extern __shared__ __align__(128) uint8_t smem[];
-  const Layout L = layout(p.Hs, p.Hk, p.Ho, p.Hv, p.DP, p.DVP, KT);
   uint8_t* sQ = smem + L.q_off;
   float* sS = reinterpret_cast<float*>(smem + L.s_off);                       // [hs4][s_pitch]
   __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(smem + L.p_off);       // [Ho][p_pitch]
@@ -102,7 +105,7 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && UNITS <= 8 ? 2 : 1) 
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int row = blockIdx.x / p.splits, split = blockIdx.x % p.splits;
-  const int per_k = p.Hs / p.Hk, per_v = p.Ho / p.Hv;
+  const int per_k = L.per_k, per_v = L.per_v;
   const int kchunks8 = (per_k + 7) >> 3, vchunks8 = (per_v + 7) >> 3;
 
   pdl_trigger();
@@ -401,7 +404,10 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && UNITS <= 8 ? 2 : 1) 
     }
     return;
   }
-  float* part = p.scratch + (static_cast<long long>(row) * p.splits + split) * p.Ho * (p.DVP + 2);
+  const long long share_row = static_cast<long long>(row) * p.splits + split;
+  float* part = p.scratch + share_row * p.Ho * p.DVP;
+  float2* stat = reinterpret_cast<float2*>(p.scratch + static_cast<long long>(p.rows) * p.splits * p.Ho * p.DVP) +
+                 share_row * p.Ho;
 #pragma unroll
   for (int i = 0; i < UNITS; ++i) {
     if (i >= u_count) continue;
@@ -409,58 +415,68 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && UNITS <= 8 ? 2 : 1) 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int hl = ch * 8 + (lane & 3) * 2 + (j & 1), d = vtile * 16 + (lane >> 2) + (j >> 1) * 8;
-      if (hl < per_v) part[(g * per_v + hl) * (p.DVP + 2) + d] = acc[i][j];
+      if (hl < per_v) part[(g * per_v + hl) * p.DVP + d] = acc[i][j];
     }
   }
   __syncthreads();                                         // (a row without a tile: the initial values are written here)
-  for (int h = tid; h < p.Ho; h += THREADS) {
-    part[h * (p.DVP + 2) + p.DVP] = sMax[h];
-    part[h * (p.DVP + 2) + p.DVP + 1] = sSum[h];
-  }
+  for (int h = tid; h < p.Ho; h += THREADS) stat[h] = make_float2(sMax[h], sSum[h]);
 }
 
-// One warp per (row, head): the shares' maxima and sums, the sink, then the columns.
-__global__ void __launch_bounds__(128) mixed_merge_kernel(const MixedAttnParams p) {
+// One CTA per (row, head): every warp works out the shares' factors, with the sink, and adds up a quarter of the shares.
+static constexpr int kMergeWarps = 4;
+
+__global__ void __launch_bounds__(kMergeWarps * 32) mixed_merge_kernel(const MixedAttnParams p) {
+  extern __shared__ float sm[];                            // [kMergeWarps][DVP]
   pdl_trigger();
   pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const long long item = blockIdx.x * 4ll + (threadIdx.x >> 5);
-  if (item >= static_cast<long long>(p.rows) * p.Ho) return;
-  const long long row = item / p.Ho;
-  const int h = static_cast<int>(item - row * p.Ho), pitch = p.DVP + 2;
-  const float* part = p.scratch + row * p.splits * p.Ho * pitch + static_cast<long long>(h) * pitch;
-  const long long step = static_cast<long long>(p.Ho) * pitch;
-  // lane s looks after share s (at most 32)
-  const float m = lane < p.splits ? part[lane * step + p.DVP] : -INFINITY;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.x;
+  const long long row = blockIdx.y;
+  const long long step = static_cast<long long>(p.Ho) * p.DVP;
+  const float* part = p.scratch + row * p.splits * step + static_cast<long long>(h) * p.DVP;
+  const float2* stat = reinterpret_cast<const float2*>(p.scratch + static_cast<long long>(p.rows) * p.splits * step) +
+                       row * p.splits * p.Ho + h;
+  // lane s looks after shares s and s + 32
+  const float2 none = make_float2(-INFINITY, 0.f);
+  const float2 a = lane < p.splits ? stat[static_cast<long long>(lane) * p.Ho] : none;
+  const float2 b = lane + 32 < p.splits ? stat[static_cast<long long>(lane + 32) * p.Ho] : none;
   const float z = p.sink ? p.sink[h] * kLog2e : -INFINITY;
-  float top = m;
+  float top = fmaxf(a.x, b.x);
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
   top = fmaxf(top, z);
-  const float f = m == -INFINITY ? 0.f : exp2f(m - top);
-  float l = f > 0.f ? f * part[lane * step + p.DVP + 1] : 0.f;
+  const float fa = a.x == -INFINITY ? 0.f : exp2f(a.x - top), fb = b.x == -INFINITY ? 0.f : exp2f(b.x - top);
+  float l = fa * a.y + fb * b.y;
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
   if (p.sink) l += exp2f(z - top);
+  for (int d = lane * 4; d - lane * 4 < p.DVP; d += 128) { // (a share without keys holds zeros)
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = warp; s < p.splits; s += kMergeWarps) {
+      const float w = __shfl_sync(0xffffffffu, s < 32 ? fa : fb, s & 31);
+      if (d < p.DVP) {
+        const float4 x = *reinterpret_cast<const float4*>(part + s * step + d);
+        o.x = fmaf(w, x.x, o.x);
+        o.y = fmaf(w, x.y, o.y);
+        o.z = fmaf(w, x.z, o.z);
+        o.w = fmaf(w, x.w, o.w);
+      }
+    }
+    if (d < p.DVP) *reinterpret_cast<float4*>(sm + warp * p.DVP + d) = o;
+  }
+  __syncthreads();
   const float inv = l > 0.f ? 1.f / l : 0.f;
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.out_stride + static_cast<long long>(h) * p.DV;
-  for (int d0 = 0; d0 < p.DV; d0 += 64) {                  // (a share without keys holds zeros)
-    const int d = d0 + lane * 2;
-    float2 o = make_float2(0.f, 0.f);
-#pragma unroll 8
-    for (int s = 0; s < p.splits; ++s) {
-      const float w = __shfl_sync(0xffffffffu, f, s);
-      const float2 x = d < p.DVP ? *reinterpret_cast<const float2*>(part + s * step + d) : make_float2(0.f, 0.f);
-      o.x = fmaf(w, x.x, o.x);
-      o.y = fmaf(w, x.y, o.y);
-    }
-    if (d < p.DV) out[d] = __float2bfloat16(o.x * inv);
-    if (d + 1 < p.DV) out[d + 1] = __float2bfloat16(o.y * inv);
+  for (int d = threadIdx.x; d < p.DV; d += kMergeWarps * 32) {
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < kMergeWarps; ++w) o += sm[w * p.DVP + d];
+    out[d] = __float2bfloat16(o * inv);
   }
 }
 
 template <int UNITS, int WARPS, int KT, int HB>
-static int launch_mixed_decode(const MixedAttnParams& p, int bytes, cudaStream_t stream) {
+static int launch_mixed_decode(const MixedAttnParams& p, const mdec::Layout& l, cudaStream_t stream) {
   auto kern = mixed_decode_kernel<UNITS, WARPS, KT, HB>;
   static DeviceOnce once;
   int dev = 0;
@@ -468,32 +484,31 @@ static int launch_mixed_decode(const MixedAttnParams& p, int bytes, cudaStream_t
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -20;
     once.mark(dev);
   }
-  return launch_pdl(kern, dim3(p.rows * p.splits), dim3(WARPS * 32), bytes, stream, 1, p) == cudaSuccess ? 0 : -21;
+  return launch_pdl(kern, dim3(p.rows * p.splits), dim3(WARPS * 32), l.bytes, stream, 1, p, l) == cudaSuccess ? 0 : -21;
 }
 
 template <int KT>
-static int launch_mixed_decode_kt(const MixedAttnParams& p, const mdec::Plan& c, int bytes, cudaStream_t stream) {
+static int launch_mixed_decode_kt(const MixedAttnParams& p, const mdec::Plan& c, cudaStream_t stream) {
+  const mdec::Layout l = mdec::layout(p.Hs, p.Hk, p.Ho, p.Hv, p.DP, p.DVP, KT);
   const int groups = c.warps * (32 / KT);                // lanes' groups that mix a head each
-  if (c.warps == 16) return launch_mixed_decode<16, 16, KT, 2>(p, bytes, stream);
+  if (c.warps == 16) return launch_mixed_decode<16, 16, KT, 2>(p, l, stream);
   if (c.units <= 4) {
-    if (p.Ho <= groups) return launch_mixed_decode<4, 8, KT, 1>(p, bytes, stream);
-    return p.Ho <= 2 * groups ? launch_mixed_decode<4, 8, KT, 2>(p, bytes, stream)
-                              : launch_mixed_decode<4, 8, KT, 4>(p, bytes, stream);
+    if (p.Ho <= groups) return launch_mixed_decode<4, 8, KT, 1>(p, l, stream);
+    return p.Ho <= 2 * groups ? launch_mixed_decode<4, 8, KT, 2>(p, l, stream)
+                              : launch_mixed_decode<4, 8, KT, 4>(p, l, stream);
   }
-  if (c.units <= 8) return p.Ho <= 2 * groups ? launch_mixed_decode<8, 8, KT, 2>(p, bytes, stream)
-                                              : launch_mixed_decode<8, 8, KT, 4>(p, bytes, stream);
-  return launch_mixed_decode<16, 8, KT, 4>(p, bytes, stream);
+  if (c.units <= 8) return p.Ho <= 2 * groups ? launch_mixed_decode<8, 8, KT, 2>(p, l, stream)
+                                              : launch_mixed_decode<8, 8, KT, 4>(p, l, stream);
+  return launch_mixed_decode<16, 8, KT, 4>(p, l, stream);
 }
 
 int mixed_decode(const MixedAttnParams& p, cudaStream_t stream) {
   const mdec::Plan c = mdec::plan(p.Hs, p.Hk, p.Ho, p.Hv, p.DP, p.DVP);
-  if (c.kt == 0 || p.splits > 32 || p.rows != p.B * p.q_len) return -2;
-  const int bytes = mdec::layout(p.Hs, p.Hk, p.Ho, p.Hv, p.DP, p.DVP, c.kt).bytes;
-  const int rc = c.kt == 32 ? launch_mixed_decode_kt<32>(p, c, bytes, stream) : launch_mixed_decode_kt<16>(p, c, bytes, stream);
+  if (c.kt == 0 || p.splits > 64 || p.rows != p.B * p.q_len) return -2;
+  const int rc = c.kt == 32 ? launch_mixed_decode_kt<32>(p, c, stream) : launch_mixed_decode_kt<16>(p, c, stream);
   if (rc != 0 || p.splits == 1) return rc;
-  const long long items = static_cast<long long>(p.rows) * p.Ho;
-  return launch_pdl(mixed_merge_kernel, dim3(static_cast<unsigned>((items + 3) / 4)), dim3(128), 0, stream, 1, p) ==
-                 cudaSuccess ? 0 : -22;
+  return launch_pdl(mixed_merge_kernel, dim3(p.Ho, p.rows), dim3(kMergeWarps * 32), kMergeWarps * p.DVP * sizeof(float), stream,
+                    1, p) == cudaSuccess ? 0 : -22;
 }
 
 }  // namespace b200

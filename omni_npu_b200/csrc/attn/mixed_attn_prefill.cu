@@ -2,9 +2,10 @@
 // heads' products of that (query, key) pair, so the work is cut twice:
 //
 //   mixed_scores_kernel   16 queries x a range of keys, all heads: Q K^T on mma.sync with the queries of a warp's heads in
-//                         registers, capped and lowered into shared memory, then the mixture as fp32 outer products
-//                         (8 output heads x 4 keys per thread); mixed scores to memory in fp32.  The distance bias of a
-//                         tile has 15 + keys values per head: a table, made while the tile before is mixed
+//                         registers; capped and lowered, a score goes to shared memory as a sum of three bf16 numbers
+//                         (24 bits: all of an fp32 significand), so that the mixture is mma.sync products with fp32
+//                         sums as well; mixed scores to memory in fp32.  The distance bias of a tile has 15 + keys
+//                         values per head: a table, made while the tile before is mixed
 //   mixed_values_kernel   128 rows = tokens x heads of a value head: online softmax over the stored scores, sink, P V
 //
 // The scores of as many query tiles as fit into the given buffer are made per call.
@@ -21,59 +22,75 @@ namespace b200 {
 
 namespace mpre {
 constexpr int BQ = 16;                   // queries of a score tile
-constexpr int RANGE = 256;               // keys of a score CTA
+constexpr int PLANES = 3;                // bf16 numbers that make up a score
 
 __device__ __forceinline__ uint32_t piece(int row, int chunk, int width) {
   return static_cast<uint32_t>(row * width * 2 + ((chunk ^ (row & 7)) << 4));
 }
 
 struct Layout {
-  int dk, ho8, s_pitch, d_pitch, k_bytes, s_off, t_off, d_off, bytes;
+  int hs16, ho16, row, head, plane;      // bytes of a query's keys, of a head, of a plane of scores
+  int t_row, t_plane;                    // bytes of a row and of a plane of the mixture
+  int d_pitch, s_off, t_off, d_off, bytes;
+  int per_k;                             // score heads of a key head
+  long long row_step;                    // floats between the rows of scores that a warp writes one after another
 };
-// ring of `stages` key tiles | scores [Hs][16][s_pitch] | talk^T [Hs][ho8] | distance bias [2][Hs][d_pitch]
-__host__ __device__ inline Layout layout(int Hs, int Hk, int Ho, int DP, int bk, int stages) {
-  Layout l;
-  l.dk = DP <= 64 ? 64 : DP <= 128 ? 128 : 256;            // 16 times the kernel's KS
-  l.ho8 = (Ho + 7) / 8 * 8;
-  l.s_pitch = bk + 8;
-  l.k_bytes = Hk * bk * l.dk * 2;
-  l.s_off = stages * l.k_bytes;
-  l.t_off = l.s_off + Hs * BQ * l.s_pitch * 4;
+// key tile [Hk][bk][dk] | scores, planes of [hs16][16][bk] | mixture, planes of [ho16][hs16] | distance bias [2][Hs][d_pitch]
+inline Layout layout(int Hs, int Hk, int Ho, int DP, int bk, int terms) {
+  Layout l{};
+  const int dk = DP <= 64 ? 64 : DP <= 128 ? 128 : 256;
+  l.hs16 = (Hs + 15) / 16 * 16;
+  l.ho16 = (Ho + 15) / 16 * 16;
+  l.row = bk * 2 + 16;                   // (the padding keeps fragment reads and writes off each other's banks)
+  l.head = BQ * l.row + 16;
+  l.plane = l.hs16 * l.head;
+  l.t_row = l.hs16 * 2 + 16;
+  l.t_plane = l.ho16 * l.t_row;
   l.d_pitch = bk + BQ;
-  l.d_off = l.t_off + Hs * l.ho8 * 4;
+  l.s_off = Hk * bk * dk * 2;
+  l.t_off = l.s_off + PLANES * l.plane;
+  l.d_off = l.t_off + terms * l.t_plane;
   l.bytes = l.d_off + 2 * Hs * l.d_pitch * 4;
   return l;
 }
 
 struct Plan {
-  int bk, stages, warps, ks;
+  int bk, warps, ks;
 };
-inline Plan plan(int Hs, int Hk, int Ho, int DP) {
-  if (DP > 256) return {0, 0, 0, 0};
+inline Plan plan(int Hs, int Hk, int Ho, int DP, int terms) {
+  if (DP > 256) return {0, 0, 0};
   const int warps = Hs <= 16 ? 8 : 16, ks = DP <= 64 ? 4 : DP <= 128 ? 8 : 16;
-  const int order[5][3] = {{32, 2, 112}, {32, 2, 226}, {32, 1, 226}, {16, 2, 226}, {16, 1, 226}};
+  const int order[4][2] = {{32, 112}, {16, 112}, {32, 226}, {16, 226}};
   for (const auto& o : order)
-    if (layout(Hs, Hk, Ho, DP, o[0], o[1]).bytes <= o[2] * 1024) return {o[0], o[1], warps, ks};
-  return {0, 0, 0, 0};
+    if ((warps == 8 || o[1] > 112) && layout(Hs, Hk, Ho, DP, o[0], terms).bytes <= o[1] * 1024) return {o[0], warps, ks};
+  return {0, 0, 0};
+}
+
+// x0, x1 as sums of three bf16 numbers each
+__device__ __forceinline__ void split3(float x0, float x1, uint32_t (&w)[PLANES]) {
+#pragma unroll
+  for (int i = 0; i < PLANES; ++i) {
+    w[i] = pack_bf16x2(x0, x1);
+    x0 -= __uint_as_float(w[i] << 16);
+    x1 -= __uint_as_float(w[i] & 0xffff0000u);
+  }
 }
 }  // namespace mpre
 
 bool mixed_prefill_fits(int Hs, int Hk, int Ho, int Hv, int DP, int DVP) {
-  return DVP <= 256 && mpre::plan(Hs, Hk, Ho, DP).bk > 0;
+  return DVP <= 256 && mpre::plan(Hs, Hk, Ho, DP, mpre::PLANES).bk > 0;
 }
 
 // ------------------------------------------------------------- scores
 // KS: steps of 16 along the head size; HPW: heads per warp and pass (16 registers of query per head and 4 steps)
 template <int WARPS, int KS, int HPW, int BK>
-__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_kernel(const MixedAttnParams p, const int stages) {
+__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_kernel(const MixedAttnParams p,
+                                                                                                const mpre::Layout L) {
   using namespace mpre;
   constexpr int THREADS = WARPS * 32, DK = KS * 16;
   extern __shared__ __align__(128) uint8_t smem[];
-  const Layout L = layout(p.Hs, p.Hk, p.Ho, p.DP, BK, stages);
-  float* sS = reinterpret_cast<float*>(smem + L.s_off);
-  float* sT = reinterpret_cast<float*>(smem + L.t_off);
   float* sD = reinterpret_cast<float*>(smem + L.d_off);
-  const uint32_t ring = smem_u32(smem);
+  const uint32_t kt = smem_u32(smem), st = kt + L.s_off, tt = kt + L.t_off;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
   pdl_trigger();
@@ -85,53 +102,66 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_k
   if (tok0 >= q_len) return;
   const int ctx = p.seq_lens[b] - q_len;
   const int hi = ctx + min(q_len, tok0 + BQ);                      // keys that some row sees
-  const int k_begin = blockIdx.y * RANGE, k_end = min(hi, k_begin + RANGE);
+  const int k_begin = blockIdx.y * p.range, k_end = min(hi, k_begin + p.range);
   if (k_begin >= k_end) return;
   const int* bt = p.block_tables + static_cast<long long>(b) * p.max_blocks;
   const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(p.q);
   const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(p.k_cache);
-  const int per = p.Hs / p.Hk;
 
-  // `1 << ll` threads share a row, a thread has the same keys of every tile and walks over the heads
-  const int chunks = p.DP >> 3;
-  int ll = 0;
-  while (ll < 5 && (1 << ll) < chunks) ++ll;
-  const int slots = THREADS >> ll, kstep = min(slots, BK), slot = tid >> ll, li = tid & ((1 << ll) - 1);
-  const int g0 = slots > BK ? slot / BK : 0, gstep = slots > BK ? slots / BK : 1;
+  // DK / 8 threads share a row (32 at most), a thread has the same keys of every tile and walks over the heads
+  constexpr int RT = DK / 8, SLOTS = THREADS / RT, KSTEP = SLOTS < BK ? SLOTS : BK, GSTEP = SLOTS > BK ? SLOTS / BK : 1;
+  const int li = tid % RT, key0 = tid / RT % KSTEP, g0 = GSTEP > 1 ? tid / RT / KSTEP : 0;
+  const bool li_used = li * 8 < p.DP;
+  const uint32_t k_dst = kt + piece(g0 * BK + key0, li, DK);       // (KSTEP is a multiple of 8)
+  const long long g_step = static_cast<long long>(GSTEP) * p.block_size * p.DP;
   auto issue = [&](int i) {
     const int n0 = k_begin + i * BK;
-    if (n0 < k_end) {
-      const uint32_t dst = ring + (stages == 2 ? i & 1 : 0) * L.k_bytes;
-      for (int j = slot & (kstep - 1); j < BK; j += kstep) {
-        const int key = n0 + j;
-        const bool ok = key < k_end;
-        const __nv_bfloat16* row0 = ok ? kc + cache_row(p, bt, key, g0, p.Hk) * p.DP : kc;
-        const long long step = ok ? static_cast<long long>(gstep) * p.block_size * p.DP : 0;
-        const int sz = ok ? 16 : 0;
-        for (int c = li; c < chunks; c += 1 << ll) {
-          const __nv_bfloat16* src = ok ? row0 + c * 8 : row0;
-          uint32_t to = dst + piece(g0 * BK + j, c, DK);
-#pragma unroll 4
-          for (int g = g0; g < p.Hk; g += gstep, src += step, to += gstep * BK * DK * 2)
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to), "l"(src), "r"(sz) : "memory");
+    if (n0 < k_end && li_used) {
+#pragma unroll
+      for (int j = 0; j < BK / KSTEP; ++j) {
+        const int key = n0 + key0 + j * KSTEP;
+        uint32_t to = k_dst + j * KSTEP * DK * 2;
+        if (key < k_end) {
+          const __nv_bfloat16* src = kc + cache_row(p, bt, key, g0, p.Hk) * p.DP + li * 8;
+          for (int g = g0; g < p.Hk; g += GSTEP, src += g_step, to += GSTEP * BK * DK * 2)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(to), "l"(src) : "memory");
+        } else {
+          for (int g = g0; g < p.Hk; g += GSTEP, to += GSTEP * BK * DK * 2)
+            asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};" ::"r"(to), "r"(0) : "memory");
         }
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (stages == 2) issue(0);
-  for (int i = tid; i < p.Hs * L.ho8; i += THREADS) {
-    const int g = i / L.ho8, h = i - g * L.ho8;
-    sT[i] = h < p.Ho ? p.talk[h * p.Hs + g] * kLog2e : 0.f;
+  issue(0);
+  // the mixture (one plane when bf16 holds it exactly), zero beyond the heads; score rows beyond the heads
+  for (int i = tid; i < L.ho16 * (L.hs16 >> 1); i += THREADS) {
+    const int h = i / (L.hs16 >> 1), g = (i - h * (L.hs16 >> 1)) * 2;
+    uint32_t w[PLANES];
+    split3(h < p.Ho && g < p.Hs ? p.talk[h * p.Hs + g] : 0.f, h < p.Ho && g + 1 < p.Hs ? p.talk[h * p.Hs + g + 1] : 0.f, w);
+#pragma unroll
+    for (int t = 0; t < PLANES; ++t)
+      if (t < p.talk_terms) *reinterpret_cast<uint32_t*>(smem + L.t_off + t * L.t_plane + h * L.t_row + g * 2) = w[t];
   }
-  // distance bias of tile i: entry x of a head is for distance base + x, base = first query - last key
+  for (int t = 0; t < PLANES; ++t)
+    for (int i = p.Hs * L.head + tid * 4; i < L.plane; i += THREADS * 4)
+      *reinterpret_cast<uint32_t*>(smem + L.s_off + t * L.plane + i) = 0u;
+  ScoreConst c = score_const(p);                           // scores in units of log2 e
+  if (c.cap > 0.f) c.cap *= kLog2e;
+  else c.in *= kLog2e;
+  // what the score of tile i starts from, cap - distance bias: entry x of a head is for distance base + x, base =
+  // first query - last key
   auto make_bias = [&](int i) {
     if (k_begin + i * BK >= k_end) return;
     const int base = ctx + tok0 - (k_begin + i * BK + BK - 1);
-    float* dst = sD + (i & 1) * p.Hs * L.d_pitch;
-    for (int e = tid; e < p.Hs * (BK + BQ); e += THREADS) {
-      const int g = e / (BK + BQ), x = e - g * (BK + BQ);
-      dst[e] = p.r1 ? distance_bias(__ldg(p.r1 + g) * kLn2, __ldg(p.r2 + g), fmaxf(static_cast<float>(base + x), 0.f)) : 0.f;
+    constexpr int W = BK + BQ, GROUP = THREADS / 16;               // 16 threads per head, W / 16 entries each
+    const int x0 = tid & 15;
+    for (int g = tid >> 4; g < p.Hs; g += GROUP) {
+      const float r1 = p.r1 ? __ldg(p.r1 + g) : 0.f, r2 = p.r1 ? __ldg(p.r2 + g) : 0.f;
+      float* dst = sD + ((i & 1) * p.Hs + g) * W + x0;
+#pragma unroll
+      for (int x = 0; x < W; x += 16)
+        dst[x] = c.cap - distance_bias(r1, r2, fmaxf(static_cast<float>(base + x0 + x), 0.f));
     }
   };
   make_bias(0);
@@ -168,21 +198,25 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_k
   const int passes = (p.Hs + WARPS * HPW - 1) / (WARPS * HPW);
   if (passes == 1) load_q(0);
 
-  const ScoreConst c = score_const(p);
+  uint32_t k_head[HPW];                                    // the key head of this warp's heads (of the first pass)
+#pragma unroll
+  for (int j = 0; j < HPW; ++j) k_head[j] = (warp * HPW + j) / L.per_k * BK * DK * 2;
+  const uint32_t k_lane = kt + ((lane & 7) + ((lane >> 4) << 3)) * DK * 2;
+  // the first row of scores that this warp writes, and where its fragments lie
+  constexpr int HALVES = BK / 16, ROWS_STEP = WARPS / HALVES;
+  const int row0 = warp / HALVES, k16 = warp % HALVES;
+  const uint32_t s_lane = st + ((lane & 7) + ((lane >> 3) & 1) * 8) * L.head + row0 * (BK * 2 + 16) + k16 * 32 + (lane >> 4) * 16;
+  const uint32_t t_lane = tt + (lane & 15) * L.t_row + (lane >> 4) * 16;
+  float* out_tile = p.scratch + (((static_cast<long long>(b) * p.tiles + blockIdx.x) * BQ + row0) * p.Ho + (lane >> 2)) * p.pitch +
+                    k_begin + k16 * 16 + (lane & 3) * 2;
   const int tiles = (k_end - k_begin + BK - 1) / BK;
   const int ks_used = p.DP >> 4;
   uint32_t kx[4];                                          // swizzled chunk of a row, by step modulo 4
 #pragma unroll
   for (int i = 0; i < 4; ++i) kx[i] = ((i * 2 + ((lane >> 3) & 1)) ^ (lane & 7)) << 4;
   for (int it = 0; it < tiles; ++it) {
-    if (stages == 1) {
-      if (it) __syncthreads();
-      issue(it);
-    }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    if (stages == 2) issue(it + 1);
-    const uint32_t kt = ring + (stages == 2 ? it & 1 : 0) * L.k_bytes;
+    __syncthreads();                                       // keys and bias are there; the scores before are used up
     const int n0 = k_begin + it * BK;
 
     for (int pass = 0; pass < passes; ++pass) {
@@ -191,77 +225,97 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_k
       for (int j = 0; j < HPW; ++j) {
         const int g = (pass * WARPS + warp) * HPW + j;
         if (g >= p.Hs) continue;
-        const uint32_t k_at = kt + ((g / per) * BK + (lane & 7) + ((lane >> 4) << 3)) * DK * 2;
+        const uint32_t k_at = k_lane + (pass == 0 ? k_head[j] : g / L.per_k * BK * DK * 2);
         float s[BK / 8][4];
 #pragma unroll
         for (int n = 0; n < BK / 8; ++n)
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
-#pragma unroll
-        for (int ks = 0; ks < KS; ++ks) {
+        const uint32_t k_of[4] = {k_at + kx[0], k_at + kx[1], k_at + kx[2], k_at + kx[3]};
+        static_for<KS>([&](auto step) {
+          constexpr int ks = decltype(step)::value;
           if (ks < ks_used) {
-#pragma unroll
-            for (int n = 0; n < BK / 16; ++n) {
+            static_for<BK / 16>([&](auto part) {
+              constexpr int n = decltype(part)::value;
               uint32_t kf[4];
-              ldmatrix_x4(kf, k_at + n * 16 * DK * 2 + (ks >> 2) * 128 + kx[ks & 3]);
+              ldmatrix_x4_at<n * 16 * DK * 2 + (ks >> 2) * 128>(kf, k_of[ks & 3]);
               mma_bf16_16816(s[2 * n], qf[j][ks], kf[0], kf[1]);
               mma_bf16_16816(s[2 * n + 1], qf[j][ks], kf[2], kf[3]);
-            }
+            });
           }
-        }
-        float* dst = sS + g * BQ * L.s_pitch + (lane >> 2) * L.s_pitch + (lane & 3) * 2;
-        const float* bias = sD + ((it & 1) * p.Hs + g) * L.d_pitch + BK - 1 + (lane >> 2) - (lane & 3) * 2;
+        });
+        uint8_t* dst = smem + L.s_off + g * L.head + (lane >> 2) * (BK * 2 + 16) + (lane & 3) * 4;
+        const float* bias = sD + ((it & 1) * p.Hs + g) * (BK + BQ) + BK - 1 + (lane >> 2) - (lane & 3) * 2;
         auto put = [&](auto cap) {
 #pragma unroll
           for (int n = 0; n < BK / 8; ++n)
 #pragma unroll
-            for (int r = 0; r < 2; ++r)
-              *reinterpret_cast<float2*>(dst + r * 8 * L.s_pitch + n * 8) =
-                  make_float2(capped_score<decltype(cap)::value>(c, s[n][2 * r]) - bias[r * 8 - n * 8],
-                              capped_score<decltype(cap)::value>(c, s[n][2 * r + 1]) - bias[r * 8 - n * 8 - 1]);
+            for (int r = 0; r < 2; ++r) {
+              uint32_t w[PLANES];
+              split3(biased_score<decltype(cap)::value>(c, s[n][2 * r], bias[r * 8 - n * 8]),
+                     biased_score<decltype(cap)::value>(c, s[n][2 * r + 1], bias[r * 8 - n * 8 - 1]), w);
+#pragma unroll
+              for (int t = 0; t < PLANES; ++t)
+                *reinterpret_cast<uint32_t*>(dst + t * L.plane + r * 8 * (BK * 2 + 16) + n * 16) = w[t];
+            }
         };
         if (c.cap > 0.f) put(std::true_type{});
         else put(std::false_type{});
       }
     }
-    __syncthreads();
+    __syncthreads();                                       // scores are there; the keys are used up
+    issue(it + 1);
     make_bias(it + 1);
 
-    // ---- mixture: an item = 8 output heads x 4 keys of a query
-    constexpr int GROUPS = BQ * BK / 4;
-    const int items = (L.ho8 >> 3) * GROUPS;
-    for (int item = tid; item < items; item += THREADS) {
-      const int hc = item / GROUPS * 8, grp = item % GROUPS;
-      const int row = grp / (BK / 4), key = grp % (BK / 4) * 4;
-      float o[8][4];
+    // ---- mixture: 16 output heads x 16 keys of a query per step
+    float* out = out_tile;
+    uint32_t s_at = s_lane;
+#pragma unroll 1
+    for (int row = row0; row < BQ; row += ROWS_STEP, out += L.row_step, s_at += ROWS_STEP * (BK * 2 + 16)) {
+      if (tok0 + row >= q_len) break;
+      uint32_t t_ob = t_lane;
+      float* o_ob = out;
+#pragma unroll 1
+      for (int left = p.Ho - (lane >> 2), ob = 0; ob < L.ho16; ob += 16, left -= 16) {
+        float o[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        uint32_t s_kb = s_at, t_kb = t_ob;
+#pragma unroll 1
+        for (int kb = 0; kb < L.hs16; kb += 16, s_kb += 16 * L.head, t_kb += 32) {
+          uint32_t sf[PLANES][4], tf[4];
 #pragma unroll
-      for (int h = 0; h < 8; ++h)
+          for (int t = 0; t < PLANES; ++t) ldmatrix_x4_trans(sf[t], s_kb + t * L.plane);
+          ldmatrix_x4(tf, t_kb);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[h][e] = 0.f;
-      const float* src = sS + row * L.s_pitch + key;
-      const float* t = sT + hc;
-#pragma unroll 4
-      for (int g = 0; g < p.Hs; ++g) {
-        const float4 a = *reinterpret_cast<const float4*>(src + g * BQ * L.s_pitch);
-        const float4 w0 = *reinterpret_cast<const float4*>(t + g * L.ho8), w1 = *reinterpret_cast<const float4*>(t + g * L.ho8 + 4);
-        const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+          for (int t = PLANES - 1; t >= 0; --t) {
+            mma_bf16_16816(o[0], tf, sf[t][0], sf[t][1]);
+            mma_bf16_16816(o[1], tf, sf[t][2], sf[t][3]);
+          }
+          if (p.talk_terms > 1) {                          // (products below 2^-24 are left out)
+            ldmatrix_x4(tf, t_kb + L.t_plane);
 #pragma unroll
-        for (int h = 0; h < 8; ++h) {
-          o[h][0] = fmaf(w[h], a.x, o[h][0]);
-          o[h][1] = fmaf(w[h], a.y, o[h][1]);
-          o[h][2] = fmaf(w[h], a.z, o[h][2]);
-          o[h][3] = fmaf(w[h], a.w, o[h][3]);
+            for (int t = 1; t >= 0; --t) {
+              mma_bf16_16816(o[0], tf, sf[t][0], sf[t][1]);
+              mma_bf16_16816(o[1], tf, sf[t][2], sf[t][3]);
+            }
+            ldmatrix_x4(tf, t_kb + 2 * L.t_plane);
+            mma_bf16_16816(o[0], tf, sf[0][0], sf[0][1]);
+            mma_bf16_16816(o[1], tf, sf[0][2], sf[0][3]);
+          }
         }
-      }
-      if (tok0 + row < q_len) {
-        float* dst = p.scratch +
-                     (((static_cast<long long>(b) * p.tiles + blockIdx.x) * BQ + row) * p.Ho + hc) * p.pitch + n0 + key;
-#pragma unroll
-        for (int h = 0; h < 8; ++h)
-          if (hc + h < p.Ho)
-            *reinterpret_cast<float4*>(dst + h * p.pitch) = make_float4(o[h][0], o[h][1], o[h][2], o[h][3]);
+        if (left > 0) {
+          *reinterpret_cast<float2*>(o_ob) = make_float2(o[0][0], o[0][1]);
+          *reinterpret_cast<float2*>(o_ob + 8) = make_float2(o[1][0], o[1][1]);
+        }
+        o_ob += 8 * p.pitch;
+        if (left > 8) {
+          *reinterpret_cast<float2*>(o_ob) = make_float2(o[0][2], o[0][3]);
+          *reinterpret_cast<float2*>(o_ob + 8) = make_float2(o[1][2], o[1][3]);
+        }
+        o_ob += 8 * p.pitch;
+        t_ob += 16 * L.t_row;
       }
     }
+    out_tile += BK;
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
@@ -303,11 +357,13 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
 
   const int rows_live = (tok_end - m0) * hc;                       // rows: (token, head of the group)
   const float* sbase = p.scratch + ((static_cast<long long>(b) * p.tiles * mpre::BQ + (m0 - first)) * p.Ho +
-                                    vh * per + head0) * p.pitch;
-  auto srow = [&](int r) {
-    const int tok = r / hc;
-    return sbase + (static_cast<long long>(tok) * p.Ho + (r - tok * hc)) * p.pitch;
-  };
+                                    vh * per + head0) * p.pitch + (tid & 15) * 4;
+  int srow[BM / 16];                                               // score rows that this thread copies from
+#pragma unroll
+  for (int i = 0; i < BM / 16; ++i) {
+    const int r = (tid >> 4) + i * 16, tok = r / hc;
+    srow[i] = r < rows_live ? tok * p.Ho + (r - tok * hc) : -1;
+  }
   auto issue = [&](int it) {
     if (it < tiles) {
       // four threads per key row, 16-byte pieces dealt out in turn
@@ -323,10 +379,9 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
       const uint32_t sdst = s0 + (it & 1) * S_BYTES + (tid & 15) * 16;
 #pragma unroll
       for (int i = 0; i < BM / 16; ++i) {
-        const int rr = (tid >> 4) + i * 16;
-        if (rows_live > rr)
-          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sdst + rr * S_PITCH * 4),
-                       "l"(srow(rr) + it * BN + (tid & 15) * 4) : "memory");
+        if (srow[i] >= 0)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sdst + ((tid >> 4) + i * 16) * S_PITCH * 4),
+                       "l"(sbase + srow[i] * p.pitch + it * BN) : "memory");
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -350,6 +405,9 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
     row_max[r] = ok && p.sink ? p.sink[h] * kLog2e : -INFINITY;
     row_sum[r] = ok && p.sink && (lane & 3) == 0 ? 1.f : 0.f;
   }
+  uint32_t vx[4];                                                  // swizzled chunk of a value row, by step modulo 4
+#pragma unroll
+  for (int i = 0; i < 4; ++i) vx[i] = (lane & 15) * DV * 2 + (((i * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
   const int w_hi = min(ctx + tok_end - 1, ctx + m0 + (warp * 16 + 15) / hc);       // last position of this warp's rows
 
   for (int it = 0; it < tiles; ++it) {
@@ -368,10 +426,16 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const float2 x = *reinterpret_cast<const float2*>(st + r * 8 * S_PITCH + i * 8);
-          const int key = n0 + i * 8 + (lane & 3) * 2;
-          s[i][2 * r] = interior || key <= pos[r] ? x.x : -INFINITY;
-          s[i][2 * r + 1] = interior || key + 1 <= pos[r] ? x.y : -INFINITY;
+          s[i][2 * r] = x.x;
+          s[i][2 * r + 1] = x.y;
         }
+      if (!interior) {
+#pragma unroll
+        for (int i = 0; i < BN / 8; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (n0 + i * 8 + (lane & 3) * 2 + (j & 1) > pos[j >> 1]) s[i][j] = -INFINITY;
+      }
       const uint32_t vt = v0 + (it & 1) * V_BYTES;
       float corr[2], m_use[2];
 #pragma unroll
@@ -398,23 +462,24 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
 #pragma unroll
           for (int j = 0; j < 4; ++j) o_acc[i][j] *= corr[j >> 1];
       }
-#pragma unroll
-      for (int ks = 0; ks < BN / 16; ++ks) {
+      const uint32_t v_of[4] = {vt + vx[0], vt + vx[1], vt + vx[2], vt + vx[3]};
+      static_for<BN / 16>([&](auto step) {
+        constexpr int ks = decltype(step)::value;
         uint32_t pa[4];
         pa[0] = pack_bf16x2(s[2 * ks][0], s[2 * ks][1]);
         pa[1] = pack_bf16x2(s[2 * ks][2], s[2 * ks][3]);
         pa[2] = pack_bf16x2(s[2 * ks + 1][0], s[2 * ks + 1][1]);
         pa[3] = pack_bf16x2(s[2 * ks + 1][2], s[2 * ks + 1][3]);
-#pragma unroll
-        for (int dt = 0; dt < DV / 16; ++dt) {
+        static_for<DV / 16>([&](auto part) {
+          constexpr int dt = decltype(part)::value;
           if (dt * 16 < p.DVP) {
             uint32_t vf[4];
-            ldmatrix_x4_trans(vf, vt + tile_offset<DV>(ks * 16 + (lane & 15), dt * 2 + (lane >> 4)));
+            ldmatrix_x4_trans_at<ks * 16 * DV * 2 + (dt >> 2) * 128>(vf, v_of[dt & 3]);
             mma_bf16_16816(o_acc[2 * dt], pa, vf[0], vf[1]);
             mma_bf16_16816(o_acc[2 * dt + 1], pa, vf[2], vf[3]);
           }
-        }
-      }
+        });
+      });
     }
     __syncthreads();
   }
@@ -445,7 +510,7 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
 }
 
 template <int WARPS, int KS, int HPW, int BK>
-static int launch_scores(const MixedAttnParams& p, int stages, cudaStream_t stream) {
+static int launch_scores(const MixedAttnParams& p, cudaStream_t stream) {
   auto kern = mixed_scores_kernel<WARPS, KS, HPW, BK>;
   static DeviceOnce once;
   int dev = 0;
@@ -453,16 +518,18 @@ static int launch_scores(const MixedAttnParams& p, int stages, cudaStream_t stre
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -20;
     once.mark(dev);
   }
-  const int bytes = mpre::layout(p.Hs, p.Hk, p.Ho, p.DP, BK, stages).bytes;
-  const dim3 grid(p.tiles, (p.max_keys + mpre::RANGE - 1) / mpre::RANGE, p.B);
-  return launch_pdl(kern, grid, dim3(WARPS * 32), bytes, stream, 1, p, stages) == cudaSuccess ? 0 : -21;
+  mpre::Layout l = mpre::layout(p.Hs, p.Hk, p.Ho, p.DP, BK, p.talk_terms);
+  l.per_k = p.Hs / p.Hk;
+  l.row_step = WARPS / (BK / 16) * p.Ho * p.pitch;
+  const dim3 grid(p.tiles, (p.max_keys + p.range - 1) / p.range, p.B);
+  return launch_pdl(kern, grid, dim3(WARPS * 32), l.bytes, stream, 1, p, l) == cudaSuccess ? 0 : -21;
 }
 
 template <int WARPS, int BK>
 static int launch_scores_ks(const MixedAttnParams& p, const mpre::Plan& c, cudaStream_t stream) {
-  if (c.ks == 4) return launch_scores<WARPS, 4, 4, BK>(p, c.stages, stream);
-  if (c.ks == 8) return launch_scores<WARPS, 8, 2, BK>(p, c.stages, stream);
-  return launch_scores<WARPS, 16, 1, BK>(p, c.stages, stream);
+  if (c.ks == 4) return launch_scores<WARPS, 4, 4, BK>(p, stream);
+  if (c.ks == 8) return launch_scores<WARPS, 8, 2, BK>(p, stream);
+  return launch_scores<WARPS, 16, 1, BK>(p, stream);
 }
 
 template <int DV>
@@ -482,9 +549,14 @@ static int launch_values(const MixedAttnParams& p, cudaStream_t stream) {
   return launch_pdl(kern, grid, dim3(mval::THREADS), SMEM, stream, 1, p, heads) == cudaSuccess ? 0 : -21;
 }
 
-int mixed_prefill(const MixedAttnParams& p, cudaStream_t stream) {
-  const mpre::Plan c = mpre::plan(p.Hs, p.Hk, p.Ho, p.DP);
-  if (c.bk == 0 || p.DVP > 256) return -2;
+int mixed_prefill(const MixedAttnParams& in, cudaStream_t stream) {
+  MixedAttnParams p = in;
+  const mpre::Plan c = mpre::plan(p.Hs, p.Hk, p.Ho, p.DP, p.talk_terms);
+  if (c.bk == 0 || p.DVP > 256 || (p.talk_terms != 1 && p.talk_terms != mpre::PLANES)) return -2;
+  // keys of a score CTA: longer ranges where there are CTAs enough
+  p.range = 128;
+  while (p.range < 1024 && static_cast<long long>(p.tiles) * p.B * ((p.max_keys + 2 * p.range - 1) / (2 * p.range)) >= 888)
+    p.range *= 2;
   int rc;
   if (c.bk == 32) rc = c.warps == 8 ? launch_scores_ks<8, 32>(p, c, stream) : launch_scores_ks<16, 32>(p, c, stream);
   else rc = c.warps == 8 ? launch_scores_ks<8, 16>(p, c, stream) : launch_scores_ks<16, 16>(p, c, stream);

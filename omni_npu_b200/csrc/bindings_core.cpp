@@ -94,8 +94,8 @@ int b200_mixed_attention(const void* q, const void* k_cache, const void* v_cache
                          const int* cu_q, const int* seq_lens, const float* r1, const float* r2, const float* talk,
                          const float* sink, int B, int rows, int q_len, int max_keys, int max_blocks, int block_size,
                          int Hs, int Hk, int Ho, int Hv, int D, int DV, int DP, int DVP, long long q_stride,
-                         long long out_stride, float scale, float softcap, int kind, int splits, float* scratch, int tile0,
-                         int tiles, long long pitch, int is_fp32, cudaStream_t stream);
+                         long long out_stride, float scale, float softcap, int kind, int talk_terms, int splits, float* scratch,
+                         int tile0, int tiles, long long pitch, int is_fp32, cudaStream_t stream);
 int b200_post_norm_residual(float* residual, long long res_stride, const int* ids, const void* table, int table_rows,
                             const void* y, long long y_stride, const void* w, int groups, const void* out_w,
                             int out_groups, void* out, long long out_stride, float eps, long long rows, int W, int n_true,
@@ -894,8 +894,8 @@ void mixed_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cac
                      const c10::optional<Tensor>& cu_q, const Tensor& seq_lens, int64_t num_seqs, int64_t q_len,
                      int64_t max_keys, int64_t head_dim, int64_t head_dim_v, double scale, double softcap,
                      const c10::optional<Tensor>& r1, const c10::optional<Tensor>& r2, const Tensor& talk,
-                     const c10::optional<Tensor>& sink, int64_t kind, int64_t splits, const c10::optional<Tensor>& scratch,
-                     int64_t tile0, int64_t tiles) {
+                     const c10::optional<Tensor>& sink, int64_t kind, int64_t talk_terms, int64_t splits,
+                     const c10::optional<Tensor>& scratch, int64_t tile0, int64_t tiles) {
   const auto dt = q.scalar_type();
   const bool f32 = is_f32(q);
   CHECK_ROWS(q, dt);
@@ -941,7 +941,7 @@ void mixed_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cac
                              (int)T, (int)q_len, (int)max_keys, (int)block_tables.stride(0), (int)k_cache.size(2), (int)Hs,
                              (int)k_cache.size(1), (int)Ho, (int)v_cache.size(1), (int)head_dim, (int)head_dim_v,
                              (int)k_cache.size(3), (int)v_cache.size(3), q.stride(0), out.stride(0), (float)scale,
-                             (float)softcap, (int)kind, (int)splits, sp, (int)tile0, (int)tiles, pitch, f32 ? 1 : 0,
+                             (float)softcap, (int)kind, (int)talk_terms, (int)splits, sp, (int)tile0, (int)tiles, pitch, f32 ? 1 : 0,
                              cur_stream()),
         "mixed_attention");
 }

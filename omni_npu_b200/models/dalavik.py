@@ -170,9 +170,11 @@ class MixedAttentionMixer(Mixer):
                                    ("r2", a.r2, False), ("sink", a.sink, True), ("talk", a.talk, True)):
             self.expect_vector(want, p + name, param, split)
 
+    @torch.no_grad()
     def clear_padding(self) -> None:
         super().clear_padding()
         self.clear(self.in_proj, self.width)
+        self.attn.talk_exact = bool((self.attn.talk.bfloat16().float() == self.attn.talk).all())
 
 
 # --------------------------------------------------------------------- the model

@@ -767,21 +767,22 @@ MIXED_SCORE_BYTES = int(os.environ.get("OMNI_B200_MIXED_SCORE_MB", "512")) << 20
 
 
 def mixed_decode_splits(num_rows: int, keys: int, sms: int = 148) -> int:
-    """CTAs that share the keys of a decode row: at least 64 keys each, two CTAs per SM."""
-    return max(1, min(32, 2 * sms // max(1, num_rows), (keys + 63) // 64))
+    """CTAs that share the keys of a decode row: at least 32 keys each, two CTAs per SM."""
+    return max(1, min(64, 2 * sms // max(1, num_rows), (keys + 31) // 32))
 
 
 def mixed_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor,
                     block_tables: torch.Tensor, cu_q: Optional[torch.Tensor], seq_lens: torch.Tensor, num_seqs: int,
                     max_q_len: int, head_dim: int, head_dim_v: int, scale: float, softcap: float, bias,
                     talk: torch.Tensor, sink: Optional[torch.Tensor], max_seq_len: int = 0, splits: int = 0,
-                    variant: int = 0) -> None:
+                    variant: int = 0, talk_exact: bool = False) -> None:
     """Attention over the paged cache whose heads mix their scores before the softmax (csrc/attn/mixed_attn.cuh),
     written into ``out`` [T, >= Ho * Dv].  q [T, Hs * Dk]; ``softcap`` 0: none; ``bias`` = (r1, r2) fp32 [Hs] or
     None: r1 ln(1 + r2 distance) is taken off; ``talk`` fp32 [Ho, Hs]; ``sink`` fp32 [Ho] or None: score of a key
     without a value.  Score head h reads key head h / (Hs / Hk), output head h value head h / (Ho / Hv).
     ``cu_q``: query offsets of prompt portions; None = decode step with ``max_q_len`` rows per sequence.
-    ``variant``: 0 = by shape, 1 = the tensor-core kernels or an error, 2 = the plain kernel."""
+    ``variant``: 0 = by shape, 1 = the tensor-core kernels or an error, 2 = the plain kernel.  ``talk_exact``: bf16
+    holds every element of ``talk`` (a third of the products of the mixture)."""
     if not q.is_cuda:
         return ref.mixed_attention(q, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len, head_dim,
                                    head_dim_v, scale, softcap, bias, talk, sink)
@@ -790,10 +791,11 @@ def mixed_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     r1, r2 = bias if bias is not None else (None, None)
     args = (q, k_cache, v_cache, out, block_tables, cu_q, seq_lens, num_seqs, max_q_len, keys, head_dim, head_dim_v, scale,
             softcap, r1, r2, talk, sink)
+    terms = 1 if talk_exact else 3
     kind = core.mixed_attention_kind(q, k_cache, v_cache, talk, cu_q is not None, variant)     # 0 plain, 1 tensor cores
     if kind == 0:
         _count(1)
-        core.mixed_attention(*args, 0, 1, None, 0, 0)
+        core.mixed_attention(*args, 0, terms, 1, None, 0, 0)
         return
     st = device_state(q.device)
     if cu_q is None:
@@ -804,7 +806,7 @@ def mixed_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             nbytes = rows * splits * talk.shape[0] * (v_cache.shape[3] + 2) * 4
             scratch = st.decode_scratch(torch.cuda.current_stream(q.device).cuda_stream, nbytes)
         _count(2 if splits > 1 else 1)
-        core.mixed_attention(*args, 1, splits, scratch, 0, 0)
+        core.mixed_attention(*args, 1, terms, splits, scratch, 0, 0)
         return
     # prompt portions: the mixed scores of a run of query tiles go through memory
     tile, tiles, pitch = 16, (max_q_len + 15) // 16, (keys + 63) // 64 * 64
@@ -812,7 +814,7 @@ def mixed_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     scores = torch.empty(num_seqs * run * tile * talk.shape[0] * pitch, dtype=torch.float32, device=q.device)
     for t0 in range(0, tiles, run):
         _count(2)
-        core.mixed_attention(*args, 1, 1, scores, t0, min(run, tiles - t0))
+        core.mixed_attention(*args, 1, terms, 1, scores, t0, min(run, tiles - t0))
 
 
 # ----------------------------------------------------------- 32-bit residual stream

@@ -859,21 +859,21 @@ def dalavik_kernels(size) -> List[dict]:
               like_prep, (t * (2 * h + 4 * kvh) * d * 2,))
         o, lo = torch.empty(t, h * e, **bf), torch.empty(t, h * d, **bf)
         r1, r2, sink = torch.rand(h, **f32), torch.rand(h, **f32) * 0.1, torch.randn(h, **f32)
-        talk = torch.eye(h, **f32) + 0.1 * torch.randn(h, h, **f32)
+        talk = (torch.eye(h, **f32) + 0.1 * torch.randn(h, h, **f32)).bfloat16().float()
         qc = q.contiguous()
 
         def like_attn():
-            if not pre:
+            if not pre and d == 128:
                 return ops.gqa_decode(qc, kc, lvc, bt, lens, n, h, d ** -0.5, 1, 0, max_seq_len=ctx)
-            if d == e and d in (64, 128):
+            if d == e == 128:
                 return ops.gqa_prefill(qc, kc, vc, bt, cu, lens, n, rows, h, d ** -0.5, True, 0)
-            return ops.gated_attention(qc, None, kc, vc, o, bt, cu, lens, n, rows, h, d, e, d ** -0.5, 0, None,
+            return ops.gated_attention(qc, None, kc, vc, o, bt, cu if pre else None, lens, n, rows, h, d, e, d ** -0.5, 0, None,
                                        max_seq_len=ctx)
         kv = n * kvh * ctx * 2
-        le = e if pre else d
+        le = e if pre or d != 128 else d
         entry("attention with mixed scores (like: grouped-query attention)",
               lambda: ops.mixed_attention(qc, kc, vc, o, bt, cu if pre else None, lens, n, rows, d, e, d ** -0.5, SOFTCAP,
-                                          (r1, r2), talk, sink, max_seq_len=ctx),
+                                          (r1, r2), talk, sink, max_seq_len=ctx, talk_exact=True),
               (kv * (d + e) + t * h * (d + e) * 2, 2.0 * pairs * (d + e), 2.0 * pairs * h), like_attn,
               (kv * (d + le) + t * h * (d + le) * 2, 2.0 * pairs * (d + le)))
         del kc, vc, lvc, y, q, kk, vv, qc, res

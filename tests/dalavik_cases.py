@@ -188,10 +188,10 @@ def score_constants(n: int, g: torch.Generator, bias=True, sink=True):
 
 
 def check_mixed_scores(device, dtype, n, kv, dim, vdim, t, bs, queries, planted, softcap=20.0, bias=True, sink=True,
-                       variant=0, splits=0, ranks=1) -> None:
+                       variant=0, splits=0, ranks=1, exact=False) -> None:
     """The last ``queries`` rows of a sequence, as a prompt portion and one by one.  Every head's score of key
     ``planted`` is close to the cap for every query that sees it, and the mixture is such that it outweighs the rest.
-    ``ranks`` > 1: the output heads of each of so many ranks."""
+    ``ranks`` > 1: the output heads of each of so many ranks.  ``exact``: a mixture that bf16 holds."""
     from omni_npu_b200 import ops
     g = torch.Generator().manual_seed(1000 * n + t + planted)
     q, k, v = (torch.randn(t, m, dd, generator=g) for m, dd in ((n, dim), (kv, dim), (kv, vdim)))
@@ -202,6 +202,8 @@ def check_mixed_scores(device, dtype, n, kv, dim, vdim, t, bs, queries, planted,
     q, k, v = (x.to(dtype) for x in (q, k, v))
     r, talk, sinks = score_constants(n, g, bias, sink)
     talk = talk + (1 - talk.sum(1, keepdim=True)).clamp(min=0) / n                       # every row adds up to one or more
+    if exact:
+        talk = talk.bfloat16().float()
     scale = dim ** -0.5
     d64 = lambda x: None if x is None else x.double()                                    # noqa: E731
     want = oracle.mixed_attend(q.double(), k.double(), v.double(), scale, softcap, *(map(d64, r) if r else (None, None)),
@@ -223,7 +225,8 @@ def check_mixed_scores(device, dtype, n, kv, dim, vdim, t, bs, queries, planted,
         def run(q_, cu, lens, b, m, sp=0):
             wide = torch.full((q_.shape[0], ho * vdim + 24), 7.0, dtype=dtype, device=device)
             ops.mixed_attention(q_, kc, vr, wide[:, : ho * vdim], bt, cu, lens, b, m, dim, vdim, scale, softcap,
-                                tuple(map(dd, r)) if r else None, *consts, max_seq_len=t, variant=variant, splits=sp)
+                                tuple(map(dd, r)) if r else None, *consts, max_seq_len=t, variant=variant, splits=sp,
+                                talk_exact=exact)
             assert float((wide[:, ho * vdim:] - 7.0).abs().max()) == 0.0
             return wide[:, : ho * vdim].double().cpu()
 

@@ -86,7 +86,8 @@ SHAPES = [(1, 1, 16, 16), (4, 2, 24, 20), (7, 1, 18, 22), (8, 2, 128, 128), (12,
 @pytest.mark.parametrize("shape", SHAPES)
 @pytest.mark.parametrize("planted", [0, 31, 32, 127, 144, 199])
 def test_mixed_scores(shape, planted):
-    cases.check_mixed_scores("cuda", torch.bfloat16, *shape, 201, 8 if planted % 2 else 64, 170, planted, splits=5)
+    cases.check_mixed_scores("cuda", torch.bfloat16, *shape, 201, 8 if planted % 2 else 64, 170, planted, splits=5,
+                             exact=planted in (0, 127, 199))
 
 
 @pytest.mark.parametrize("shape", SHAPES[1:6])
@@ -112,7 +113,7 @@ def test_mixed_scores_in_32_bit(shape):
 def test_mixed_scores_of_long_sequences():
     """Far keys over many key ranges and shares."""
     for planted in (3, 1030, 2040):
-        cases.check_mixed_scores("cuda", torch.bfloat16, 6, 3, 64, 32, 2050, 16, 40, planted, splits=32)
+        cases.check_mixed_scores("cuda", torch.bfloat16, 6, 3, 64, 32, 2050, 16, 40, planted, splits=61)
 
 
 @pytest.mark.parametrize("dtype", sorted(DTYPES))

@@ -108,6 +108,64 @@ __global__ void __launch_bounds__(kLatentThreads) latent_prep_kernel(const Laten
   }
 }
 
+// The norms alone (no queries to rotate), rows of whole 16-byte pieces: one warp per (token, part), part 0 the cache row,
+// the last part the queries' latent.
+static constexpr int kNormVecs = 8;                      // vectors of eight elements per lane at most
+
+template <typename T>
+__device__ __forceinline__ void warp_norm_row(const T* src, const T* w, T* dst, int n, float eps, int lane) {
+  float x[kNormVecs][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kNormVecs; ++i) {
+    const int v = lane + i * 32;
+    if (v * 8 >= n) continue;
+    Row8<T>::load(src, v, x[i]);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(x[i][j], x[i][j], ss);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(n) + eps);
+#pragma unroll
+  for (int i = 0; i < kNormVecs; ++i) {
+    const int v = lane + i * 32;
+    if (v * 8 >= n) continue;
+    float g[8];
+    Row8<T>::load(w, v, g);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[i][j] = x[i][j] * inv * g[j];
+    Row8<T>::store(dst, v, x[i]);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kLatentThreads) latent_norm_kernel(const LatentPrepParams p, const int T_rows) {
+  pdl_trigger();
+  pdl_wait();
+  const int parts = (p.kv ? 1 : 0) + (p.low ? 1 : 0), lane = threadIdx.x & 31;
+  const int item = blockIdx.x * (kLatentThreads / 32) + (threadIdx.x >> 5);
+  if (item >= T_rows * parts) return;
+  const int part = item / T_rows;
+  const long long t = item - part * T_rows;
+  if (p.low && part == parts - 1) {
+    warp_norm_row<T>(static_cast<const T*>(p.low) + t * p.low_stride, static_cast<const T*>(p.low_w),
+                     static_cast<T*>(p.low_out) + t * p.low_width, p.low_rank, p.eps, lane);
+    return;
+  }
+  const int slot = p.slots[t];
+  if (slot < 0) return;
+  int pos = p.positions[t];
+  pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
+  const T* kv = static_cast<const T*>(p.kv) + t * p.kv_stride;
+  T* dst = static_cast<T*>(p.cache) + static_cast<long long>(slot) * p.row;
+  const int half = p.rot >> 1;
+  const float* cs = p.cos_sin + static_cast<long long>(pos) * p.rot;
+  for (int i = lane; i < half; i += 32) rotate_pair<T>(kv + p.rank, dst + p.rank, i, half, p.neox, cs);
+  for (int d = p.rank + p.rot + lane; d < p.row; d += 32) dst[d] = from_float<T>(0.f);
+  warp_norm_row<T>(kv, static_cast<const T*>(p.norm_w), dst, p.rank, p.eps, lane);
+}
+
 // ------------------------------------------------------------- per-head products
 struct HeadGemmParams {
   const void* a;               // [T, H, K]
@@ -279,6 +337,19 @@ extern "C" int b200_latent_prep(void* q, long long q_stride, const void* kv, lon
                      low_width};
   int ny = q ? (H * rot / 2 + 4 * kLatentThreads - 1) / (4 * kLatentThreads) : (kv && low ? 2 : 1);
   if (T >= 1024 || ny < 1) ny = 1;
+  const auto whole = [&](const void* ptr, long long stride, int n) {
+    return ptr == nullptr || ((reinterpret_cast<uintptr_t>(ptr) & (is_fp32 ? 31 : 15)) == 0 && stride % 8 == 0 && n % 8 == 0 &&
+                              n <= kNormVecs * 256);
+  };
+  if (q == nullptr && whole(kv, kv_stride, rank) && whole(norm_w, 0, rank) && whole(low, low_stride, low_rank) &&
+      whole(low_w, 0, low_rank) && whole(low_out, low_width, low_rank) && whole(kv ? cache : nullptr, row, rank) &&
+      (low == nullptr || low_rank == low_width)) {
+    const int items = T * ((kv ? 1 : 0) + (low ? 1 : 0)), per = kLatentThreads / 32;
+    const dim3 grid((items + per - 1) / per), block(kLatentThreads);
+    const cudaError_t e = is_fp32 ? launch_pdl(latent_norm_kernel<float>, grid, block, 0, stream, 1, p, T)
+                                  : launch_pdl(latent_norm_kernel<__nv_bfloat16>, grid, block, 0, stream, 1, p, T);
+    return e == cudaSuccess ? 0 : -3;
+  }
   const dim3 grid(T, ny), block(kLatentThreads);
   const cudaError_t e = is_fp32 ? launch_pdl(latent_prep_kernel<float>, grid, block, 0, stream, 1, p)
                                 : launch_pdl(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, stream, 1, p);

@@ -267,51 +267,63 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_k
     issue(it + 1);
     make_bias(it + 1);
 
-    // ---- mixture: 16 output heads x 16 keys of a query per step
+    // ---- mixture: 16 output heads x 16 keys of one or two queries per step
+    constexpr int UNITS = BQ / ROWS_STEP >= 2 ? 2 : 1;
     float* out = out_tile;
     uint32_t s_at = s_lane;
 #pragma unroll 1
-    for (int row = row0; row < BQ; row += ROWS_STEP, out += L.row_step, s_at += ROWS_STEP * (BK * 2 + 16)) {
+    for (int row = row0; row < BQ; row += UNITS * ROWS_STEP, out += UNITS * L.row_step, s_at += UNITS * ROWS_STEP * (BK * 2 + 16)) {
       if (tok0 + row >= q_len) break;
+      const bool second = tok0 + row + ROWS_STEP < q_len;
       uint32_t t_ob = t_lane;
       float* o_ob = out;
 #pragma unroll 1
       for (int left = p.Ho - (lane >> 2), ob = 0; ob < L.ho16; ob += 16, left -= 16) {
-        float o[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        float o[UNITS][2][4];
+#pragma unroll
+        for (int u = 0; u < UNITS; ++u)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) o[u][0][e] = o[u][1][e] = 0.f;
         uint32_t s_kb = s_at, t_kb = t_ob;
 #pragma unroll 1
         for (int kb = 0; kb < L.hs16; kb += 16, s_kb += 16 * L.head, t_kb += 32) {
-          uint32_t sf[PLANES][4], tf[4];
-#pragma unroll
-          for (int t = 0; t < PLANES; ++t) ldmatrix_x4_trans(sf[t], s_kb + t * L.plane);
+          uint32_t sf[PLANES][UNITS][4], tf[4];
           ldmatrix_x4(tf, t_kb);
 #pragma unroll
-          for (int t = PLANES - 1; t >= 0; --t) {
-            mma_bf16_16816(o[0], tf, sf[t][0], sf[t][1]);
-            mma_bf16_16816(o[1], tf, sf[t][2], sf[t][3]);
-          }
+          for (int t = PLANES - 1; t >= 0; --t)
+#pragma unroll
+            for (int u = 0; u < UNITS; ++u) ldmatrix_x4_trans(sf[t][u], s_kb + t * L.plane + u * ROWS_STEP * (BK * 2 + 16));
+          const auto add = [&](int t) {
+#pragma unroll
+            for (int u = 0; u < UNITS; ++u) {
+              mma_bf16_16816(o[u][0], tf, sf[t][u][0], sf[t][u][1]);
+              mma_bf16_16816(o[u][1], tf, sf[t][u][2], sf[t][u][3]);
+            }
+          };
+#pragma unroll
+          for (int t = PLANES - 1; t >= 0; --t) add(t);
           if (p.talk_terms > 1) {                          // (products below 2^-24 are left out)
             ldmatrix_x4(tf, t_kb + L.t_plane);
-#pragma unroll
-            for (int t = 1; t >= 0; --t) {
-              mma_bf16_16816(o[0], tf, sf[t][0], sf[t][1]);
-              mma_bf16_16816(o[1], tf, sf[t][2], sf[t][3]);
-            }
+            add(1);
+            add(0);
             ldmatrix_x4(tf, t_kb + 2 * L.t_plane);
-            mma_bf16_16816(o[0], tf, sf[0][0], sf[0][1]);
-            mma_bf16_16816(o[1], tf, sf[0][2], sf[0][3]);
+            add(0);
           }
         }
-        if (left > 0) {
-          *reinterpret_cast<float2*>(o_ob) = make_float2(o[0][0], o[0][1]);
-          *reinterpret_cast<float2*>(o_ob + 8) = make_float2(o[1][0], o[1][1]);
+        float* o_low = o_ob + 8 * p.pitch;
+#pragma unroll
+        for (int u = 0; u < UNITS; ++u) {
+          if (u == 1 && !second) continue;
+          if (left > 0) {
+            *reinterpret_cast<float2*>(o_ob + u * L.row_step) = make_float2(o[u][0][0], o[u][0][1]);
+            *reinterpret_cast<float2*>(o_ob + u * L.row_step + 8) = make_float2(o[u][1][0], o[u][1][1]);
+          }
+          if (left > 8) {
+            *reinterpret_cast<float2*>(o_low + u * L.row_step) = make_float2(o[u][0][2], o[u][0][3]);
+            *reinterpret_cast<float2*>(o_low + u * L.row_step + 8) = make_float2(o[u][1][2], o[u][1][3]);
+          }
         }
-        o_ob += 8 * p.pitch;
-        if (left > 8) {
-          *reinterpret_cast<float2*>(o_ob) = make_float2(o[0][2], o[0][3]);
-          *reinterpret_cast<float2*>(o_ob + 8) = make_float2(o[1][2], o[1][3]);
-        }
-        o_ob += 8 * p.pitch;
+        o_ob += 16 * p.pitch;
         t_ob += 16 * L.t_row;
       }
     }

@@ -247,6 +247,8 @@ LOW_RANK = 128
 TAPS = 4
 # fp32 multiply-adds per second of the CUDA cores at the maximum clock: what bounds the recurrences
 FP32_FLOPS = 148 * 128 * 2 * 1.965e9
+# exponentials, logarithms and reciprocals per second of the special function units at that clock
+SPECIAL_OPS = 148 * 16 * 1.965e9
 
 
 def fuvirax(size) -> ModelConfig:
@@ -700,8 +702,8 @@ def dalavik_kernels(size) -> List[dict]:
     f32 = dict(dtype=torch.float32, device="cuda")
     i32 = dict(dtype=torch.int32, device="cuda")
 
-    def bound(nbytes: float, flops: float = 0.0, fp32: float = 0.0) -> float:
-        return max(nbytes / bw, flops / fl, fp32 / FP32_FLOPS) * 1e3
+    def bound(nbytes: float, flops: float = 0.0, fp32: float = 0.0, special: float = 0.0) -> float:
+        return max(nbytes / bw, flops / fl, fp32 / FP32_FLOPS, special / SPECIAL_OPS) * 1e3
 
     def entry(name: str, fn, cost, like=None, like_cost=None):
         ms, b = _time(fn), bound(*cost)
@@ -744,9 +746,10 @@ def dalavik_kernels(size) -> List[dict]:
         product("gate / up + relu (like: gate / up + silu)", x, 2 * ff, 2 * ff, act=dict(swiglu=True, act=ops.RELU),
                 like_act=dict(swiglu=True))
         sp = (side + 7) // 8 * 8
-        product("token input: gate (like: both latents of MLA)", x, sp, qr + row)
+        product("token input: gate (like: router of 128 experts)", x, sp, 128)
         z = torch.randn(t, sp, **bf)
-        product("token input: back (like: queries from their latent)", z, w, h * qk, zq)
+        low = torch.randn(t, 2 * LOW_RANK, **bf)
+        product("token input: back (like: low-rank product of Fuvirax)", z, w, h * 2 * hd, low)
         ids, table = torch.randint(0, VOCAB, (t,), **i32), torch.randn(VOCAB, side * DALAVIK_LAYERS, **bf)
         gu = torch.randn(t, 2 * sp, **bf)
         entry("token input: gated rows (like: silu(gate) * up)", lambda: ops.gelu_rows(z, ids, table, side, side),
@@ -874,8 +877,8 @@ def dalavik_kernels(size) -> List[dict]:
         entry("attention with mixed scores (like: grouped-query attention)",
               lambda: ops.mixed_attention(qc, kc, vc, o, bt, cu if pre else None, lens, n, rows, d, e, d ** -0.5, SOFTCAP,
                                           (r1, r2), talk, sink, max_seq_len=ctx, talk_exact=True),
-              (kv * (d + e) + t * h * (d + e) * 2, 2.0 * pairs * (d + e), 2.0 * pairs * h), like_attn,
-              (kv * (d + le) + t * h * (d + le) * 2, 2.0 * pairs * (d + le)))
+              (kv * (d + e) + t * h * (d + e) * 2, 2.0 * pairs * (d + e), 2.0 * pairs * h, 3.0 * pairs), like_attn,
+              (kv * (d + le) + t * h * (d + le) * 2, 2.0 * pairs * (d + le), 0.0, 1.0 * pairs))
         del kc, vc, lvc, y, q, kk, vv, qc, res
         gc.collect()
         torch.cuda.empty_cache()

@@ -35,8 +35,8 @@ struct MixedAttnParams {
   float scale, softcap;
   int splits;                  // decode: CTAs that share a row's keys
   float* scratch;              // decode: [rows, splits, Ho, DVP], then [rows, splits, Ho, 2]; prompts: see pitch
-  // prompts: the query tiles of 16 rows tile0 .. tile0 + tiles - 1 of every sequence; their mixed scores (times
-  // log2 e) are [B, tiles, 16, Ho, pitch]
+  // prompts: portions are cut into tiles of 16 queries, numbered through all sequences; this call makes tiles
+  // tile0 .. tile0 + tiles - 1, whose mixed scores (times log2 e) are [tiles, 16, Ho, pitch]
   int tile0, tiles, max_q_len, max_keys;
   int range;                   // keys of a score CTA
   int talk_terms;              // 1: bf16 holds every element of talk exactly, 3: it does not

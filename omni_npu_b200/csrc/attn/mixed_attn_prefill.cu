@@ -66,6 +66,36 @@ inline Plan plan(int Hs, int Hk, int Ho, int DP, int terms) {
   return {0, 0, 0};
 }
 
+// Query tiles of the sequences before b.
+__device__ __forceinline__ int tiles_before(const int* cu_q, int b, int lane) {
+  int n = 0;
+  for (int i = lane; i < b; i += 32) n += (cu_q[i + 1] - cu_q[i] + BQ - 1) / BQ;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) n += __shfl_xor_sync(0xffffffffu, n, o);
+  return n;
+}
+// The sequence that query tile `tile` belongs to (-1: none), and the tile's number in it.
+__device__ __forceinline__ int tile_owner(const int* cu_q, int B, int tile, int lane, int* local) {
+  for (int base = 0; base < B; base += 32) {
+    const int i = base + lane;
+    const int mine = i < B ? (cu_q[i + 1] - cu_q[i] + BQ - 1) / BQ : 0;
+    int upto = mine;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, upto, o);
+      if (lane >= o) upto += v;
+    }
+    const unsigned past = __ballot_sync(0xffffffffu, upto > tile);
+    if (past) {
+      const int l = __ffs(past) - 1;
+      *local = tile - __shfl_sync(0xffffffffu, upto - mine, l);
+      return base + l;
+    }
+    tile -= __shfl_sync(0xffffffffu, upto, 31);
+  }
+  return -1;
+}
+
 // x0, x1 as sums of three bf16 numbers each
 __device__ __forceinline__ void split3(float x0, float x1, uint32_t (&w)[PLANES]) {
 #pragma unroll
@@ -95,11 +125,13 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_k
 
   pdl_trigger();
   pdl_wait();
-  const int b = blockIdx.z;
+  const int tile = gridDim.x - 1 - blockIdx.x;             // (the tiles with most keys first)
+  int local = 0;
+  const int b = tile_owner(p.cu_q, p.B, p.tile0 + tile, lane, &local);
+  if (b < 0) return;
   const long long q_begin = p.cu_q[b];
   const int q_len = static_cast<int>(p.cu_q[b + 1] - q_begin);
-  const int tok0 = (p.tile0 + blockIdx.x) * BQ;
-  if (tok0 >= q_len) return;
+  const int tok0 = local * BQ;
   const int ctx = p.seq_lens[b] - q_len;
   const int hi = ctx + min(q_len, tok0 + BQ);                      // keys that some row sees
   const int k_begin = blockIdx.y * p.range, k_end = min(hi, k_begin + p.range);
@@ -207,7 +239,7 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_k
   const int row0 = warp / HALVES, k16 = warp % HALVES;
   const uint32_t s_lane = st + ((lane & 7) + ((lane >> 3) & 1) * 8) * L.head + row0 * (BK * 2 + 16) + k16 * 32 + (lane >> 4) * 16;
   const uint32_t t_lane = tt + (lane & 15) * L.t_row + (lane >> 4) * 16;
-  float* out_tile = p.scratch + (((static_cast<long long>(b) * p.tiles + blockIdx.x) * BQ + row0) * p.Ho + (lane >> 2)) * p.pitch +
+  float* out_tile = p.scratch + ((static_cast<long long>(tile) * BQ + row0) * p.Ho + (lane >> 2)) * p.pitch +
                     k_begin + k16 * 16 + (lane & 3) * 2;
   const int tiles = (k_end - k_begin + BK - 1) / BK;
   const int ks_used = p.DP >> 4;
@@ -357,8 +389,10 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
   const int tt = BM / hc;
   const long long q_begin = p.cu_q[b];
   const int q_len = static_cast<int>(p.cu_q[b + 1] - q_begin);
-  const int first = p.tile0 * mpre::BQ;
-  const int last = min(q_len, first + p.tiles * mpre::BQ);
+  // this sequence's share of the call's query tiles
+  const int before = mpre::tiles_before(p.cu_q, b, lane);
+  const int first = max(0, p.tile0 - before) * mpre::BQ;
+  const int last = min(q_len, (p.tile0 + p.tiles - before) * mpre::BQ);
   const int m0 = first + (gridDim.x - 1 - blockIdx.x) * tt;        // (the tiles with most keys first)
   if (m0 >= last) return;
   const int tok_end = min(last, m0 + tt);
@@ -368,14 +402,10 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
   const int tiles = (hi + BN - 1) / BN;
 
   const int rows_live = (tok_end - m0) * hc;                       // rows: (token, head of the group)
-  const float* sbase = p.scratch + ((static_cast<long long>(b) * p.tiles * mpre::BQ + (m0 - first)) * p.Ho +
-                                    vh * per + head0) * p.pitch + (tid & 15) * 4;
-  int srow[BM / 16];                                               // score rows that this thread copies from
-#pragma unroll
-  for (int i = 0; i < BM / 16; ++i) {
-    const int r = (tid >> 4) + i * 16, tok = r / hc;
-    srow[i] = r < rows_live ? tok * p.Ho + (r - tok * hc) : -1;
-  }
+  const float* sbase = p.scratch + ((static_cast<long long>(before - p.tile0) * mpre::BQ + m0) * p.Ho + vh * per + head0) * p.pitch + (tid & 15) * 4;
+  __shared__ int srow[BM];                                         // where the tile's rows of scores lie, -1: nowhere
+  if (tid < BM) srow[tid] = tid < rows_live ? tid / hc * p.Ho + tid % hc : -1;
+  __syncthreads();
   auto issue = [&](int it) {
     if (it < tiles) {
       // four threads per key row, 16-byte pieces dealt out in turn
@@ -391,9 +421,10 @@ __global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_
       const uint32_t sdst = s0 + (it & 1) * S_BYTES + (tid & 15) * 16;
 #pragma unroll
       for (int i = 0; i < BM / 16; ++i) {
-        if (srow[i] >= 0)
+        const int at = srow[(tid >> 4) + i * 16];
+        if (at >= 0)
           asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sdst + ((tid >> 4) + i * 16) * S_PITCH * 4),
-                       "l"(sbase + srow[i] * p.pitch + it * BN) : "memory");
+                       "l"(sbase + at * p.pitch + it * BN) : "memory");
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -533,7 +564,7 @@ static int launch_scores(const MixedAttnParams& p, cudaStream_t stream) {
   mpre::Layout l = mpre::layout(p.Hs, p.Hk, p.Ho, p.DP, BK, p.talk_terms);
   l.per_k = p.Hs / p.Hk;
   l.row_step = WARPS / (BK / 16) * p.Ho * p.pitch;
-  const dim3 grid(p.tiles, (p.max_keys + p.range - 1) / p.range, p.B);
+  const dim3 grid(p.tiles, (p.max_keys + p.range - 1) / p.range);
   return launch_pdl(kern, grid, dim3(WARPS * 32), l.bytes, stream, 1, p, l) == cudaSuccess ? 0 : -21;
 }
 
@@ -556,7 +587,7 @@ static int launch_values(const MixedAttnParams& p, cudaStream_t stream) {
   }
   const int per = p.Ho / p.Hv, heads = per < mval::BM ? per : mval::BM;
   const int hchunks = (per + heads - 1) / heads, tt = mval::BM / heads;
-  const int toks = p.tiles * mpre::BQ;
+  const int own = (p.max_q_len + mpre::BQ - 1) / mpre::BQ, toks = (p.tiles < own ? p.tiles : own) * mpre::BQ;
   const dim3 grid((toks + tt - 1) / tt, p.Hv * hchunks, p.B);
   return launch_pdl(kern, grid, dim3(mval::THREADS), SMEM, stream, 1, p, heads) == cudaSuccess ? 0 : -21;
 }
@@ -567,7 +598,7 @@ int mixed_prefill(const MixedAttnParams& in, cudaStream_t stream) {
   if (c.bk == 0 || p.DVP > 256 || (p.talk_terms != 1 && p.talk_terms != mpre::PLANES)) return -2;
   // keys of a score CTA: longer ranges where there are CTAs enough
   p.range = 128;
-  while (p.range < 1024 && static_cast<long long>(p.tiles) * p.B * ((p.max_keys + 2 * p.range - 1) / (2 * p.range)) >= 888)
+  while (p.range < 1024 && static_cast<long long>(p.tiles) * ((p.max_keys + 2 * p.range - 1) / (2 * p.range)) >= 888)
     p.range *= 2;
   int rc;
   if (c.bk == 32) rc = c.warps == 8 ? launch_scores_ks<8, 32>(p, c, stream) : launch_scores_ks<16, 32>(p, c, stream);

@@ -888,8 +888,8 @@ int64_t mixed_attention_kind(const Tensor& q, const Tensor& k_cache, const Tenso
   return kind;
 }
 
-// out [T, >= Ho * Dv].  kind 1: `scratch` holds the partial results of a split decode row, or the mixed scores of the
-// query tiles tile0 .. tile0 + tiles - 1 of every portion.
+// out [T, >= Ho * Dv].  kind 1: `scratch` holds the partial results of split decode rows, or the mixed scores of the
+// query tiles tile0 .. tile0 + tiles - 1, numbered through all portions.
 void mixed_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, Tensor out, const Tensor& block_tables,
                      const c10::optional<Tensor>& cu_q, const Tensor& seq_lens, int64_t num_seqs, int64_t q_len,
                      int64_t max_keys, int64_t head_dim, int64_t head_dim_v, double scale, double softcap,
@@ -930,7 +930,7 @@ void mixed_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_cac
   const int64_t pitch = (max_keys + 63) / 64 * 64;
   float* sp = nullptr;
   if (scratch.has_value()) {
-    const int64_t need = cu ? num_seqs * tiles * 16 * Ho * pitch : T * splits * Ho * (v_cache.size(3) + 2);
+    const int64_t need = cu ? tiles * 16 * Ho * pitch : T * splits * Ho * (v_cache.size(3) + 2);
     TORCH_CHECK(scratch->is_cuda() && scratch->is_contiguous() && (int64_t)scratch->nbytes() >= need * 4,
                 "mixed_attention: scratch");
     sp = static_cast<float*>(scratch->data_ptr());

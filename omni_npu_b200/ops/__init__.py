@@ -763,7 +763,7 @@ def gated_attention(q: torch.Tensor, gate: Optional[torch.Tensor], k_cache: torc
 
 
 # --------------------------------------------------- attention whose heads share their scores
-MIXED_SCORE_BYTES = int(os.environ.get("OMNI_B200_MIXED_SCORE_MB", "512")) << 20
+MIXED_SCORE_BYTES = int(os.environ.get("OMNI_B200_MIXED_SCORE_MB", "1152")) << 20
 
 
 def mixed_decode_splits(num_rows: int, keys: int, sms: int = 148) -> int:
@@ -808,10 +808,13 @@ def mixed_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         _count(2 if splits > 1 else 1)
         core.mixed_attention(*args, 1, terms, splits, scratch, 0, 0)
         return
-    # prompt portions: the mixed scores of a run of query tiles go through memory
-    tile, tiles, pitch = 16, (max_q_len + 15) // 16, (keys + 63) // 64 * 64
-    run = max(1, min(tiles, MIXED_SCORE_BYTES // (num_seqs * tile * talk.shape[0] * pitch * 4)))
-    scores = torch.empty(num_seqs * run * tile * talk.shape[0] * pitch, dtype=torch.float32, device=q.device)
+    # prompt portions: the mixed scores of a run of query tiles (of 16 rows, numbered through all portions) go through
+    # memory
+    tiles, pitch = (rows + 15 * num_seqs) // 16, (keys + 63) // 64 * 64
+    row_floats = talk.shape[0] * pitch
+    most = max(1, MIXED_SCORE_BYTES // (16 * row_floats * 4))
+    run = -(-tiles // -(-tiles // most))                    # runs of equal length
+    scores = torch.empty(run * 16 * row_floats, dtype=torch.float32, device=q.device)
     for t0 in range(0, tiles, run):
         _count(2)
         core.mixed_attention(*args, 1, terms, 1, scores, t0, min(run, tiles - t0))

@@ -279,8 +279,9 @@ def check_mixed_batch(device, dtype, n, kv, dim, vdim, lens, portions, bs=16) ->
     run(portions, cu)
     keep = ops.MIXED_SCORE_BYTES
     try:
-        ops.MIXED_SCORE_BYTES = 1                        # one query tile of each portion at a time
-        run(portions, cu)
+        for tiles in (1, 3):                             # so many query tiles at a time
+            ops.MIXED_SCORE_BYTES = tiles * 16 * n * ((max(lens) + 63) // 64 * 64) * 4
+            run(portions, cu)
     finally:
         ops.MIXED_SCORE_BYTES = keep
     run([1] * len(lens), None)

@@ -122,6 +122,12 @@ def test_mixed_scores_of_a_batch(dtype, shape):
     cases.check_mixed_batch("cuda", DTYPES[dtype], *shape, [140, 7, 325, 64, 33], [100, 7, 2, 17, 1])
 
 
+def test_mixed_scores_of_many_portions():
+    """More sequences than a warp has lanes."""
+    lens = [1 + (37 * i) % 50 for i in range(45)]
+    cases.check_mixed_batch("cuda", torch.bfloat16, 4, 2, 32, 32, lens, [1 + n // 2 for n in lens])
+
+
 @pytest.mark.parametrize("dtype", sorted(DTYPES))
 @pytest.mark.parametrize("shape", [(3, 20, 8, 12, 28, 18), (4, 128, 64, 128, 512, 384), (18, 16, 6, 24, 136, 72)])
 @pytest.mark.parametrize("planted", [0, 15, 49, 51])

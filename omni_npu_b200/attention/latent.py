@@ -28,6 +28,8 @@ class LatentAttention(nn.Module):
     """``num_heads``: heads of this rank.  ``w_uk`` [heads * nope, rank] and ``w_uv`` [heads * v, rank] are
     set before ``build_absorbed``."""
 
+    layer_idx = -1           # (the cache is named at each call; what looks for attention layers finds this one)
+
     def __init__(self, num_heads: int, nope_dim: int, rope_dim: int, v_head_dim: int, kv_rank: int, scale: float,
                  neox: bool, eps: float, dtype: torch.dtype, device, q_rank: int = 0, own_rows: bool = True,
                  rows_shared: bool = False) -> None:

@@ -88,8 +88,8 @@ bool mixed_decode_fits(int Hs, int Hk, int Ho, int Hv, int DP, int DVP) {
 
 // UNITS: accumulator tiles (8 heads x 16 columns) per warp.  HB: output heads that a lane mixes at a time
 template <int UNITS, int WARPS, int KT, int HB>
-__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && UNITS <= 8 ? 2 : 1) mixed_decode_kernel(const MixedAttnParams p,
-                                                                                                       const mdec::Layout L) {
+__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && UNITS <= 8 ? 2 : 1)
+mixed_decode_kernel(const MixedAttnParams p, const mdec::Layout L) {
   using namespace mdec;
   constexpr int THREADS = WARPS * 32, SUB = 32 / KT;
   extern __shared__ __align__(128) uint8_t smem[];

@@ -114,8 +114,8 @@ bool mixed_prefill_fits(int Hs, int Hk, int Ho, int Hv, int DP, int DVP) {
 // ------------------------------------------------------------- scores
 // KS: steps of 16 along the head size; HPW: heads per warp and pass (16 registers of query per head and 4 steps)
 template <int WARPS, int KS, int HPW, int BK>
-__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) mixed_scores_kernel(const MixedAttnParams p,
-                                                                                                const mpre::Layout L) {
+__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1)
+mixed_scores_kernel(const MixedAttnParams p, const mpre::Layout L) {
   using namespace mpre;
   constexpr int THREADS = WARPS * 32, DK = KS * 16;
   extern __shared__ __align__(128) uint8_t smem[];
@@ -373,8 +373,8 @@ constexpr int S_BYTES = BM * S_PITCH * 4;
 
 // DV: upper bound of the padded value size
 template <int DV>
-__global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2) mixed_values_kernel(const MixedAttnParams p,
-                                                                                       const int heads_per_tile) {
+__global__ void __launch_bounds__(mval::THREADS, DV > 128 ? 1 : 2)
+mixed_values_kernel(const MixedAttnParams p, const int heads_per_tile) {
   using namespace mval;
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int V_BYTES = BN * DV * 2;

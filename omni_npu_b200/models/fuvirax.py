@@ -26,7 +26,6 @@ from typing import Any, Dict, Iterable, List, Optional, Tuple
 import torch
 from torch import nn
 
-from .. import ops
 from ..attention.latent import LatentAttention
 from ..attention.metadata import get_forward_context
 from ..attention.recurrent import DeltaRuleAttention, GatedLinearAttention

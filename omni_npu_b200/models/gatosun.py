@@ -31,7 +31,6 @@ from torch import nn
 
 from .. import ops
 from ..attention.gqa import NormedGQAAttention
-from ..attention.metadata import get_forward_context
 from ..attention.recurrent import DecayLinearAttention, TimeMixAttention
 from ..config import (AttentionSpec, DecayLinearSpec, DenseSpec, EngineConfig, ExpertSpec, LayerSpec, ModelConfig, MoESpec,
                       ParallelSpec, TimeMixSpec, to_dtype)

@@ -2,7 +2,7 @@
 checkpoint's tensors (name -> shape and how it is placed), and the base of their mixers."""
 from __future__ import annotations
 
-from typing import Any, Callable, Dict, Iterable, List, Optional, Tuple
+from typing import Any, Callable, Dict, Iterable, List, Tuple
 
 import torch
 from torch import nn
